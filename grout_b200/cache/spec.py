@@ -36,12 +36,15 @@ class KVSpec:
     token's value is read from its key row (a latent that serves as both), so the
     store holds one tensor and hands it out as keys and as values.  ``keep_first``:
     with a window, a sequence's first ``keep_first`` tokens stay visible to every
-    later query, so the pages that hold them are never given back."""
+    later query, so the pages that hold them are never given back.  ``chunk``: queries see
+    the tokens of their own chunk of that many positions only (positions count from the
+    sequence's start), so what lies in front of the next token's chunk is given back."""
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     values_in_keys: bool = False
     keep_first: int = 0
+    chunk: Optional[int] = None
 
     def make_store(self, n_layers: int, sizes: StoreSizes, dtype, device, allocate: bool = True):
         from .stores import KVStore

@@ -6,8 +6,8 @@
 change after construction, so a captured CUDA graph stays valid.  Pages are
 zero-filled once and never cleared again: a sequence's length gates every read.  (The reference keeps one
 ``[kv heads, S, D]`` pair per layer for its single sequence,
-src/model.rs:1450-1455.)  A store with a window gives pages back as soon as
-every token in them has left the window of all later queries.
+src/model.rs:1450-1455.)  A store with a window (or chunks) gives pages back as soon
+as every token in them has left the window (the chunk) of all later queries.
 
 ``StateStore``: ``[layers, slots + 1, *shape]`` of fixed-size state, zeroed when a
 slot is opened; the last row belongs to no sequence and is where padding rows
@@ -88,14 +88,16 @@ class KVStore:
             self._dirty[slot] = min(self._dirty.get(slot, first), first)
 
     def trim(self, slot: int, length: int) -> None:
-        """With a window: frees pages whose tokens no query at position >= length
+        """With a window or chunks: frees pages whose tokens no query at position >= length
         can see any more (all their positions are <= length - window, and none of
-        them is among the first ``keep_first``)."""
-        w = self.spec.window
-        if w is None:
+        them is among the first ``keep_first``; or all lie in front of the chunk of
+        position ``length``)."""
+        w, c = self.spec.window, self.spec.chunk
+        if w is None and c is None:
             return
         pages = self.pages_of[slot]
-        dead = max(0, length - w + 1) // PAGE_TOKENS   # pages [0, dead) are out of reach
+        first = max(0, length - w + 1 if w is not None else 0, length // c * c if c is not None else 0)
+        dead = first // PAGE_TOKENS                    # pages [0, dead) are out of reach
         kept = pages_for(self.spec.keep_first)         # ... but for those with kept first tokens
         for i in range(kept, min(dead, len(pages))):
             if pages[i] is not None:

@@ -5,9 +5,10 @@ from .suvazen import SuvazenConfig
 from .sonalorn import SonalornConfig
 from .zutazen import ZutazenConfig
 from .mananex import MananexConfig
+from .kakotar import KakotarConfig
 from .registry import (Architecture, known_architectures, load_config, register_architecture,
                        resolve_architecture, unregister_architecture)
 
-__all__ = ["ConfigError", "ModelConfig", "GenerationConfig", "Qwen3Config", "SuvazenConfig", "SonalornConfig", "ZutazenConfig", "MananexConfig", "Architecture",
+__all__ = ["ConfigError", "ModelConfig", "GenerationConfig", "Qwen3Config", "SuvazenConfig", "SonalornConfig", "ZutazenConfig", "MananexConfig", "KakotarConfig", "Architecture",
            "known_architectures", "load_config", "register_architecture",
            "resolve_architecture", "unregister_architecture", "read_json"]

@@ -40,6 +40,7 @@ struct DecodeArgs {
   const float* sinks;      // [nq] one more logit of every head's denominator, or null
   ScoreCap cap;            // the score cap (off when cap_log2 == 0)
   int keep_first;          // with a window: a sequence's first keep_first keys stay visible behind it
+  int chunk;               // > 0: a query sees the keys of its own chunk of positions only
 };
 
 template <int DT>
@@ -59,7 +60,7 @@ __global__ void __launch_bounds__(DC_THREADS) attn_decode_kernel(const DecodeArg
 
   // key tiles of this split
   const int pos = kv_len - 1;
-  const int key_lo = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+  const int key_lo = first_key(pos, a.window, a.chunk);
   const int tile_lo = key_lo / DC_BN;
   // With kept first keys the tiles in front of the window that hold some are visited too:
   // the splits divide the list v = 0 .. n_tiles - 1, the kept tiles first, then the window's.
@@ -322,6 +323,7 @@ static int launch(const DecodeArgs& a, cudaStream_t s) {
 // 128, groups of more than 16 query heads per kv head, and pages that are no
 // multiple of 32 tokens; the caller then uses the plain kernel.
 GB_EXPORT int gb_attn_decode_bf16(const DecodeArgs* a, int D, cudaStream_t s) {
+  if (a->chunk < 0) return GB_ERR_BAD_ARG;
   if (a->n_seqs < 0 || a->nq <= 0 || a->nkv <= 0 || a->nq % a->nkv || a->max_pages <= 0 ||
       a->n_splits <= 0)
     return GB_ERR_BAD_ARG;

@@ -53,6 +53,7 @@ struct DecodeTmaArgs {
   const float* sinks;      // [nq] one more logit of every head's denominator, or null
   ScoreCap cap;            // the score cap (off when cap_log2 == 0)
   int keep_first;          // with a window: a sequence's first keep_first keys stay visible behind it
+  int chunk;               // > 0: a query sees the keys of its own chunk of positions only
 };
 
 #define DA_STAMP(slot)                                                                          \
@@ -96,7 +97,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k,
 
   // key tiles of this split
   const int pos = kv_len - 1;
-  const int key_lo = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+  const int key_lo = first_key(pos, a.window, a.chunk);
   const int tile_lo = key_lo / DA_BN;
   // With kept first keys the tiles in front of the window that hold some are visited too:
   // the splits divide the list v = 0 .. n_tiles - 1, the kept tiles first, then the window's.
@@ -428,6 +429,7 @@ static int launch(const CUtensorMap& mk, const CUtensorMap& mv, const DecodeTmaA
 GB_EXPORT int gb_attn_decode_tma(const void* k_pages, const void* v_pages, long long n_pages,
                                  const DecodeTmaArgs* a, int D, int page, int stages,
                                  cudaStream_t s) {
+  if (a->chunk < 0) return GB_ERR_BAD_ARG;
   if (a->n_seqs < 0 || a->nq <= 0 || a->nkv <= 0 || a->nq % a->nkv || a->max_pages <= 0 ||
       a->n_splits <= 0 || n_pages <= 0 || !k_pages || !v_pages || !a->error)
     return GB_ERR_BAD_ARG;

@@ -11,7 +11,8 @@
 // when j > pos - W (the reference masks with -1e30 instead of skipping,
 // src/kernels.rs:1190-1191, 1256; same result) or, with `keep_first` F, when j < F:
 // the first F tokens of a sequence stay visible behind the window, at their own
-// positions; they are visited first, then the window.  With a cap c > 0 a score s
+// positions; they are visited first, then the window.  With a chunk size C, key j is visible
+// only when it lies in the query's own chunk, j / C == pos / C.  With a cap c > 0 a score s
 // becomes c * tanh(s / c); with sinks, exp(sinks[h]) is one more term of query
 // head h's denominator, without a value.
 #include "common.cuh"
@@ -28,7 +29,7 @@ __global__ void attn_generic_kernel(const T* __restrict__ q, const T* __restrict
                                     const int* __restrict__ slots, T* __restrict__ out, int nq,
                                     int nkv, int D, int page, float scale, int window,
                                     float softcap, const float* __restrict__ sinks,
-                                    int keep_first) {
+                                    int keep_first, int chunk) {
   extern __shared__ float sm[];
   __shared__ float scratch[32];
   float* q_s = sm;       // [D]
@@ -41,7 +42,7 @@ __global__ void attn_generic_kernel(const T* __restrict__ q, const T* __restrict
     return;
   }
   const int pos = token_pos[t];
-  const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int lo = first_key(pos, window, chunk);
   const int kvh = h / (nq / nkv);
   const int* table = block_table + (size_t)slot * max_pages;
   const T* qr = q + ((size_t)t * nq + h) * D;
@@ -111,8 +112,9 @@ template <typename T>
 static int launch(const void* q, const void* k_pages, const void* v_pages, const int* block_table,
                   int max_pages, const int* token_seq, const int* token_pos, const int* slots,
                   void* out, int n_tokens, int nq, int nkv, int D, int page, float scale,
-                  int window, float softcap, const float* sinks, int keep_first,
+                  int window, float softcap, const float* sinks, int keep_first, int chunk,
                   cudaStream_t stream) {
+  if (chunk < 0) return GB_ERR_BAD_ARG;
   if (keep_first < 0) return GB_ERR_BAD_ARG;
   if (n_tokens < 0 || nq <= 0 || nkv <= 0 || nq % nkv || D <= 0 || page <= 0 || max_pages <= 0)
     return GB_ERR_BAD_ARG;
@@ -122,7 +124,7 @@ static int launch(const void* q, const void* k_pages, const void* v_pages, const
   attn_generic_kernel<T><<<dim3(n_tokens, nq), ATT_THREADS, smem, stream>>>(
       (const T*)q, (const T*)k_pages, (const T*)v_pages, block_table, max_pages, token_seq,
       token_pos, slots, (T*)out, nq, nkv, D, page, scale, window, softcap, sinks,
-      window > 0 ? keep_first : 0);
+      window > 0 ? keep_first : 0, chunk);
   return gb_status();
 }
 
@@ -131,16 +133,16 @@ GB_EXPORT int gb_attn_generic_f32(const void* q, const void* k_pages, const void
                                   const int* token_pos, const int* slots, void* out, int n_tokens,
                                   int nq, int nkv, int D, int page, float scale, int window,
                                   float softcap, const float* sinks, int keep_first,
-                                  cudaStream_t s) {
+                                  int chunk, cudaStream_t s) {
   return launch<float>(q, k_pages, v_pages, block_table, max_pages, token_seq, token_pos, slots,
-                       out, n_tokens, nq, nkv, D, page, scale, window, softcap, sinks, keep_first, s);
+                       out, n_tokens, nq, nkv, D, page, scale, window, softcap, sinks, keep_first, chunk, s);
 }
 GB_EXPORT int gb_attn_generic_bf16(const void* q, const void* k_pages, const void* v_pages,
                                    const int* block_table, int max_pages, const int* token_seq,
                                    const int* token_pos, const int* slots, void* out, int n_tokens,
                                    int nq, int nkv, int D, int page, float scale, int window,
                                    float softcap, const float* sinks, int keep_first,
-                                  cudaStream_t s) {
+                                  int chunk, cudaStream_t s) {
   return launch<bf16>(q, k_pages, v_pages, block_table, max_pages, token_seq, token_pos, slots,
-                      out, n_tokens, nq, nkv, D, page, scale, window, softcap, sinks, keep_first, s);
+                      out, n_tokens, nq, nkv, D, page, scale, window, softcap, sinks, keep_first, chunk, s);
 }

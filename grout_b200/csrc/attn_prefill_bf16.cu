@@ -4,7 +4,7 @@
 // pages (64 keys), fetched with asynchronous copies two tiles deep while the
 // tensor cores work on the one before.  Queries start at the position that the
 // sequence had before the step, so a prompt that continues an earlier one works;
-// a window limits every row to its last `window` keys.
+// a window limits every row to its last `window` keys, a chunk size to the keys of its own chunk.
 //
 // Blocks are ordered longest first: the last query block of a long prompt visits
 // the most key tiles and is launched first (the idea of the reference's
@@ -31,6 +31,7 @@ struct PrefillArgs {
   const float* sinks;      // [nq] one more logit of every head's denominator, or null
   ScoreCap cap;            // the score cap (off when cap_log2 == 0)
   int keep_first;          // with a window: a sequence's first keep_first keys stay visible behind it
+  int chunk;               // > 0: a query sees the keys of its own chunk of positions only
 };
 
 template <int DT>
@@ -73,7 +74,7 @@ __global__ void __launch_bounds__(PF_THREADS) attn_prefill_kernel(const PrefillA
 
   // the block's key range
   const int key_hi = pos0 + rows - 1;
-  const int key_lo = (a.window > 0 && pos0 - a.window + 1 > 0) ? pos0 - a.window + 1 : 0;
+  const int key_lo = first_key(pos0, a.window, a.chunk);
   const int tile_lo = key_lo / PF_BN, tile_hi = key_hi / PF_BN;
   // The tiles in front of the window that hold kept first keys are visited first: the block
   // walks v = 0 .. n_visit - 1, tile v of the kept ones, then the window's.
@@ -120,11 +121,12 @@ __global__ void __launch_bounds__(PF_THREADS) attn_prefill_kernel(const PrefillA
     const int row = warp * 16 + g + r * 8;
     const int pos = pos0 + row;
     hi[r] = row < rows ? pos : -1;  // rows beyond the block see nothing
-    lo[r] = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+    lo[r] = first_key(pos, a.window, a.chunk);
   }
   // the warp can skip tiles that none of its rows sees
   const int warp_hi = pos0 + min(rows - 1, warp * 16 + 15);
-  const int warp_lo = (a.window > 0) ? max(0, pos0 + warp * 16 - a.window + 1) : 0;
+  const int warp_lo = first_key(pos0 + warp * 16, a.window, a.chunk);
+  const int warp_lo_last = first_key(pos0 + warp * 16 + 15, a.window, a.chunk);
 
   for (int v = 0; v < n_visit; ++v) {
     const int tile = tile_of(v);
@@ -138,8 +140,8 @@ __global__ void __launch_bounds__(PF_THREADS) attn_prefill_kernel(const PrefillA
     if (warp * 16 < rows && key0 <= warp_hi && (key0 + PF_BN - 1 >= warp_lo || key0 < keep)) {
       const bf16* kt = k_s + stage * PF_BN * LD;
       const bf16* vt = v_s + stage * PF_BN * LD;
-      // tiles strictly below every row's own position and above every window edge need no mask
-      const bool need_mask = (key0 + PF_BN - 1 > pos0 + warp * 16) || (a.window > 0) ||
+      // tiles strictly below every row's own position and above every row's first key need no mask
+      const bool need_mask = (key0 + PF_BN - 1 > pos0 + warp * 16) || key0 < warp_lo_last ||
                              (warp * 16 + 15 >= rows);
       if (need_mask) w.template tile<PF_BN, true>(kt, vt, key0, lo, hi, a.scale_log2);
       else w.template tile<PF_BN, false>(kt, vt, key0, lo, hi, a.scale_log2);
@@ -181,6 +183,7 @@ static int launch(const PrefillArgs& a, cudaStream_t s) {
 // head_dim must be a multiple of 16 up to 128 and the page 64 tokens; other
 // shapes are refused (the caller then uses the plain kernel).
 GB_EXPORT int gb_attn_prefill_bf16(const PrefillArgs* a, int D, int page, cudaStream_t s) {
+  if (a->chunk < 0) return GB_ERR_BAD_ARG;
   if (a->n_seqs <= 0 || a->nq <= 0 || a->nkv <= 0 || a->nq % a->nkv || a->max_pages <= 0 ||
       a->n_qblocks < 0)
     return GB_ERR_BAD_ARG;

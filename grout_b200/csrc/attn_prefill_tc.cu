@@ -72,6 +72,7 @@ struct AttnTcArgs {
   const float* sinks;      // [nq] one more logit of every head's denominator, or null
   ScoreCap cap;            // the score cap (off when cap_log2 == 0)
   int keep_first;          // with a window: a sequence's first keep_first keys stay visible behind it
+  int chunk;               // > 0: a query sees the keys of its own chunk of positions only
 };
 
 // V tile as the B operand of R = P V: N (head_dim) is the contiguous direction
@@ -244,7 +245,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   const int* table = a.block_table + (size_t)slot * a.max_pages;
   const bool has_b = G == 2 && rows > AT_BM;
   const int rows_a = min(rows, AT_BM), rows_b = rows - AT_BM;
-  const int key_lo = (a.window > 0 && pos0 - a.window + 1 > 0) ? pos0 - a.window + 1 : 0;
+  const int key_lo = first_key(pos0, a.window, a.chunk);
   const int tile_lo = key_lo / AT_BN;
   // With kept first keys the tiles in front of the window that hold some come first in the
   // list of tiles: entry j is tile j of the kept ones, then the window's tiles.
@@ -448,14 +449,17 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     const int pos = pos0 + g * AT_BM + r;
     const int rows_mine = g ? rows_b : rows_a;
     const int hi = r < rows_mine ? pos : -1;       // rows beyond the step see nothing
-    const int lo = (a.window > 0 && pos - a.window + 1 > 0) ? pos - a.window + 1 : 0;
+    const int lo = first_key(pos, a.window, a.chunk);
     const uint32_t lane_addr = tmem_base + ((uint32_t)(q * 32) << 16);
     const uint32_t o_addr = lane_addr + Cfg::TMEM_O + g * D;
     const uint32_t s_addr = lane_addr + Cfg::TMEM_S + g * AT_BN;
     const int n_mine = g ? n_b : n_a;
-    // a tile wholly at or below the block's first position P (and inside every row's
-    // window) needs no mask: the first that does is the one whose last key lies beyond P
-    const int j_mask = (a.window > 0 || rows_mine < AT_BM) ? 0 : max(0, (pos0 + g * AT_BM + 1) / AT_BN - tile_lo);
+    // a tile wholly at or below the block's first position P and not below the first key of
+    // the block's last row needs no mask: the first that does on the upper side is the one
+    // whose last key lies beyond P
+    const bool bounded = a.window > 0 || a.chunk > 0;
+    const int j_mask = rows_mine < AT_BM ? 0 : max(0, n_kept + (pos0 + g * AT_BM + 1) / AT_BN - tile_lo);
+    const int lo_last = first_key(pos0 + g * AT_BM + AT_BM - 1, a.window, a.chunk);
     const uint32_t p_row = smem_u32(p_s + (g * 2) * Cfg::P_BYTES + r * 128), p_swz = (uint32_t)(r & 7) << 4;
     float m_used = -INFINITY, l = 0.f;             // base of the exponent (scaled), row sum
     const bool capped = a.cap.cap_log2 != 0.f;     // capped scores are in the log2 domain already
@@ -496,7 +500,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       float s[AT_BN];
       float mx;
       const int key0 = tile_of(j) * AT_BN;
-      const bool need_mask = j >= j_mask;
+      const bool need_mask = j >= j_mask || key0 < lo_last;
       AT_STAMP(stamp_buf, (g * 4 + (j - 8)) * 8 + 0)
       if (!wait_warp(&s_full[g], ((uint32_t)j) & 1)) { ok = false; break; }
       {
@@ -519,7 +523,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         }
         if (need_mask) {
           const int last = hi - key0, first = lo - key0;   // this row's keys of the tile
-          if (a.window > 0) {
+          if (bounded) {
             const int kept_below = keep - key0;            // keys of the tile that a window keeps
 #pragma unroll
             for (int c = 0; c < AT_BN; ++c)
@@ -680,6 +684,7 @@ static int launch(const CUtensorMap& mk, const CUtensorMap& mv, const bf16* q, c
 GB_EXPORT int gb_attn_prefill_tc(const void* q, const void* k_pages, const void* v_pages,
                                  const AttnTcArgs* a, int n_tokens, long long n_pages, int D, int page,
                                  int rows_per_block, cudaStream_t s) {
+  if (a->chunk < 0) return GB_ERR_BAD_ARG;
   if (!q || !k_pages || !v_pages || !a->out || !a->error || a->n_seqs <= 0 || a->nq <= 0 ||
       a->nkv <= 0 || a->nq % a->nkv || a->max_pages <= 0 || a->n_qblocks < 0 || n_tokens <= 0 ||
       n_pages <= 0)

@@ -140,6 +140,15 @@ static inline int gb_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, siz
   return gb_launch_cluster(kernel, grid, block, smem, stream, 1, args...);
 }
 
+// The first key that a query at position `pos` sees: with a window W its last W keys, with
+// chunks of C positions (counted from the sequence's start) the keys of its own chunk;
+// 0 stands for no bound.  Never falls as `pos` grows.
+__device__ __forceinline__ int first_key(int pos, int window, int chunk) {
+  int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  if (chunk > 0) lo = max(lo, pos - pos % chunk);
+  return lo;
+}
+
 // Address of row `pos` of kv head `h` of a sequence in a paged cache laid out
 // [n_pages, n_kv_heads, page, D]; `table` is the sequence's row of the block table.
 __device__ __forceinline__ size_t paged_row(const int* table, int pos, int h, int nkv, int page,

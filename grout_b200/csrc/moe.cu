@@ -18,6 +18,12 @@
 // y = expert(s x): gate and up have no bias, so their 32-bit sums are multiplied by s
 // before the activation, and the second product is stored as it is.
 //
+// Further forms: `group_top2` scores a group by the sum of its two largest c (of its only
+// one where a group has a single output); `normalize` makes a token's weights s / (sum of
+// the chosen s + 1e-20) * weight_scale (without it they are s * weight_scale); with no
+// gate weights an expert is ungated, y = max(x Wu_e^T, 0)^2 Wd_e^T (no limit, slope or
+// offset).
+//
 // Nothing here needs the host to know how many tokens an expert got, so a step
 // can be captured: `route` chooses and counts, and its last block turns the counts into a
 // list of (token, choice) pairs ordered by expert; the two products walk
@@ -33,7 +39,7 @@ struct MoeArgs {
   const void* x;            // [T, W] activations
   const float* router_w;    // [E + n_identity, W]
   const float* correction;  // [E + n_identity]
-  const void* w_gate;       // [E, F, W]
+  const void* w_gate;       // [E, F, W], or null: the experts have no gate
   const void* w_up;         // [E, F, W]
   const void* w_down;       // [E, W, F]
   int* ids;                 // [T, top] chosen outputs
@@ -43,13 +49,16 @@ struct MoeArgs {
   int* offsets;             // [E + 1]
   int* perm;                // [T top] pairs (t * top + j) ordered by expert
   void* act;                // [T top, F] activations of the experts' inner layer, in list order
-  float* out;               // [top, T, W]
+  float* out;               // [top, T, W] (rows beyond it, if any, are the caller's)
   int T, W, F, E, n_identity, top, n_groups, keep_groups;
   float limit, slope;
   int score_fn;              // 0: softmax over the outputs, 1: sigmoid of each, 2: softmax over the chosen
   int weigh_input;           // the weight multiplies the expert's input, not its result
   float up_offset;           // y = act(g) (u + up_offset)
   const float* router_bias;  // [E + n_identity] added to z, or null
+  int group_top2;            // a group's score is the sum of its two largest c, not its largest
+  int normalize;             // the chosen outputs' weights are divided by their sum
+  float weight_scale;        // and multiplied by this
 };
 
 #define MOE_MAX_OUTPUTS 1024
@@ -59,9 +68,8 @@ struct MoeArgs {
 
 template <typename T>
 __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeArgs a) {
-  extern __shared__ float sm[];   // z [n_all], c [n_all]
+  extern __shared__ float sm[];   // z [n_all], c [n_all], a score per group
   __shared__ float part[MOE_ROUTE_THREADS / 32][MOE_ROUTE_CHUNK];
-  __shared__ float gbest[MOE_MAX_OUTPUTS];
   pdl_launch_dependents_if_small();
   pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -69,6 +77,7 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
   const int n_all = a.E + a.n_identity, W = a.W;
   float* z = sm;
   float* c = sm + n_all;
+  float* gval = c + n_all;         // [n_groups] scores of the groups
   const T* x = (const T*)a.x + (size_t)t * W;
   // every thread takes a slice of the row against a few router rows at a time, so that
   // all of a slice's loads are under way together; the sums are put together in a fixed
@@ -98,53 +107,75 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
     }
     __syncthreads();
   }
-  if (tid == 0) {
-    float mx = -INFINITY, sum = 0.f;
+  if (warp == 0) {        // one warp turns logits into scores and chooses
     if (a.score_fn == 1) {
-      for (int e = 0; e < n_all; ++e) z[e] = 1.0f / (1.0f + expf(-z[e]));
-    } else if (a.score_fn == 2) {
-      // the logits themselves choose; the chosen ones' weights are worked out below
-    } else {
-      for (int e = 0; e < n_all; ++e) mx = fmaxf(mx, z[e]);
-      for (int e = 0; e < n_all; ++e) { z[e] = expf(z[e] - mx); sum += z[e]; }
-      for (int e = 0; e < n_all; ++e) z[e] = z[e] / sum;
-    }
-    for (int e = 0; e < n_all; ++e) c[e] = z[e] + (a.correction ? a.correction[e] : 0.f);
+      for (int e = lane; e < n_all; e += 32) z[e] = 1.0f / (1.0f + expf(-z[e]));
+    } else if (a.score_fn == 0) {
+      float mx = -INFINITY, sum = 0.f;
+      for (int e = lane; e < n_all; e += 32) mx = fmaxf(mx, z[e]);
+      mx = warp_max(mx);
+      for (int e = lane; e < n_all; e += 32) { z[e] = expf(z[e] - mx); sum += z[e]; }
+      sum = warp_sum(sum);
+      for (int e = lane; e < n_all; e += 32) z[e] = z[e] / sum;
+    }   // score_fn 2: the logits themselves choose; the chosen ones' weights are worked out below
+    for (int e = lane; e < n_all; e += 32) c[e] = z[e] + (a.correction ? a.correction[e] : 0.f);
+    __syncwarp();
     if (a.n_groups > 1 && a.keep_groups < a.n_groups) {
       const int per = n_all / a.n_groups;
-      // drop the groups that are not among the best: n_groups - keep_groups times the worst
-      // remaining one (of equal groups the later one goes first)
-      float* best = gbest;                       // a group's best choice score; NaN once dropped
-      for (int g = 0; g < a.n_groups; ++g) {
-        float b = -INFINITY;
-        for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, c[e]);
-        best[g] = b;
+      for (int g = lane; g < a.n_groups; g += 32) {
+        float b1 = -INFINITY, b2 = -INFINITY;           // the group's two largest
+        for (int e = g * per; e < (g + 1) * per; ++e) {
+          const float v = c[e];
+          b2 = fmaxf(b2, fminf(b1, v));
+          b1 = fmaxf(b1, v);
+        }
+        gval[g] = a.group_top2 && per > 1 ? b1 + b2 : b1;
       }
-      for (int d = 0; d < a.n_groups - a.keep_groups; ++d) {
-        int worst = -1;
-        float worst_v = INFINITY;
-        for (int g = 0; g < a.n_groups; ++g)
-          if (!isnan(best[g]) && best[g] <= worst_v) { worst_v = best[g]; worst = g; }
-        best[worst] = NAN;
-        for (int e = worst * per; e < (worst + 1) * per; ++e) c[e] = -INFINITY;
+      __syncwarp();
+      // a group that `keep_groups` others come before (larger, or equal and earlier) is dropped
+      for (int g = lane; g < a.n_groups; g += 32) {
+        const float v = gval[g];
+        int before = 0;
+        for (int o = 0; o < a.n_groups; ++o) before += gval[o] > v || (gval[o] == v && o < g);
+        if (before >= a.keep_groups)
+          for (int e = g * per; e < (g + 1) * per; ++e) c[e] = -INFINITY;
       }
+      __syncwarp();
     }
+    float chosen_sum = 0.f, first_z = 0.f;
     for (int j = 0; j < a.top; ++j) {   // the largest first; of equal ones the earlier
-      int best = 0;
-      float best_v = -INFINITY;
-      bool found = false;
-      for (int e = 0; e < n_all; ++e)
-        if (!isnan(c[e]) && (!found || c[e] > best_v)) { best = e; best_v = c[e]; found = true; }
-      c[best] = NAN;                    // taken
-      a.ids[(size_t)t * a.top + j] = best;
-      a.wts[(size_t)t * a.top + j] = z[best];
+      float bv = -INFINITY;
+      int bi = 0x7fffffff;
+      for (int e = lane; e < n_all; e += 32) {         // (one that is taken is NaN: no comparison holds)
+        const float v = c[e];
+        if (v > bv || (v == bv && e < bi)) { bv = v; bi = e; }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+      }
+      const int best = bi < n_all ? bi : 0;
+      const float w = z[best];
+      if (j == 0) first_z = w;
+      chosen_sum += a.score_fn == 2 ? expf(w - first_z) : w;   // (the first logit is the largest)
+      __syncwarp();
+      if (lane == 0) {
+        c[best] = NAN;                  // taken
+        a.ids[(size_t)t * a.top + j] = best;
+        a.wts[(size_t)t * a.top + j] = w;
+      }
+      __syncwarp();
     }
-    if (a.score_fn == 2) {              // softmax over the chosen logits alone; the first is the largest
+    if (lane == 0) {
       float* w = a.wts + (size_t)t * a.top;
-      const float top_z = w[0];
-      float sum = 0.f;
-      for (int j = 0; j < a.top; ++j) { w[j] = expf(w[j] - top_z); sum += w[j]; }
-      for (int j = 0; j < a.top; ++j) w[j] = w[j] / sum;
+      for (int j = 0; j < a.top; ++j) {
+        // softmax over the chosen logits alone, or the scores, as they are or as shares of their sum
+        const float v = a.score_fn == 2 ? expf(w[j] - first_z) / chosen_sum
+                        : a.normalize   ? w[j] / (chosen_sum + 1e-20f) : w[j];
+        w[j] = v * a.weight_scale;
+      }
     }
   }
   __syncthreads();
@@ -223,7 +254,8 @@ __global__ void __launch_bounds__(256) moe_up_kernel(const MoeArgs a) {
   const int f0 = blockIdx.y * MOE_BN;
   if (tid < MOE_BM) tok[tid] = tid < n_rows ? a.perm[first + tid] / a.top : -1;
   __syncthreads();
-  const T* wg = (const T*)a.w_gate + (size_t)e * F * W;
+  const bool gated = a.w_gate != nullptr;
+  const T* wg = gated ? (const T*)a.w_gate + (size_t)e * F * W : nullptr;
   const T* wu = (const T*)a.w_up + (size_t)e * F * W;
   const int tx = tid & 63, ty = tid >> 6;      // column, group of four rows
   float accg[4] = {0.f, 0.f, 0.f, 0.f}, accu[4] = {0.f, 0.f, 0.f, 0.f};
@@ -235,13 +267,13 @@ __global__ void __launch_bounds__(256) moe_up_kernel(const MoeArgs a) {
     for (int i = tid; i < MOE_BN * MOE_BK; i += 256) {
       const int n = i / MOE_BK, k = i % MOE_BK;
       const bool ok = f0 + n < F && k0 + k < W;
-      Gs[n][k] = ok ? to_f32<T>(wg[(size_t)(f0 + n) * W + k0 + k]) : 0.f;
+      if (gated) Gs[n][k] = ok ? to_f32<T>(wg[(size_t)(f0 + n) * W + k0 + k]) : 0.f;
       Us[n][k] = ok ? to_f32<T>(wu[(size_t)(f0 + n) * W + k0 + k]) : 0.f;
     }
     __syncthreads();
 #pragma unroll
     for (int k = 0; k < MOE_BK; ++k) {
-      const float g = Gs[tx][k], u = Us[tx][k];
+      const float g = gated ? Gs[tx][k] : 0.f, u = Us[tx][k];
 #pragma unroll
       for (int r = 0; r < 4; ++r) {
         const float x = As[ty * 4 + r][k];
@@ -259,9 +291,15 @@ __global__ void __launch_bounds__(256) moe_up_kernel(const MoeArgs a) {
     if (row >= n_rows) continue;
     float g = accg[r], u = accu[r];
     if (a.weigh_input) { const float w = a.wts[a.perm[first + row]]; g *= w; u *= w; }
-    g = fminf(g, a.limit);
-    u = fminf(fmaxf(u, -a.limit), a.limit);
-    const float y = g / (1.0f + expf(-a.slope * g)) * (u + a.up_offset);
+    float y;
+    if (gated) {
+      g = fminf(g, a.limit);
+      u = fminf(fmaxf(u, -a.limit), a.limit);
+      y = g / (1.0f + expf(-a.slope * g)) * (u + a.up_offset);
+    } else {
+      u = fmaxf(u, 0.f);
+      y = u * u;
+    }
     ((T*)a.act)[(size_t)(first + row) * F + f0 + tx] = from_f32<T>(y);
   }
 }
@@ -334,9 +372,14 @@ __device__ __forceinline__ void ldmatrix_x2(uint32_t (&r)[2], const void* smem) 
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(s));
 }
 
-template <bool UP, int BM>
+// The three products: an expert's second, its first with gate and up side by side, its first
+// without a gate.
+enum MoeMode { MOE_DOWN = 0, MOE_GATED = 1, MOE_UNGATED = 2 };
+
+template <int MODE, int BM>
 struct MoeTile {
-  static constexpr int NB = UP ? 2 : 1;
+  static constexpr bool UP = MODE != MOE_DOWN;
+  static constexpr int NB = MODE == MOE_GATED ? 2 : 1;
   static constexpr int BN = BM >= 64 ? MT_BN : 32;
   static constexpr int THREADS = 128;
   // a warp's share of the tile: MI pieces of 16 rows by NJ pieces of 8 columns.  Many rows:
@@ -350,9 +393,10 @@ struct MoeTile {
   static constexpr size_t SMEM = (size_t)STAGES * STAGE_ELEMS * sizeof(bf16);
 };
 
-template <bool UP, int BM>
+template <int MODE, int BM>
 __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
-  using Tile = MoeTile<UP, BM>;
+  using Tile = MoeTile<MODE, BM>;
+  constexpr bool UP = Tile::UP, GATED = MODE == MOE_GATED;
   constexpr int NB = Tile::NB, STAGES = Tile::STAGES, BN = Tile::BN, NT = Tile::THREADS;
   constexpr int MI = Tile::MI, NJ = Tile::NJ;
   extern __shared__ __align__(16) bf16 tiles[];
@@ -371,8 +415,8 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
   }
   __syncthreads();
   const bf16* A = (const bf16*)(UP ? a.x : a.act);
-  const bf16* B0 = (const bf16*)(UP ? a.w_gate : a.w_down) + (size_t)e * N * K;
-  const bf16* B1 = UP ? (const bf16*)a.w_up + (size_t)e * N * K : nullptr;
+  const bf16* B0 = (const bf16*)(GATED ? a.w_gate : UP ? a.w_up : a.w_down) + (size_t)e * N * K;
+  const bf16* B1 = GATED ? (const bf16*)a.w_up + (size_t)e * N * K : nullptr;
   auto load = [&](int stage, int k0) {
     bf16* As = tiles + stage * Tile::STAGE_ELEMS;
     bf16* Bs = As + BM * MT_LD;
@@ -386,7 +430,7 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
       const int c = tid + i * NT, r = c >> 3, pc = (c & 7) * 8, kc = k0 + pc;
       const bool ok = n0 + r < N && kc < K;
       cp_async16(Bs + r * MT_LD + pc, ok ? B0 + (size_t)(n0 + r) * K + kc : B0, ok);
-      if (UP) cp_async16(Bs + (BN + r) * MT_LD + pc, ok ? B1 + (size_t)(n0 + r) * K + kc : B1, ok);
+      if (GATED) cp_async16(Bs + (BN + r) * MT_LD + pc, ok ? B1 + (size_t)(n0 + r) * K + kc : B1, ok);
     }
   };
   float acc[NB][MI][NJ][4];
@@ -461,9 +505,14 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
           float y[2];
 #pragma unroll
           for (int x = 0; x < 2; ++x) {
-            const float gt = fminf(wi * acc[0][m][j][half * 2 + x], a.limit);
-            const float up = fminf(fmaxf(wi * acc[NB - 1][m][j][half * 2 + x], -a.limit), a.limit);
-            y[x] = gt / (1.0f + expf(-a.slope * gt)) * (up + a.up_offset);
+            if (GATED) {
+              const float gt = fminf(wi * acc[0][m][j][half * 2 + x], a.limit);
+              const float up = fminf(fmaxf(wi * acc[NB - 1][m][j][half * 2 + x], -a.limit), a.limit);
+              y[x] = gt / (1.0f + expf(-a.slope * gt)) * (up + a.up_offset);
+            } else {
+              const float up = fmaxf(wi * acc[0][m][j][half * 2 + x], 0.f);
+              y[x] = up * up;
+            }
           }
           if (col + 1 < N) *reinterpret_cast<uint32_t*>(dst + col) = pack_bf16(y[0], y[1]);
           else if (col < N) dst[col] = from_f32<bf16>(y[0]);
@@ -483,16 +532,22 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
     }
 }
 
-template <bool UP, int BM>
+template <int MODE, int BM>
 static int moe_tc_launch(const MoeArgs& a, long long pairs, cudaStream_t s) {
   const long long tiles = pairs / BM + (pairs < a.E ? pairs : a.E);
   if (tiles > 0x7fffffffLL) return GB_ERR_UNSUPPORTED;
-  const size_t smem = MoeTile<UP, BM>::SMEM;
-  cudaError_t ce = cudaFuncSetAttribute(moe_tc_kernel<UP, BM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const size_t smem = MoeTile<MODE, BM>::SMEM;
+  cudaError_t ce = cudaFuncSetAttribute(moe_tc_kernel<MODE, BM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (ce != cudaSuccess) return (int)ce;
-  const int N = UP ? a.F : a.W, BN = MoeTile<UP, BM>::BN;
-  return gb_launch(moe_tc_kernel<UP, BM>, dim3((unsigned)tiles, (N + BN - 1) / BN),
-                   dim3(MoeTile<UP, BM>::THREADS), smem, s, a);
+  const int N = MODE != MOE_DOWN ? a.F : a.W, BN = MoeTile<MODE, BM>::BN;
+  return gb_launch(moe_tc_kernel<MODE, BM>, dim3((unsigned)tiles, (N + BN - 1) / BN),
+                   dim3(MoeTile<MODE, BM>::THREADS), smem, s, a);
+}
+
+template <int BM>
+static int moe_tc_products(const MoeArgs& a, long long pairs, cudaStream_t s) {
+  int e = a.w_gate ? moe_tc_launch<MOE_GATED, BM>(a, pairs, s) : moe_tc_launch<MOE_UNGATED, BM>(a, pairs, s);
+  return e ? e : moe_tc_launch<MOE_DOWN, BM>(a, pairs, s);
 }
 
 static int moe_check(const MoeArgs& a) {
@@ -503,7 +558,7 @@ static int moe_check(const MoeArgs& a) {
   if (n_all % a.n_groups || a.top > n_all) return GB_ERR_BAD_ARG;
   if (n_all > MOE_MAX_OUTPUTS) return GB_ERR_UNSUPPORTED;
   if (a.score_fn < 0 || a.score_fn > 2) return GB_ERR_BAD_ARG;
-  if (!a.x || !a.router_w || !a.w_gate || !a.w_up || !a.w_down || !a.ids || !a.wts ||
+  if (!a.x || !a.router_w || !a.w_up || !a.w_down || !a.ids || !a.wts ||
       !a.rank || !a.counts || !a.offsets || !a.perm || !a.act || !a.out)
     return GB_ERR_BAD_ARG;
   return 0;
@@ -515,27 +570,18 @@ static int moe_forward(const MoeArgs& a, cudaStream_t s) {
   if (e) return e;
   if (a.T == 0) return 0;
   const int n_all = a.E + a.n_identity;
-  e = gb_launch(moe_route_kernel<T>, dim3(a.T), dim3(MOE_ROUTE_THREADS), (size_t)2 * n_all * sizeof(float), s, a);
+  e = gb_launch(moe_route_kernel<T>, dim3(a.T), dim3(MOE_ROUTE_THREADS), (size_t)(2 * n_all + a.n_groups) * sizeof(float), s, a);
   if (e) return e;
   // the most tiles the pairs can make: every expert may end in a tile that is not full
   const long long pairs = (long long)a.T * a.top;
   if (sizeof(T) == 2 && a.W % 8 == 0 && a.F % 8 == 0 &&
       ((((uintptr_t)a.x) | ((uintptr_t)a.act) | ((uintptr_t)a.w_gate) | ((uintptr_t)a.w_up) |
         ((uintptr_t)a.w_down) | ((uintptr_t)a.out)) & 15) == 0) {
-    // few pairs per expert (a decode step): narrow tiles, deeper pipeline
-    if (pairs <= 4LL * a.E) {
-      e = moe_tc_launch<true, 16>(a, pairs, s);
-      if (e) return e;
-      return moe_tc_launch<false, 16>(a, pairs, s);
-    }
-    if (pairs >= 64LL * a.E) {      // 64 pairs an expert and more: tiles of 128 rows
-      e = moe_tc_launch<true, 128>(a, pairs, s);
-      if (e) return e;
-      return moe_tc_launch<false, 128>(a, pairs, s);
-    }
-    e = moe_tc_launch<true, 64>(a, pairs, s);
-    if (e) return e;
-    return moe_tc_launch<false, 64>(a, pairs, s);
+    // few pairs per expert (a decode step): narrow tiles, deeper pipeline; 64 pairs an expert
+    // and more: tiles of 128 rows
+    if (pairs <= 4LL * a.E) return moe_tc_products<16>(a, pairs, s);
+    if (pairs >= 64LL * a.E) return moe_tc_products<128>(a, pairs, s);
+    return moe_tc_products<64>(a, pairs, s);
   }
   const long long tiles = pairs / MOE_BM + (pairs < a.E ? pairs : a.E);
   if (tiles > 0x7fffffffLL) return GB_ERR_UNSUPPORTED;

@@ -6,7 +6,15 @@
 // (and/or to a dense kv_out).  The normalised value is not rounded before the
 // rotation: one rounding at the store, as in the reference's
 // qk_norm_rope_kv_prefill_raw_f16 (src/kernels.rs:3415-3732, maths 3576-3652).
-// angle = float(pos) * inv_freq[j] in 32-bit with the accurate sincosf.
+// angle = float(pos) * inv_freq[j] in 32-bit with the accurate sincosf; sine and cosine
+// are multiplied by `rot_scale` (1 for a plain rotation).
+//
+// With `maps` M > 1 every head has M query and M key vectors of D elements that share the
+// head's one value: the projection has nq = heads * M query vectors and nkv * M key
+// vectors.  A stored key row holds the M keys of its kv head side by side, and query vector
+// m of a head becomes a row of its own whose elements m D .. (m + 1) D are the query and
+// whose rest is zeros, so that its product with a stored row is its product with key m.
+// Attention then sees nq query heads and nkv kv heads.
 #include "common.cuh"
 
 struct QkPrepareArgs {
@@ -33,6 +41,8 @@ struct QkPrepareArgs {
   float q_temp_coef;        // with q_temp_every > 0 a query at position p is multiplied, after its
   int q_temp_every;         //   norm, by 1 + coef * ln(floor((p + 1) / every) + 1)
   int interleaved;          // the rotation pairs element 2j with 2j + 1 instead of j with j + rot_dim / 2
+  int maps;                 // query and key vectors of a head that share its value (1: the ordinary head)
+  float rot_scale;          // factor of the rotation's sine and cosine
 };
 
 __device__ __forceinline__ float query_temperature(const QkPrepareArgs& a, int pos) {
@@ -49,18 +59,19 @@ __global__ void qk_prepare_kernel(const QkPrepareArgs a) {
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
-  const int n_heads = a.nq + (a.v_from_k ? 1 : 2) * a.nkv;
+  const int nk = a.nkv * a.maps;            // key vectors of the projection
+  const int n_heads = a.nq + nk + (a.v_from_k ? 0 : a.nkv);
   const int head = blockIdx.y * (blockDim.x >> 5) + warp;
   if (head >= n_heads) return;  // warps are independent below
   const int Dv = a.Dv > 0 ? a.Dv : a.D;     // a value head's size in the projection
   const int Ds = a.Ds > 0 ? a.Ds : a.D;     // a stored row's width
-  const int kind = head < a.nq ? 0 : (head < a.nq + a.nkv ? 1 : 2);
+  const int kind = head < a.nq ? 0 : (head < a.nq + nk ? 1 : 2);
   const int D = kind == 2 ? Dv : a.D;
   const int wider = a.D > Dv ? a.D : Dv;
   float* x = sm + warp * (wider > Ds ? wider : Ds);
   // columns of the projection: q heads, k heads (both of a.D), then v heads of Dv
-  const size_t width = (size_t)(a.nq + a.nkv) * a.D + (a.v_from_k ? 0 : (size_t)a.nkv * Dv);
-  const size_t col0 = kind == 2 ? (size_t)(a.nq + a.nkv) * a.D + (size_t)(head - a.nq - a.nkv) * Dv
+  const size_t width = (size_t)(a.nq + nk) * a.D + (a.v_from_k ? 0 : (size_t)a.nkv * Dv);
+  const size_t col0 = kind == 2 ? (size_t)(a.nq + nk) * a.D + (size_t)(head - a.nq - nk) * Dv
                                 : (size_t)head * a.D;
   if (a.qkv_parts) {
     const float* ps = a.qkv_parts + (size_t)t * width + col0;
@@ -115,6 +126,7 @@ __global__ void qk_prepare_kernel(const QkPrepareArgs a) {
       const float angle = (float)pos * a.inv_freq[j];
       float s, c;
       sincosf(angle, &s, &c);
+      s *= a.rot_scale, c *= a.rot_scale;
       const int i0 = a.interleaved ? 2 * j : j, i1 = a.interleaved ? 2 * j + 1 : j + half;
       const float lo = x[i0], hi = x[i1];
       x[i0] = lo * c - hi * s;
@@ -122,15 +134,23 @@ __global__ void qk_prepare_kernel(const QkPrepareArgs a) {
     }
     __syncwarp();
   }
+  // the elements at0 .. at1 - 1 of a stored row are this warp's, x[] from at0 - shift on
+  int at0 = 0, at1 = Ds, shift = 0;
+  if (a.maps > 1 && kind != 2) {
+    const int m = (kind == 0 ? head : head - a.nq) % a.maps;
+    shift = m * D;
+    if (kind == 1) at0 = shift, at1 = m + 1 == a.maps ? Ds : shift + D;
+  }
+  auto stored = [&](int d) { return d >= shift && d < shift + Ds ? x[d - shift] : 0.f; };
   if (kind == 0) {
     T* dst = (T*)a.q_out + ((size_t)t * a.nq + head) * Ds;
-    for (int d = lane; d < Ds; d += 32) dst[d] = from_f32<T>(x[d]);
+    for (int d = lane; d < Ds; d += 32) dst[d] = from_f32<T>(stored(d));
     return;
   }
-  const int hh = kind == 1 ? head - a.nq : head - a.nq - a.nkv;
+  const int hh = kind == 1 ? (head - a.nq) / a.maps : head - a.nq - nk;
   if (a.kv_out) {
     T* dst = (T*)a.kv_out + ((size_t)t * 2 * a.nkv + (kind == 1 ? hh : a.nkv + hh)) * Ds;
-    for (int d = lane; d < Ds; d += 32) dst[d] = from_f32<T>(x[d]);
+    for (int d = at0 + lane; d < at1; d += 32) dst[d] = from_f32<T>(stored(d));
   }
   if (a.k_pages) {
     const int slot = a.slots[a.token_seq[t]];
@@ -138,7 +158,7 @@ __global__ void qk_prepare_kernel(const QkPrepareArgs a) {
     const int* table = a.block_table + (size_t)slot * a.max_pages;
     T* base = (T*)(kind == 1 ? a.k_pages : a.v_pages);
     T* dst = base + paged_row(table, pos, hh, a.nkv, a.page, Ds);
-    for (int d = lane; d < Ds; d += 32) dst[d] = from_f32<T>(x[d]);
+    for (int d = at0 + lane; d < at1; d += 32) dst[d] = from_f32<T>(stored(d));
   }
 }
 
@@ -171,6 +191,7 @@ __global__ void qk_prepare_fast_kernel(const QkPrepareArgs a) {
       for (int e = 0; e < 2; ++e) {
         sn[p][e] = 0.f, cs[p][e] = 1.f;
         if (j < HALF) sincosf((float)pos * a.inv_freq[j + e], &sn[p][e], &cs[p][e]);
+        sn[p][e] *= a.rot_scale, cs[p][e] *= a.rot_scale;
       }
     }
   }
@@ -316,7 +337,10 @@ __global__ void __launch_bounds__(128, 8) qk_prepare_wide_kernel(const QkPrepare
   __shared__ __align__(16) float sn_s[HALF], cs_s[HALF], wq_s[D], wk_s[D];
   for (int j = threadIdx.x; j < HALF; j += blockDim.x) {
     float sj = 0.f, cj = 1.f;
-    if (a.inv_freq) sincosf((float)pos * a.inv_freq[j], &sj, &cj);
+    if (a.inv_freq) {
+      sincosf((float)pos * a.inv_freq[j], &sj, &cj);
+      sj *= a.rot_scale, cj *= a.rot_scale;
+    }
     sn_s[j] = sj, cs_s[j] = cj;
   }
   for (int j = threadIdx.x; j < D; j += blockDim.x) {
@@ -452,8 +476,11 @@ __global__ void __launch_bounds__(128) qk_prepare_chunk_kernel(const QkPrepareAr
   // what no kernel of this step writes comes before the wait for the projection
   const int pos = a.token_pos[t];
   if (a.inv_freq) {
-    for (int j = threadIdx.x; j < half; j += blockDim.x)
-      sincosf((float)pos * a.inv_freq[j], &sc_s[j], &sc_s[half + j]);
+    for (int j = threadIdx.x; j < half; j += blockDim.x) {
+      float s, c;
+      sincosf((float)pos * a.inv_freq[j], &s, &c);
+      sc_s[j] = s * a.rot_scale, sc_s[half + j] = c * a.rot_scale;
+    }
   }
   size_t page_row0 = 0;   // row of (page of pos, kv head 0, pos in page)
   bool paged = false;
@@ -576,6 +603,159 @@ __global__ void __launch_bounds__(128) qk_prepare_chunk_kernel(const QkPrepareAr
   pdl_launch_dependents_if_large();
 }
 
+// Heads without norms in every other layout (bf16 activations): heads whose size is no
+// power of two, values of another size than the keys, rows filled up with zeros, several
+// maps.  A thread makes eight consecutive elements of a stored row at a time: it finds the
+// eight projection columns they come from and, where they turn, the eight columns of their
+// partners (the same row of the projection, in L1 by then), so no thread waits for another.
+// The token's sines and cosines are computed once per block and shared.
+__global__ void __launch_bounds__(128) qk_prepare_piece_kernel(const QkPrepareArgs a) {
+  extern __shared__ float sc_s[];                // [rot_dim / 2] sines, then as many cosines
+  const int D = a.D, Dv = a.Dv > 0 ? a.Dv : a.D, Ds = a.Ds > 0 ? a.Ds : a.D, half = a.rot_dim >> 1;
+  const int t = blockIdx.x, nk = a.nkv * a.maps;
+  const size_t width = (size_t)(a.nq + nk) * D + (size_t)a.nkv * Dv;
+  pdl_launch_dependents_if_small();
+  // what no kernel of this step writes comes before the wait for the projection
+  const int pos = a.token_pos[t];
+  if (a.inv_freq) {
+    for (int j = threadIdx.x; j < half; j += blockDim.x) {
+      float s, c;
+      sincosf((float)pos * a.inv_freq[j], &s, &c);
+      sc_s[j] = s * a.rot_scale, sc_s[half + j] = c * a.rot_scale;
+    }
+  }
+  size_t page_row0 = 0;   // row of (page of pos, kv head 0, pos in page)
+  bool paged = false;
+  if (a.k_pages) {
+    const int slot = a.slots[a.token_seq[t]];
+    if (slot >= 0) {
+      page_row0 = paged_row(a.block_table + (size_t)slot * a.max_pages, pos, 0, a.nkv, a.page, Ds);
+      paged = true;
+    }
+  }
+  __syncthreads();
+  const float q_temp = query_temperature(a, pos);
+  pdl_wait();
+  // eight projection columns from `at` on (a row's partial sums added in order)
+  auto load8 = [&](size_t at, float (&x)[8]) {
+    if (a.qkv_parts) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = 0.f;
+      for (int k0 = 0; k0 < a.n_parts; k0 += 4) {   // four partials requested at once, added in order
+        float4 pa[4], pb[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          const int k = k0 + u < a.n_parts ? k0 + u : a.n_parts - 1;
+          const float4* ps = reinterpret_cast<const float4*>(a.qkv_parts + (size_t)k * a.part_stride + at);
+          pa[u] = ps[0], pb[u] = ps[1];
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+          if (k0 + u < a.n_parts) {
+            x[0] += pa[u].x, x[1] += pa[u].y, x[2] += pa[u].z, x[3] += pa[u].w;
+            x[4] += pb[u].x, x[5] += pb[u].y, x[6] += pb[u].z, x[7] += pb[u].w;
+          }
+      }
+    } else {
+      const uint4 raw = *reinterpret_cast<const uint4*>((const bf16*)a.qkv + at);
+      const uint32_t rw[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const __nv_bfloat162 v2 = *reinterpret_cast<const __nv_bfloat162*>(&rw[i]);
+        x[2 * i] = __low2float(v2), x[2 * i + 1] = __high2float(v2);
+      }
+    }
+  };
+  const int per_row = Ds >> 3, n_rows = a.nq + (a.k_pages ? 2 * a.nkv : 0), n_items = n_rows * per_row;
+#pragma unroll 2
+  for (int item = blockIdx.y * blockDim.x + threadIdx.x; item < n_items; item += gridDim.y * blockDim.x) {
+    const int row = item / per_row, col = (item - row * per_row) * 8;
+    const int kind = row < a.nq ? 0 : (row < a.nq + a.nkv ? 1 : 2);
+    // where the eight elements come from: element `in_head` on of a vector at `src`
+    int in_head = col;
+    size_t src;
+    bool zero;
+    if (kind == 2) {
+      src = (size_t)(a.nq + nk) * D + (size_t)(row - a.nq - a.nkv) * Dv;
+      zero = col >= Dv;
+    } else if (kind == 1) {
+      const int m = col / D;
+      in_head = col - m * D;
+      src = (size_t)(a.nq + (row - a.nq) * a.maps + m) * D;
+      zero = m >= a.maps;
+    } else {
+      in_head = col - (row % a.maps) * D;
+      src = (size_t)row * D;
+      zero = in_head < 0 || in_head >= D;
+    }
+    float x[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] = 0.f;
+    if (!zero) {
+      const size_t at = (size_t)t * width + src + in_head;
+      load8(at, x);
+      if (kind != 2 && a.inv_freq && in_head < a.rot_dim) {
+        if (a.interleaved) {
+#pragma unroll
+          for (int e = 0; e < 8; e += 2) {
+            if (in_head + e >= a.rot_dim) break;
+            const float s = sc_s[(in_head + e) >> 1], c = sc_s[half + ((in_head + e) >> 1)];
+            const float u = x[e], v = x[e + 1];
+            x[e] = u * c - v * s;
+            x[e + 1] = v * c + u * s;
+          }
+        } else {
+          const bool first = in_head < half;      // (half is a multiple of eight)
+          float y[8];
+          load8(first ? at + half : at - half, y);
+          const int j0 = first ? in_head : in_head - half;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const float s = sc_s[j0 + e], c = sc_s[half + j0 + e];
+            x[e] = first ? x[e] * c - y[e] * s : x[e] * c + y[e] * s;
+          }
+        }
+      }
+      if (kind == 0 && a.q_temp_every > 0) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] *= q_temp;
+      }
+    }
+    uint32_t w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const __nv_bfloat162 p2 = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+      w[i] = *reinterpret_cast<const uint32_t*>(&p2);
+    }
+    const uint4 o8 = make_uint4(w[0], w[1], w[2], w[3]);
+    if (kind == 0) {
+      *reinterpret_cast<uint4*>((bf16*)a.q_out + ((size_t)t * a.nq + row) * Ds + col) = o8;
+    } else if (paged) {
+      const int hh = kind == 1 ? row - a.nq : row - a.nq - a.nkv;
+      *reinterpret_cast<uint4*>((bf16*)(kind == 1 ? a.k_pages : a.v_pages) + page_row0 +
+                                (size_t)hh * a.page * Ds + col) = o8;
+    }
+  }
+  pdl_launch_dependents_if_large();
+}
+
+static bool piece_ok(const QkPrepareArgs& a) {
+  auto al = [](const void* p) { return (((uintptr_t)p) & 15) == 0; };
+  const int Dv = a.Dv > 0 ? a.Dv : a.D, Ds = a.Ds > 0 ? a.Ds : a.D;
+  return !a.q_w && !a.k_w && !a.v_from_k && !a.kv_out && a.D % 8 == 0 && Dv % 8 == 0 && Ds % 8 == 0 &&
+         (!a.inv_freq || ((a.interleaved || (a.rot_dim / 2) % 8 == 0) && a.rot_dim <= 1024)) && al(a.qkv) &&
+         al(a.q_out) && al(a.k_pages) && al(a.v_pages) && al(a.qkv_parts) && (a.part_stride & 3) == 0;
+}
+
+static int launch_piece(const QkPrepareArgs& a, cudaStream_t stream) {
+  const int Ds = a.Ds > 0 ? a.Ds : a.D;
+  const int items = (a.nq + (a.k_pages ? 2 * a.nkv : 0)) * (Ds / 8);
+  // few tokens: a thread per piece; many: a block walks all of a token's rows
+  const int gy = a.n_tokens >= 128 ? 1 : (items + 127) / 128;
+  const size_t smem = a.inv_freq ? (size_t)a.rot_dim * sizeof(float) : 0;
+  return gb_launch(qk_prepare_piece_kernel, dim3(a.n_tokens, gy), dim3(128), smem, stream, a);
+}
+
 static bool chunk_ok(const QkPrepareArgs& a) {
   auto al = [](const void* p) { return (((uintptr_t)p) & 15) == 0; };
   const int lph = a.D / 8;
@@ -640,7 +820,7 @@ static bool fast_ok(const QkPrepareArgs& a) {
 template <typename T, typename WT>
 static int launch(const QkPrepareArgs& a, cudaStream_t stream) {
   const int warps = 4;
-  const int n_heads = a.nq + (a.v_from_k ? 1 : 2) * a.nkv;
+  const int n_heads = a.nq + a.nkv * a.maps + (a.v_from_k ? 0 : a.nkv);
   dim3 grid(a.n_tokens, (n_heads + warps - 1) / warps);
   int widest = a.D;
   if (a.Dv > widest) widest = a.Dv;
@@ -663,14 +843,18 @@ static int check(const QkPrepareArgs& a) {
   if (a.v_from_k && (a.k_w || a.nkv <= 0)) return GB_ERR_UNSUPPORTED;
   if (a.Dv < 0 || a.Ds < 0 || (a.Ds > 0 && (a.Ds < a.D || a.Ds < a.Dv))) return GB_ERR_BAD_ARG;
   if (a.q_temp_every < 0) return GB_ERR_BAD_ARG;
+  if (a.maps < 1 || a.nq % a.maps) return GB_ERR_BAD_ARG;
+  // (several maps: rows that hold all of a kv head's keys, and no dense copy of keys and values)
+  if (a.maps > 1 && (a.kv_out || a.v_from_k || a.Ds < a.maps * a.D)) return GB_ERR_BAD_ARG;
   return 0;
 }
 
 // The kernels that keep a head in registers know one head size, and the query
-// temperature as a factor of the query norm's; heads of two sizes, filled-up rows
-// and a temperature without a query norm take the plain kernel.
+// temperature as a factor of the query norm's; heads of two sizes, filled-up rows, several
+// maps and a temperature without a query norm take the kernel of 8-element pieces where
+// there are no norms, else the plain one.
 static bool plain_only(const QkPrepareArgs& a) {
-  return (a.Dv > 0 && a.Dv != a.D) || (a.Ds > 0 && a.Ds != a.D) || (a.q_temp_every > 0 && !a.q_w);
+  return (a.Dv > 0 && a.Dv != a.D) || (a.Ds > 0 && a.Ds != a.D) || (a.q_temp_every > 0 && !a.q_w) || a.maps > 1;
 }
 
 GB_EXPORT int gb_qk_prepare_f32(const QkPrepareArgs* a, int w_is_f32, cudaStream_t s) {
@@ -684,10 +868,12 @@ GB_EXPORT int gb_qk_prepare_bf16(const QkPrepareArgs* a, int w_is_f32, cudaStrea
   int e = check(*a);
   if (e) return e;
   if (a->n_tokens == 0) return 0;
+  if (plain_only(*a) && piece_ok(*a)) return launch_piece(*a, s);
   if (plain_only(*a)) return w_is_f32 ? launch<bf16, float>(*a, s) : launch<bf16, bf16>(*a, s);
   if (fast_ok(*a) && wide_ok(*a)) return w_is_f32 ? launch_wide<float>(*a, s) : launch_wide<bf16>(*a, s);
   if (fast_ok(*a)) return w_is_f32 ? launch_fast<float>(*a, s) : launch_fast<bf16>(*a, s);
   if (chunk_ok(*a)) return w_is_f32 ? launch_chunk<float>(*a, s) : launch_chunk<bf16>(*a, s);
+  if (piece_ok(*a)) return launch_piece(*a, s);
   return w_is_f32 ? launch<bf16, float>(*a, s) : launch<bf16, bf16>(*a, s);
 }
 

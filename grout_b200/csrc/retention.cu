@@ -11,7 +11,13 @@
 // mixer's one projection (columns q [H dk] | k [H dk] | v [H dv] | gate [H dv]),
 // and only y is rounded to the activation type.
 //
-// Three kernels.  `rotate` writes the turned q and scaled k of every row.  `scan`
+// The same recurrence with other ends ("lightning attention"): with `silu` q, k and v all
+// pass x sigmoid(x) and nothing turns, and with `joint_norm` the read-outs of all heads are
+// normalised together, over H dv elements, times a weight, and gated by a sigmoid:
+//
+//   y = o / sqrt(mean over all heads(o^2) + eps) * norm_w * sigmoid(gate)
+//
+// Three kernels.  `rotate` (with `silu`: `activate`, which leaves v beside them) writes the turned q and scaled k of every row.  `scan`
 // walks a sequence's rows in order: a block owns one (sequence, head) and RT_COLS
 // columns of S; a column's dk elements live in the registers of eight lanes, the
 // rows' q, k and v are staged in shared memory RT_STAGE rows at a time, and the
@@ -51,7 +57,18 @@ struct RetentionArgs {
   int n_tokens, n_seqs, H, dk, dv, rot_dim;
   float k_scale, norm_eps;
   int max_rows;           // the most rows a sequence brings (0: unknown)
+  int silu;               // q, k and v pass a silu
+  int joint_norm;         // one norm over all heads' read-outs, weight norm_w, sigmoid gate
+  const float* norm_w;    // [H dv]
+  float* v;               // [T, H dv] scratch of a step with `silu`: the activated values
 };
+
+__device__ __forceinline__ float rt_silu(float x) { return x / (1.0f + expf(-x)); }
+// Row t's values of head h: the projection's columns, or where `activate` left them.
+__device__ __forceinline__ const float* rt_values(const RetentionArgs& a, int t, int h) {
+  return a.silu ? a.v + ((size_t)t * a.H + h) * a.dv
+                : a.proj + (size_t)t * (2 * a.H * a.dk + 2 * a.H * a.dv) + 2 * a.H * a.dk + h * a.dv;
+}
 
 #define RT_LANES 8      // lanes that share a column of the state
 #define RT_COLS 16      // columns a block owns
@@ -83,6 +100,31 @@ __global__ void __launch_bounds__(256) retention_rotate_kernel(const RetentionAr
     const float u = row[i], v = row[i + half];
     out[i] = (u * c - v * s) * mul;
     out[i + half] = (v * c + u * s) * mul;
+  }
+  pdl_launch_dependents_if_large();
+}
+
+// silu of every q, k and v of the step, four elements a thread where the sizes allow it.
+__global__ void __launch_bounds__(256) retention_activate_kernel(const RetentionArgs a) {
+  pdl_launch_dependents_if_small();
+  pdl_wait();
+  const int nqk = 2 * a.H * a.dk, nv = a.H * a.dv, C = nqk + 2 * nv, t = blockIdx.x;
+  const float* row = a.proj + (size_t)t * C;
+  float* qk = a.qk + (size_t)t * nqk;
+  float* v = a.v + (size_t)t * nv;
+  if (((nqk | nv) & 3) == 0) {
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * 4; i < nqk + nv; i += gridDim.y * blockDim.x * 4) {
+      float4 x = *reinterpret_cast<const float4*>(row + i);
+      const float mul = i >= a.H * a.dk && i < nqk ? a.k_scale : 1.0f;
+      x.x = rt_silu(x.x) * mul, x.y = rt_silu(x.y) * mul, x.z = rt_silu(x.z) * mul, x.w = rt_silu(x.w) * mul;
+      *reinterpret_cast<float4*>(i < nqk ? qk + i : v + (i - nqk)) = x;
+    }
+  } else {
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < nqk + nv; i += gridDim.y * blockDim.x) {
+      const float x = rt_silu(row[i]) * (i >= a.H * a.dk && i < nqk ? a.k_scale : 1.0f);
+      if (i < nqk) qk[i] = x;
+      else v[i - nqk] = x;
+    }
   }
   pdl_launch_dependents_if_large();
 }
@@ -124,7 +166,6 @@ __global__ void __launch_bounds__(RT_COLS* RT_LANES) retention_scan_kernel(const
     const int i = rt_row<KPL>(lane, r);
     S[r] = (sp && live && i < dk) ? sp[(size_t)i * dv + col] : 0.f;
   }
-  const int C = 2 * H * dk + 2 * H * dv;
   for (int t0 = 0; t0 < n; t0 += RT_STAGE) {
     const int nt = min(RT_STAGE, n - t0);
     __syncthreads();
@@ -136,7 +177,7 @@ __global__ void __launch_bounds__(RT_COLS* RT_LANES) retention_scan_kernel(const
     }
     for (int i = tid; i < nt * RT_COLS; i += blockDim.x) {
       const int tt = i / RT_COLS, c = c0 + i % RT_COLS;
-      vs[tt][i % RT_COLS] = c < dv ? a.proj[(size_t)(first + t0 + tt) * C + 2 * H * dk + h * dv + c] : 0.f;
+      vs[tt][i % RT_COLS] = c < dv ? rt_values(a, first + t0 + tt, h)[c] : 0.f;
     }
     __syncthreads();
     for (int tt = 0; tt < nt; ++tt) {
@@ -201,7 +242,6 @@ __global__ void __launch_bounds__(256) retention_chunk_kernel(const RetentionArg
   if (z * RT_CHUNK >= n) return;
   const int rows = min(RT_CHUNK, n - z * RT_CHUNK), r0 = first + z * RT_CHUNK;
   const int tid = threadIdx.x, ty = tid / 16, tx = tid % 16;
-  const int C = 2 * H * dk + 2 * H * dv;
   const float decay = a.decay[h];
   if (tid <= RT_CT) dpow[tid] = powf(decay, (float)tid);
   float acc[4][4];
@@ -250,7 +290,7 @@ __global__ void __launch_bounds__(256) retention_chunk_kernel(const RetentionArg
 #pragma unroll
     for (int i = 0; i < RT_CT * RT_CT / 256; ++i) {
       const int idx = tid + i * 256, t = idx / RT_CT, c = idx % RT_CT;
-      Vs[t][c] = (t < rows && c0 + c < dv) ? a.proj[(size_t)(r0 + t) * C + 2 * H * dk + h * dv + c0 + c] : 0.f;
+      Vs[t][c] = (t < rows && c0 + c < dv) ? rt_values(a, r0 + t, h)[c0 + c] : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -438,6 +478,40 @@ __global__ void __launch_bounds__(128) retention_finish_kernel(const RetentionAr
   }
 }
 
+// y[t, :] = o / sqrt(mean over the row(o^2) + eps) * norm_w * sigmoid(gate): one block per row
+template <typename T>
+__global__ void __launch_bounds__(256) retention_joint_finish_kernel(const RetentionArgs a) {
+  __shared__ float scratch[32];
+  pdl_launch_dependents_if_small();
+  pdl_wait();
+  const int t = blockIdx.x, n = a.H * a.dv;
+  const float* o = a.o + (size_t)t * n;
+  const float* g = a.proj + (size_t)t * (2 * a.H * a.dk + 2 * n) + 2 * a.H * a.dk + n;
+  T* y = (T*)a.y + (size_t)t * n;
+  float ss = 0.f;
+  if ((n & 3) == 0 && ((2 * a.H * a.dk) & 3) == 0) {
+    for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+      const float4 x = *reinterpret_cast<const float4*>(o + i);
+      ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, ss))));
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + a.norm_eps);
+    for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+      const float4 x = *reinterpret_cast<const float4*>(o + i), w = *reinterpret_cast<const float4*>(a.norm_w + i),
+                   gv = *reinterpret_cast<const float4*>(g + i);
+      y[i] = from_f32<T>(x.x * inv * w.x / (1.0f + expf(-gv.x)));
+      y[i + 1] = from_f32<T>(x.y * inv * w.y / (1.0f + expf(-gv.y)));
+      y[i + 2] = from_f32<T>(x.z * inv * w.z / (1.0f + expf(-gv.z)));
+      y[i + 3] = from_f32<T>(x.w * inv * w.w / (1.0f + expf(-gv.w)));
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(o[i], o[i], ss);
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + a.norm_eps);
+    for (int i = threadIdx.x; i < n; i += blockDim.x)
+      y[i] = from_f32<T>(o[i] * inv * a.norm_w[i] / (1.0f + expf(-g[i])));
+  }
+  pdl_launch_dependents_if_large();
+}
+
 #define RT_STEP_WARPS 8
 
 // One row per sequence.  DVJ: columns a lane holds (dv <= 32 DVJ).
@@ -463,6 +537,7 @@ __global__ void __launch_bounds__(RT_STEP_WARPS * 32) retention_step_kernel(cons
   for (int e = tid; e < dk; e += blockDim.x) {
     const float* q = row + h * dk;
     const float* k = row + H * dk + h * dk;
+    if (a.silu) { qs[e] = rt_silu(q[e]); ks[e] = rt_silu(k[e]) * a.k_scale; continue; }
     if (e >= a.rot_dim) { qs[e] = q[e]; ks[e] = k[e] * a.k_scale; continue; }
     if (e >= half) continue;
     float sn, cs;
@@ -472,7 +547,10 @@ __global__ void __launch_bounds__(RT_STEP_WARPS * 32) retention_step_kernel(cons
     ks[e] = (k[e] * cs - k[e + half] * sn) * a.k_scale;
     ks[e + half] = (k[e + half] * cs + k[e] * sn) * a.k_scale;
   }
-  for (int c = tid; c < dv; c += blockDim.x) vs[c] = row[2 * H * dk + h * dv + c];
+  for (int c = tid; c < dv; c += blockDim.x) {
+    const float v = row[2 * H * dk + h * dv + c];
+    vs[c] = a.silu ? rt_silu(v) : v;
+  }
   __syncthreads();
   const int slot = a.slots[seq];
   float* sp = slot >= 0 ? a.state + (size_t)slot * a.state_stride + (size_t)h * dk * dv : nullptr;
@@ -525,6 +603,14 @@ __global__ void __launch_bounds__(RT_STEP_WARPS * 32) retention_step_kernel(cons
       ss = fmaf(o[j], o[j], ss);
     }
   }
+  if (a.joint_norm) {          // the norm is over all heads: another kernel finishes the row
+#pragma unroll
+    for (int j = 0; j < (int)(sizeof(o) / sizeof(float)); ++j) {
+      const int c = tid + j * RT_STEP_WARPS * 32;
+      if (c < dv) a.o[((size_t)t * H + h) * dv + c] = o[j];
+    }
+    return;
+  }
   const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dv + a.norm_eps);
   const float* g = row + 2 * H * dk + H * dv + h * dv;
   T* y = (T*)a.y + ((size_t)t * H + h) * dv;
@@ -562,6 +648,14 @@ static int retention_chunk_launch(const RetentionArgs& a, cudaStream_t s, int ch
 }
 
 template <typename T>
+static int retention_finish(const RetentionArgs& a, cudaStream_t s) {
+  if (a.joint_norm)
+    return gb_launch(retention_joint_finish_kernel<T>, dim3(a.n_tokens), dim3(256), 0, s, a);
+  const long long warps = (long long)a.n_tokens * a.H;
+  return gb_launch(retention_finish_kernel<T>, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, s, a);
+}
+
+template <typename T>
 static int retention_forward(const RetentionArgs& a, cudaStream_t s) {
   if (a.n_tokens < 0 || a.n_seqs < 0 || a.H <= 0 || a.dk <= 0 || a.dv <= 0 || a.rot_dim < 0 ||
       a.rot_dim > a.dk || a.rot_dim % 2 || a.n_seqs > 65535)
@@ -569,15 +663,18 @@ static int retention_forward(const RetentionArgs& a, cudaStream_t s) {
   if (!a.proj || !a.decay || !a.token_pos || !a.cu_q || !a.slots || !a.state || !a.qk || !a.o ||
       !a.y || (a.rot_dim && !a.inv_freq))
     return GB_ERR_BAD_ARG;
+  if ((a.silu && (!a.v || a.rot_dim)) || (a.joint_norm && !a.norm_w)) return GB_ERR_BAD_ARG;
   if (a.dk > 256) return GB_ERR_UNSUPPORTED;
   if (a.n_tokens == 0 || a.n_seqs == 0) return 0;
   if (a.max_rows == 1 && a.dv <= 256 && a.H <= 65535) {
-    if (a.dv <= 32) return retention_step_launch<T, 1>(a, s);
-    if (a.dv <= 64) return retention_step_launch<T, 2>(a, s);
-    if (a.dv <= 128) return retention_step_launch<T, 4>(a, s);
-    return retention_step_launch<T, 8>(a, s);
+    int e = a.dv <= 32    ? retention_step_launch<T, 1>(a, s)
+            : a.dv <= 64  ? retention_step_launch<T, 2>(a, s)
+            : a.dv <= 128 ? retention_step_launch<T, 4>(a, s)
+                          : retention_step_launch<T, 8>(a, s);
+    return e || !a.joint_norm ? e : retention_finish<T>(a, s);
   }
-  int e = gb_launch(retention_rotate_kernel, dim3(a.n_tokens), dim3(256), 0, s, a);
+  int e = a.silu ? gb_launch(retention_activate_kernel, dim3(a.n_tokens, 2), dim3(256), 0, s, a)
+                 : gb_launch(retention_rotate_kernel, dim3(a.n_tokens), dim3(256), 0, s, a);
   if (e) return e;
   // a sequence of many rows goes chunk by chunk: every chunk alone from zeros and all at
   // once, then the states at the chunks' starts, then what those add to the read-outs
@@ -599,8 +696,7 @@ static int retention_forward(const RetentionArgs& a, cudaStream_t s) {
                   dim3(chunks * (RT_CHUNK / RT_TM) * ((a.dv + RT_TN - 1) / RT_TN), a.H, a.n_seqs), dim3(256), 0, s, a);
     if (e) return e;
   }
-  const long long warps = (long long)a.n_tokens * a.H;
-  return gb_launch(retention_finish_kernel<T>, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, s, a);
+  return retention_finish<T>(a, s);
 }
 
 GB_EXPORT int gb_retention_forward_f32(const RetentionArgs* a, cudaStream_t s) {

@@ -157,6 +157,7 @@ def _cost_attention(out, q, k_pages, *args, **kw):
     nq, D = q.shape[1], q.shape[2]
     nkv, item = k_pages.shape[1], k_pages.element_size()
     kv_len, slots, cu_q, window = kw.get("kv_len"), kw.get("slots"), kw.get("cu_q"), kw.get("window")
+    chunk = kw.get("chunk")
     if kv_len is None:
         return _nbytes(q, out), 0
     live = (slots >= 0)
@@ -169,6 +170,11 @@ def _cost_attention(out, q, k_pages, *args, **kw):
     if window:
         pairs = torch.minimum(pairs, rows * float(window))
         lens = torch.minimum(lens, rows + float(window))
+    elif chunk:          # keys a query sees: its place in its chunk, plus one; read: from the first row's chunk on
+        tri = lambda n: torch.floor(n / chunk) * (chunk * (chunk + 1) / 2) + (n % chunk) * (n % chunk + 1) / 2
+        pairs = tri(lens) - tri(lens - rows)
+        first = torch.clamp(lens - rows, min=0)
+        lens = lens - torch.floor(first / chunk) * chunk
     kv_bytes = (lens.sum() * (2 * nkv * D * item))
     pair_sum = pairs.sum()
     base = _nbytes(q, out)
@@ -413,6 +419,62 @@ def add_layernorm(res_in: Optional[torch.Tensor], delta: Optional[torch.Tensor],
     return res_out, y
 
 
+class _DytArgs(ctypes.Structure):
+    _fields_ = [("res_in", _P), ("delta", _P), ("parts", _P), ("n_parts", _I), ("part_stride", _L),
+                ("rows", _P), ("alpha", _P), ("w", _P), ("b", _P), ("res_out", _P), ("y", _P),
+                ("n_rows", _I), ("N", _I)]
+
+
+@_profiled("add_dyt", _cost_io)
+def add_dyt(res_in: Optional[torch.Tensor], delta: Optional[torch.Tensor], alpha: torch.Tensor,
+            weight: torch.Tensor, bias: torch.Tensor, *, dtype: torch.dtype,
+            rows: Optional[torch.Tensor] = None, write_res: bool = True
+            ) -> Tuple[Optional[torch.Tensor], torch.Tensor]:
+    """v = res_in + delta in 32-bit -> (v, tanh(alpha v) * weight + bias).  ``alpha`` is one
+    32-bit number on the device, ``weight`` and ``bias`` are 32-bit [N]; ``delta`` is [T, N] in
+    ``dtype`` or a stack of 32-bit partial sums [S, T, N], added in order.  Without ``rows`` the
+    residual is updated in place when ``res_in`` is given."""
+    parts = None
+    if delta is not None and delta.dim() == 3:
+        _need(delta, "partial sums", torch.float32, 3)
+        parts, delta = delta, None
+    src = res_in if res_in is not None else (delta if delta is not None else
+                                             (parts[0] if parts is not None else None))
+    if src is None:
+        raise KernelError("add_dyt needs a residual or a delta")
+    if res_in is not None:
+        _need(res_in, "residual", torch.float32, 2)
+    if delta is not None:
+        _need(delta, "delta", dtype, 2)
+    for t in (delta, parts[0] if parts is not None else None):
+        if t is not None and tuple(t.shape) != tuple(src.shape):
+            raise KernelError(f"residual {tuple(src.shape)} and delta {tuple(t.shape)} differ")
+    N = src.shape[1]
+    for t, nm, n in ((alpha, "alpha", 1), (weight, "norm weight", N), (bias, "norm bias", N)):
+        _need(t, nm, torch.float32, 1)
+        if t.shape[0] != n:
+            raise KernelError(f"{nm} has {t.shape[0]} elements for rows of {N}")
+    if rows is not None:
+        _need(rows, "row list", torch.int32, 1)
+    n_rows = rows.shape[0] if rows is not None else src.shape[0]
+    res_out = None
+    if write_res:
+        nothing_added = delta is None and parts is None
+        if rows is None and res_in is not None:
+            res_out = None if nothing_added else res_in
+        else:
+            res_out = torch.empty((n_rows, N), dtype=torch.float32, device=src.device)
+    y = torch.empty((n_rows, N), dtype=dtype, device=src.device)
+    a = _DytArgs()
+    a.res_in, a.delta, a.parts = _ptr(res_in), _ptr(delta), _ptr(parts)
+    a.n_parts = 0 if parts is None else parts.shape[0]
+    a.part_stride = 0 if parts is None else parts.stride(0)
+    a.rows, a.alpha, a.w, a.b = _ptr(rows), alpha.data_ptr(), weight.data_ptr(), bias.data_ptr()
+    a.res_out, a.y, a.n_rows, a.N = _ptr(res_out), y.data_ptr(), n_rows, N
+    _check(_fn("dyt", f"gb_add_dyt_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()), "add_dyt")
+    return (res_in if res_out is None and rows is None and write_res else res_out), y
+
+
 class _PostNormArgs(ctypes.Structure):
     _fields_ = [("res_in", _P), ("delta", _P), ("parts", _P), ("n_parts", _I), ("part_stride", _L),
                 ("rows", _P), ("post_w", _P), ("post_eps", _F), ("scale", _P), ("w", _P),
@@ -481,7 +543,8 @@ class _QkPrepareArgs(ctypes.Structure):
                 ("n_tokens", _I), ("nq", _I), ("nkv", _I), ("D", _I), ("rot_dim", _I),
                 ("max_pages", _I), ("page", _I), ("qkv_parts", _P), ("n_parts", _I),
                 ("part_stride", _L), ("v_from_k", _I), ("Dv", _I), ("Ds", _I),
-                ("q_temp_coef", _F), ("q_temp_every", _I), ("interleaved", _I)]
+                ("q_temp_coef", _F), ("q_temp_every", _I), ("interleaved", _I), ("maps", _I),
+                ("rot_scale", _F)]
 
 
 @_profiled("qk_prepare", lambda out, qkv, nq, nkv, D, **k: _cost_qk_prepare(out, qkv, nq, nkv, D))
@@ -490,7 +553,8 @@ def qk_prepare(qkv: torch.Tensor, nq: int, nkv: int, D: int, *, q_w=None, k_w=No
                block_table=None, k_pages=None, v_pages=None, page: int = 0,
                want_kv_out: bool = False, values_are_keys: bool = False,
                v_dim: Optional[int] = None, q_temp: Optional[Tuple[float, int]] = None,
-               interleaved: bool = False):
+               interleaved: bool = False, rot_scale: float = 1.0, maps: int = 1,
+               row_width: Optional[int] = None):
     """Returns (q [T, nq, Ds], kv_out or None); writes k, v into the pages when given.
     ``qkv`` may be a stack of 32-bit partial sums [S, T, width] of the projection
     (bf16 engines only): they are added in order.  ``values_are_keys``: the
@@ -500,7 +564,12 @@ def qk_prepare(qkv: torch.Tensor, nq: int, nkv: int, D: int, *, q_w=None, k_w=No
     row width (at least D and ``v_dim``) or, without pages, the larger of the two,
     and end in zeros.  ``q_temp`` = (coef, every): a query at position p is
     multiplied, after its norm, by 1 + coef * ln(floor((p + 1) / every) + 1).
-    ``interleaved``: the rotation pairs element 2j with 2j + 1 (else j with j + rot_dim / 2)."""
+    ``interleaved``: the rotation pairs element 2j with 2j + 1 (else j with j + rot_dim / 2);
+    ``rot_scale`` multiplies its sine and cosine.  ``row_width``: Ds of queries that are made
+    without pages (for pages that another layer wrote).  ``maps`` M: a head has M query and M
+    key vectors of D that share its value: the projection holds ``nq`` = heads * M queries and
+    nkv * M keys; a stored key row is the M keys side by side, and query vector m of a head is
+    a row of its own that is zero but for its elements m D .. (m + 1) D."""
     parts = None
     if qkv.dim() == 3:
         _need(qkv, "qkv partial sums", torch.float32, 3)
@@ -512,14 +581,17 @@ def qk_prepare(qkv: torch.Tensor, nq: int, nkv: int, D: int, *, q_w=None, k_w=No
         dt = qkv.dtype
     T = qkv.shape[-2]
     Dv = int(v_dim) if v_dim else D
-    if Dv != D and (values_are_keys or nkv == 0):
+    maps = int(maps)
+    if maps < 1 or nq % maps or (maps > 1 and (values_are_keys or want_kv_out)):
+        raise KernelError(f"{nq} queries do not form heads of {maps} maps with values of their own")
+    if Dv != D and values_are_keys:
         raise KernelError("values of another size than the keys need a v projection")
-    Ds = int(k_pages.shape[-1]) if k_pages is not None else max(D, Dv)
-    if Ds < max(D, Dv):
-        raise KernelError(f"pages with rows of {Ds} cannot hold heads of {D} and {Dv}")
-    width = (nq + nkv) * D + (0 if values_are_keys else nkv * Dv)
+    Ds = int(k_pages.shape[-1]) if k_pages is not None else int(row_width or max(maps * D, Dv))
+    if Ds < max(maps * D, Dv):
+        raise KernelError(f"rows of {Ds} cannot hold {maps} times {D} and {Dv} elements")
+    width = (nq + nkv * maps) * D + (0 if values_are_keys else nkv * Dv)
     if qkv.shape[-1] != width:
-        raise KernelError(f"the projection has {qkv.shape[-1]} columns, expected {nq} + {nkv} heads of "
+        raise KernelError(f"the projection has {qkv.shape[-1]} columns, expected {nq} + {nkv * maps} heads of "
                           f"{D}" + ("" if values_are_keys else f" and {nkv} of {Dv}") + f" = {width}")
     w_is_f32 = int(dt == torch.float32)      # without norm weights: whatever the entry point takes
     for w, nm in ((q_w, "q norm weight"), (k_w, "k norm weight")):
@@ -549,7 +621,7 @@ def qk_prepare(qkv: torch.Tensor, nq: int, nkv: int, D: int, *, q_w=None, k_w=No
     a.eps, a.n_tokens, a.nq, a.nkv, a.D, a.rot_dim = float(eps), T, nq, nkv, D, int(rot_dim)
     a.v_from_k = int(values_are_keys)
     a.interleaved = int(bool(interleaved) and inv_freq is not None)
-    a.Dv, a.Ds = Dv, Ds
+    a.Dv, a.Ds, a.maps, a.rot_scale = Dv, Ds, maps, float(rot_scale)
     if q_temp:
         a.q_temp_coef, a.q_temp_every = float(q_temp[0]), int(q_temp[1])
     if k_pages is not None:
@@ -600,6 +672,15 @@ def _attn_common(q, k_pages, v_pages, block_table, token_seq, token_pos, slots, 
     return T, nq, nkv, D
 
 
+def _chunk_arg(chunk: Optional[int], keep_first: int) -> int:
+    """The kernels' chunk argument: a query sees the keys of its own chunk of that many
+    positions (0: no chunks)."""
+    chunk = int(chunk or 0)
+    if chunk < 0 or (chunk and keep_first):
+        raise KernelError("a chunk size is positive and goes without kept first keys")
+    return chunk
+
+
 def _check_sinks(sinks, nq: int) -> None:
     if sinks is not None:
         _need(sinks, "sinks", torch.float32, 1)
@@ -610,30 +691,41 @@ def _check_sinks(sinks, nq: int) -> None:
 @_profiled("attn_generic", lambda out, q, *a, **k: (_nbytes(q, out), 0))
 def attn_generic(q, k_pages, v_pages, block_table, *, token_seq, token_pos, slots, page: int,
                  scale: float, window: Optional[int] = None, softcap: Optional[float] = None,
-                 sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                 sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
+                    chunk: int = 0) -> torch.Tensor:
     T, nq, nkv, D = _attn_common(q, k_pages, v_pages, block_table, token_seq, token_pos, slots, page)
     _check_sinks(sinks, nq)
     out = torch.empty_like(q)
     sfx = _suffix(q.dtype)
-    _check(_fn("attn_generic", f"gb_attn_generic_{sfx}", "ppppippppiiiiififpip")(
+    _check(_fn("attn_generic", f"gb_attn_generic_{sfx}", "ppppippppiiiiififpiip")(
         q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), block_table.data_ptr(),
         block_table.shape[1], token_seq.data_ptr(), token_pos.data_ptr(), slots.data_ptr(),
         out.data_ptr(), T, nq, nkv, D, page, float(scale), int(window or 0), float(softcap or 0.0),
-        _ptr(sinks), int(keep_first or 0), _stream()), "attn_generic")
+        _ptr(sinks), int(keep_first or 0), _chunk_arg(chunk, keep_first), _stream()), "attn_generic")
     return out
 
 
 # ---------------------------------------------------------------- matrix products
+def _result(shape, dtype, device, into: Optional[torch.Tensor]) -> torch.Tensor:
+    """A new tensor, or the caller's (contiguous, of that shape and type)."""
+    if into is None:
+        return torch.empty(shape, dtype=dtype, device=device)
+    _need(into, "result", dtype)
+    if into.numel() != math.prod(shape):
+        raise KernelError(f"the result is {tuple(into.shape)}, expected {tuple(shape)}")
+    return into.view(shape)
+
+
 @_profiled("gemm_f32", _cost_gemm)
-def gemm_f32(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """a [M, K] . w [N, K]^T in true 32-bit on the CUDA cores."""
+def gemm_f32(a: torch.Tensor, w: torch.Tensor, into: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """a [M, K] . w [N, K]^T in true 32-bit on the CUDA cores (written into ``into`` when given)."""
     _need(a, "activations", torch.float32, 2)
     _need(w, "weight", torch.float32, 2)
     M, K = a.shape
     N = w.shape[0]
     if w.shape[1] != K:
         raise KernelError(f"weight is {tuple(w.shape)} for activations of width {K}")
-    c = torch.empty((M, N), dtype=torch.float32, device=a.device)
+    c = _result((M, N), torch.float32, a.device, into)
     _check(_fn("gemm_f32", "gb_gemm_nt_f32", "pppiiiiiip")(
         a.data_ptr(), w.data_ptr(), c.data_ptr(), M, N, K, K, K, N, _stream()), "gemm_f32")
     return c
@@ -752,12 +844,16 @@ def cast(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
 
 
 @_profiled("library_mm", _cost_gemm)
-def library_mm(x: torch.Tensor, w: torch.Tensor, out_dtype=None) -> torch.Tensor:
+def library_mm(x: torch.Tensor, w: torch.Tensor, out_dtype=None,
+               into: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x [M, K] . w [N, K]^T by the library's matrix product (cuBLAS through
     torch.mm): the prompt products for which the reference calls a library too
     (src/cublas.rs:287-307).  It is here so that the profile sees it."""
     _need(x, "activations", torch.bfloat16, 2)
     _need(w, "weight", torch.bfloat16, 2)
+    if into is not None:
+        y = _result((x.shape[0], w.shape[0]), out_dtype or torch.bfloat16, x.device, into)
+        return torch.mm(x, w.t(), out_dtype=y.dtype, out=y) if y.dtype == torch.float32 else torch.mm(x, w.t(), out=y)
     if out_dtype == torch.float32:
         return torch.mm(x, w.t(), out_dtype=torch.float32)
     return torch.mm(x, w.t())
@@ -813,7 +909,7 @@ def skinny_plan(M: int, N: int, K: int, out_f32: bool, silu: bool):
 
 @_profiled("gemm_skinny_bf16", _cost_gemm)
 def gemm_skinny_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype=torch.bfloat16,
-                     silu_mul: bool = False) -> torch.Tensor:
+                     silu_mul: bool = False, into: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x [M <= 64, K] . w [N, K]^T, bf16 in, 32-bit accumulate; the decode-time
     linear.  With ``silu_mul`` the rows of ``w`` are gate and up rows interleaved
     in groups of 8 and the result is silu(gate) * up, [M, N / 2]."""
@@ -831,7 +927,7 @@ def gemm_skinny_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype=torch.bfloat16,
         raise KernelError(f"output must be bfloat16 or float32, not {out_dtype}")
     if silu_mul and N % 16:
         raise KernelError(f"the interleaved gate|up product needs N to be a multiple of 16, got {N}")
-    y = torch.empty((M, N // 2 if silu_mul else N), dtype=out_dtype, device=x.device)
+    y = _result((M, N // 2 if silu_mul else N), out_dtype, x.device, into)
     if M == 0:
         return y
     with torch.cuda.device(x.device):
@@ -916,12 +1012,33 @@ def tc_wait_selftest(device, limit_us: int = 1000) -> int:
     return int(left.item())
 
 
+def _tc_plan(rows_a: int, rows_b: int, K: int):
+    """(tile columns, ..., scratch floats, counters, partial sums of a split result) of the
+    tcgen05 product of this shape on the current device."""
+    key = (rows_a, rows_b, K, torch.cuda.current_device())
+    plan = _TC_PLANS.get(key)
+    if plan is None:
+        out = (c_int * 5)()
+        _check(_fn("gemm_tc", "gb_gemm_tc_plan", "iiip")(rows_a, rows_b, K, ctypes.addressof(out)),
+               "gemm_tc_plan", 0)
+        plan = _TC_PLANS[key] = (out[0], out[1], out[2], out[3], out[4])
+    return plan
+
+
+def gemm_tc_parts(M: int, N: int, K: int, device) -> int:
+    """How many partial sums ``gemm_tc_bf16(swap=True, split_out=True)`` returns for x [M, K]
+    and w [N, K] (0: an ordinary result)."""
+    with torch.cuda.device(device):
+        return _tc_plan(N, M, K)[4]
+
+
 @_profiled("gemm_tc_bf16", _cost_gemm)
 def gemm_tc_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype=torch.bfloat16,
                  swap: Optional[bool] = None, silu_mul: bool = False,
                  stamps: Optional[torch.Tensor] = None, split_out: bool = False,
                  relu_squared: bool = False, gate_act: str = "silu",
-                 bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 bias: Optional[torch.Tensor] = None,
+                 into: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x [M, K] . w [N, K]^T on the tcgen05 tensor cores (TMA-fed, accumulator in
     tensor memory).  ``swap``: put the weight rows on the 128-row side of the MMA
     and the activation rows on the narrow side (the layout for few rows); by
@@ -953,21 +1070,14 @@ def gemm_tc_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype=torch.bfloat16,
     if relu_squared and (silu_mul or split_out):
         raise KernelError("the squared relu goes with neither the gate|up epilogue nor partial sums")
     n_out = N // 2 if silu_mul else N
-    y = torch.empty((M, n_out), dtype=out_dtype, device=x.device)
     if M == 0:
-        return y
+        return _result((M, n_out), out_dtype, x.device, into)
     A, B = (w, x) if swap else (x, w)
     with torch.cuda.device(x.device):
-        key = (A.shape[0], B.shape[0], K, torch.cuda.current_device())
-        plan = _TC_PLANS.get(key)
-        if plan is None:
-            out = (c_int * 5)()
-            _check(_fn("gemm_tc", "gb_gemm_tc_plan", "iiip")(
-                A.shape[0], B.shape[0], K, ctypes.addressof(out)), "gemm_tc_plan", 0)
-            plan = _TC_PLANS[key] = (out[0], out[1], out[2], out[3], out[4])
+        plan = _tc_plan(A.shape[0], B.shape[0], K)
         split = plan[4] if (split_out and swap and not silu_mul) else 0
-        if split:
-            y = torch.empty((split, M, N), dtype=torch.float32, device=x.device)
+        y = (_result((split, M, N), torch.float32, x.device, into) if split
+             else _result((M, n_out), out_dtype, x.device, into))
         ws = _WORKSPACES.setdefault(x.device.index or 0, _Workspace())
         scratch, counters = ws.get(x.device, plan[2], plan[3])
         a = _TcArgs()
@@ -1025,7 +1135,8 @@ def gemm_tc2_pays(M: int, N: int, device, fused_silu: bool) -> bool:
 def gemm_tc2_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype=torch.bfloat16,
                   silu_mul: bool = False, tile_cols: int = 0,
                   relu_squared: bool = False, gate_act: str = "silu",
-                  bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  bias: Optional[torch.Tensor] = None,
+                  into: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x [M, K] . w [N, K]^T for many rows on pairs of SMs (tcgen05.mma.cta_group::2,
     tiles of 256 rows and ``tile_cols`` columns: a multiple of 16 up to 256, by
     default chosen by the kernel's launcher for the shape).  ``silu_mul``: the rows of ``w`` are gate and up rows
@@ -1051,7 +1162,7 @@ def gemm_tc2_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype=torch.bfloat16,
     n_out = N // 2 if silu_mul else N
     if (n_out * (4 if out_dtype == torch.float32 else 2)) % 16:
         raise KernelError(f"gemm_tc2_bf16 stores 16 bytes at a time: {n_out} output columns do not allow it")
-    y = torch.empty((M, n_out), dtype=out_dtype, device=x.device)
+    y = _result((M, n_out), out_dtype, x.device, into)
     if M == 0:
         return y
     a = _Tc2Args()
@@ -1072,7 +1183,7 @@ class _PrefillArgs(ctypes.Structure):
                 ("slots", _P), ("kv_len", _P), ("out", _P), ("n_seqs", _I), ("nq", _I),
                 ("nkv", _I), ("max_pages", _I), ("window", _I), ("n_qblocks", _I),
                 ("scale_log2", _F), ("sinks", _P), ("cap_log2", _F), ("cap_inv", _F),
-                ("keep_first", _I)]
+                ("keep_first", _I), ("chunk", _I)]
 
 
 class _DecodeArgs(ctypes.Structure):
@@ -1080,7 +1191,7 @@ class _DecodeArgs(ctypes.Structure):
                 ("kv_len", _P), ("out", _P), ("part_o", _P), ("part_ml", _P), ("n_seqs", _I),
                 ("nq", _I), ("nkv", _I), ("max_pages", _I), ("page", _I), ("window", _I),
                 ("n_splits", _I), ("scale_log2", _F), ("sinks", _P), ("cap_log2", _F),
-                ("cap_inv", _F), ("keep_first", _I)]
+                ("cap_inv", _F), ("keep_first", _I), ("chunk", _I)]
 
 
 def _set_cap_and_sinks(a, scale: float, softcap: Optional[float], sinks, nq: int) -> None:
@@ -1140,7 +1251,8 @@ def _q_blocks(q_lens, n_qblocks, rows: int, T: int, n_seqs: int) -> int:
 def attn_prefill_bf16(q, k_pages, v_pages, block_table, *, cu_q, slots, kv_len, q_lens=(),
                       page: int, scale: float, window: Optional[int] = None,
                       n_qblocks: Optional[int] = None, softcap: Optional[float] = None,
-                      sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                      sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
+                    chunk: int = 0) -> torch.Tensor:
     """Causal attention of whole prompts (or their continuation) on the tensor
     cores.  ``keep_first``: with a window, a sequence's first keys that stay visible behind it.  The grid is sized from ``q_lens``, the host's copy of the sequences'
     row counts, or, without them, from ``n_qblocks`` (an upper bound of the
@@ -1165,7 +1277,7 @@ def attn_prefill_bf16(q, k_pages, v_pages, block_table, *, cu_q, slots, kv_len, 
     a.window = int(window or 0)
     a.n_qblocks = _q_blocks(q_lens, n_qblocks, PREFILL_ROWS, T, n_seqs)
     a.scale_log2 = float(scale) * _LOG2E
-    a.keep_first = int(keep_first or 0)
+    a.keep_first, a.chunk = int(keep_first or 0), _chunk_arg(chunk, keep_first)
     _set_cap_and_sinks(a, scale, softcap, sinks, nq)
     _check(_fn("attn_prefill_bf16", "gb_attn_prefill_bf16", "piip")(
         ctypes.addressof(a), D, page, _stream()), "attn_prefill_bf16")
@@ -1176,7 +1288,7 @@ class _AttnTcArgs(ctypes.Structure):
     _fields_ = [("block_table", _P), ("cu_q", _P), ("slots", _P), ("kv_len", _P), ("out", _P),
                 ("error", _P), ("n_seqs", _I), ("nq", _I), ("nkv", _I), ("max_pages", _I),
                 ("window", _I), ("n_qblocks", _I), ("scale_log2", _F), ("sinks", _P),
-                ("cap_log2", _F), ("cap_inv", _F), ("keep_first", _I)]
+                ("cap_log2", _F), ("cap_inv", _F), ("keep_first", _I), ("chunk", _I)]
 
 
 PREFILL_TC_ROWS = 0        # query rows per block of the tcgen05 prefill kernel: 128, 256 or 0 = by size
@@ -1201,7 +1313,8 @@ def attn_prefill_tc(q, k_pages, v_pages, block_table, *, cu_q, slots, kv_len, q_
                     page: int, scale: float, window: Optional[int] = None,
                     rows_per_block: int = 0, n_qblocks: Optional[int] = None,
                     softcap: Optional[float] = None,
-                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
+                    chunk: int = 0) -> torch.Tensor:
     """Causal attention of whole prompts (or their continuation) with both
     products on the tcgen05 tensor cores.  Pages must hold finite values in the
     rows beyond a sequence's length (the cache zero-fills its pages).  The grid is
@@ -1230,7 +1343,7 @@ def attn_prefill_tc(q, k_pages, v_pages, block_table, *, cu_q, slots, kv_len, q_
         prefill_tc_rows(_q_blocks(q_lens, None, 256, T, n_seqs), nq, q.device)
     a.n_qblocks = _q_blocks(q_lens, n_qblocks, rows, T, n_seqs)
     a.scale_log2 = float(scale) * _LOG2E
-    a.keep_first = int(keep_first or 0)
+    a.keep_first, a.chunk = int(keep_first or 0), _chunk_arg(chunk, keep_first)
     _set_cap_and_sinks(a, scale, softcap, sinks, nq)
     _check(_fn("attn_prefill_tc", "gb_attn_prefill_tc", "ppppiliiip")(
         q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr(), ctypes.addressof(a), T,
@@ -1258,9 +1371,13 @@ def decode_splits(n_seqs: int, nkv: int, max_kv_len: int, device) -> int:
     return min(s for s, c in cost.items() if c <= 1.03 * best)
 
 
-def _keys_visited(max_kv_len: int, window: Optional[int], page: int, keep_first: int = 0) -> int:
+def _keys_visited(max_kv_len: int, window: Optional[int], page: int, keep_first: int = 0,
+                  chunk: int = 0) -> int:
     """The most keys a decode row reads: its sequence's, or with a window the
-    window's and the kept first ones, rounded out to the tiles that hold them."""
+    window's and the kept first ones, with chunks its chunk's, rounded out to the tiles
+    that hold them."""
+    if chunk:
+        max_kv_len = min(max_kv_len, chunk + page - 1)
     if not window:
         return max_kv_len
     kept = (int(keep_first or 0) + page - 1) // page * page
@@ -1271,7 +1388,8 @@ def _keys_visited(max_kv_len: int, window: Optional[int], page: int, keep_first:
 def attn_decode_bf16(q, k_pages, v_pages, block_table, *, slots, kv_len, page: int, scale: float,
                      max_kv_len: int, window: Optional[int] = None,
                      n_splits: Optional[int] = None, softcap: Optional[float] = None,
-                     sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                     sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
+                    chunk: int = 0) -> torch.Tensor:
     """Attention of one new token per sequence over its cached keys (split-K).
     ``keep_first``: with a window, a sequence's first keys that stay visible behind it."""
     _need(q, "q", torch.bfloat16, 3)
@@ -1287,7 +1405,7 @@ def attn_decode_bf16(q, k_pages, v_pages, block_table, *, slots, kv_len, page: i
         raise KernelError("one slot and one length per query row are needed")
     # (a window bounds the keys a row visits, whatever its sequence's length)
     ns = int(n_splits) if n_splits else decode_splits(
-        B, nkv, _keys_visited(max_kv_len, window, page, keep_first), q.device)
+        B, nkv, _keys_visited(max_kv_len, window, page, keep_first, chunk), q.device)
     out = torch.empty_like(q)
     part_o = part_ml = None
     if ns > 1:
@@ -1302,7 +1420,7 @@ def attn_decode_bf16(q, k_pages, v_pages, block_table, *, slots, kv_len, page: i
     a.part_o, a.part_ml = _ptr(part_o), _ptr(part_ml)
     a.n_seqs, a.nq, a.nkv, a.max_pages, a.page = B, nq, nkv, block_table.shape[1], page
     a.window, a.n_splits, a.scale_log2 = int(window or 0), ns, float(scale) * _LOG2E
-    a.keep_first = int(keep_first or 0)
+    a.keep_first, a.chunk = int(keep_first or 0), _chunk_arg(chunk, keep_first)
     _set_cap_and_sinks(a, scale, softcap, sinks, nq)
     _check(_fn("attn_decode_bf16", "gb_attn_decode_bf16", "pip")(
         ctypes.addressof(a), D, _stream()), "attn_decode_bf16", 2 if ns > 1 else 1)
@@ -1314,7 +1432,7 @@ class _DecodeTmaArgs(ctypes.Structure):
                 ("part_o", _P), ("part_ml", _P), ("counters", _P), ("error", _P), ("n_seqs", _I),
                 ("nq", _I), ("nkv", _I), ("max_pages", _I), ("window", _I), ("n_splits", _I),
                 ("scale_log2", _F), ("stamps", _P), ("sinks", _P), ("cap_log2", _F),
-                ("cap_inv", _F), ("keep_first", _I)]
+                ("cap_inv", _F), ("keep_first", _I), ("chunk", _I)]
 
 
 DECODE_TMA_STAMPS: Optional[torch.Tensor] = None      # int64 [blocks, 12] for tuning, or None
@@ -1368,7 +1486,8 @@ def attn_decode_tma(q, k_pages, v_pages, block_table, *, slots, kv_len, page: in
                     max_kv_len: int, window: Optional[int] = None,
                     n_splits: Optional[int] = None, stages: int = 0,
                     softcap: Optional[float] = None,
-                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
+                    chunk: int = 0) -> torch.Tensor:
     """Attention of one new token per sequence over its cached keys, the tiles
     brought in by TMA and the splits combined by the block that finishes last (one
     launch).  Heads of 64 or 128, pages of 64 tokens."""
@@ -1386,7 +1505,7 @@ def attn_decode_tma(q, k_pages, v_pages, block_table, *, slots, kv_len, page: in
     stages = int(stages or DECODE_TMA_STAGES) or (2 if B * nkv < DECODE_TMA_DEEP_PAIRS else 3)
     per_sm = {2: 3, 3: 2, 4: 1}.get(stages, 2) if D == 128 else 3
     ns = int(n_splits) if n_splits else decode_tma_splits(
-        B, nkv, _keys_visited(max_kv_len, window, page, keep_first), q.device, per_sm)
+        B, nkv, _keys_visited(max_kv_len, window, page, keep_first, chunk), q.device, per_sm)
     out = torch.empty_like(q)
     a = _DecodeTmaArgs()
     if ns > 1:
@@ -1404,7 +1523,7 @@ def attn_decode_tma(q, k_pages, v_pages, block_table, *, slots, kv_len, page: in
     a.n_seqs, a.nq, a.nkv, a.max_pages = B, nq, nkv, block_table.shape[1]
     a.window, a.n_splits, a.scale_log2 = int(window or 0), ns, float(scale) * _LOG2E
     a.stamps = _ptr(DECODE_TMA_STAMPS)
-    a.keep_first = int(keep_first or 0)
+    a.keep_first, a.chunk = int(keep_first or 0), _chunk_arg(chunk, keep_first)
     _set_cap_and_sinks(a, scale, softcap, sinks, nq)
     with torch.cuda.device(q.device):
         _check(_fn("attn_decode_tma", "gb_attn_decode_tma", "pplpiiip")(
@@ -1416,16 +1535,19 @@ def attn_decode_tma(q, k_pages, v_pages, block_table, *, slots, kv_len, page: in
 # ---------------------------------------------------------------- attention dispatch
 def attention(q, k_pages, v_pages, block_table, *, step, page: int, scale: float,
               window: Optional[int] = None, softcap: Optional[float] = None,
-              sinks: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+              sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
+                    chunk: int = 0) -> torch.Tensor:
     """Attention of the step's queries over their sequences' cached keys.
     32-bit tensors take the plain 32-bit kernel; bfloat16 takes the tensor-core
     kernels where they accept the shape and the plain kernel elsewhere.
     ``softcap`` c: scores become c * tanh(score / c); ``sinks`` [nq] float32: one
     more term exp(sinks[h]) in the denominator of query head h; ``keep_first`` F: with a
-    window, key j < F stays visible to every later query (at its own position)."""
+    window, key j < F stays visible to every later query (at its own position); ``chunk`` C: a
+    query at position p sees the keys of its own chunk only, j // C == p // C (positions count
+    from the sequence's start)."""
     _T, nq, D = q.shape
     keep_first = int(keep_first or 0) if window else 0
-    extra = dict(softcap=softcap, sinks=sinks, keep_first=keep_first)
+    extra = dict(softcap=softcap, sinks=sinks, keep_first=keep_first, chunk=chunk)
     if q.dtype == torch.bfloat16 and fast_attention_takes(D, nq, k_pages.shape[1], page):
         nkv = k_pages.shape[1]
         if step.decode and attn_decode_tma_takes(D, nq, nkv, page) and (
@@ -1449,7 +1571,31 @@ def attention(q, k_pages, v_pages, block_table, *, step, page: int, scale: float
                                  page=page, scale=scale, window=window, **extra)
     return attn_generic(q, k_pages, v_pages, block_table, token_seq=step.token_seq,
                         token_pos=step.token_pos, slots=step.slots, page=page, scale=scale,
-                        window=window, softcap=softcap, sinks=sinks, keep_first=keep_first)
+                        window=window, **extra)
+
+
+# ---------------------------------------------------------------- differential attention
+class _DiffHeadsArgs(ctypes.Structure):
+    _fields_ = [("x", _P), ("out", _P), ("n_rows", _I), ("heads", _I), ("Ds", _I), ("Dv", _I),
+                ("lam", _F), ("eps", _F), ("mult", _F)]
+
+
+@_profiled("diff_heads", lambda out, x, v_dim, *a: (2 * _nbytes(out) + _nbytes(out), 0))
+def diff_heads(x: torch.Tensor, v_dim: int, lam: float, eps: float, mult: float) -> torch.Tensor:
+    """x [T, 2 heads, Ds], the outputs of a head's two attention maps side by side, ->
+    [T, heads * v_dim]: per head o = map 1 - lam * map 2 over the first ``v_dim`` elements, then
+    o / sqrt(mean(o^2) + eps) * mult (32-bit)."""
+    _need(x, "the maps' outputs", ndim=3)
+    T, n2, Ds = x.shape
+    if n2 % 2 or v_dim > Ds:
+        raise KernelError(f"{tuple(x.shape)} does not hold two maps a head of {v_dim} elements")
+    out = torch.empty((T, n2 // 2 * v_dim), dtype=x.dtype, device=x.device)
+    a = _DiffHeadsArgs()
+    a.x, a.out, a.n_rows, a.heads, a.Ds, a.Dv = x.data_ptr(), out.data_ptr(), T, n2 // 2, Ds, int(v_dim)
+    a.lam, a.eps, a.mult = float(lam), float(eps), float(mult)
+    _check(_fn("diff_heads", f"gb_diff_heads_{_suffix(x.dtype)}", "pp")(ctypes.addressof(a), _stream()),
+           "diff_heads")
+    return out
 
 
 # ---------------------------------------------------------------- gated delta rule
@@ -1549,7 +1695,8 @@ class _RetentionArgs(ctypes.Structure):
                 ("slots", _P), ("state", _P), ("state_stride", _L), ("qk", _P), ("o", _P), ("chunk_state", _P),
                 ("y", _P),
                 ("n_tokens", _I), ("n_seqs", _I), ("H", _I), ("dk", _I), ("dv", _I), ("rot_dim", _I),
-                ("k_scale", _F), ("norm_eps", _F), ("max_rows", _I)]
+                ("k_scale", _F), ("norm_eps", _F), ("max_rows", _I), ("silu", _I), ("joint_norm", _I),
+                ("norm_w", _P), ("v", _P)]
 
 
 RETENTION_CHUNK = 64         # rows of a chunk of the kernel's chunked form
@@ -1567,13 +1714,16 @@ def _cost_retention(out, proj, state, *a, H, dk, dv, **k):
 def retention_forward(proj: torch.Tensor, state: torch.Tensor, decay: torch.Tensor,
                       inv_freq: Optional[torch.Tensor], *, H: int, dk: int, dv: int, rot_dim: int,
                       k_scale: float, norm_eps: float, token_pos, cu_q, slots,
-                      dtype: torch.dtype, max_rows: Optional[int] = None) -> torch.Tensor:
+                      dtype: torch.dtype, max_rows: Optional[int] = None, silu: bool = False,
+                      joint_norm: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Retention on the rows of a step.  ``proj`` [T, 2 H dk + 2 H dv] 32-bit: the columns
     q | k | v | gate of the mixer's one projection; ``state`` [slots, H dk dv] 32-bit, updated
     in place for the sequences whose slot is not negative; ``decay`` [H] 32-bit; ``inv_freq``
     [rot_dim / 2] the rotation's frequencies (element i of a head goes with element
     i + rot_dim / 2).  Returns y [T, H dv] in ``dtype``: every head's read-out S^T q,
     divided by its root mean square over dv (``norm_eps`` under the root), times silu(gate).
+    ``silu``: q, k and v pass x sigmoid(x) (and nothing turns); ``joint_norm`` [H dv] 32-bit: the
+    read-outs of all heads are normalised together, times this weight and sigmoid(gate).
     ``max_rows``: the most rows any sequence of the step brings, when the caller knows it (a
     step of one row a sequence is one kernel; a step with a sequence of many rows runs all
     chunks of 64 rows side by side and joins them through the states at their starts)."""
@@ -1607,12 +1757,23 @@ def retention_forward(proj: torch.Tensor, state: torch.Tensor, decay: torch.Tens
     a.n_tokens, a.n_seqs, a.H, a.dk, a.dv, a.rot_dim = T, n_seqs, H, dk, dv, int(rot_dim)
     a.k_scale, a.norm_eps = float(k_scale), float(norm_eps)
     a.max_rows = int(max_rows) if max_rows else 0
+    if silu:
+        if rot_dim:
+            raise KernelError("activated queries and keys do not turn")
+        values = torch.empty((T, H * dv), dtype=torch.float32, device=dev)
+        a.silu, a.v = 1, values.data_ptr()
+    if joint_norm is not None:
+        _need(joint_norm, "norm weight", torch.float32, 1)
+        if joint_norm.shape[0] != H * dv:
+            raise KernelError(f"the norm weight has {joint_norm.shape[0]} elements, expected {H * dv}")
+        a.joint_norm, a.norm_w = 1, joint_norm.data_ptr()
     chunked = a.max_rows >= RETENTION_CHUNK_MIN
     if chunked:   # one matrix a head for every chunk of every sequence
         chunk_state = torch.empty((T // RETENTION_CHUNK + n_seqs, H * dk * dv), dtype=torch.float32, device=dev)
         a.chunk_state = chunk_state.data_ptr()
     _check(_fn("retention", f"gb_retention_forward_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
-           "retention_forward", 1 if a.max_rows == 1 and dv <= 256 else 5 if chunked else 3)
+           "retention_forward", (2 if a.joint_norm else 1) if a.max_rows == 1 and dv <= 256
+           else 5 if chunked else 3)
     return y
 
 
@@ -1788,7 +1949,8 @@ class _MoeArgs(ctypes.Structure):
                 ("offsets", _P), ("perm", _P), ("act", _P), ("out", _P), ("T", _I), ("W", _I),
                 ("F", _I), ("E", _I), ("n_identity", _I), ("top", _I), ("n_groups", _I),
                 ("keep_groups", _I), ("limit", _F), ("slope", _F), ("score_fn", _I),
-                ("weigh_input", _I), ("up_offset", _F), ("router_bias", _P)]
+                ("weigh_input", _I), ("up_offset", _F), ("router_bias", _P), ("group_top2", _I),
+                ("normalize", _I), ("weight_scale", _F)]
 
 
 _MOE_COUNTS = {}
@@ -1797,18 +1959,19 @@ MOE_SCORE_FNS = {"softmax": 0, "sigmoid": 1, "softmax_top": 2}     # the route k
 
 def _cost_moe(out, x, router_w, correction, w_gate, w_up, w_down, *, top, **k):
     T, W = x.shape
-    E, F = w_gate.shape[0], w_gate.shape[1]
-    used = min(E, T * top)
-    return (_nbytes(x, out) + used * 3 * F * W * w_gate.element_size(), 6.0 * T * top * F * W)
+    E, F = w_up.shape[0], w_up.shape[1]
+    used, mats = min(E, T * top), 2 if w_gate is None else 3
+    return (_nbytes(x, out) + used * mats * F * W * w_up.element_size(), 2.0 * mats * T * top * F * W)
 
 
 @_profiled("moe_forward", _cost_moe)
 def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[torch.Tensor],
-                w_gate: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, *, top: int,
+                w_gate: Optional[torch.Tensor], w_up: torch.Tensor, w_down: torch.Tensor, *, top: int,
                 n_identity: int = 0, n_groups: int = 1, keep_groups: int = 1,
                 limit: float = math.inf, slope: float = 1.0, score_fn: str = "softmax",
                 weigh_input: bool = False, up_offset: float = 1.0, want_choice: bool = False,
-                router_bias: Optional[torch.Tensor] = None):
+                router_bias: Optional[torch.Tensor] = None, group_top2: bool = False,
+                normalize: bool = False, weight_scale: float = 1.0, extra: int = 0):
     """A feed-forward of routed experts on rows x [T, W] -> 32-bit partial sums
     [top, T, W], choice j of every token in [j], already weighted; their sum is the
     feed-forward's output.  ``router_w`` [E + n_identity, W] and ``correction`` are
@@ -1819,7 +1982,10 @@ def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[to
     logits alone; ``router_bias`` (32-bit) is added to the logits;
     ``correction`` may be None; ``weigh_input`` multiplies the expert's input, not its
     result, by the weight; an expert is Wd (g sigmoid(slope g) (u + up_offset)) with g
-    and u clamped at ``limit``.
+    and u clamped at ``limit``; without ``w_gate`` it is Wd max(u, 0)^2.  ``group_top2``: a
+    group's score is the sum of its two largest choice scores, not its largest; ``normalize``: the
+    chosen outputs' weights are divided by their sum; ``weight_scale`` multiplies the weights.
+    ``extra``: that many more [T, W] terms are appended to the result for the caller to fill.
     With ``want_choice`` also returns (ids [T, top] int32, weights [T, top])."""
     _need(x, "activations", ndim=2)
     T, W = x.shape
@@ -1833,10 +1999,11 @@ def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[to
         if router_bias.shape[0] != router_w.shape[0]:
             raise KernelError("the router's bias and its weight do not fit together")
     for t, nm in ((w_gate, "gate weights"), (w_up, "up weights"), (w_down, "down weights")):
-        _need(t, nm, x.dtype, 3)
-    E, F = w_gate.shape[0], w_gate.shape[1]
+        if t is not None or nm != "gate weights":
+            _need(t, nm, x.dtype, 3)
+    E, F = w_up.shape[0], w_up.shape[1]
     n_all = E + n_identity
-    if tuple(w_gate.shape) != (E, F, W) or tuple(w_up.shape) != (E, F, W) or \
+    if (w_gate is not None and tuple(w_gate.shape) != (E, F, W)) or tuple(w_up.shape) != (E, F, W) or \
             tuple(w_down.shape) != (E, W, F) or tuple(router_w.shape) != (n_all, W) or \
             (correction is not None and correction.shape[0] != n_all):
         raise KernelError("the experts' weights, the router and the correction do not fit together")
@@ -1847,20 +2014,21 @@ def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[to
     offsets = torch.empty((E + 1,), dtype=torch.int32, device=dev)
     perm = torch.empty((T * top,), dtype=torch.int32, device=dev)
     act = torch.empty((T * top, F), dtype=x.dtype, device=dev)
-    out = torch.empty((top, T, W), dtype=torch.float32, device=dev)
+    out = torch.empty((top + extra, T, W), dtype=torch.float32, device=dev)
     key = (dev.index or 0, E)
     counts = _MOE_COUNTS.get(key)      # zero between calls: the kernels leave it so
     if counts is None:
         counts = _MOE_COUNTS[key] = torch.zeros((E + 1,), dtype=torch.int32, device=dev)
     a = _MoeArgs()
     a.x, a.router_w, a.correction = x.data_ptr(), router_w.data_ptr(), _ptr(correction)
-    a.w_gate, a.w_up, a.w_down = w_gate.data_ptr(), w_up.data_ptr(), w_down.data_ptr()
+    a.w_gate, a.w_up, a.w_down = _ptr(w_gate), w_up.data_ptr(), w_down.data_ptr()
     a.ids, a.wts, a.rank, a.counts = ids.data_ptr(), wts.data_ptr(), rank.data_ptr(), counts.data_ptr()
     a.offsets, a.perm, a.act, a.out = offsets.data_ptr(), perm.data_ptr(), act.data_ptr(), out.data_ptr()
     a.T, a.W, a.F, a.E, a.n_identity, a.top = T, W, F, E, int(n_identity), int(top)
     a.n_groups, a.keep_groups, a.limit, a.slope = int(n_groups), int(keep_groups), float(limit), float(slope)
     a.score_fn, a.weigh_input, a.up_offset = MOE_SCORE_FNS[score_fn], int(weigh_input), float(up_offset)
     a.router_bias = _ptr(router_bias)
+    a.group_top2, a.normalize, a.weight_scale = int(group_top2), int(normalize), float(weight_scale)
     _check(_fn("moe", f"gb_moe_forward_{_suffix(x.dtype)}", "pp")(ctypes.addressof(a), _stream()),
            "moe_forward", 3)
     return (out, ids, wts) if want_choice else out

@@ -195,15 +195,25 @@ class RoutedExperts(FeedForward):
         ``weigh_input``: the weight multiplies the expert's input instead of its
         result, out = sum of expert(s x)
 
+    ``gated`` False: an expert has no gate, y = Wd max(Wu x, 0)^2 (then ``limit`` and
+    ``gate_slope`` have nothing to act on); ``group_score`` "top2": a group's score is the sum
+    of its two largest c; ``normalize``: the weights are the chosen outputs' s divided by their
+    sum (+ 1e-20); ``weight_scale`` multiplies the weights.  ``shared_intermediate``: one more
+    ungated expert of that size, ``shared.up`` / ``shared.down``, that runs for every token
+    with weight 1.
+
     Tensors: ``router`` [n_experts + n_identity, hidden], ``correction``, and per
     expert j ``e<j>.gate`` / ``e<j>.up`` [intermediate, hidden], ``e<j>.down``.  The
-    result leaves as ``top`` weighted 32-bit partial sums, which the next norm adds."""
+    result leaves as ``top`` weighted 32-bit partial sums (and the shared expert's behind
+    them), which the next norm adds."""
 
     def __init__(self, ctx: BuildContext, hidden: int, intermediate: int, n_experts: int, top: int,
-                 limit: Optional[float], gate_slope: float, n_identity: int = 0, n_groups: int = 1,
+                 limit: Optional[float] = None, gate_slope: float = 1.0, n_identity: int = 0, n_groups: int = 1,
                  keep_groups: int = 1, score_fn: str = "softmax", correction: bool = True,
                  weigh_input: bool = False, up_offset: float = 1.0, router_bias: bool = False,
-                 router_bias_name: str = "router.b"):
+                 router_bias_name: str = "router.b", gated: bool = True, group_score: str = "max",
+                 normalize: bool = False, weight_scale: float = 1.0,
+                 shared_intermediate: Optional[int] = None):
         super().__init__(ctx)
         self.hidden, self.intermediate = int(hidden), int(intermediate)
         self.E, self.n_identity, self.top = int(n_experts), int(n_identity), int(top)
@@ -215,6 +225,13 @@ class RoutedExperts(FeedForward):
         self.score_fn, self.has_correction, self.weigh_input = score_fn, bool(correction), bool(weigh_input)
         self.has_router_bias, self.router_bias_name = bool(router_bias), router_bias_name
         self.router_b = None
+        if group_score not in ("max", "top2"):
+            raise ValueError(f"group score '{group_score}': 'max' or 'top2'")
+        self.gated, self.group_top2 = bool(gated), group_score == "top2"
+        self.normalize, self.weight_scale = bool(normalize), float(weight_scale)
+        self.shared = (ReluSquaredMLP(ctx, hidden, int(shared_intermediate),
+                                      names={"up": "shared.up", "down": "shared.down"})
+                       if shared_intermediate else None)
         n_all = self.E + self.n_identity
         if n_all % self.n_groups or not 1 <= self.keep_groups <= self.n_groups:
             raise ValueError(f"{n_all} router outputs do not form {self.n_groups} equal groups "
@@ -231,10 +248,16 @@ class RoutedExperts(FeedForward):
         if self.has_router_bias:
             specs[self.router_bias_name] = ParamSpec((n_all,), "offset")
         for j in range(self.E):
-            specs[f"e{j}.gate"] = ParamSpec((self.intermediate, self.hidden))
+            if self.gated:
+                specs[f"e{j}.gate"] = ParamSpec((self.intermediate, self.hidden))
             specs[f"e{j}.up"] = ParamSpec((self.intermediate, self.hidden))
             specs[f"e{j}.down"] = ParamSpec((self.hidden, self.intermediate))
+        if self.shared:
+            specs.update(self.shared.param_specs())
         return specs
+
+    def children(self):
+        return (self.shared,) if self.shared else ()
 
     def load(self, params):
         # the router is 32-bit whatever the checkpoint stores
@@ -244,7 +267,10 @@ class RoutedExperts(FeedForward):
                          if self.has_router_bias else None)
         stack = lambda what: torch.stack([params[f"e{j}.{what}"] for j in range(self.E)]).to(
             self.ctx.dtype).contiguous()
-        self.w_gate, self.w_up, self.w_down = stack("gate"), stack("up"), stack("down")
+        self.w_gate = stack("gate") if self.gated else None
+        self.w_up, self.w_down = stack("up"), stack("down")
+        if self.shared:
+            self.shared.load({n: params[n] for n in self.shared.param_specs()})
 
     def kernel_modules(self):
         return ("moe",)
@@ -253,9 +279,15 @@ class RoutedExperts(FeedForward):
         return True
 
     def forward(self, x, step):
-        return ops.moe_forward(x, self.router_w, self.correction, self.w_gate, self.w_up,
-                               self.w_down, top=self.top, n_identity=self.n_identity,
-                               n_groups=self.n_groups, keep_groups=self.keep_groups,
-                               limit=self.limit, slope=self.gate_slope, score_fn=self.score_fn,
-                               weigh_input=self.weigh_input, up_offset=self.up_offset,
-                               router_bias=self.router_b)
+        # the shared expert leaves its 32-bit sums behind the routed ones
+        extra = self.shared.down.n_parts(x.shape[0]) if self.shared else 0
+        out = ops.moe_forward(x, self.router_w, self.correction, self.w_gate, self.w_up, self.w_down,
+                              top=self.top, n_identity=self.n_identity, n_groups=self.n_groups,
+                              keep_groups=self.keep_groups, limit=self.limit, slope=self.gate_slope,
+                              score_fn=self.score_fn, weigh_input=self.weigh_input,
+                              up_offset=self.up_offset, router_bias=self.router_b,
+                              group_top2=self.group_top2, normalize=self.normalize,
+                              weight_scale=self.weight_scale, extra=extra)
+        if self.shared:
+            self.shared.down(self.shared.up.relu_squared(x), into=out[self.top:])
+        return out

@@ -57,14 +57,18 @@ class Linear:
         return mods
 
     def __call__(self, x: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-                 partial_ok: bool = False) -> torch.Tensor:
-        """``partial_ok``: the caller hands the result to a kernel that can add
+                 partial_ok: bool = False, into: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``into``: a contiguous 32-bit tensor for the result ([``n_parts(M)``, M, N]; implies
+        32-bit partial sums).  ``partial_ok``: the caller hands the result to a kernel that can add
         32-bit partial sums (a norm's residual add, the q/k preparation); a product
         with few rows and few tiles may then come back as [S, M, N] float32, its
         split-K reduction left to that kernel."""
-        out_dtype = out_dtype or x.dtype
+        out_dtype = torch.float32 if into is not None else (out_dtype or x.dtype)
+        partial_ok = partial_ok or into is not None
         w = self.weight
         if w.dtype == torch.float32:
+            if into is not None:
+                return ops.gemm_f32(ops.cast(x, torch.float32), w, into=into)
             y = ops.gemm_f32(ops.cast(x, torch.float32), w)
             return ops.cast(y, out_dtype)
         if x.dtype != torch.bfloat16:
@@ -73,16 +77,25 @@ class Linear:
         if self.in_features % 8 == 0:
             if M <= ops.SKINNY_MAX_ROWS:
                 if self.decode_kernel == "tc":
-                    return ops.gemm_tc_bf16(x, w, out_dtype, swap=True, split_out=partial_ok)
-                return ops.gemm_skinny_bf16(x, w, out_dtype)
+                    return ops.gemm_tc_bf16(x, w, out_dtype, swap=True, split_out=partial_ok, into=into)
+                return ops.gemm_skinny_bf16(x, w, out_dtype, into=into)
             if self.prefill_kernel == "tc":
-                return ops.gemm_tc_bf16(x, w, out_dtype, swap=False)
+                return ops.gemm_tc_bf16(x, w, out_dtype, swap=False, into=into)
             if ops.gemm_tc2_takes(self.out_features, out_dtype) and (
                     self.prefill_kernel == "pair" or
                     (self.prefill_kernel == "auto" and
                      ops.gemm_tc2_pays(M, self.out_features, x.device, fused_silu=False))):
-                return ops.gemm_tc2_bf16(x, w, out_dtype)
-        return ops.library_mm(x, w, out_dtype)
+                return ops.gemm_tc2_bf16(x, w, out_dtype, into=into)
+        return ops.library_mm(x, w, out_dtype, into=into)
+
+    def n_parts(self, M: int) -> int:
+        """How many 32-bit partial sums the product with M rows makes when it is asked to
+        leave them (``partial_ok``): 1 where it leaves its finished sum."""
+        w = self.weight
+        if (w.dtype == torch.bfloat16 and self.in_features % 8 == 0 and M <= ops.SKINNY_MAX_ROWS
+                and self.decode_kernel == "tc"):
+            return max(1, ops.gemm_tc_parts(M, self.out_features, self.in_features, w.device))
+        return 1
 
     def silu_mul(self, x: torch.Tensor, interleave: int, activation: str = "silu",
                  bias: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -65,7 +65,12 @@ class GQAAttention(Mixer):
     are then as wide as the larger of the two, filled up with zeros, and the o
     projection's columns likewise, so that every attention kernel serves.
     ``keep_first`` F: with a window, the sequence's first F tokens stay visible to every
-    later query, at their own positions (their pages are kept).  ``head_gate``: every
+    later query, at their own positions (their pages are kept).  ``chunk`` C: position i sees
+    keys of its own chunk only, j // C == i // C.  ``shares_kv``: the layer has no key and value
+    projections and attends over the keys and values that another layer has stored (its cache
+    is given by the schedule), with queries, window and all else of its own;  ``reach``: how far
+    back the layers that read this one's cache look, when that is further than its own window
+    (a number of keys, or None: all of them).  ``head_gate``: every
     head's output is multiplied by sigmoid(Wg h)_head, one number a head (tensor ``g``
     [heads, hidden]; 32-bit sums, 32-bit sigmoid), before the o projection.  A rotation
     of neighbouring pairs (``rotary_interleaved``) is folded into the q/k kernel as the
@@ -88,8 +93,14 @@ class GQAAttention(Mixer):
                  shares_kv: bool = False, softcap: Optional[float] = None, sinks: bool = False,
                  values_are_keys: bool = False, names: Optional[dict] = None,
                  v_head_dim: Optional[int] = None, q_temp: Optional[tuple] = None,
-                 sink_logit: Optional[float] = None, keep_first: int = 0, head_gate: bool = False):
+                 sink_logit: Optional[float] = None, keep_first: int = 0, head_gate: bool = False,
+                 chunk: Optional[int] = None, reach: Optional[int] = 0):
         super().__init__(ctx)
+        self.chunk = int(chunk or 0)
+        # the keys that must stay in the cache: this layer's window or what its readers need
+        self.kept_window = None if window is None or reach is None else max(int(window), int(reach))
+        if self.chunk and (keep_first or reach != 0):
+            raise ValueError("chunks go with neither kept first keys nor readers of another reach")
         self.keep_first = int(keep_first or 0) if window else 0
         self.head_gate = bool(head_gate)
         self.beside = False          # set by a SideBySide parent before load
@@ -101,9 +112,8 @@ class GQAAttention(Mixer):
         # the width of a cached row, of a query and of the attention's output
         self.Ds = max(self.D, self.Dv)
         if self.Ds != self.D or self.Ds != self.Dv:
-            if values_are_keys or shares_kv:
-                raise ValueError("values of another size than the keys go with a v projection "
-                                 "and a cache of the layer's own")
+            if values_are_keys:
+                raise ValueError("values of another size than the keys go with a v projection")
             if ctx.dtype == torch.bfloat16:       # the tensor-core kernels take multiples of 16
                 self.Ds = (self.Ds + 15) // 16 * 16
         self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp else None
@@ -191,9 +201,8 @@ class GQAAttention(Mixer):
     def cache_spec(self):
         if self.shares_kv:
             return None
-        if self.keep_first:
-            return KVSpec(self.nkv, self.Ds, self.window, keep_first=self.keep_first)
-        return KVSpec(self.nkv, self.Ds, self.window)
+        return KVSpec(self.nkv, self.Ds, self.kept_window, keep_first=self.keep_first,
+                      chunk=self.chunk or None)
 
     # -- beside another mixer ------------------------------------------------
     @property
@@ -238,19 +247,20 @@ class GQAAttention(Mixer):
             raise ValueError("a position encoding with arithmetic of its own goes with neither "
                              "values of another size nor a query temperature")
         # the q/k preparation can add the partial sums of a split-K projection itself
-        qkv = self.qkv(x, partial_ok=fused and x.dtype == torch.bfloat16 and not self.shares_kv)
+        qkv = self.qkv(x, partial_ok=fused and x.dtype == torch.bfloat16)
+        seen = dict(step=step, page=cache.page, scale=self.scale, window=self.window, softcap=self.softcap,
+                    sinks=self.sink, keep_first=self.keep_first, chunk=self.chunk)
         if self.shares_kv:
-            q, _ = ops.qk_prepare(qkv, self.nq, 0, self.D, q_w=self.q_norm_w,
+            q, _ = ops.qk_prepare(qkv, self.nq, 0, self.D, row_width=self.Ds, q_w=self.q_norm_w,
                                   eps=self.qk_norm_eps or 0.0,
                                   inv_freq=rot.inv_freq if rot else None,
                                   rot_dim=rot.rot_dim if rot else 0, token_seq=step.token_seq,
                                   token_pos=step.token_pos, slots=step.slots, q_temp=self.q_temp,
-                                  interleaved=bool(rot and rot.interleaved))
+                                  interleaved=bool(rot and rot.interleaved),
+                                  rot_scale=rot.amplitude if rot else 1.0)
             if rot is None:
                 q, _k = self.position.apply_qk(q, q[:, :0], step.token_pos)
-            return ops.attention(q.contiguous(), cache.k_pages, cache.v_pages, cache.block_table,
-                                 step=step, page=cache.page, scale=self.scale, window=self.window,
-                                 softcap=self.softcap, sinks=self.sink, keep_first=self.keep_first)
+            return ops.attention(q.contiguous(), cache.k_pages, cache.v_pages, cache.block_table, **seen)
         common = dict(q_w=self.q_norm_w, k_w=self.k_norm_w, eps=self.qk_norm_eps or 0.0,
                       values_are_keys=self.values_are_keys, token_seq=step.token_seq, token_pos=step.token_pos, slots=step.slots)
         if fused:
@@ -260,7 +270,7 @@ class GQAAttention(Mixer):
                                   block_table=cache.block_table, k_pages=cache.k_pages,
                                   v_pages=cache.v_pages, page=cache.page, v_dim=self.Dv,
                                   q_temp=self.q_temp, interleaved=bool(rot and rot.interleaved),
-                                  **common)
+                                  rot_scale=rot.amplitude if rot else 1.0, **common)
         else:
             # a position encoding with its own arithmetic: normalise, hand q and k
             # over, then store
@@ -272,9 +282,104 @@ class GQAAttention(Mixer):
                          slots=step.slots, block_table=cache.block_table, k_pages=cache.k_pages,
                          v_pages=cache.v_pages, page=cache.page)
             q = q.contiguous()
-        return ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, step=step,
-                             page=cache.page, scale=self.scale, window=self.window,
-                             softcap=self.softcap, sinks=self.sink, keep_first=self.keep_first)
+        return ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, **seen)
+
+
+@register_part("mixer", "differential_attention")
+class DifferentialAttention(Mixer):
+    """Attention with two maps a head over the same values, the second subtracted from the
+    first.  With h the mixer's input,
+
+        q = Wq h  (n_heads x [map 1 | map 2] x head_dim),  k = Wk h  (n_kv_heads x 2 x head_dim),
+        v = Wv h  (n_kv_heads x v_head_dim);   q and k of each map turned by ``position``
+        a_n = softmax(q_n . k_n * scale over the keys the query sees) v                   n = 1, 2
+        lambda = exp(sum(lq1 lk1)) - exp(sum(lq2 lk2)) + diff           (one number for the layer)
+        o = a_1 - lambda a_2;   o <- o / sqrt(mean(o^2) + norm_eps) * (1 - diff)         per head
+        y = Wo [ o ]
+
+    A query sees the keys of its own chunk of ``chunk`` positions (counted from the sequence's
+    start; None: no chunks), the last ``window`` of them if given; query head i reads kv head
+    i // (n_heads / n_kv_heads).
+
+    A cached key row holds both maps' keys of a kv head side by side, next to its one value; a
+    head's two queries become two query rows, each zero where the other map's key lies.  So
+    the attention kernels see 2 n_heads query heads on n_kv_heads kv heads, read every key and
+    value once for both maps, and know nothing of maps; one more kernel takes the difference,
+    the norm and the factor (32-bit).  ``names`` replaces local tensor names (keys q, k, v, o,
+    lq1, lk1, lq2, lk2)."""
+
+    NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "lq1": "lq1", "lk1": "lk1", "lq2": "lq2", "lk2": "lk2"}
+
+    def __init__(self, ctx: BuildContext, hidden: int, n_heads: int, n_kv_heads: int, head_dim: int,
+                 v_head_dim: int, position: PartSpec, scale: float, diff: float, norm_eps: float,
+                 chunk: Optional[int] = None, window: Optional[int] = None, names: Optional[dict] = None):
+        super().__init__(ctx)
+        if n_heads % n_kv_heads:
+            raise ValueError(f"{n_heads} heads cannot share {n_kv_heads} kv heads")
+        self.hidden, self.H, self.G = int(hidden), int(n_heads), int(n_kv_heads)
+        self.D, self.Dv = int(head_dim), int(v_head_dim)
+        self.scale, self.diff, self.norm_eps = float(scale), float(diff), float(norm_eps)
+        self.chunk, self.window = int(chunk or 0), (int(window) if window else None)
+        # the width of a cached row, of a query and of the attention's output
+        self.Ds = max(2 * self.D, self.Dv)
+        if ctx.dtype == torch.bfloat16:       # the tensor-core kernels take multiples of 16
+            self.Ds = (self.Ds + 15) // 16 * 16
+        self.names = dict(self.NAMES, **(names or {}))
+        self.position = build_part("position", position, ctx)
+        if self.position.rotary() is None and type(self.position).apply_qk is not PositionEncoding.apply_qk:
+            raise ValueError("differential attention takes a rotation (or no position encoding)")
+        self.qkv = self.o = None
+        self.lam = 0.0
+
+    def children(self):
+        return (self.position,)
+
+    def param_specs(self):
+        W, H, G, D, nm = self.hidden, self.H, self.G, self.D, self.names
+        specs = {nm["q"]: ParamSpec((H * 2 * D, W)), nm["k"]: ParamSpec((G * 2 * D, W)),
+                 nm["v"]: ParamSpec((G * self.Dv, W)), nm["o"]: ParamSpec((W, H * self.Dv))}
+        specs.update({nm[n]: ParamSpec((D,), "offset") for n in ("lq1", "lk1", "lq2", "lk2")})
+        return specs
+
+    def load(self, params):
+        nm = self.names
+        ws = [params[nm[k]] for k in ("q", "k", "v")]
+        if len({w.dtype for w in ws}) != 1:
+            raise ValueError("q, k and v projections must be stored in one dtype to be fused")
+        self.qkv = Linear(torch.cat(ws, dim=0), self.ctx.products)
+        self.o = Linear(params[nm["o"]], self.ctx.products)
+        # a constant of the layer once its tensors are known
+        dot = lambda a, b: float((params[nm[a]].double() * params[nm[b]].double()).sum())
+        self.lam = math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + self.diff
+
+    def kernel_modules(self):
+        mods = ("qk_prepare", "attn_generic", "diff_heads") + self.qkv.kernel_modules() + self.o.kernel_modules()
+        if self.ctx.dtype == torch.bfloat16:
+            mods += ops.fast_attention_modules(self.Ds, 2 * self.H, self.G)
+        return mods
+
+    def cache_spec(self):
+        return KVSpec(self.G, self.Ds, self.window, chunk=self.chunk or None)
+
+    def captures_prompts(self):
+        return True
+
+    def forward(self, x, step, cache):
+        if cache is None or cache.spec != self.cache_spec():
+            raise ValueError(f"differential attention with {self.G} kv heads of {self.Ds} was given the "
+                             f"cache {None if cache is None else cache.spec}")
+        rot = self.position.rotary()
+        qkv = self.qkv(x, partial_ok=x.dtype == torch.bfloat16)
+        q, _ = ops.qk_prepare(qkv, 2 * self.H, self.G, self.D, maps=2, v_dim=self.Dv,
+                              inv_freq=rot.inv_freq if rot else None, rot_dim=rot.rot_dim if rot else 0,
+                              interleaved=bool(rot and rot.interleaved), rot_scale=rot.amplitude if rot else 1.0,
+                              token_seq=step.token_seq, token_pos=step.token_pos, slots=step.slots,
+                              block_table=cache.block_table, k_pages=cache.k_pages, v_pages=cache.v_pages,
+                              page=cache.page)
+        maps = ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, step=step, page=cache.page,
+                             scale=self.scale, window=self.window, chunk=self.chunk)
+        y = ops.diff_heads(maps, self.Dv, self.lam, self.norm_eps, 1.0 - self.diff)
+        return self.o(y, partial_ok=True)
 
 
 @register_part("mixer", "side_by_side")

@@ -310,3 +310,47 @@ class LayerNorm(Norm):
                                  post_bias=post.bias if post else None,
                                  post_eps=post.eps if post else 0.0,
                                  post_center=post.center if post else True)
+
+
+@register_part("norm", "dynamic_tanh")
+class DynamicTanh(Norm):
+    """y = tanh(alpha * x) * w + b, alpha one number (tensor ``<name><alpha_suffix>``, a
+    scalar), w and b vectors: a norm without mean or variance, so no element depends on
+    another.  The sum into the stream, the tanh and the scaling are 32-bit and one kernel.
+    ``name``: the weight's local name; ``alpha_suffix`` and ``bias_suffix`` follow it."""
+
+    def __init__(self, ctx: BuildContext, dim: int, name: str = "weight",
+                 alpha_suffix: str = ".alpha", bias_suffix: str = ".b"):
+        super().__init__(ctx)
+        self.dim = int(dim)
+        self.names = (name, name + alpha_suffix, name + bias_suffix)
+        self.weight = self.alpha = self.bias = None
+
+    def param_specs(self):
+        w, alpha, b = self.names
+        return {w: ParamSpec((self.dim,), "vector"), alpha: ParamSpec((), "vector"),
+                b: ParamSpec((self.dim,), "offset")}
+
+    def load(self, params):
+        # 32-bit whatever the checkpoint stores: the norm's arithmetic is 32-bit
+        w, alpha, b = (params[n].float().contiguous() for n in self.names)
+        self.weight, self.alpha, self.bias = w, alpha.reshape(1), b
+
+    def kernel_modules(self):
+        return ("dyt",)
+
+    def captures_prompts(self):
+        return True
+
+    def forward(self, x):
+        _res, y = ops.add_dyt(None, x, self.alpha, self.weight, self.bias, dtype=self.ctx.dtype,
+                              write_res=False)
+        return y
+
+    def add_norm(self, res, delta, rows=None):
+        if isinstance(delta, Averaged):          # resolved step by step, then normalised
+            res, delta, rows = delta.resolve(res, rows), None, None
+        elif isinstance(delta, (Contribution, tuple, list)):
+            res, delta = residual_add(res, resolve_terms(delta)), None
+        return ops.add_dyt(res, delta, self.alpha, self.weight, self.bias, dtype=self.ctx.dtype,
+                           rows=rows)

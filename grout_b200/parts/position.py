@@ -14,6 +14,7 @@ An encoding that is added to the embeddings is not of this family: it is an
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Optional
 
@@ -28,6 +29,7 @@ class RotaryTable:
     inv_freq: torch.Tensor   # float32 [rot_dim / 2] on the device
     rot_dim: int
     interleaved: bool = False   # element 2j goes with 2j + 1 instead of j with j + rot_dim / 2
+    amplitude: float = 1.0      # factor of every sine and cosine
 
 
 class PositionEncoding(Part):
@@ -50,11 +52,18 @@ class NoPosition(PositionEncoding):
 
 
 def scaled_inverse_frequencies(rot_dim: int, theta: float, scaling: Optional[dict]) -> np.ndarray:
-    """theta^(-2j / rot_dim) for j < rot_dim / 2 in float64, with the band-wise
-    scaling of ``RotaryHalfSplit`` when ``scaling`` is given."""
+    """theta^(-2j / rot_dim) for j < rot_dim / 2 in float64, with one of the scalings of
+    ``RotaryHalfSplit`` when ``scaling`` is given."""
     j = np.arange(rot_dim // 2, dtype=np.float64)
     f = np.power(np.float64(theta), -2.0 * j / rot_dim)
-    if scaling:
+    if scaling and "fast" in scaling:
+        factor, original, fast, slow = (float(scaling[k]) for k in ("factor", "original", "fast", "slow"))
+        element = lambda turns: rot_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+        lo = max(math.floor(element(fast)), 0)
+        hi = min(math.ceil(element(slow)), rot_dim - 1)
+        ramp = np.clip((j - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+        f = f / factor * ramp + f * (1.0 - ramp)
+    elif scaling:
         factor, low, high, original = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
         wave = 2.0 * np.pi / f
         s = (original / wave - low) / (high - low)
@@ -75,8 +84,14 @@ class RotaryHalfSplit(PositionEncoding):
     rule that Llama 3.1 introduced): with wavelength l = 2 pi / f, a frequency
     with l < original / high stays, one with l > original / low becomes
     f / factor, and between the two f / factor and f are mixed with weights
-    1 - s and s, s = (original / l - low) / (high - low).  With ``scaling``, or
-    with ``exact_table``, the table is computed in float64 and rounded once."""
+    1 - s and s, s = (original / l - low) / (high - low).
+
+    ``scaling`` = dict(factor, original, fast, slow) is the rule named YaRN: with
+    e(t) = rot_dim ln(original / (2 pi t)) / (2 ln theta), the element that turns t times
+    within the original length, frequency j becomes f / factor * r + f (1 - r), r rising from
+    0 at element floor(e(fast)) to 1 at ceil(e(slow)) in a straight line, and every sine and
+    cosine is multiplied by 0.1 ln(factor) + 1 (``RotaryTable.amplitude``).  With ``scaling``,
+    or with ``exact_table``, the table is computed in float64 and rounded once."""
 
     def __init__(self, ctx: BuildContext, head_dim: int, theta: float,
                  rot_dim: Optional[int] = None, scaling: Optional[dict] = None,
@@ -93,8 +108,10 @@ class RotaryHalfSplit(PositionEncoding):
         self.scaling = dict(scaling) if scaling else None
         if self.scaling or exact_table:
             inv = scaled_inverse_frequencies(self.rot_dim, self.theta, self.scaling)
+        amplitude = (0.1 * math.log(float(self.scaling["factor"])) + 1.0
+                     if self.scaling and "fast" in self.scaling else 1.0)
         self._table = RotaryTable(torch.from_numpy(inv.astype(np.float32)).to(ctx.device),
-                                  self.rot_dim)
+                                  self.rot_dim, amplitude=amplitude)
 
     def rotary(self):
         return self._table

@@ -178,6 +178,72 @@ class Retention(Mixer):
         return self.o(y, partial_ok=True)
 
 
+@register_part("mixer", "lightning_attention")
+class LightningAttention(Mixer):
+    """Linear attention with a fixed decay per head, activated queries, keys and values, and
+    one norm over all heads.  With h the mixer's input,
+
+        q = silu(Wq h), k = silu(Wk h)  (n_heads x key_dim),  v = silu(Wv h)  (n_heads x value_dim)
+        S <- decay_i S + k v^T;  o = S^T q                                    per head i
+        y = Wo [ (all heads' o) / sqrt(mean(o^2) + norm_eps) * w * sigmoid(Wg h) ]
+
+    the mean over the n_heads * value_dim numbers of a token, w as long.  ``decay`` holds one
+    constant per head.  The state, the projections' product and the kernels are those of
+    ``Retention`` (which turns q and k, normalises every head by itself and gates by a silu);
+    all that lies between the projections' 32-bit sums and y is 32-bit.  ``names`` replaces
+    local tensor names (keys q, k, v, g, norm, o)."""
+
+    NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "norm": "norm", "o": "o"}
+
+    def __init__(self, ctx: BuildContext, hidden: int, n_heads: int, key_dim: int, value_dim: int,
+                 decay, norm_eps: float, names=None):
+        super().__init__(ctx)
+        self.hidden, self.H, self.dk, self.dv = int(hidden), int(n_heads), int(key_dim), int(value_dim)
+        self.decay_values = tuple(float(d) for d in decay)
+        if len(self.decay_values) != self.H:
+            raise ValueError(f"{len(self.decay_values)} decays for {self.H} heads")
+        self.norm_eps = float(norm_eps)
+        self.names = dict(self.NAMES, **(names or {}))
+        self.proj = self.o = self.decay = self.norm_w = None
+
+    def param_specs(self):
+        W, H, dk, dv, nm = self.hidden, self.H, self.dk, self.dv, self.names
+        return {nm["q"]: ParamSpec((H * dk, W)), nm["k"]: ParamSpec((H * dk, W)),
+                nm["v"]: ParamSpec((H * dv, W)), nm["g"]: ParamSpec((H * dv, W)),
+                nm["norm"]: ParamSpec((H * dv,), "vector"), nm["o"]: ParamSpec((W, H * dv))}
+
+    def load(self, params):
+        nm = self.names
+        ws = [params[nm[k]] for k in ("q", "k", "v", "g")]
+        if len({w.dtype for w in ws}) != 1:
+            raise ValueError("the projections of one mixer must be stored in one dtype to be fused")
+        self.proj = Linear(torch.cat(ws, dim=0), self.ctx.products)
+        self.o = Linear(params[nm["o"]], self.ctx.products)
+        self.norm_w = params[nm["norm"]].float().contiguous()
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=ws[0].device)
+
+    def kernel_modules(self):
+        return ("retention",) + self.proj.kernel_modules() + self.o.kernel_modules()
+
+    def cache_spec(self):
+        return StateSpec((self.H * self.dk * self.dv,), torch.float32)
+
+    def captures_prompts(self):
+        return True
+
+    def forward(self, x, step, cache):
+        if cache is None or tuple(cache.spec.shape) != tuple(self.cache_spec().shape):
+            raise ValueError(f"lightning attention was given the cache "
+                             f"{None if cache is None else cache.spec}")
+        proj = self.proj(x, out_dtype=torch.float32)
+        y = ops.retention_forward(proj, cache.state, self.decay, None, H=self.H, dk=self.dk, dv=self.dv,
+                                  rot_dim=0, k_scale=1.0, norm_eps=self.norm_eps,
+                                  token_pos=step.token_pos, cu_q=step.cu_q, slots=step.slots,
+                                  dtype=self.ctx.dtype, max_rows=step.max_q_len, silu=True,
+                                  joint_norm=self.norm_w)
+        return self.o(y, partial_ok=True)
+
+
 @register_part("mixer", "gated_linear_recurrence")
 class GatedLinearRecurrence(Mixer):
     """The recurrent block of Griffin: two branches of ``width`` channels,
