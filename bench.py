@@ -21,7 +21,7 @@ weights, far more than the 126 MB L2, so nothing is flushed between timed steps.
                                        decode steps (launched one by one, an event pair
                                        around each): calls, time, GB/s, TFLOP/s, fractions
     python bench.py --requests S       the reference's request grid
-    python bench.py --designs [--design suvazen|sonalorn|zutazen|mananex] [--design-sizes 1b,4b,8b] [--batch B] [--design-ops]
+    python bench.py --designs [--design suvazen|sonalorn|zutazen|mananex|kakotar] [--design-sizes 1b,4b,8b] [--batch B] [--design-ops]
                                        prefill and decode throughput of the Suvazen (or Sonalorn)
                                        design beside the Qwen3 decoder at equal layer sizes (random weights), and
                                        with --design-ops the per-kernel tables of both
@@ -247,6 +247,34 @@ def mananex_config(size: str) -> dict:
     return dict(architecture="Mananex", vocab=V, width=W, norm={"eps": 1e-6}, layers=layers)
 
 
+def kakotar_config(size: str) -> dict:
+    """The Kakotar model of a size: the width, heads, head size, layers and vocabulary of
+    the Qwen3 model; the layers mix in turn by differential attention in chunks of 1,280
+    (a token behind a prompt of 2,048 then sees 768 keys and more; the Qwen3 model's heads, two maps of half the head size over values of the head size),
+    by lightning attention (as many heads, keys and values of the head size, decays from
+    1 - 2^-5 to 1 - 2^-10), by attention over a window of 1,024 with a YaRN-stretched
+    rotation, and by attention over the keys and values of the layer before; every layer
+    routes two of eight experts (four groups of which two are kept) beside a shared one,
+    each of 3/8 the Qwen3 model's feed-forward rows (two matrices instead of three: the
+    weights of a gated expert of a quarter of the rows)."""
+    W, nq, nkv, D, I, L, V = DESIGN_SIZES[size]
+    ff = 3 * I // 8 // 64 * 64
+    diff = dict(heads=nq, kv_heads=nkv, dim=D // 2, vdim=D, scale=(D // 2) ** -0.5, diff=0.5, mask={"size": 1280},
+                rot={"base": 500000.0, "dims": D // 2,
+                     "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}})
+    light = dict(heads=nq, dim=D, vdim=D,
+                 decay=[1.0 - 2.0 ** (-5.0 - 5.0 * h / max(nq - 1, 1)) for h in range(nq)])
+    attn = dict(heads=nq, kv_heads=nkv, dim=D, vdim=D, scale=D ** -0.5, mask={"size": 1024},
+                rot={"base": 1000000.0, "dims": D,
+                     "scaling": {"factor": 4.0, "fast": 32.0, "slow": 1.0, "original": 8192}})
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": ff},
+           "router": {"experts": 8, "top": 2, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    kinds = lambda i: (("attention_2", diff), ("lightning", light), ("attention", attn),
+                       ("attention", dict(attn, kv_from=i - 1)))[i % 4]
+    layers = [dict(type=kinds(i)[0], mixer=kinds(i)[1], mlp=mlp) for i in range(L)]
+    return dict(architecture="Kakotar", vocab=V, width=W, norm={"eps": 1e-6}, layers=layers)
+
+
 def design_configs(size: str, design: str = "suvazen"):
     W, nq, nkv, D, I, L, V = DESIGN_SIZES[size]
     qwen = dict(QWEN3_4B, hidden_size=W, num_attention_heads=nq, num_key_value_heads=nkv, head_dim=D,
@@ -264,6 +292,8 @@ def design_configs(size: str, design: str = "suvazen"):
         return {"qwen3": qwen, "sonalorn": sonalorn_config(size), "zutazen": zutazen_config(size)}
     if design == "mananex":       # beside the attention model and beside the design with matrix states and experts
         return {"qwen3": qwen, "zutazen": zutazen_config(size), "mananex": mananex_config(size)}
+    if design == "kakotar":       # the same two: attention, and matrix states, windows and experts
+        return {"qwen3": qwen, "zutazen": zutazen_config(size), "kakotar": kakotar_config(size)}
     return {"qwen3": qwen, "suvazen": suv}
 
 
@@ -325,14 +355,19 @@ def run_designs(sizes, batch: int, steps: int, warm: int, with_ops: bool, pk,
             dec_ms = a.elapsed_time(b) / steps
             n_weights = sum(t.numel() for t in _weights_of(eng))
             stores = [x for st in eng.cache.stores for x in getattr(st, "stores", [st])]   # (a layer may have two needs)
-            kv_bytes = sum(st.k[:, :1].numel() * 2 * 2 // 64 for st in stores
-                           if hasattr(st, "k") and not st.spec.window)
-            # a window bounds the keys a step reads, whatever the sequence holds
-            win_bytes = sum(st.k[:, :1].numel() * 2 * 2 // 64 * (st.spec.window + st.spec.keep_first)
-                            for st in stores if hasattr(st, "k") and st.spec.window)
+            # every layer reads the keys and values its query sees once, those of another layer's
+            # cache too; a window or a chunk bounds them, whatever the sequence holds
+            layout, ctx_mid = eng.cache.layout, PROMPT + warm + steps / 2
+            kv_bytes = 0
+            for k, e in enumerate(eng.model.plan.schedule):
+                owner = k if e.cache_of is None else e.cache_of
+                if owner in layout.where:
+                    st = eng.cache.stores[layout.where[owner][0]]
+                    kv_bytes += sum(x.k[:1, :1].numel() * 2 * 2 // 64 * _keys_seen(x.spec, ctx_mid)
+                                    for x in getattr(st, "stores", [st]) if hasattr(x, "k"))
             # a recurrent mixer reads and writes its whole state every step
             state_bytes = sum(2 * st.state[:, :1].numel() * 4 for st in stores if hasattr(st, "state"))
-            step_bytes = 2 * n_weights + batch * ((PROMPT + warm + steps / 2) * kv_bytes + win_bytes + state_bytes)
+            step_bytes = 2 * n_weights + batch * (kv_bytes + state_bytes)
             out[size][design] = {
                 "prefill_ms": round(pre_ms, 3), "prefill_tok_s": round(PROMPT / pre_ms * 1e3, 1),
                 "decode_ms_per_step": round(dec_ms, 4), "decode_tok_s": round(batch / dec_ms * 1e3, 1),
@@ -379,6 +414,14 @@ def run_designs(sizes, batch: int, steps: int, warm: int, with_ops: bool, pk,
                       "prompt_len": PROMPT, "steps": steps, "warmup": warm, "peaks": pk["source"],
                       "sizes": out}))
     return 0
+
+
+def _keys_seen(spec, length: float) -> float:
+    """The keys that the last token of a sequence of ``length`` sees in this store: all of them, its
+    window with the first tokens the window keeps, or those of its chunk so far."""
+    if spec.window:
+        return min(length, spec.window + spec.keep_first)
+    return (length - 1) % spec.chunk + 1 if spec.chunk else length
 
 
 def _weights_of(eng):
@@ -500,9 +543,7 @@ def decode_timeline(eng, slots, V, g, pk, steps: int = 3) -> str:
         print(f"bench.py: {len(labels)} launches were logged for a step of {len(ev) // n} kernels; "
               f"rows are named by kernel", file=sys.stderr)
     kv_spec = next((x.spec for st in eng.cache.stores for x in getattr(st, "stores", [st]) if hasattr(x, "k")), None)
-    # (a window, with the first tokens it keeps, bounds the keys a step reads)
-    reach = kv_spec.window + kv_spec.keep_first if kv_spec is not None and kv_spec.window else None
-    kv = sum(min(eng.cache.length[s], reach) if reach else eng.cache.length[s] for s in slots)
+    kv = sum(int(_keys_seen(kv_spec, eng.cache.length[s])) if kv_spec is not None else 0 for s in slots)
 
     def must_read(name):
         """Bytes a call of this kernel has to read: a product its weights, the decode
@@ -558,7 +599,7 @@ def main() -> int:
     ap.add_argument("--designs", action="store_true",
                     help="instead of the default run: the Suvazen design beside the Qwen3 decoder at "
                          "equal layer sizes (--design-sizes), prefill and decode at --batch")
-    ap.add_argument("--design", default="suvazen", choices=["suvazen", "sonalorn", "zutazen", "mananex"],
+    ap.add_argument("--design", default="suvazen", choices=["suvazen", "sonalorn", "zutazen", "mananex", "kakotar"],
                     help="which design --designs sets beside Qwen3")
     ap.add_argument("--design-sizes", default="1b,4b,8b",
                     help=f"which of {sorted(DESIGN_SIZES)} --designs runs")
