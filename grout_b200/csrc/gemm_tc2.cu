@@ -26,7 +26,7 @@
 // No copy in this file is a multicast copy.  All waits are bounded (tc_common.cuh);
 // on expiry a block records a code in args.error and leaves; its partner's waits
 // run out the same way.
-#include "tc_common.cuh"
+#include "tc_pair.cuh"
 
 #define T2_BM 128      // rows of X per block (256 per pair)
 #define T2_BNH 128     // rows of W per block (256 per pair)
@@ -59,51 +59,6 @@ static constexpr int T2_STAGE_BYTES = T2_A_BYTES + T2_B_BYTES;
 static constexpr size_t T2_SMEM = (size_t)T2_STAGES * T2_STAGE_BYTES + 1024 + 256;
 // f32 accumulate, bf16 x bf16, both K-major, M = 256 (over the pair); N is added at run time
 static constexpr uint32_t T2_IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(256 >> 4) << 24);
-
-__device__ __forceinline__ uint32_t cluster_rank() {
-  uint32_t r;
-  asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
-  return r;
-}
-__device__ __forceinline__ void cluster_sync_all() {
-  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-// shared::cluster address of the same variable in block `rank` of the cluster
-__device__ __forceinline__ uint32_t map_to_rank(const void* p, uint32_t rank) {
-  uint32_t out;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(out) : "r"(smem_u32(p)), "r"(rank));
-  return out;
-}
-__device__ __forceinline__ void mbar_arrive_cluster(uint32_t cluster_addr) {
-  asm volatile("mbarrier.arrive.shared::cluster.b64 _, [%0];" ::"r"(cluster_addr) : "memory");
-}
-// A tile copy of one block of a pair whose bytes are counted on a barrier of the pair's first block
-__device__ __forceinline__ void tma_load_2d_pair(void* dst, const CUtensorMap* map, int x, int y,
-                                                 uint32_t bar_cluster_addr) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.cta_group::2.shared::cluster.global.mbarrier::complete_tx::bytes "
-      "[%0], [%1, {%3, %4}], [%2];" ::"r"(smem_u32(dst)),
-      "l"(map), "r"(bar_cluster_addr), "r"(x), "r"(y)
-      : "memory");
-}
-__device__ __forceinline__ void tc_mma_pair(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc,
-                                            uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n\t}" ::"r"(tmem_d),
-      "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-// Arrives (once the MMAs issued so far are complete) on the barrier at this
-// offset in both blocks of the pair.
-__device__ __forceinline__ void tc_commit_pair(void* bar) {
-  asm volatile(
-      "tcgen05.commit.cta_group::2.mbarrier::arrive::one.shared::cluster.multicast::cluster.b64 [%0], %1;" ::"r"(
-          smem_u32(bar)),
-      "h"((uint16_t)3)
-      : "memory");
-}
 
 // silu, (kind 3) the tanh form of gelu with tanh(x) = 1 - 2 / (e^2x + 1), or (kind 5) relu
 __device__ __forceinline__ float t2_gate(float g, int kind) {

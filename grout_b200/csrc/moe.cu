@@ -24,6 +24,10 @@
 // gate weights an expert is ungated, y = max(x Wu_e^T, 0)^2 Wd_e^T (no limit, slope or
 // offset).
 //
+// A shared expert (ungated, weights ws_up [Fs, W] and ws_down [W, Fs]) runs for every token with
+// weight 1 in the same two launches: its tiles come first in the tensor-core kernels' grid,
+// its rows are the tokens as they lie in x, its result is out[top, token, :].
+//
 // Nothing here needs the host to know how many tokens an expert got, so a step
 // can be captured: `route` chooses and counts, and its last block turns the counts into a
 // list of (token, choice) pairs ordered by expert; the two products walk
@@ -59,6 +63,11 @@ struct MoeArgs {
   int group_top2;            // a group's score is the sum of its two largest c, not its largest
   int normalize;             // the chosen outputs' weights are divided by their sum
   float weight_scale;        // and multiplied by this
+  const void* ws_up;         // [Fs, W] the shared expert, or null
+  const void* ws_down;       // [W, Fs]
+  void* act_s;               // [T, Fs] its inner activations
+  int Fs;
+  int route_only;            // stop behind `route` (the products are another source's kernels)
 };
 
 #define MOE_MAX_OUTPUTS 1024
@@ -201,18 +210,35 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
   __syncthreads();
   if (!is_last) return;
   __threadfence();
-  if (tid == 0) {          // few experts: a serial scan is shorter than its set-up
+  // (all counts are requested at once; the choices' shared memory holds them and their offsets)
+  int* cnt = reinterpret_cast<int*>(sm);               // [E]
+  int* off = cnt + a.E;                                // [E]
+  for (int e = tid; e < a.E; e += blockDim.x) cnt[e] = __ldcg(&a.counts[e]);
+  __syncthreads();
+  if (warp == 0) {                                     // exclusive sums, 32 experts a turn
     int run = 0;
-    for (int e = 0; e < a.E; ++e) { a.offsets[e] = run; run += __ldcg(&a.counts[e]); }
-    a.offsets[a.E] = run;
+    for (int e0 = 0; e0 < a.E; e0 += 32) {
+      const int c0 = e0 + lane < a.E ? cnt[e0 + lane] : 0;
+      int v = c0;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int u = __shfl_up_sync(0xffffffffu, v, o);
+        if (lane >= o) v += u;
+      }
+      if (e0 + lane < a.E) {
+        off[e0 + lane] = run + v - c0;
+        a.offsets[e0 + lane] = run + v - c0;
+      }
+      run += __shfl_sync(0xffffffffu, v, 31);
+    }
+    if (lane == 0) a.offsets[a.E] = run;
   }
   __syncthreads();
   const int n_pairs = a.T * a.top;
   for (int p = tid; p < n_pairs; p += blockDim.x) {
-    const int e = __ldcg(&a.ids[p]);
-    if (e < a.E) a.perm[a.offsets[e] + __ldcg(&a.rank[p])] = p;
+    const int e = __ldcg(&a.ids[p]), r = __ldcg(&a.rank[p]);
+    if (e < a.E) a.perm[off[e] + r] = p;
   }
-  __syncthreads();
   for (int e = tid; e <= a.E; e += blockDim.x) a.counts[e] = 0;
 }
 
@@ -403,19 +429,29 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
   __shared__ int src_row[BM];
   pdl_launch_dependents_if_small();
   pdl_wait();
-  int e, first, n_rows;
-  if (!moe_find_tile<BM>(a.offsets, a.E, blockIdx.x, e, first, n_rows)) return;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int K = UP ? a.W : a.F, N = UP ? a.F : a.W;
+  int e = 0, first, n_rows;
+  const int shared_tiles = a.Fs > 0 ? (a.T + BM - 1) / BM : 0;
+  const bool shared = (int)blockIdx.x < shared_tiles;      // a tile of the shared expert: tokens as they come
+  const int F = shared ? a.Fs : a.F;
+  const int K = UP ? a.W : F, N = UP ? F : a.W;
   const int n0 = blockIdx.y * BN;
+  if (n0 >= N) return;
+  if (shared) {
+    first = blockIdx.x * BM;
+    n_rows = min(BM, a.T - first);
+  } else if (!moe_find_tile<BM>(a.offsets, a.E, blockIdx.x - shared_tiles, e, first, n_rows)) {
+    return;
+  }
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   for (int i = tid; i < BM; i += NT) {
     int r = -1;
-    if (i < n_rows) r = UP ? a.perm[first + i] / a.top : first + i;
+    if (i < n_rows) r = UP && !shared ? a.perm[first + i] / a.top : first + i;
     src_row[i] = r;
   }
   __syncthreads();
-  const bf16* A = (const bf16*)(UP ? a.x : a.act);
-  const bf16* B0 = (const bf16*)(GATED ? a.w_gate : UP ? a.w_up : a.w_down) + (size_t)e * N * K;
+  const bf16* A = (const bf16*)(UP ? a.x : shared ? a.act_s : a.act);
+  const bf16* B0 = shared ? (const bf16*)(UP ? a.ws_up : a.ws_down)
+                          : (const bf16*)(GATED ? a.w_gate : UP ? a.w_up : a.w_down) + (size_t)e * N * K;
   const bf16* B1 = GATED ? (const bf16*)a.w_up + (size_t)e * N * K : nullptr;
   auto load = [&](int stage, int k0) {
     bf16* As = tiles + stage * Tile::STAGE_ELEMS;
@@ -497,8 +533,8 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
       const int row = row_w + m * 16 + g + half * 8;
       if (row >= n_rows) continue;
       if (UP) {
-        bf16* dst = (bf16*)a.act + (size_t)(first + row) * N;
-        const float wi = a.weigh_input ? a.wts[a.perm[first + row]] : 1.0f;
+        bf16* dst = (bf16*)(shared ? a.act_s : a.act) + (size_t)(first + row) * N;
+        const float wi = a.weigh_input && !shared ? a.wts[a.perm[first + row]] : 1.0f;
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
           const int col = n0 + col_w + j * 8 + t * 2;
@@ -518,8 +554,9 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
           else if (col < N) dst[col] = from_f32<bf16>(y[0]);
         }
       } else {
-        const int p = a.perm[first + row], tok = p / a.top, jc = p % a.top;
-        const float w = a.weigh_input ? 1.0f : a.wts[p];
+        const int p = shared ? 0 : a.perm[first + row];
+        const int tok = shared ? first + row : p / a.top, jc = shared ? a.top : p % a.top;
+        const float w = a.weigh_input || shared ? 1.0f : a.wts[p];
         float* dst = a.out + ((size_t)jc * a.T + tok) * N;
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
@@ -534,12 +571,12 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
 
 template <int MODE, int BM>
 static int moe_tc_launch(const MoeArgs& a, long long pairs, cudaStream_t s) {
-  const long long tiles = pairs / BM + (pairs < a.E ? pairs : a.E);
+  const long long tiles = pairs / BM + (pairs < a.E ? pairs : a.E) + (a.Fs > 0 ? (a.T + BM - 1) / BM : 0);
   if (tiles > 0x7fffffffLL) return GB_ERR_UNSUPPORTED;
   const size_t smem = MoeTile<MODE, BM>::SMEM;
   cudaError_t ce = cudaFuncSetAttribute(moe_tc_kernel<MODE, BM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (ce != cudaSuccess) return (int)ce;
-  const int N = MODE != MOE_DOWN ? a.F : a.W, BN = MoeTile<MODE, BM>::BN;
+  const int N = MODE == MOE_DOWN ? a.W : (a.Fs > a.F ? a.Fs : a.F), BN = MoeTile<MODE, BM>::BN;
   return gb_launch(moe_tc_kernel<MODE, BM>, dim3((unsigned)tiles, (N + BN - 1) / BN),
                    dim3(MoeTile<MODE, BM>::THREADS), smem, s, a);
 }
@@ -558,6 +595,7 @@ static int moe_check(const MoeArgs& a) {
   if (n_all % a.n_groups || a.top > n_all) return GB_ERR_BAD_ARG;
   if (n_all > MOE_MAX_OUTPUTS) return GB_ERR_UNSUPPORTED;
   if (a.score_fn < 0 || a.score_fn > 2) return GB_ERR_BAD_ARG;
+  if (a.Fs < 0 || (a.Fs > 0 && (!a.ws_up || !a.ws_down || !a.act_s || a.w_gate))) return GB_ERR_BAD_ARG;
   if (!a.x || !a.router_w || !a.w_up || !a.w_down || !a.ids || !a.wts ||
       !a.rank || !a.counts || !a.offsets || !a.perm || !a.act || !a.out)
     return GB_ERR_BAD_ARG;
@@ -571,11 +609,11 @@ static int moe_forward(const MoeArgs& a, cudaStream_t s) {
   if (a.T == 0) return 0;
   const int n_all = a.E + a.n_identity;
   e = gb_launch(moe_route_kernel<T>, dim3(a.T), dim3(MOE_ROUTE_THREADS), (size_t)(2 * n_all + a.n_groups) * sizeof(float), s, a);
-  if (e) return e;
+  if (e || a.route_only) return e;
   // the most tiles the pairs can make: every expert may end in a tile that is not full
   const long long pairs = (long long)a.T * a.top;
-  if (sizeof(T) == 2 && a.W % 8 == 0 && a.F % 8 == 0 &&
-      ((((uintptr_t)a.x) | ((uintptr_t)a.act) | ((uintptr_t)a.w_gate) | ((uintptr_t)a.w_up) |
+  if (sizeof(T) == 2 && a.W % 8 == 0 && a.F % 8 == 0 && a.Fs % 8 == 0 &&
+      ((((uintptr_t)a.ws_up) | ((uintptr_t)a.ws_down) | ((uintptr_t)a.act_s) | ((uintptr_t)a.x) | ((uintptr_t)a.act) | ((uintptr_t)a.w_gate) | ((uintptr_t)a.w_up) |
         ((uintptr_t)a.w_down) | ((uintptr_t)a.out)) & 15) == 0) {
     // few pairs per expert (a decode step): narrow tiles, deeper pipeline; 64 pairs an expert
     // and more: tiles of 128 rows
@@ -583,6 +621,7 @@ static int moe_forward(const MoeArgs& a, cudaStream_t s) {
     if (pairs >= 64LL * a.E) return moe_tc_products<128>(a, pairs, s);
     return moe_tc_products<64>(a, pairs, s);
   }
+  if (a.Fs > 0) return GB_ERR_UNSUPPORTED;       // the plain kernels know no shared expert
   const long long tiles = pairs / MOE_BM + (pairs < a.E ? pairs : a.E);
   if (tiles > 0x7fffffffLL) return GB_ERR_UNSUPPORTED;
   e = gb_launch(moe_up_kernel<T>, dim3((unsigned)tiles, (a.F + MOE_BN - 1) / MOE_BN), dim3(256), 0, s, a);

@@ -1950,7 +1950,30 @@ class _MoeArgs(ctypes.Structure):
                 ("F", _I), ("E", _I), ("n_identity", _I), ("top", _I), ("n_groups", _I),
                 ("keep_groups", _I), ("limit", _F), ("slope", _F), ("score_fn", _I),
                 ("weigh_input", _I), ("up_offset", _F), ("router_bias", _P), ("group_top2", _I),
-                ("normalize", _I), ("weight_scale", _F)]
+                ("normalize", _I), ("weight_scale", _F), ("ws_up", _P), ("ws_down", _P), ("act_s", _P),
+                ("Fs", _I), ("route_only", _I)]
+
+
+class _MoePairArgs(ctypes.Structure):
+    _fields_ = [("x", _P), ("xg", _P), ("w_gate", _P), ("w_up", _P), ("w_down", _P), ("ws_up", _P),
+                ("ws_down", _P), ("offsets", _P), ("perm", _P), ("wts", _P), ("act", _P), ("act_s", _P),
+                ("out", _P), ("error", _P), ("T", _I), ("W", _I), ("F", _I), ("Fs", _I), ("E", _I),
+                ("top", _I), ("limit", _F), ("slope", _F), ("up_offset", _F), ("weigh_input", _I)]
+
+
+_TC_ERROR_NAMES.update({141: "the experts' MMA lane waited 2 s for a stage that never arrived",
+                        142: "the experts' loads waited 2 s for a stage that was never released",
+                        143: "the experts' epilogue waited 2 s for an accumulator",
+                        144: "the experts' MMA lane waited 2 s for an accumulator to be drained"})
+# From how many (token, choice) pairs an expert on the products run on pairs of SMs
+# ("auto"); "pair" takes them wherever the sizes allow, "tiles" never.
+MOE_PRODUCTS = "auto"
+MOE_PAIR_ROWS = 64
+
+
+def moe_tensor_cores_take(W: int, F: int, Fs: int = 0) -> bool:
+    """Whether the tensor-core kernels take experts of these widths (bfloat16)."""
+    return W % 8 == 0 and F % 8 == 0 and Fs % 8 == 0
 
 
 _MOE_COUNTS = {}
@@ -1961,7 +1984,9 @@ def _cost_moe(out, x, router_w, correction, w_gate, w_up, w_down, *, top, **k):
     T, W = x.shape
     E, F = w_up.shape[0], w_up.shape[1]
     used, mats = min(E, T * top), 2 if w_gate is None else 3
-    return (_nbytes(x, out) + used * mats * F * W * w_up.element_size(), 2.0 * mats * T * top * F * W)
+    Fs = k["shared"][0].shape[0] if k.get("shared") else 0
+    return (_nbytes(x, out) + (used * mats * F + 2 * Fs) * W * w_up.element_size(),
+            2.0 * T * W * (mats * top * F + 2 * Fs))
 
 
 @_profiled("moe_forward", _cost_moe)
@@ -1971,7 +1996,7 @@ def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[to
                 limit: float = math.inf, slope: float = 1.0, score_fn: str = "softmax",
                 weigh_input: bool = False, up_offset: float = 1.0, want_choice: bool = False,
                 router_bias: Optional[torch.Tensor] = None, group_top2: bool = False,
-                normalize: bool = False, weight_scale: float = 1.0, extra: int = 0):
+                normalize: bool = False, weight_scale: float = 1.0, extra: int = 0, shared=None):
     """A feed-forward of routed experts on rows x [T, W] -> 32-bit partial sums
     [top, T, W], choice j of every token in [j], already weighted; their sum is the
     feed-forward's output.  ``router_w`` [E + n_identity, W] and ``correction`` are
@@ -1986,6 +2011,9 @@ def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[to
     group's score is the sum of its two largest choice scores, not its largest; ``normalize``: the
     chosen outputs' weights are divided by their sum; ``weight_scale`` multiplies the weights.
     ``extra``: that many more [T, W] terms are appended to the result for the caller to fill.
+    ``shared`` = (up [Fs, W], down [W, Fs]): one more ungated expert that runs for every token with
+    weight 1 in the same launches and leaves its term behind the ``top`` others (bfloat16, ungated
+    experts, widths that ``moe_tensor_cores_take``).
     With ``want_choice`` also returns (ids [T, top] int32, weights [T, top])."""
     _need(x, "activations", ndim=2)
     T, W = x.shape
@@ -2007,6 +2035,17 @@ def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[to
             tuple(w_down.shape) != (E, W, F) or tuple(router_w.shape) != (n_all, W) or \
             (correction is not None and correction.shape[0] != n_all):
         raise KernelError("the experts' weights, the router and the correction do not fit together")
+    Fs = 0
+    if shared is not None:
+        Fs = shared[0].shape[0]
+        for t, nm, shape in ((shared[0], "shared up weight", (Fs, W)), (shared[1], "shared down weight", (W, Fs))):
+            _need(t, nm, x.dtype, 2)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"{nm} is {tuple(t.shape)}, expected {shape}")
+        if x.dtype != torch.bfloat16 or w_gate is not None or extra or not moe_tensor_cores_take(W, F, Fs):
+            raise KernelError("a shared expert in the experts' launches goes with bfloat16, ungated experts and "
+                              "widths that are multiples of eight")
+        extra = 1
     dev = x.device
     ids = torch.empty((T, top), dtype=torch.int32, device=dev)
     wts = torch.empty((T, top), dtype=torch.float32, device=dev)
@@ -2029,8 +2068,27 @@ def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[to
     a.score_fn, a.weigh_input, a.up_offset = MOE_SCORE_FNS[score_fn], int(weigh_input), float(up_offset)
     a.router_bias = _ptr(router_bias)
     a.group_top2, a.normalize, a.weight_scale = int(group_top2), int(normalize), float(weight_scale)
+    act_s = None
+    if Fs:
+        act_s = torch.empty((T, Fs), dtype=x.dtype, device=dev)
+        a.ws_up, a.ws_down, a.act_s, a.Fs = shared[0].data_ptr(), shared[1].data_ptr(), act_s.data_ptr(), Fs
+    pair = (x.dtype == torch.bfloat16 and T > 0 and moe_tensor_cores_take(W, F, Fs) and MOE_PRODUCTS != "tiles"
+            and (MOE_PRODUCTS == "pair" or T * top >= MOE_PAIR_ROWS * E))
+    a.route_only = int(pair)
     _check(_fn("moe", f"gb_moe_forward_{_suffix(x.dtype)}", "pp")(ctypes.addressof(a), _stream()),
-           "moe_forward", 3)
+           "moe_forward", 1 if pair else 3)
+    if pair:
+        xg = torch.empty((T * top, W), dtype=x.dtype, device=dev)
+        b = _MoePairArgs()
+        b.x, b.xg, b.w_gate, b.w_up, b.w_down = x.data_ptr(), xg.data_ptr(), _ptr(w_gate), w_up.data_ptr(), w_down.data_ptr()
+        if Fs:
+            b.ws_up, b.ws_down, b.act_s, b.Fs = a.ws_up, a.ws_down, a.act_s, Fs
+        b.offsets, b.perm, b.wts = offsets.data_ptr(), perm.data_ptr(), wts.data_ptr()
+        b.act, b.out, b.error = act.data_ptr(), out.data_ptr(), _tc_error_flag(dev).data_ptr()
+        b.T, b.W, b.F, b.E, b.top = T, W, F, E, int(top)
+        b.limit, b.slope, b.up_offset, b.weigh_input = float(limit), float(slope), float(up_offset), int(weigh_input)
+        with torch.cuda.device(dev):
+            _check(_fn("moe_pair", "gb_moe_pair_bf16", "pp")(ctypes.addressof(b), _stream()), "moe_pair", 3)
     return (out, ids, wts) if want_choice else out
 
 

@@ -273,21 +273,28 @@ class RoutedExperts(FeedForward):
             self.shared.load({n: params[n] for n in self.shared.param_specs()})
 
     def kernel_modules(self):
+        if self.ctx.dtype == torch.bfloat16 and ops.moe_tensor_cores_take(self.hidden, self.intermediate):
+            return ("moe", "moe_pair")
         return ("moe",)
 
     def captures_prompts(self):
         return True
 
     def forward(self, x, step):
-        # the shared expert leaves its 32-bit sums behind the routed ones
-        extra = self.shared.down.n_parts(x.shape[0]) if self.shared else 0
+        # the shared expert runs in the routed ones' launches where their kernels take it; else it
+        # leaves its 32-bit sums behind theirs
+        fused = (self.shared is not None and not self.gated and x.dtype == torch.bfloat16
+                 and self.shared.up.weight.dtype == self.shared.down.weight.dtype == torch.bfloat16
+                 and ops.moe_tensor_cores_take(self.hidden, self.intermediate, self.shared.intermediate))
+        extra = self.shared.down.n_parts(x.shape[0]) if self.shared and not fused else 0
         out = ops.moe_forward(x, self.router_w, self.correction, self.w_gate, self.w_up, self.w_down,
                               top=self.top, n_identity=self.n_identity, n_groups=self.n_groups,
                               keep_groups=self.keep_groups, limit=self.limit, slope=self.gate_slope,
                               score_fn=self.score_fn, weigh_input=self.weigh_input,
                               up_offset=self.up_offset, router_bias=self.router_b,
                               group_top2=self.group_top2, normalize=self.normalize,
-                              weight_scale=self.weight_scale, extra=extra)
-        if self.shared:
+                              weight_scale=self.weight_scale, extra=extra,
+                              shared=(self.shared.up.weight, self.shared.down.weight) if fused else None)
+        if self.shared and not fused:
             self.shared.down(self.shared.up.relu_squared(x), into=out[self.top:])
         return out

@@ -320,7 +320,7 @@ def test_stores_give_back_pages_and_keep_a_readers(engines):
     assert eng.cache.tokens_held() == 0
     eng = engines("P", "float32")
     s = eng.open_sequence()
-    eng.step([(s, toks[:200])], [[0]])
+    eng.step([(s, random_tokens(200, KAK["P"]["vocab"], 411))], [[0]])
     # layer 0's own window is 9, its reader's 40: positions 161.. stay (pages 2 and 3); chunks of 7: page 3
     held = sorted(st.pool.n_held for st in eng.cache.stores if hasattr(st, "pool"))
     assert held == [1, 2], held

@@ -601,24 +601,64 @@ def _moe(m, dtype, seed=0, correction=None):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("T", [1, 5, 70, 600])
 @pytest.mark.parametrize("m", MOE_SHAPES)
-def test_ungated_experts_groups_and_the_shared_expert(dtype, T, m):
+def test_ungated_experts_groups_and_the_shared_expert(monkeypatch, dtype, T, m):
     """Choice scores that are mostly negative (a dropped group must count as minus infinity, not as
     zero); few rows and many (the products' kernels differ)."""
     part, w, mlp = _moe(m, dtype)
     x = rnd(T, m["W"], seed=5).to(dtype)
     pw = {"m." + k: v for k, v in w.items()}
     want = plain.experts_ff(x.double(), pw, "m.", mlp)
-    got = part.forward(x.to(DEV), None)
-    assert got.dtype == torch.float32 and got.shape[0] >= m["top"] + (1 if m["shared"] else 0)
-    got = got.sum(0).double().cpu()
-    if dtype == torch.float32:
-        close(got, want, dtype, scale=float(want.abs().max()))
-    else:      # a near tie between two experts may fall the other way after rounding: most rows agree
-        rows = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
-        assert float(rows.median()) < 0.02 and float((rows < 0.06).double().mean()) > 0.9
-    if T == 70:     # a token's result does not depend on the rows around it
-        alone = part.forward(x[11:12].to(DEV), None).sum(0).double().cpu()
-        close(alone[0], got[11], dtype, scale=float(want.abs().max()) / (1 if dtype == torch.float32 else 8))
+    from grout_b200.kernels import ops
+    for products in ("auto", "tiles", "pair") if dtype == torch.bfloat16 else ("auto",):
+        monkeypatch.setattr(ops, "MOE_PRODUCTS", products)
+        got = part.forward(x.to(DEV), None)
+        assert got.dtype == torch.float32 and got.shape[0] >= m["top"] + (1 if m["shared"] else 0)
+        got = got.sum(0).double().cpu()
+        if dtype == torch.float32:
+            close(got, want, dtype, scale=float(want.abs().max()))
+        else:      # a near tie between two experts may fall the other way after rounding: most rows agree
+            rows = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
+            assert float(rows.median()) < 0.02 and float((rows < 0.06).double().mean()) > 0.9, products
+        if T == 70:     # a token's result does not depend on the rows around it
+            alone = part.forward(x[11:12].to(DEV), None).sum(0).double().cpu()
+            close(alone[0], got[11], dtype, products, scale=float(want.abs().max()) / (1 if dtype == torch.float32 else 8))
+    ops.check_kernel_errors()
+
+
+@pytest.mark.parametrize("T", [1, 130, 700])
+@pytest.mark.parametrize("shape", [(6, 2, 24, 64, 0, 0), (3, 3, 200, 96, 2, 1), (1, 1, 136, 40, 0, 0), (40, 4, 72, 264, 0, 1)])
+def test_experts_on_pairs_of_SMs_and_in_tiles_agree(T, shape):
+    """The grouped product on pairs of SMs against the tile kernels, gated and ungated, with a clamp, an
+    offset, outputs that hand the input on and weights on the input; experts without rows, with fewer
+    than a tile's and with more; widths that end inside a tile."""
+    from grout_b200.kernels import ops
+    E, top, F, W, identity, weigh = shape
+    bf = torch.bfloat16
+    x = rnd(T, W, seed=1).to(bf).to(DEV)
+    router = g32(rnd(E + identity, W, seed=2, scale=0.5))
+    if E > 5:
+        router[4] = -router[0]                              # (an expert that is chosen rarely)
+        router[5] = -1.0e3 * router[1].abs() * x[0].float().sign()
+    wg, wu, wd = (rnd(*s, seed=3 + i, scale=0.3).to(bf).to(DEV) for i, s in enumerate(((E, F, W), (E, F, W), (E, W, F))))
+    shared = (rnd(88, W, seed=7, scale=0.3).to(bf).to(DEV), rnd(W, 88, seed=8, scale=0.3).to(bf).to(DEV))
+    for gate in (wg, None):
+        for sh in ((None, shared) if gate is None else (None,)):
+            outs = []
+            for products in ("tiles", "pair"):
+                ops.MOE_PRODUCTS = products
+                try:
+                    outs.append(ops.moe_forward(x, router, None, gate, wu, wd, top=top, n_identity=identity,
+                                                limit=1.5 if gate is not None else math.inf, slope=1.3,
+                                                weigh_input=bool(weigh), up_offset=0.5, shared=sh))
+                finally:
+                    ops.MOE_PRODUCTS = "auto"
+            assert outs[0].shape[0] == top + (1 if sh else 0)
+            scale = float(outs[0].abs().max())
+            assert scale > 0.1 and not torch.isnan(outs[1]).any()
+            # the inner activations are rounded to bfloat16 from sums taken in another order
+            assert float((outs[0] - outs[1]).abs().max()) < 0.02 * scale
+            assert float((outs[0] - outs[1]).pow(2).mean().sqrt()) < 0.002 * scale
+    ops.check_kernel_errors()
 
 
 def test_the_choice_goes_by_corrected_scores_and_the_weights_do_not():
