@@ -33,7 +33,11 @@
 // list of (token, choice) pairs ordered by expert; the two products walk
 // tiles of that list; a block finds its expert from the counts, and blocks
 // beyond the last tile return.  A pair's row is computed the same way wherever it
-// lands in the list, so a token's result does not depend on the batch.  The
+// lands in the list, so a token's result does not depend on the batch.  A step of few rows
+// (`small`, a decode step) needs no list: a block of the products belongs to an expert and
+// finds the expert's pairs among the step's few choices itself, pair p's inner activations
+// lie in row p, and since its weights are known from the start it asks for the first of them
+// before it waits for the choices.  The
 // weighted results are left as `top` 32-bit partial sums [top, T, W]
 // (choice j of token t in out[j, t, :]), which the norm that follows adds in
 // order.
@@ -67,6 +71,9 @@ struct MoeArgs {
   const void* ws_down;       // [W, Fs]
   void* act_s;               // [T, Fs] its inner activations
   int Fs;
+  int small;                 // a step of few rows: no ordered list, blocks of the products by expert
+  int early;                 // with `small`: a block's first weights are requested before the choices are known
+  int stage_router;          // the router's rows fit in a block's shared memory and are fetched before the wait
   int route_only;            // stop behind `route` (the products are another source's kernels)
 };
 
@@ -80,14 +87,25 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
   extern __shared__ float sm[];   // z [n_all], c [n_all], a score per group
   __shared__ float part[MOE_ROUTE_THREADS / 32][MOE_ROUTE_CHUNK];
   pdl_launch_dependents_if_small();
-  pdl_wait();
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int nwarps = blockDim.x >> 5;
   const int n_all = a.E + a.n_identity, W = a.W;
   float* z = sm;
   float* c = sm + n_all;
   float* gval = c + n_all;         // [n_groups] scores of the groups
+  const float* router = a.router_w;
+  if (a.stage_router) {            // (no kernel's output: before the wait)
+    float* rs = sm + ((2 * n_all + a.n_groups + 3) & ~3);
+    for (int i = tid * 4; i < n_all * W; i += MOE_ROUTE_THREADS * 4) cp_async16(rs + i, a.router_w + i, true);
+    cp_async_commit();
+    router = rs;
+  }
+  pdl_wait();
   const T* x = (const T*)a.x + (size_t)t * W;
+  if (a.stage_router) {
+    cp_async_wait<0>();
+    __syncthreads();
+  }
   // every thread takes a slice of the row against a few router rows at a time, so that
   // all of a slice's loads are under way together; the sums are put together in a fixed
   // order (lanes by the shuffle tree, then warp after warp)
@@ -101,7 +119,7 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
       const float xv = to_f32<T>(x[i]);
 #pragma unroll
       for (int u = 0; u < MOE_ROUTE_CHUNK; ++u)
-        if (u < nu) acc[u] = fmaf(xv, a.router_w[(size_t)(e0 + u) * W + i], acc[u]);
+        if (u < nu) acc[u] = fmaf(xv, router[(size_t)(e0 + u) * W + i], acc[u]);
     }
 #pragma unroll
     for (int u = 0; u < MOE_ROUTE_CHUNK; ++u) {
@@ -187,10 +205,13 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
       }
     }
   }
+  if (a.small && a.n_identity == 0) return;          // the products' blocks read the choices themselves
   __syncthreads();
+  if (!a.small) {
   for (int j = tid; j < a.top; j += blockDim.x) {   // the choices' places among their experts' pairs
     const int e = a.ids[(size_t)t * a.top + j];
     a.rank[(size_t)t * a.top + j] = e < a.E ? atomicAdd(&a.counts[e], 1) : -1;
+  }
   }
   pdl_launch_dependents_if_large();
   for (int j = 0; j < a.top; ++j) {     // experts that hand their input on
@@ -199,6 +220,7 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
     float* o = a.out + ((size_t)j * a.T + t) * W;
     for (int i = tid; i < W; i += blockDim.x) o[i] = w * to_f32<T>(x[i]);
   }
+  if (a.small) return;
   // The block that finishes last turns the counts into the list of pairs ordered by expert:
   // every block publishes its choices, then draws a ticket (counts[E]); the one that draws
   // the last ticket sees all of them.  It leaves the counts and the ticket at zero for the
@@ -419,7 +441,7 @@ struct MoeTile {
   static constexpr size_t SMEM = (size_t)STAGES * STAGE_ELEMS * sizeof(bf16);
 };
 
-template <int MODE, int BM>
+template <int MODE, int BM, bool SMALL>
 __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
   using Tile = MoeTile<MODE, BM>;
   constexpr bool UP = Tile::UP, GATED = MODE == MOE_GATED;
@@ -427,9 +449,10 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
   constexpr int MI = Tile::MI, NJ = Tile::NJ;
   extern __shared__ __align__(16) bf16 tiles[];
   __shared__ int src_row[BM];
+  __shared__ int pair_of[BM];                  // the tile's pairs
   pdl_launch_dependents_if_small();
-  pdl_wait();
-  int e = 0, first, n_rows;
+  if (!SMALL) pdl_wait();
+  int e = 0, first = 0, n_rows = 0;
   const int shared_tiles = a.Fs > 0 ? (a.T + BM - 1) / BM : 0;
   const bool shared = (int)blockIdx.x < shared_tiles;      // a tile of the shared expert: tokens as they come
   const int F = shared ? a.Fs : a.F;
@@ -439,28 +462,59 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
   if (shared) {
     first = blockIdx.x * BM;
     n_rows = min(BM, a.T - first);
+  } else if (SMALL) {
+    const int per_expert = (a.T + BM - 1) / BM;            // an expert has at most one pair a token
+    e = (blockIdx.x - shared_tiles) / per_expert;
+    first = ((blockIdx.x - shared_tiles) % per_expert) * BM;   // its pairs from this one on
   } else if (!moe_find_tile<BM>(a.offsets, a.E, blockIdx.x - shared_tiles, e, first, n_rows)) {
     return;
   }
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  for (int i = tid; i < BM; i += NT) {
-    int r = -1;
-    if (i < n_rows) r = UP && !shared ? a.perm[first + i] / a.top : first + i;
-    src_row[i] = r;
-  }
-  __syncthreads();
+  auto list_rows = [&] {       // which rows of A the tile has: from the list, from the choices, or as tokens come
+    if (SMALL && !shared) {
+      __shared__ int found_s[NT / 32];
+      int seen = 0;
+      for (int p0 = 0; p0 < a.T * a.top; p0 += NT) {
+        const int p = p0 + tid;
+        const bool mine = p < a.T * a.top && __ldcg(&a.ids[p]) == e;
+        const unsigned votes = __ballot_sync(0xffffffffu, mine);
+        if (lane == 0) found_s[warp] = __popc(votes);
+        __syncthreads();
+        int at = seen;
+        for (int w = 0; w < NT / 32; ++w) {
+          if (w < warp) at += found_s[w];
+          seen += found_s[w];
+        }
+        at += __popc(votes & ((1u << lane) - 1)) - first;
+        if (mine && at >= 0 && at < BM) pair_of[at] = p;
+        __syncthreads();
+      }
+      n_rows = min(BM, seen - first);
+    } else {
+      for (int i = tid; i < n_rows; i += NT) pair_of[i] = shared ? 0 : a.perm[first + i];
+      __syncthreads();
+    }
+    for (int i = tid; i < BM; i += NT) {
+      int r = -1;
+      if (i < n_rows) r = shared ? first + i : UP ? pair_of[i] / a.top : SMALL ? pair_of[i] : first + i;
+      src_row[i] = r;
+    }
+    __syncthreads();
+  };
   const bf16* A = (const bf16*)(UP ? a.x : shared ? a.act_s : a.act);
   const bf16* B0 = shared ? (const bf16*)(UP ? a.ws_up : a.ws_down)
                           : (const bf16*)(GATED ? a.w_gate : UP ? a.w_up : a.w_down) + (size_t)e * N * K;
   const bf16* B1 = GATED ? (const bf16*)a.w_up + (size_t)e * N * K : nullptr;
-  auto load = [&](int stage, int k0) {
+  auto load_a = [&](int stage, int k0) {
     bf16* As = tiles + stage * Tile::STAGE_ELEMS;
-    bf16* Bs = As + BM * MT_LD;
     for (int c = tid; c < BM * 8; c += NT) {             // rows x 8 pieces of 8 elements
       const int r = c >> 3, pc = (c & 7) * 8, kc = k0 + pc;
       const bool ok = src_row[r] >= 0 && kc < K;
       cp_async16(As + r * MT_LD + pc, ok ? A + (size_t)src_row[r] * K + kc : A, ok);
     }
+  };
+  auto load_b = [&](int stage, int k0) {
+    bf16* Bs = tiles + stage * Tile::STAGE_ELEMS + BM * MT_LD;
 #pragma unroll
     for (int i = 0; i < BN * 8 / NT; ++i) {
       const int c = tid + i * NT, r = c >> 3, pc = (c & 7) * 8, kc = k0 + pc;
@@ -484,15 +538,34 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
   // two 8-column pieces at a time (four 8 x 8 blocks), or one (two blocks: lanes 0-15 give the rows)
   const int brow = col_w + (lane & 7) + (NJ > 1 ? (lane >> 4) * 8 : 0), bcol = ((lane >> 3) & 1) * 8;
   const int nk = (K + MT_BK - 1) / MT_BK;
+  const bool early = SMALL && (a.early || shared);
+  if (early) {                                   // weights, which no kernel writes: before the wait
+#pragma unroll
+    for (int st = 0; st < STAGES - 1; ++st)
+      if (st < nk) load_b(st, st * MT_BK);
+    cp_async_commit();
+  }
+  if (SMALL) pdl_wait();
+  list_rows();
+  if (SMALL && n_rows <= 0) {                    // an expert nobody chose (the copies under way land first)
+    cp_async_wait<0>();
+    return;
+  }
 #pragma unroll
   for (int st = 0; st < STAGES - 1; ++st) {      // a group per stage, empty beyond the end
-    if (st < nk) load(st, st * MT_BK);
+    if (st < nk) {
+      load_a(st, st * MT_BK);
+      if (!early) load_b(st, st * MT_BK);
+    }
     cp_async_commit();
   }
   for (int kt = 0; kt < nk; ++kt) {
     cp_async_wait<STAGES - 2>();                  // chunk kt has landed
     __syncthreads();                              // ... for every thread; chunk kt - 1 is done with
-    if (kt + STAGES - 1 < nk) load((kt + STAGES - 1) % STAGES, (kt + STAGES - 1) * MT_BK);
+    if (kt + STAGES - 1 < nk) {
+      load_a((kt + STAGES - 1) % STAGES, (kt + STAGES - 1) * MT_BK);
+      load_b((kt + STAGES - 1) % STAGES, (kt + STAGES - 1) * MT_BK);
+    }
     cp_async_commit();
     const bf16* As = tiles + (kt % STAGES) * Tile::STAGE_ELEMS;
     const bf16* Bs = As + BM * MT_LD;
@@ -533,8 +606,8 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
       const int row = row_w + m * 16 + g + half * 8;
       if (row >= n_rows) continue;
       if (UP) {
-        bf16* dst = (bf16*)(shared ? a.act_s : a.act) + (size_t)(first + row) * N;
-        const float wi = a.weigh_input && !shared ? a.wts[a.perm[first + row]] : 1.0f;
+        bf16* dst = (bf16*)(shared ? a.act_s : a.act) + (size_t)(SMALL && !shared ? pair_of[row] : first + row) * N;
+        const float wi = a.weigh_input && !shared ? a.wts[pair_of[row]] : 1.0f;
 #pragma unroll
         for (int j = 0; j < NJ; ++j) {
           const int col = n0 + col_w + j * 8 + t * 2;
@@ -554,7 +627,7 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
           else if (col < N) dst[col] = from_f32<bf16>(y[0]);
         }
       } else {
-        const int p = shared ? 0 : a.perm[first + row];
+        const int p = pair_of[row];
         const int tok = shared ? first + row : p / a.top, jc = shared ? a.top : p % a.top;
         const float w = a.weigh_input || shared ? 1.0f : a.wts[p];
         float* dst = a.out + ((size_t)jc * a.T + tok) * N;
@@ -569,22 +642,32 @@ __global__ void __launch_bounds__(128) moe_tc_kernel(const MoeArgs a) {
     }
 }
 
-template <int MODE, int BM>
+template <int MODE, int BM, bool SMALL = false>
 static int moe_tc_launch(const MoeArgs& a, long long pairs, cudaStream_t s) {
-  const long long tiles = pairs / BM + (pairs < a.E ? pairs : a.E) + (a.Fs > 0 ? (a.T + BM - 1) / BM : 0);
+  const long long tiles = (SMALL ? (long long)a.E * ((a.T + BM - 1) / BM) : pairs / BM + (pairs < a.E ? pairs : a.E)) +
+                          (a.Fs > 0 ? (a.T + BM - 1) / BM : 0);
   if (tiles > 0x7fffffffLL) return GB_ERR_UNSUPPORTED;
   const size_t smem = MoeTile<MODE, BM>::SMEM;
-  cudaError_t ce = cudaFuncSetAttribute(moe_tc_kernel<MODE, BM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  cudaError_t ce = cudaFuncSetAttribute(moe_tc_kernel<MODE, BM, SMALL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (ce != cudaSuccess) return (int)ce;
   const int N = MODE == MOE_DOWN ? a.W : (a.Fs > a.F ? a.Fs : a.F), BN = MoeTile<MODE, BM>::BN;
-  return gb_launch(moe_tc_kernel<MODE, BM>, dim3((unsigned)tiles, (N + BN - 1) / BN),
+  return gb_launch(moe_tc_kernel<MODE, BM, SMALL>, dim3((unsigned)tiles, (N + BN - 1) / BN),
                    dim3(MoeTile<MODE, BM>::THREADS), smem, s, a);
 }
 
-template <int BM>
+template <int BM, bool SMALL = false>
 static int moe_tc_products(const MoeArgs& a, long long pairs, cudaStream_t s) {
-  int e = a.w_gate ? moe_tc_launch<MOE_GATED, BM>(a, pairs, s) : moe_tc_launch<MOE_UNGATED, BM>(a, pairs, s);
-  return e ? e : moe_tc_launch<MOE_DOWN, BM>(a, pairs, s);
+  int e = a.w_gate ? moe_tc_launch<MOE_GATED, BM, SMALL>(a, pairs, s) : moe_tc_launch<MOE_UNGATED, BM, SMALL>(a, pairs, s);
+  return e ? e : moe_tc_launch<MOE_DOWN, BM, SMALL>(a, pairs, s);
+}
+
+// A step whose products need no ordered list: few rows, few choices to look through, and
+// hardly more blocks (one tile of 16 pairs an expert and 16 rows) than the list would give.
+#define MOE_SMALL_ROWS 64
+#define MOE_SMALL_PAIRS 512
+static bool moe_small(const MoeArgs& a, long long pairs) {
+  return a.T <= MOE_SMALL_ROWS && pairs <= MOE_SMALL_PAIRS && pairs <= 4LL * a.E &&
+         (long long)a.E * ((a.T + 15) / 16) <= 256;
 }
 
 static int moe_check(const MoeArgs& a) {
@@ -603,18 +686,34 @@ static int moe_check(const MoeArgs& a) {
 }
 
 template <typename T>
-static int moe_forward(const MoeArgs& a, cudaStream_t s) {
+static int moe_forward(MoeArgs a, cudaStream_t s) {
   int e = moe_check(a);
   if (e) return e;
   if (a.T == 0) return 0;
   const int n_all = a.E + a.n_identity;
-  e = gb_launch(moe_route_kernel<T>, dim3(a.T), dim3(MOE_ROUTE_THREADS), (size_t)(2 * n_all + a.n_groups) * sizeof(float), s, a);
+  const long long pairs = (long long)a.T * a.top;
+  const bool tensor_cores =
+      sizeof(T) == 2 && a.W % 8 == 0 && a.F % 8 == 0 && a.Fs % 8 == 0 &&
+      ((((uintptr_t)a.ws_up) | ((uintptr_t)a.ws_down) | ((uintptr_t)a.act_s) | ((uintptr_t)a.x) |
+        ((uintptr_t)a.act) | ((uintptr_t)a.w_gate) | ((uintptr_t)a.w_up) | ((uintptr_t)a.w_down) |
+        ((uintptr_t)a.out)) & 15) == 0;
+  a.small = tensor_cores && !a.route_only && moe_small(a, pairs);
+  // (where most experts would be asked for weights in vain they wait for the choices)
+  a.early = a.small && pairs >= a.E;
+  const size_t choice = (size_t)(2 * n_all + a.n_groups) * sizeof(float);
+  const size_t staged = ((choice + 15) & ~(size_t)15) + (size_t)n_all * a.W * sizeof(float);
+  a.stage_router = a.T <= 64 && a.W % 4 == 0 && ((uintptr_t)a.router_w & 15) == 0 && staged <= 160 * 1024;
+  static bool raised = false;      // more than the 48 KB a kernel gets without asking
+  if (a.stage_router && !raised) {
+    cudaError_t ce = cudaFuncSetAttribute(moe_route_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+    if (ce != cudaSuccess) return (int)ce;
+    raised = true;
+  }
+  e = gb_launch(moe_route_kernel<T>, dim3(a.T), dim3(MOE_ROUTE_THREADS), a.stage_router ? staged : choice, s, a);
   if (e || a.route_only) return e;
   // the most tiles the pairs can make: every expert may end in a tile that is not full
-  const long long pairs = (long long)a.T * a.top;
-  if (sizeof(T) == 2 && a.W % 8 == 0 && a.F % 8 == 0 && a.Fs % 8 == 0 &&
-      ((((uintptr_t)a.ws_up) | ((uintptr_t)a.ws_down) | ((uintptr_t)a.act_s) | ((uintptr_t)a.x) | ((uintptr_t)a.act) | ((uintptr_t)a.w_gate) | ((uintptr_t)a.w_up) |
-        ((uintptr_t)a.w_down) | ((uintptr_t)a.out)) & 15) == 0) {
+  if (tensor_cores) {
+    if (a.small) return moe_tc_products<16, true>(a, pairs, s);
     // few pairs per expert (a decode step): narrow tiles, deeper pipeline; 64 pairs an expert
     // and more: tiles of 128 rows
     if (pairs <= 4LL * a.E) return moe_tc_products<16>(a, pairs, s);

@@ -1951,7 +1951,8 @@ class _MoeArgs(ctypes.Structure):
                 ("keep_groups", _I), ("limit", _F), ("slope", _F), ("score_fn", _I),
                 ("weigh_input", _I), ("up_offset", _F), ("router_bias", _P), ("group_top2", _I),
                 ("normalize", _I), ("weight_scale", _F), ("ws_up", _P), ("ws_down", _P), ("act_s", _P),
-                ("Fs", _I), ("route_only", _I)]
+                ("Fs", _I), ("small", _I), ("early", _I),
+                ("stage_router", _I), ("route_only", _I)]
 
 
 class _MoePairArgs(ctypes.Structure):

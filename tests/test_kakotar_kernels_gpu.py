@@ -599,7 +599,7 @@ def _moe(m, dtype, seed=0, correction=None):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("T", [1, 5, 70, 600])
+@pytest.mark.parametrize("T", [1, 5, 33, 70, 600])
 @pytest.mark.parametrize("m", MOE_SHAPES)
 def test_ungated_experts_groups_and_the_shared_expert(monkeypatch, dtype, T, m):
     """Choice scores that are mostly negative (a dropped group must count as minus infinity, not as
@@ -625,7 +625,7 @@ def test_ungated_experts_groups_and_the_shared_expert(monkeypatch, dtype, T, m):
     ops.check_kernel_errors()
 
 
-@pytest.mark.parametrize("T", [1, 130, 700])
+@pytest.mark.parametrize("T", [1, 12, 64, 130, 700])
 @pytest.mark.parametrize("shape", [(6, 2, 24, 64, 0, 0), (3, 3, 200, 96, 2, 1), (1, 1, 136, 40, 0, 0), (40, 4, 72, 264, 0, 1)])
 def test_experts_on_pairs_of_SMs_and_in_tiles_agree(T, shape):
     """The grouped product on pairs of SMs against the tile kernels, gated and ungated, with a clamp, an
