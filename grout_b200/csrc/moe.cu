@@ -82,6 +82,134 @@ struct MoeArgs {
 #define MOE_ROUTE_THREADS 256
 #define MOE_ROUTE_CHUNK 8     // router outputs whose sums a thread carries side by side
 
+// What one warp does with a token's logits z [n_all]: turns them into scores, chooses, and writes
+// the choices and their weights.  c [n_all] and gval [n_groups] are shared-memory scratch.
+__device__ __forceinline__ void moe_choose(const MoeArgs& a, float* z, float* c, float* gval, int t, int lane) {
+  const int n_all = a.E + a.n_identity;
+  if (a.score_fn == 1) {
+    for (int e = lane; e < n_all; e += 32) z[e] = 1.0f / (1.0f + expf(-z[e]));
+  } else if (a.score_fn == 0) {
+    float mx = -INFINITY, sum = 0.f;
+    for (int e = lane; e < n_all; e += 32) mx = fmaxf(mx, z[e]);
+    mx = warp_max(mx);
+    for (int e = lane; e < n_all; e += 32) { z[e] = expf(z[e] - mx); sum += z[e]; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < n_all; e += 32) z[e] = z[e] / sum;
+  }   // score_fn 2: the logits themselves choose; the chosen ones' weights are worked out below
+  for (int e = lane; e < n_all; e += 32) c[e] = z[e] + (a.correction ? a.correction[e] : 0.f);
+  __syncwarp();
+  if (a.n_groups > 1 && a.keep_groups < a.n_groups) {
+    const int per = n_all / a.n_groups;
+    for (int g = lane; g < a.n_groups; g += 32) {
+      float b1 = -INFINITY, b2 = -INFINITY;           // the group's two largest
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float v = c[e];
+        b2 = fmaxf(b2, fminf(b1, v));
+        b1 = fmaxf(b1, v);
+      }
+      gval[g] = a.group_top2 && per > 1 ? b1 + b2 : b1;
+    }
+    __syncwarp();
+    // a group that `keep_groups` others come before (larger, or equal and earlier) is dropped
+    for (int g = lane; g < a.n_groups; g += 32) {
+      const float v = gval[g];
+      int before = 0;
+      for (int o = 0; o < a.n_groups; ++o) before += gval[o] > v || (gval[o] == v && o < g);
+      if (before >= a.keep_groups)
+        for (int e = g * per; e < (g + 1) * per; ++e) c[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  float chosen_sum = 0.f, first_z = 0.f;
+  for (int j = 0; j < a.top; ++j) {   // the largest first; of equal ones the earlier
+    float bv = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < n_all; e += 32) {         // (one that is taken is NaN: no comparison holds)
+      const float v = c[e];
+      if (v > bv || (v == bv && e < bi)) { bv = v; bi = e; }
+    }
+  #pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+    }
+    const int best = bi < n_all ? bi : 0;
+    const float w = z[best];
+    if (j == 0) first_z = w;
+    chosen_sum += a.score_fn == 2 ? expf(w - first_z) : w;   // (the first logit is the largest)
+    __syncwarp();
+    if (lane == 0) {
+      c[best] = NAN;                  // taken
+      a.ids[(size_t)t * a.top + j] = best;
+      a.wts[(size_t)t * a.top + j] = w;
+    }
+    __syncwarp();
+  }
+  if (lane == 0) {
+    float* w = a.wts + (size_t)t * a.top;
+    for (int j = 0; j < a.top; ++j) {
+      // softmax over the chosen logits alone, or the scores, as they are or as shares of their sum
+      const float v = a.score_fn == 2 ? expf(w[j] - first_z) / chosen_sum
+                      : a.normalize   ? w[j] / (chosen_sum + 1e-20f) : w[j];
+      w[j] = v * a.weight_scale;
+    }
+  }
+}
+
+// What the block that finishes last does: the counts become the list of pairs ordered by
+// expert.  cnt and off [E] are shared-memory scratch; the counts and the blocks' tickets are
+// left at zero for the next call.
+__device__ __forceinline__ void moe_order_pairs(const MoeArgs& a, int* cnt, int* off) {
+  const int tid = threadIdx.x, lane = tid & 31, nt = blockDim.x;
+  for (int e = tid; e < a.E; e += nt) cnt[e] = __ldcg(&a.counts[e]);   // (all requested at once)
+  __syncthreads();
+  if (tid < 32) {                                      // exclusive sums, 32 experts a turn
+    int run = 0;
+    for (int e0 = 0; e0 < a.E; e0 += 32) {
+      const int c0 = e0 + lane < a.E ? cnt[e0 + lane] : 0;
+      int v = c0;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int u = __shfl_up_sync(0xffffffffu, v, o);
+        if (lane >= o) v += u;
+      }
+      if (e0 + lane < a.E) {
+        off[e0 + lane] = run + v - c0;
+        a.offsets[e0 + lane] = run + v - c0;
+      }
+      run += __shfl_sync(0xffffffffu, v, 31);
+    }
+    if (lane == 0) a.offsets[a.E] = run;
+  }
+  __syncthreads();
+  const int n_pairs = a.T * a.top;
+  for (int p0 = tid; p0 < n_pairs; p0 += 8 * nt) {     // eight pairs' loads are requested together
+    int e[8], r[8];
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+      const int p = p0 + u * nt < n_pairs ? p0 + u * nt : p0;
+      e[u] = __ldcg(&a.ids[p]), r[u] = __ldcg(&a.rank[p]);
+    }
+#pragma unroll
+    for (int u = 0; u < 8; ++u)
+      if (p0 + u * nt < n_pairs && e[u] < a.E) a.perm[off[e[u]] + r[u]] = p0 + u * nt;
+  }
+  for (int e = tid; e <= a.E; e += nt) a.counts[e] = 0;
+}
+
+// True in every thread of the block that draws the last ticket of the grid (counts[E]): every
+// block publishes its choices before it draws, so the last one sees all of them.
+__device__ __forceinline__ bool moe_last_block(const MoeArgs& a) {
+  __shared__ int is_last;
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) is_last = atomicAdd(&a.counts[a.E], 1) == (int)gridDim.x - 1;
+  __syncthreads();
+  if (is_last) __threadfence();
+  return is_last != 0;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeArgs a) {
   extern __shared__ float sm[];   // z [n_all], c [n_all], a score per group
@@ -135,84 +263,15 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
     __syncthreads();
   }
   if (warp == 0) {        // one warp turns logits into scores and chooses
-    if (a.score_fn == 1) {
-      for (int e = lane; e < n_all; e += 32) z[e] = 1.0f / (1.0f + expf(-z[e]));
-    } else if (a.score_fn == 0) {
-      float mx = -INFINITY, sum = 0.f;
-      for (int e = lane; e < n_all; e += 32) mx = fmaxf(mx, z[e]);
-      mx = warp_max(mx);
-      for (int e = lane; e < n_all; e += 32) { z[e] = expf(z[e] - mx); sum += z[e]; }
-      sum = warp_sum(sum);
-      for (int e = lane; e < n_all; e += 32) z[e] = z[e] / sum;
-    }   // score_fn 2: the logits themselves choose; the chosen ones' weights are worked out below
-    for (int e = lane; e < n_all; e += 32) c[e] = z[e] + (a.correction ? a.correction[e] : 0.f);
-    __syncwarp();
-    if (a.n_groups > 1 && a.keep_groups < a.n_groups) {
-      const int per = n_all / a.n_groups;
-      for (int g = lane; g < a.n_groups; g += 32) {
-        float b1 = -INFINITY, b2 = -INFINITY;           // the group's two largest
-        for (int e = g * per; e < (g + 1) * per; ++e) {
-          const float v = c[e];
-          b2 = fmaxf(b2, fminf(b1, v));
-          b1 = fmaxf(b1, v);
-        }
-        gval[g] = a.group_top2 && per > 1 ? b1 + b2 : b1;
-      }
-      __syncwarp();
-      // a group that `keep_groups` others come before (larger, or equal and earlier) is dropped
-      for (int g = lane; g < a.n_groups; g += 32) {
-        const float v = gval[g];
-        int before = 0;
-        for (int o = 0; o < a.n_groups; ++o) before += gval[o] > v || (gval[o] == v && o < g);
-        if (before >= a.keep_groups)
-          for (int e = g * per; e < (g + 1) * per; ++e) c[e] = -INFINITY;
-      }
-      __syncwarp();
-    }
-    float chosen_sum = 0.f, first_z = 0.f;
-    for (int j = 0; j < a.top; ++j) {   // the largest first; of equal ones the earlier
-      float bv = -INFINITY;
-      int bi = 0x7fffffff;
-      for (int e = lane; e < n_all; e += 32) {         // (one that is taken is NaN: no comparison holds)
-        const float v = c[e];
-        if (v > bv || (v == bv && e < bi)) { bv = v; bi = e; }
-      }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-        if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
-      }
-      const int best = bi < n_all ? bi : 0;
-      const float w = z[best];
-      if (j == 0) first_z = w;
-      chosen_sum += a.score_fn == 2 ? expf(w - first_z) : w;   // (the first logit is the largest)
-      __syncwarp();
-      if (lane == 0) {
-        c[best] = NAN;                  // taken
-        a.ids[(size_t)t * a.top + j] = best;
-        a.wts[(size_t)t * a.top + j] = w;
-      }
-      __syncwarp();
-    }
-    if (lane == 0) {
-      float* w = a.wts + (size_t)t * a.top;
-      for (int j = 0; j < a.top; ++j) {
-        // softmax over the chosen logits alone, or the scores, as they are or as shares of their sum
-        const float v = a.score_fn == 2 ? expf(w[j] - first_z) / chosen_sum
-                        : a.normalize   ? w[j] / (chosen_sum + 1e-20f) : w[j];
-        w[j] = v * a.weight_scale;
-      }
-    }
+    moe_choose(a, z, c, gval, t, lane);
   }
   if (a.small && a.n_identity == 0) return;          // the products' blocks read the choices themselves
   __syncthreads();
-  if (!a.small) {
-  for (int j = tid; j < a.top; j += blockDim.x) {   // the choices' places among their experts' pairs
-    const int e = a.ids[(size_t)t * a.top + j];
-    a.rank[(size_t)t * a.top + j] = e < a.E ? atomicAdd(&a.counts[e], 1) : -1;
-  }
-  }
+  if (!a.small)
+    for (int j = tid; j < a.top; j += blockDim.x) {   // the choices' places among their experts' pairs
+      const int e = a.ids[(size_t)t * a.top + j];
+      a.rank[(size_t)t * a.top + j] = e < a.E ? atomicAdd(&a.counts[e], 1) : -1;
+    }
   pdl_launch_dependents_if_large();
   for (int j = 0; j < a.top; ++j) {     // experts that hand their input on
     if (a.ids[(size_t)t * a.top + j] < a.E) continue;
@@ -221,47 +280,115 @@ __global__ void __launch_bounds__(MOE_ROUTE_THREADS) moe_route_kernel(const MoeA
     for (int i = tid; i < W; i += blockDim.x) o[i] = w * to_f32<T>(x[i]);
   }
   if (a.small) return;
-  // The block that finishes last turns the counts into the list of pairs ordered by expert:
-  // every block publishes its choices, then draws a ticket (counts[E]); the one that draws
-  // the last ticket sees all of them.  It leaves the counts and the ticket at zero for the
-  // next call.
-  __shared__ int is_last;
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) is_last = atomicAdd(&a.counts[a.E], 1) == (int)gridDim.x - 1;
-  __syncthreads();
-  if (!is_last) return;
-  __threadfence();
-  // (all counts are requested at once; the choices' shared memory holds them and their offsets)
-  int* cnt = reinterpret_cast<int*>(sm);               // [E]
-  int* off = cnt + a.E;                                // [E]
-  for (int e = tid; e < a.E; e += blockDim.x) cnt[e] = __ldcg(&a.counts[e]);
-  __syncthreads();
-  if (warp == 0) {                                     // exclusive sums, 32 experts a turn
-    int run = 0;
-    for (int e0 = 0; e0 < a.E; e0 += 32) {
-      const int c0 = e0 + lane < a.E ? cnt[e0 + lane] : 0;
-      int v = c0;
+  if (!moe_last_block(a)) return;
+  int* cnt = reinterpret_cast<int*>(sm);               // (the choices' shared memory is free)
+  moe_order_pairs(a, cnt, cnt + a.E);
+}
+
+// The same for many rows: the block brings eight router rows at a time into shared memory, a
+// warp makes the logits of TPW tokens side by side (four neighbouring elements a lane) and
+// chooses for one after the other; the block counts its choices per expert in shared memory and adds them to the
+// experts' counts in one go.
+#define MOE_ROWS_WARPS 8
+template <typename T> __device__ __forceinline__ void moe_load4(const T* p, float (&v)[4]);
+template <> __device__ __forceinline__ void moe_load4<float>(const float* p, float (&v)[4]) {
+  const float4 x = *reinterpret_cast<const float4*>(p);
+  v[0] = x.x, v[1] = x.y, v[2] = x.z, v[3] = x.w;
+}
+template <> __device__ __forceinline__ void moe_load4<bf16>(const bf16* p, float (&v)[4]) {
+  const uint2 x = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&x.x), b = *reinterpret_cast<const __nv_bfloat162*>(&x.y);
+  v[0] = __low2float(a), v[1] = __high2float(a), v[2] = __low2float(b), v[3] = __high2float(b);
+}
+
+template <typename T, int TPW>
+__global__ void __launch_bounds__(MOE_ROWS_WARPS * 32) moe_route_rows_kernel(const MoeArgs a) {
+  extern __shared__ float sm[];
+  pdl_launch_dependents_if_small();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int n_all = a.E + a.n_identity, W = a.W, top = a.top;
+  const int per_tok = 2 * n_all + a.n_groups;
+  float* mine = sm + (size_t)warp * TPW * per_tok;
+  int* cnt = reinterpret_cast<int*>(sm + (size_t)MOE_ROWS_WARPS * TPW * per_tok);   // [E]
+  int* base = cnt + a.E;                                                            // [E]
+  float* rs = sm + (((size_t)MOE_ROWS_WARPS * TPW * per_tok + 2 * a.E + 3) & ~(size_t)3);   // [MOE_ROUTE_CHUNK, W]
+  auto stage = [&](int e0) {       // (no kernel's output)
+    const int n = min(MOE_ROUTE_CHUNK, n_all - e0) * W;
+    for (int i = tid * 4; i < n; i += MOE_ROWS_WARPS * 32 * 4) cp_async16(rs + i, a.router_w + (size_t)e0 * W + i, true);
+    cp_async_commit();
+  };
+  stage(0);
+  for (int e = tid; e < a.E; e += blockDim.x) cnt[e] = 0;
+  pdl_wait();
+  const int t0 = (blockIdx.x * MOE_ROWS_WARPS + warp) * TPW;
+  const T* x = (const T*)a.x;
+  for (int e0 = 0; e0 < n_all; e0 += MOE_ROUTE_CHUNK) {
+    float acc[TPW][MOE_ROUTE_CHUNK];
 #pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const int u = __shfl_up_sync(0xffffffffu, v, o);
-        if (lane >= o) v += u;
-      }
-      if (e0 + lane < a.E) {
-        off[e0 + lane] = run + v - c0;
-        a.offsets[e0 + lane] = run + v - c0;
-      }
-      run += __shfl_sync(0xffffffffu, v, 31);
+    for (int k = 0; k < TPW; ++k)
+#pragma unroll
+      for (int u = 0; u < MOE_ROUTE_CHUNK; ++u) acc[k][u] = 0.f;
+    if (e0) {
+      __syncthreads();             // everyone is done with the rows before these
+      stage(e0);
     }
-    if (lane == 0) a.offsets[a.E] = run;
+    cp_async_wait<0>();
+    __syncthreads();
+    const int last = min(MOE_ROUTE_CHUNK, n_all - e0) - 1;
+#pragma unroll 4
+    for (int i = lane * 4; i < W; i += 128) {
+      float xv[TPW][4];
+#pragma unroll
+      for (int k = 0; k < TPW; ++k) moe_load4<T>(x + (size_t)min(t0 + k, a.T - 1) * W + i, xv[k]);
+#pragma unroll
+      for (int u = 0; u < MOE_ROUTE_CHUNK; ++u) {
+        const float4 w = *reinterpret_cast<const float4*>(rs + (size_t)min(u, last) * W + i);
+#pragma unroll
+        for (int k = 0; k < TPW; ++k)
+          acc[k][u] = fmaf(xv[k][3], w.w, fmaf(xv[k][2], w.z, fmaf(xv[k][1], w.y, fmaf(xv[k][0], w.x, acc[k][u]))));
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < TPW; ++k)
+#pragma unroll
+      for (int u = 0; u < MOE_ROUTE_CHUNK; ++u) {
+        const float v = warp_sum(acc[k][u]);
+        if (lane == 0 && e0 + u < n_all)
+          mine[k * per_tok + e0 + u] = v + (a.router_bias ? a.router_bias[e0 + u] : 0.f);
+      }
   }
   __syncthreads();
-  const int n_pairs = a.T * a.top;
-  for (int p = tid; p < n_pairs; p += blockDim.x) {
-    const int e = __ldcg(&a.ids[p]), r = __ldcg(&a.rank[p]);
-    if (e < a.E) a.perm[off[e] + r] = p;
+  for (int k = 0; k < TPW; ++k) {
+    const int t = t0 + k;
+    if (t >= a.T) break;
+    float* z = mine + k * per_tok;
+    moe_choose(a, z, z + n_all, z + 2 * n_all, t, lane);
+    __syncwarp();
+    for (int j = lane; j < top; j += 32) {             // the pair's place among the block's for its expert
+      const int e = a.ids[(size_t)t * top + j];
+      a.rank[(size_t)t * top + j] = e < a.E ? atomicAdd(&cnt[e], 1) : -1;
+    }
   }
-  for (int e = tid; e <= a.E; e += blockDim.x) a.counts[e] = 0;
+  __syncthreads();
+  for (int e = tid; e < a.E; e += blockDim.x) base[e] = cnt[e] ? atomicAdd(&a.counts[e], cnt[e]) : 0;
+  __syncthreads();
+  for (int k = 0; k < TPW; ++k) {
+    const int t = t0 + k;
+    if (t >= a.T) break;
+    for (int j = lane; j < top; j += 32) {
+      const int e = a.ids[(size_t)t * top + j];
+      if (e < a.E) a.rank[(size_t)t * top + j] += base[e];
+    }
+    for (int j = 0; j < top; ++j) {                    // experts that hand their input on
+      if (a.ids[(size_t)t * top + j] < a.E) continue;
+      const float w = a.wts[(size_t)t * top + j];
+      float* o = a.out + ((size_t)j * a.T + t) * W;
+      for (int i = lane; i < W; i += 32) o[i] = w * to_f32<T>(x[(size_t)t * W + i]);
+    }
+  }
+  pdl_launch_dependents_if_large();
+  if (!moe_last_block(a)) return;
+  moe_order_pairs(a, cnt, base);
 }
 
 #define MOE_BM 16
@@ -709,7 +836,24 @@ static int moe_forward(MoeArgs a, cudaStream_t s) {
     if (ce != cudaSuccess) return (int)ce;
     raised = true;
   }
-  e = gb_launch(moe_route_kernel<T>, dim3(a.T), dim3(MOE_ROUTE_THREADS), a.stage_router ? staged : choice, s, a);
+  const int TPW = 2;
+  const size_t by_rows = ((MOE_ROWS_WARPS * TPW * choice + (size_t)2 * a.E * sizeof(int) + 15) & ~(size_t)15) +
+                         (size_t)(n_all < MOE_ROUTE_CHUNK ? n_all : MOE_ROUTE_CHUNK) * a.W * sizeof(float);
+  static bool raised_rows = false;
+  // (its logits are summed in another order; in the 32-bit path a token's are the same to the bit
+  // whatever the step brings, so that path keeps to the kernel of a block a token)
+  if (sizeof(T) == 2 && a.T > 64 && a.W % 4 == 0 && (((uintptr_t)a.router_w | (uintptr_t)a.x) & 15) == 0 &&
+      by_rows <= 200 * 1024) {
+    if (!raised_rows) {
+      cudaError_t ce = cudaFuncSetAttribute(moe_route_rows_kernel<T, TPW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+      if (ce != cudaSuccess) return (int)ce;
+      raised_rows = true;
+    }
+    e = gb_launch(moe_route_rows_kernel<T, TPW>, dim3((a.T + MOE_ROWS_WARPS * TPW - 1) / (MOE_ROWS_WARPS * TPW)),
+                  dim3(MOE_ROWS_WARPS * 32), by_rows, s, a);
+  } else {
+    e = gb_launch(moe_route_kernel<T>, dim3(a.T), dim3(MOE_ROUTE_THREADS), a.stage_router ? staged : choice, s, a);
+  }
   if (e || a.route_only) return e;
   // the most tiles the pairs can make: every expert may end in a tile that is not full
   if (tensor_cores) {

@@ -73,15 +73,23 @@ static constexpr size_t MP_SMEM = (size_t)MP_STAGES * MP_STAGE_BYTES + 1024 + 25
 static constexpr uint32_t MP_IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(MP_BN >> 3) << 17) |
                                      ((uint32_t)(256 >> 4) << 24);
 
+#define MP_GATHER_ROWS 4   // rows a block copies side by side: that many loads of a thread under way
 __global__ void __launch_bounds__(128) moe_gather_kernel(const MoePairArgs a) {
   pdl_launch_dependents_if_small();
   pdl_wait();
-  const int i = blockIdx.x;
-  if (i < a.offsets[a.E]) {
-    const int n = a.W / 8;
-    const uint4* src = reinterpret_cast<const uint4*>((const bf16*)a.x + (size_t)(a.perm[i] / a.top) * a.W);
-    uint4* dst = reinterpret_cast<uint4*>((bf16*)a.xg + (size_t)i * a.W);
-    for (int c = threadIdx.x; c < n; c += blockDim.x) dst[c] = src[c];
+  const int i0 = blockIdx.x * MP_GATHER_ROWS, n = a.W / 8, listed = a.offsets[a.E];
+  const uint4* src[MP_GATHER_ROWS];
+#pragma unroll
+  for (int r = 0; r < MP_GATHER_ROWS; ++r)
+    src[r] = reinterpret_cast<const uint4*>((const bf16*)a.x + (size_t)(i0 + r < listed ? a.perm[i0 + r] / a.top : 0) * a.W);
+  uint4* dst = reinterpret_cast<uint4*>((bf16*)a.xg + (size_t)i0 * a.W);
+  for (int c = threadIdx.x; c < n; c += blockDim.x) {
+    uint4 v[MP_GATHER_ROWS];
+#pragma unroll
+    for (int r = 0; r < MP_GATHER_ROWS; ++r) v[r] = src[r][c];
+#pragma unroll
+    for (int r = 0; r < MP_GATHER_ROWS; ++r)
+      if (i0 + r < listed) dst[(size_t)r * n + c] = v[r];
   }
   pdl_launch_dependents_if_large();
 }
@@ -413,7 +421,7 @@ GB_EXPORT int gb_moe_pair_bf16(const MoePairArgs* args, cudaStream_t s) {
     if (e != cudaSuccess) return (int)e;
   }
   if (sms < 2) return GB_ERR_UNSUPPORTED;
-  int e = gb_launch(moe_gather_kernel, dim3((unsigned)(a.T * a.top)), dim3(128), 0, s, a);
+  int e = gb_launch(moe_gather_kernel, dim3((unsigned)((a.T * a.top + MP_GATHER_ROWS - 1) / MP_GATHER_ROWS)), dim3(128), 0, s, a);
   if (e) return e;
   e = a.w_gate ? launch<MP_GATED>(a, sms, s) : launch<MP_UNGATED>(a, sms, s);
   if (e) return e;

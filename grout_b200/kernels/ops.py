@@ -1966,10 +1966,13 @@ _TC_ERROR_NAMES.update({141: "the experts' MMA lane waited 2 s for a stage that 
                         142: "the experts' loads waited 2 s for a stage that was never released",
                         143: "the experts' epilogue waited 2 s for an accumulator",
                         144: "the experts' MMA lane waited 2 s for an accumulator to be drained"})
-# From how many (token, choice) pairs an expert on the products run on pairs of SMs
-# ("auto"); "pair" takes them wherever the sizes allow, "tiles" never.
+# Which kernels the experts' products run on: "auto" takes the grouped product on pairs of SMs
+# with more than MOE_PAIR_ROWS (token, choice) pairs an expert and the tile kernels below,
+# "pair" and "tiles" the one wherever the sizes allow.  Measured (us for both products with
+# the routing, tiles / pair; 8 experts of 3,648 x 2,560, two a token): 16 tokens 80 / 99, 32 tokens
+# 122 / 98, 256 249 / 112, 2,048 768 / 223; gated 16 tokens 100 / 134, 32 167 / 136, 2,048 980 / 290.
 MOE_PRODUCTS = "auto"
-MOE_PAIR_ROWS = 64
+MOE_PAIR_ROWS = 4
 
 
 def moe_tensor_cores_take(W: int, F: int, Fs: int = 0) -> bool:
@@ -2074,7 +2077,7 @@ def moe_forward(x: torch.Tensor, router_w: torch.Tensor, correction: Optional[to
         act_s = torch.empty((T, Fs), dtype=x.dtype, device=dev)
         a.ws_up, a.ws_down, a.act_s, a.Fs = shared[0].data_ptr(), shared[1].data_ptr(), act_s.data_ptr(), Fs
     pair = (x.dtype == torch.bfloat16 and T > 0 and moe_tensor_cores_take(W, F, Fs) and MOE_PRODUCTS != "tiles"
-            and (MOE_PRODUCTS == "pair" or T * top >= MOE_PAIR_ROWS * E))
+            and (MOE_PRODUCTS == "pair" or T * top > MOE_PAIR_ROWS * E))
     a.route_only = int(pair)
     _check(_fn("moe", f"gb_moe_forward_{_suffix(x.dtype)}", "pp")(ctypes.addressof(a), _stream()),
            "moe_forward", 1 if pair else 3)
