@@ -7,8 +7,9 @@
 // s = rows[r] when a row list is given (the gather before the last norm), else r.  Every
 // element stands for itself: there is nothing to sum over a row, so a row is cut into as
 // many blocks as keep the GPU busy and no block waits for another.  A thread takes four
-// neighbouring elements (one where the width or an address does not allow that); the order
-// in which partial sums are added depends on nothing but their number.
+// neighbouring elements of a row, or of four rows (one element where the width or an address
+// does not allow that); the order in which partial sums are added depends on nothing but
+// their number.
 #include "common.cuh"
 
 struct DytArgs {
@@ -51,10 +52,13 @@ template <> __device__ __forceinline__ void store4<bf16>(bf16* p, const float (&
 
 #define DYT_THREADS 128
 
-template <typename T>
+// ROWS rows a thread, one after the other in memory, with PU partial sums of each requested at
+// once: a step of many rows keeps more loads under way per thread (one row a thread left the
+// kernel waiting for memory in waves), a step of few spreads its rows over the blocks.
+template <typename T, int ROWS, int PU>
 __global__ void __launch_bounds__(DYT_THREADS) add_dyt_vec_kernel(const DytArgs a) {
   pdl_launch_dependents_if_small();
-  const int N = a.N, i = (blockIdx.y * DYT_THREADS + threadIdx.x) * 4, r = blockIdx.x;
+  const int N = a.N, i = (blockIdx.y * DYT_THREADS + threadIdx.x) * 4, r0 = blockIdx.x * ROWS;
   float wv[4], bv[4], alpha = 0.f;
   if (i < N) {                    // no kernel's output: before the wait
     alpha = *a.alpha;
@@ -63,33 +67,47 @@ __global__ void __launch_bounds__(DYT_THREADS) add_dyt_vec_kernel(const DytArgs 
   }
   pdl_wait();
   if (i < N) {
-    const size_t s = a.rows ? (size_t)a.rows[r] : (size_t)r;
-    float v[4] = {0.f, 0.f, 0.f, 0.f}, d[4] = {0.f, 0.f, 0.f, 0.f};
-    if (a.res_in) load4<float>(a.res_in + s * N + i, v);
-    if (a.delta) load4<T>((const T*)a.delta + s * N + i, d);
-    if (a.parts) {
-      const float* p = a.parts + s * N + i;
-      for (int k0 = 0; k0 < a.n_parts; k0 += 8) {   // eight requested at once, added in order
-        float pk[8][4];
+    float v[ROWS][4], d[ROWS][4];
+    size_t at[ROWS];
 #pragma unroll
-        for (int u = 0; u < 8; ++u)
-          if (k0 + u < a.n_parts) load4<float>(p + (size_t)(k0 + u) * a.part_stride, pk[u]);
+    for (int k = 0; k < ROWS; ++k) {
+      const int r = min(r0 + k, a.n_rows - 1);
+      at[k] = (a.rows ? (size_t)a.rows[r] : (size_t)r) * N + i;
 #pragma unroll
-        for (int u = 0; u < 8; ++u)
-          if (k0 + u < a.n_parts) {
+      for (int e = 0; e < 4; ++e) v[k][e] = d[k][e] = 0.f;
+      if (a.res_in) load4<float>(a.res_in + at[k], v[k]);
+      if (a.delta) load4<T>((const T*)a.delta + at[k], d[k]);
+    }
+    for (int k0 = 0; k0 < a.n_parts; k0 += PU) {   // PU of them requested at once, added in order
+      float pk[PU][ROWS][4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) d[e] += pk[u][e];
-          }
+      for (int u = 0; u < PU; ++u)
+        if (k0 + u < a.n_parts) {
+#pragma unroll
+          for (int k = 0; k < ROWS; ++k) load4<float>(a.parts + (size_t)(k0 + u) * a.part_stride + at[k], pk[u][k]);
+        }
+#pragma unroll
+      for (int u = 0; u < PU; ++u)
+        if (k0 + u < a.n_parts) {
+#pragma unroll
+          for (int k = 0; k < ROWS; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) d[k][e] += pk[u][k][e];
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < ROWS; ++k) {
+      if (r0 + k >= a.n_rows) break;
+      float o[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        v[k][e] += d[k][e];
+        o[e] = tanhf(alpha * v[k][e]) * wv[e] + bv[e];
       }
+      const size_t to = (size_t)(r0 + k) * N + i;
+      if (a.res_out) store4<float>(a.res_out + to, v[k]);
+      store4<T>((T*)a.y + to, o);
     }
-    float o[4];
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      v[e] += d[e];
-      o[e] = tanhf(alpha * v[e]) * wv[e] + bv[e];
-    }
-    if (a.res_out) store4<float>(a.res_out + (size_t)r * N + i, v);
-    store4<T>((T*)a.y + (size_t)r * N + i, o);
   }
   pdl_launch_dependents_if_large();
 }
@@ -124,8 +142,10 @@ static int launch(const DytArgs& a, cudaStream_t s) {
   const int per = vec ? 4 * DYT_THREADS : DYT_THREADS;
   const long long gy = ((long long)a.N + per - 1) / per;
   if (gy > 65535) return GB_ERR_UNSUPPORTED;
+  if (vec && a.n_rows >= 512)
+    return gb_launch(add_dyt_vec_kernel<T, 4, 3>, dim3((a.n_rows + 3) / 4, (unsigned)gy), dim3(DYT_THREADS), 0, s, a);
   const dim3 grid(a.n_rows, (unsigned)gy);
-  return vec ? gb_launch(add_dyt_vec_kernel<T>, grid, dim3(DYT_THREADS), 0, s, a)
+  return vec ? gb_launch(add_dyt_vec_kernel<T, 1, 8>, grid, dim3(DYT_THREADS), 0, s, a)
              : gb_launch(add_dyt_kernel<T>, grid, dim3(DYT_THREADS), 0, s, a);
 }
 

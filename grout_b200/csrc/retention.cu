@@ -33,13 +33,16 @@
 // sum_t decay^(rows-1-t) k_t v_t^T.  `prefix` turns those into the states at the chunks'
 // starts (S <- decay^rows S + added, in the chunks' order) and stores the last; `cross`
 // adds decay^(j+1) S_start^T q to row j of every chunk, a tiled 32-bit product too.  The
-// recurrence is linear, so this is the same sum in another order.
+// recurrence is linear, so this is the same sum in another order.  Heads of 64 or 128 keys and
+// values take `chunk` and `cross` in a form that brings the chunk's rows (and the state it
+// starts from) into shared memory whole, skips what the mask hides and keeps larger tiles of
+// sums in registers.
 //
 // A step in which every sequence brings one row (decoding) is one kernel, `step`:
 // a block owns one (sequence, head), turns the row's q and k itself, streams the
 // head's whole state through once (a warp reads and writes whole rows of S), adds
 // up the warps' partial read-outs in shared memory and finishes the head.
-#include "common.cuh"
+#include "attn_mma.cuh"   // cp_async16
 
 struct RetentionArgs {
   const float* proj;      // [T, 2 H dk + 2 H dv]
@@ -352,6 +355,155 @@ __global__ void __launch_bounds__(256) retention_chunk_kernel(const RetentionArg
   pdl_launch_dependents_if_large();
 }
 
+// The same for heads of DK keys and DV values (64 or 128 each): the chunk's q, k and v come whole,
+// by asynchronous 16-byte copies.  Rows of q and k are DK + 4 floats apart, so that sixteen rows
+// read at one column fall into different banks; P takes q's place once it is computed.  A
+// thread owns 4 x 4 elements of P (rows and columns sixteen apart, so that a group of them
+// above the diagonal is left out whole), 4 x DV/16 of the read-outs and DK/16 x DV/16 of what
+// the chunk adds to the state.
+template <int DK, int DV>
+__global__ void __launch_bounds__(256, 2) retention_chunk_tile_kernel(const RetentionArgs a) {
+  extern __shared__ __align__(16) float rc_sm[];
+  constexpr int LDK = DK + 4, LDP = RT_CT + 4, NK = DK / 64, NV = DV / 64;
+  float* Qs = rc_sm;                       // [64][LDK]
+  float* Ks = Qs + RT_CT * LDK;            // [64][LDK]
+  float* Vs = Ks + RT_CT * LDK;            // [64][DV]
+  float* dpow = Vs + RT_CT * DV;           // decay^0 .. decay^64
+  float* PsT = Qs;                         // [key row][LDP query rows]
+  pdl_launch_dependents_if_small();
+  const int tid = threadIdx.x, ty = tid / 16, tx = tid % 16;
+  const int h = blockIdx.x, seq = blockIdx.y, z = blockIdx.z, H = a.H;
+  const float decay = a.decay[h];
+  if (tid <= RT_CT) dpow[tid] = powf(decay, (float)tid);
+  pdl_wait();
+  const int first = a.cu_q[seq], n = a.cu_q[seq + 1] - first;
+  if (z * RT_CHUNK >= n) return;
+  const int rows = min(RT_CHUNK, n - z * RT_CHUNK), r0 = first + z * RT_CHUNK;
+  for (int i = tid; i < RT_CT * DK / 4; i += 256) {
+    const int m = i / (DK / 4), e = (i % (DK / 4)) * 4;
+    const bool ok = m < rows;
+    const float* src = ok ? a.qk + ((size_t)(r0 + m) * 2 * H + h) * DK + e : a.qk;
+    cp_async16(Qs + m * LDK + e, src, ok);
+    cp_async16(Ks + m * LDK + e, ok ? src + (size_t)H * DK : src, ok);
+  }
+  for (int i = tid; i < RT_CT * DV / 4; i += 256) {
+    const int m = i / (DV / 4), c = (i % (DV / 4)) * 4;
+    const bool ok = m < rows;
+    cp_async16(Vs + m * DV + c, ok ? rt_values(a, r0 + m, h) + c : a.qk, ok);
+  }
+  cp_async_commit();
+  cp_async_wait<0>();
+  __syncthreads();
+  {
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+#pragma unroll 2
+    for (int k = 0; k < DK; k += 4) {
+      float4 q[4], kk[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        q[i] = *reinterpret_cast<const float4*>(Qs + (ty + 16 * i) * LDK + k);
+        kk[i] = *reinterpret_cast<const float4*>(Ks + (tx + 16 * i) * LDK + k);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j <= i; ++j)
+          acc[i][j] = fmaf(q[i].w, kk[j].w, fmaf(q[i].z, kk[j].z, fmaf(q[i].y, kk[j].y, fmaf(q[i].x, kk[j].x, acc[i][j]))));
+    }
+    __syncthreads();                       // q has been read for the last time
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int qi = ty + 16 * i, kj = tx + 16 * j;
+        PsT[kj * LDP + qi] = kj <= qi ? acc[i][j] * dpow[qi - kj] : 0.f;
+      }
+    // k under the decay that is left of it at the chunk's end
+    for (int i = tid; i < RT_CT * DK / 4; i += 256) {
+      const int m = i / (DK / 4), e = (i % (DK / 4)) * 4;
+      if (m < rows) {
+        float4* k4 = reinterpret_cast<float4*>(Ks + m * LDK + e);
+        const float f = dpow[rows - 1 - m];
+        k4->x *= f, k4->y *= f, k4->z *= f, k4->w *= f;
+      }
+    }
+    __syncthreads();
+  }
+  {
+    float acc[4][4 * NV];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4 * NV; ++j) acc[i][j] = 0.f;
+    const int t_end = min(rows, ((tid >> 5) * 2 + 2) * 4);     // no row of this warp sees keys beyond
+#pragma unroll 4
+    for (int t = 0; t < t_end; ++t) {
+      const float4 p4 = *reinterpret_cast<const float4*>(PsT + t * LDP + ty * 4);
+      const float p[4] = {p4.x, p4.y, p4.z, p4.w};
+#pragma unroll
+      for (int nv = 0; nv < NV; ++nv) {
+        const float4 v = *reinterpret_cast<const float4*>(Vs + t * DV + nv * 64 + tx * 4);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          acc[i][nv * 4] = fmaf(p[i], v.x, acc[i][nv * 4]);
+          acc[i][nv * 4 + 1] = fmaf(p[i], v.y, acc[i][nv * 4 + 1]);
+          acc[i][nv * 4 + 2] = fmaf(p[i], v.z, acc[i][nv * 4 + 2]);
+          acc[i][nv * 4 + 3] = fmaf(p[i], v.w, acc[i][nv * 4 + 3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int m = ty * 4 + i;
+      if (m >= rows) continue;
+      float* o = a.o + ((size_t)(r0 + m) * H + h) * DV + tx * 4;
+#pragma unroll
+      for (int nv = 0; nv < NV; ++nv)
+        *reinterpret_cast<float4*>(o + nv * 64) =
+            make_float4(acc[i][nv * 4], acc[i][nv * 4 + 1], acc[i][nv * 4 + 2], acc[i][nv * 4 + 3]);
+    }
+  }
+  {
+    float acc[4 * NK][4 * NV];
+#pragma unroll
+    for (int i = 0; i < 4 * NK; ++i)
+#pragma unroll
+      for (int j = 0; j < 4 * NV; ++j) acc[i][j] = 0.f;
+#pragma unroll 2
+    for (int t = 0; t < rows; ++t) {
+      float kv[4 * NK], vv[4 * NV];
+#pragma unroll
+      for (int nk = 0; nk < NK; ++nk) {
+        const float4 k4 = *reinterpret_cast<const float4*>(Ks + t * LDK + nk * 64 + ty * 4);
+        kv[nk * 4] = k4.x, kv[nk * 4 + 1] = k4.y, kv[nk * 4 + 2] = k4.z, kv[nk * 4 + 3] = k4.w;
+      }
+#pragma unroll
+      for (int nv = 0; nv < NV; ++nv) {
+        const float4 v4 = *reinterpret_cast<const float4*>(Vs + t * DV + nv * 64 + tx * 4);
+        vv[nv * 4] = v4.x, vv[nv * 4 + 1] = v4.y, vv[nv * 4 + 2] = v4.z, vv[nv * 4 + 3] = v4.w;
+      }
+#pragma unroll
+      for (int i = 0; i < 4 * NK; ++i)
+#pragma unroll
+        for (int j = 0; j < 4 * NV; ++j) acc[i][j] = fmaf(kv[i], vv[j], acc[i][j]);
+    }
+    float* sp = a.chunk_state + (rt_entry(first, z, seq) * H + h) * (size_t)DK * DV + tx * 4;
+#pragma unroll
+    for (int i = 0; i < 4 * NK; ++i) {
+      const int e = (i >> 2) * 64 + ty * 4 + (i & 3);
+#pragma unroll
+      for (int nv = 0; nv < NV; ++nv)
+        *reinterpret_cast<float4*>(sp + (size_t)e * DV + nv * 64) =
+            make_float4(acc[i][nv * 4], acc[i][nv * 4 + 1], acc[i][nv * 4 + 2], acc[i][nv * 4 + 3]);
+    }
+  }
+  pdl_launch_dependents_if_large();
+}
+
 // The states at the chunks' starts: a thread owns one element of a (sequence, head)'s
 // matrix, walks the chunks in order, leaves in every chunk's entry the state the chunk
 // starts from in place of what the chunk adds, and stores the state after the last.
@@ -451,6 +603,74 @@ __global__ void __launch_bounds__(256) retention_cross_kernel(const RetentionArg
     for (int j = 0; j < 8; ++j) {
       const int c = c0 + (j < 4 ? tx * 4 + j : 64 + tx * 4 + j - 4);
       if (c < dv) o[c] = fmaf(f, acc[i][j], o[c]);
+    }
+  }
+}
+
+// The same for heads of DK keys and DV values: a block owns a whole chunk of one head, with its q
+// and the state it starts from in shared memory.
+template <int DK, int DV>
+__global__ void __launch_bounds__(256, 2) retention_cross_tile_kernel(const RetentionArgs a) {
+  extern __shared__ __align__(16) float rc_sm[];
+  constexpr int LDK = DK + 4, NV = DV / 64;
+  float* Qs = rc_sm;                       // [64][LDK]
+  float* Ss = Qs + RT_CT * LDK;            // [DK][DV]
+  pdl_launch_dependents_if_small();
+  const int tid = threadIdx.x, ty = tid / 16, tx = tid % 16;
+  const int h = blockIdx.x, seq = blockIdx.y, z = blockIdx.z, H = a.H;
+  const float decay = a.decay[h];
+  pdl_wait();
+  const int first = a.cu_q[seq], n = a.cu_q[seq + 1] - first;
+  if (z * RT_CHUNK >= n) return;
+  const int rows = min(RT_CHUNK, n - z * RT_CHUNK), r0 = first + z * RT_CHUNK;
+  const float* S = a.chunk_state + (rt_entry(first, z, seq) * H + h) * (size_t)DK * DV;
+  for (int i = tid; i < RT_CT * DK / 4; i += 256) {
+    const int m = i / (DK / 4), e = (i % (DK / 4)) * 4;
+    const bool ok = m < rows;
+    cp_async16(Qs + m * LDK + e, ok ? a.qk + ((size_t)(r0 + m) * 2 * H + h) * DK + e : a.qk, ok);
+  }
+  for (int i = tid * 4; i < DK * DV; i += 256 * 4) cp_async16(Ss + i, S + i, true);
+  cp_async_commit();
+  cp_async_wait<0>();
+  __syncthreads();
+  float acc[4][4 * NV];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4 * NV; ++j) acc[i][j] = 0.f;
+#pragma unroll 2
+  for (int k = 0; k < DK; k += 4) {
+    float4 q[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) q[i] = *reinterpret_cast<const float4*>(Qs + (ty + 16 * i) * LDK + k);
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk)
+#pragma unroll
+      for (int nv = 0; nv < NV; ++nv) {
+        const float4 s = *reinterpret_cast<const float4*>(Ss + (k + kk) * DV + nv * 64 + tx * 4);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float qv = kk == 0 ? q[i].x : kk == 1 ? q[i].y : kk == 2 ? q[i].z : q[i].w;
+          acc[i][nv * 4] = fmaf(qv, s.x, acc[i][nv * 4]);
+          acc[i][nv * 4 + 1] = fmaf(qv, s.y, acc[i][nv * 4 + 1]);
+          acc[i][nv * 4 + 2] = fmaf(qv, s.z, acc[i][nv * 4 + 2]);
+          acc[i][nv * 4 + 3] = fmaf(qv, s.w, acc[i][nv * 4 + 3]);
+        }
+      }
+  }
+  pdl_launch_dependents_if_large();
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = ty + 16 * i;
+    if (m >= rows) continue;
+    const float f = powf(decay, (float)(m + 1));
+    float* o = a.o + ((size_t)(r0 + m) * H + h) * DV + tx * 4;
+#pragma unroll
+    for (int nv = 0; nv < NV; ++nv) {
+      float4 v = *reinterpret_cast<const float4*>(o + nv * 64);
+      v.x = fmaf(f, acc[i][nv * 4], v.x), v.y = fmaf(f, acc[i][nv * 4 + 1], v.y);
+      v.z = fmaf(f, acc[i][nv * 4 + 2], v.z), v.w = fmaf(f, acc[i][nv * 4 + 3], v.w);
+      *reinterpret_cast<float4*>(o + nv * 64) = v;
     }
   }
 }
@@ -636,6 +856,34 @@ static int retention_scan_launch(const RetentionArgs& a, cudaStream_t s) {
                    dim3(RT_COLS * RT_LANES), 0, s, a);
 }
 
+// Whether the chunk and cross kernels of whole heads take these heads; then their launches.
+static bool retention_tiled(const RetentionArgs& a, int chunks) {
+  const uintptr_t all = (uintptr_t)a.qk | (uintptr_t)a.proj | (uintptr_t)a.v | (uintptr_t)a.o | (uintptr_t)a.chunk_state;
+  return (a.dk == 64 || a.dk == 128) && (a.dv == 64 || a.dv == 128) && (all & 15) == 0 && chunks <= 65535;
+}
+template <int DK, int DV>
+static int retention_tile_launch(const RetentionArgs& a, cudaStream_t s, int chunks, bool cross) {
+  const size_t smem = (size_t)(cross ? RT_CT * (DK + 4) + DK * DV : 2 * RT_CT * (DK + 4) + RT_CT * DV + RT_CT + 4) * sizeof(float);
+  static bool raised = false;    // more than the 48 KB a kernel gets without asking
+  if (!raised) {
+    const int most = 112 * 1024;
+    cudaError_t ce = cudaFuncSetAttribute(retention_chunk_tile_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
+    if (ce == cudaSuccess)
+      ce = cudaFuncSetAttribute(retention_cross_tile_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
+    if (ce != cudaSuccess) return (int)ce;
+    raised = true;
+  }
+  const dim3 grid(a.H, a.n_seqs, chunks);
+  return cross ? gb_launch(retention_cross_tile_kernel<DK, DV>, grid, dim3(256), smem, s, a)
+               : gb_launch(retention_chunk_tile_kernel<DK, DV>, grid, dim3(256), smem, s, a);
+}
+static int retention_tile(const RetentionArgs& a, cudaStream_t s, int chunks, bool cross) {
+  if (a.dk == 64) return a.dv == 64 ? retention_tile_launch<64, 64>(a, s, chunks, cross)
+                                    : retention_tile_launch<64, 128>(a, s, chunks, cross);
+  return a.dv == 64 ? retention_tile_launch<128, 64>(a, s, chunks, cross)
+                    : retention_tile_launch<128, 128>(a, s, chunks, cross);
+}
+
 static int retention_chunk_launch(const RetentionArgs& a, cudaStream_t s, int chunks) {
   const size_t smem = (size_t)(3 * RT_CT * RT_CT + 2 * RT_TK * RT_CT + RT_CT + 1) * sizeof(float);
   static bool raised = false;    // more than the 48 KB a kernel gets without asking
@@ -681,7 +929,9 @@ static int retention_forward(const RetentionArgs& a, cudaStream_t s) {
   int chunks = a.max_rows >= RT_CHUNK_MIN && a.chunk_state ? (a.max_rows + RT_CHUNK - 1) / RT_CHUNK : 0;
   if (chunks > 65535 || (long long)chunks * (RT_CHUNK / RT_TM) * ((a.dv + RT_TN - 1) / RT_TN) > 0x7fffffffLL) chunks = 0;
   const int kpl = (a.dk + RT_LANES - 1) / RT_LANES;
-  if (chunks) e = retention_chunk_launch(a, s, chunks);
+  const bool tiled = chunks && retention_tiled(a, chunks);
+  if (tiled) e = retention_tile(a, s, chunks, false);
+  else if (chunks) e = retention_chunk_launch(a, s, chunks);
   else if (kpl <= 1) e = retention_scan_launch<1>(a, s);
   else if (kpl <= 2) e = retention_scan_launch<2>(a, s);
   else if (kpl <= 4) e = retention_scan_launch<4>(a, s);
@@ -692,8 +942,9 @@ static int retention_forward(const RetentionArgs& a, cudaStream_t s) {
   if (chunks) {
     e = gb_launch(retention_prefix_kernel, dim3((a.dk * a.dv + 255) / 256, a.H, a.n_seqs), dim3(256), 0, s, a);
     if (e) return e;
-    e = gb_launch(retention_cross_kernel,
-                  dim3(chunks * (RT_CHUNK / RT_TM) * ((a.dv + RT_TN - 1) / RT_TN), a.H, a.n_seqs), dim3(256), 0, s, a);
+    e = tiled ? retention_tile(a, s, chunks, true)
+              : gb_launch(retention_cross_kernel,
+                          dim3(chunks * (RT_CHUNK / RT_TM) * ((a.dv + RT_TN - 1) / RT_TN), a.H, a.n_seqs), dim3(256), 0, s, a);
     if (e) return e;
   }
   return retention_finish<T>(a, s);

@@ -57,7 +57,7 @@ g32 = lambda t: t.float().to(DEV).contiguous()
 
 # ------------------------------------------------------------------ dynamic tanh
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("T,N,parts", [(1, 96, 0), (5, 100, 3), (3, 7, 2), (70, 2560, 1), (300, 640, 13), (2, 4099, 9)])
+@pytest.mark.parametrize("T,N,parts", [(1, 96, 0), (5, 100, 3), (3, 7, 2), (70, 2560, 1), (514, 640, 13), (2, 4099, 9)])
 def test_dynamic_tanh_with_the_sum_in_front(dtype, T, N, parts):
     w = {"n": 1 + rnd(N, seed=1, scale=0.3), "n.b": rnd(N, seed=2, scale=0.5), "n.alpha": torch.tensor(0.7)}
     w = {k: v.to(dtype) for k, v in w.items()}
@@ -506,7 +506,8 @@ def test_lightning_attention_whole_in_portions_and_token_by_token(m):
 
 
 @pytest.mark.parametrize("m", [_light(3, 40, 20), _light(2, 64, 130, lo=0.9), _light(1, 128, 128, lo=0.97),
-                               _light(2, 18, 30, lo=0.5, hi=0.9999)])
+                               _light(2, 18, 30, lo=0.5, hi=0.9999), _light(3, 64, 64), _light(2, 64, 128, lo=0.99),
+                               _light(2, 128, 64, lo=0.8, hi=1.0)])
 def test_lightning_attention_long_sequences_go_chunk_by_chunk(m):
     """Long sequences beside short ones and a padding sequence, lengths at a chunk's edge, from states
     an earlier portion left; then single steps from the kept states; slots used again."""
