@@ -249,14 +249,15 @@ def mananex_config(size: str) -> dict:
 
 def kakotar_config(size: str) -> dict:
     """The Kakotar model of a size: the width, heads, head size, layers and vocabulary of
-    the Qwen3 model; the layers mix in turn by differential attention in chunks of 1,280
-    (a token behind a prompt of 2,048 then sees 768 keys and more; the Qwen3 model's heads, two maps of half the head size over values of the head size),
-    by lightning attention (as many heads, keys and values of the head size, decays from
-    1 - 2^-5 to 1 - 2^-10), by attention over a window of 1,024 with a YaRN-stretched
-    rotation, and by attention over the keys and values of the layer before; every layer
-    routes two of eight experts (four groups of which two are kept) beside a shared one,
-    each of 3/8 the Qwen3 model's feed-forward rows (two matrices instead of three: the
-    weights of a gated expert of a quarter of the rows)."""
+    the Qwen3 model; the layers mix in turn by differential attention in chunks of 1,280 (a
+    token behind a prompt of 2,048 then sees 768 keys and more; the Qwen3 model's heads, two
+    maps of half the head size over values of the head size), by lightning attention (as
+    many heads, keys and values of the head size, decays from 1 - 2^-5 to 1 - 2^-10), by
+    attention over a window of 1,024 with a YaRN-stretched rotation, and by attention over
+    the keys and values of the layer before; every layer routes two of eight experts (four
+    groups of which two are kept) beside a shared one, each of 3/8 the Qwen3 model's
+    feed-forward rows (two matrices instead of three: the weights of a gated expert of a
+    quarter of the rows)."""
     W, nq, nkv, D, I, L, V = DESIGN_SIZES[size]
     ff = 3 * I // 8 // 64 * 64
     diff = dict(heads=nq, kv_heads=nkv, dim=D // 2, vdim=D, scale=(D // 2) ** -0.5, diff=0.5, mask={"size": 1280},

@@ -603,8 +603,8 @@ def _moe(m, dtype, seed=0, correction=None):
 @pytest.mark.parametrize("T", [1, 5, 33, 70, 600])
 @pytest.mark.parametrize("m", MOE_SHAPES)
 def test_ungated_experts_groups_and_the_shared_expert(monkeypatch, dtype, T, m):
-    """Choice scores that are mostly negative (a dropped group must count as minus infinity, not as
-    zero); few rows and many (the products' kernels differ)."""
+    """Choice scores that are mostly negative, so that a dropped group that were left at zero would win;
+    few rows and many (the products' kernels differ)."""
     part, w, mlp = _moe(m, dtype)
     x = rnd(T, m["W"], seed=5).to(dtype)
     pw = {"m." + k: v for k, v in w.items()}
