@@ -1,0 +1,378 @@
+// The delta rule with one decay per key channel (Kimi delta attention): a mixer whose memory is
+// one matrix S [dk, dv] per head and sequence, updated token by token,
+//
+//   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+//
+// with g in (0, 1)^dk, beta in (0, 1), k a unit vector and q a unit vector times dk^(-1/2).  q, k and
+// v come out of short causal convolutions over time (one filter per channel, no bias) followed by
+// silu; g = exp(-exp(A_log) softplus(z + dt_bias)) with logits z from a product of two thin
+// matrices; the read-out is RMS-normalised over dv, multiplied by a weight shared by the heads
+// and by the sigmoid of a gate that comes from two thin matrices, too.
+//
+// Everything here is 32-bit whatever the activation type: the projection and the second thin
+// product arrive as 32-bit sums, and only y, the o projection's input, is rounded (and the thin
+// products' inner values, where activations are 16-bit).
+//
+//   prepare  one block per token and kv head (its q, its k and their product) or run of value
+//            channels: convolution, silu, unit vectors, beta; the thin products' inner values go
+//            to a tensor of their own, the second thin product's input
+//   step     a step in which every sequence brings one row: a block per (sequence, head) streams the
+//            head's state through registers once (a column's dk elements in eight lanes), and then
+//            normalises and gates the head's read-out; the heads' blocks share the new tail
+//   scan     any other step of short sequences: the columns of S are independent recurrences; a
+//            column is held in the registers of eight lanes, 16 columns a block, and the rows are
+//            walked in order, their q, k and g staged in shared memory 16 at a time
+//   finish   after scan: one warp per (token, head) normalises and gates; the block of a sequence's
+//            first row keeps the new tail
+//
+// With s' = g s the two sums over dk that a row needs, s' . k and s' . q, are taken together:
+// u = beta (v - s' . k) and o = s' . q + u (k . q), so a row costs one round of shuffles.
+//
+// Columns of the projection: q [G dk] | k [G dk] | v [H dv] | beta logits [H] | inner values [n_low].
+// Columns of the second thin product: z [H dk] | gate logits [H dv].  A sequence's state is one row of
+// floats: the convolutions' tail [taps - 1, Cc] (Cc = the convolved channels q | k | v), then S as
+// [H, dv, dk], a column's dk elements side by side.  Rows of slot < 0 (padding) start from zeros
+// and store nothing.
+#include "short_conv.cuh"
+
+struct ChannelDeltaArgs {
+  const float* proj;       // [n_tokens, C_all]
+  const float* conv_w;     // [Cc, taps], the last column is the current token's
+  const float* a_log;      // [H]
+  const float* dt_bias;    // [H dk]
+  const float* norm_w;     // [dv]
+  const int* token_seq;    // [n_tokens]
+  const int* cu_q;         // [n_seqs + 1]
+  const int* slots;        // [n_seqs]
+  float* state;            // [slots, state_stride]
+  long long state_stride;
+  float* prep;             // [n_tokens, prep_stride]: unit q | unit k | v | beta [H] | k . q [G]
+  void* low;               // [n_tokens, n_low] in the activation type
+  const float* wide;       // [n_tokens, H dk + H dv]: z | gate logits
+  float* o;                // [n_tokens, H, dv]
+  void* y;                 // [n_tokens, H dv] in the activation type
+  int n_tokens, n_seqs, H, G, dk, dv, taps, n_low;
+  float unit_eps, norm_eps;
+  int prep_stride;         // floats between rows of prep: round4(Cc + H + G)
+  int max_rows;            // the most rows any sequence brings (0: unknown)
+};
+
+__device__ __forceinline__ int cd_channels(const ChannelDeltaArgs& a) { return 2 * a.G * a.dk + a.H * a.dv; }
+__device__ __forceinline__ int cd_columns(const ChannelDeltaArgs& a) { return cd_channels(a) + a.H + a.n_low; }
+__device__ __forceinline__ float cd_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+// the logarithm of a channel's decay; `rate` = exp(A_log) of its head
+__device__ __forceinline__ float cd_log_decay(float z, float bias, float rate) { return -rate * softplus_f(z + bias); }
+
+#define CD_PREP_V 256
+
+template <typename T>
+__global__ void __launch_bounds__(256) channel_delta_prepare_kernel(const ChannelDeltaArgs a) {
+  extern __shared__ float row[];   // [2 dk]: a kv head's q and k after the convolution
+  __shared__ float scratch[32];
+  pdl_launch_dependents_if_small();
+  const int t = blockIdx.x, unit = blockIdx.y, tid = threadIdx.x;
+  const int H = a.H, G = a.G, dk = a.dk;
+  const int Cc = cd_channels(a), C_all = cd_columns(a), P = a.prep_stride;
+  const int seq = a.token_seq[t];
+  const int slot = a.slots[seq];
+  const int r = t - a.cu_q[seq];                 // the token's place among its sequence's rows
+  const float* tail = slot >= 0 ? a.state + (size_t)slot * a.state_stride : nullptr;
+  float* out = a.prep + (size_t)t * P;
+  pdl_wait();
+  if (unit >= G) {                               // value channels: convolution and silu
+    const int c = 2 * G * dk + (unit - G) * CD_PREP_V + tid;
+    if (tid < CD_PREP_V && c < Cc) out[c] = short_conv_silu(a.proj, C_all, a.conv_w, a.taps, tail, Cc, t, r, c);
+    return;
+  }
+  float sq = 0.f, sk = 0.f;
+  for (int i = tid; i < 2 * dk; i += blockDim.x) {
+    const int c = i < dk ? unit * dk + i : (G + unit) * dk + (i - dk);
+    const float v = short_conv_silu(a.proj, C_all, a.conv_w, a.taps, tail, Cc, t, r, c);
+    row[i] = v;
+    if (i < dk) sq += v * v; else sk += v * v;
+  }
+  sq = block_sum(sq, scratch);
+  sk = block_sum(sk, scratch);
+  const float iq = 1.0f / sqrtf(sq + a.unit_eps) * (1.0f / sqrtf((float)dk));
+  const float ik = 1.0f / sqrtf(sk + a.unit_eps);
+  float kq = 0.f;
+  for (int d = tid; d < dk; d += blockDim.x) {
+    const float q = row[d] * iq, k = row[dk + d] * ik;
+    out[unit * dk + d] = q;
+    out[(G + unit) * dk + d] = k;
+    kq = fmaf(q, k, kq);
+  }
+  kq = block_sum(kq, scratch);
+  if (tid == 0) out[Cc + H + unit] = kq;
+  if (unit == 0) {
+    const float* rest = a.proj + (size_t)t * C_all + Cc;
+    for (int h = tid; h < H; h += blockDim.x) out[Cc + h] = cd_sigmoid(rest[h]);
+    T* low = (T*)a.low + (size_t)t * a.n_low;
+    for (int i = tid; i < a.n_low; i += blockDim.x) low[i] = from_f32<T>(rest[H + i]);
+  }
+  pdl_launch_dependents_if_large();
+}
+
+#define CD_LANES 8       // lanes that share a column of S
+#define CD_COLS 16       // columns of S per block of the scan
+#define CD_TT 16         // rows staged together
+
+// R floats of a column per lane, in pieces of four: piece i of lane l holds the elements
+// (i * 8 + l) * 4 .. + 3, so that the lanes of a column read contiguous bytes at a time.
+template <int R>
+__device__ __forceinline__ void cd_load_column(float (&S)[R], const float* sp, int dk, int l, bool wide) {
+#pragma unroll
+  for (int i = 0; i < R / 4; ++i) {
+    const int e = (i * CD_LANES + l) * 4;
+    if (wide) {
+      const float4 x = sp && e < dk ? *reinterpret_cast<const float4*>(sp + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[4 * i] = x.x, S[4 * i + 1] = x.y, S[4 * i + 2] = x.z, S[4 * i + 3] = x.w;
+    } else {
+#pragma unroll
+      for (int x = 0; x < 4; ++x) S[4 * i + x] = sp && e + x < dk ? sp[e + x] : 0.f;
+    }
+  }
+}
+template <int R>
+__device__ __forceinline__ void cd_store_column(const float (&S)[R], float* sp, int dk, int l, bool wide) {
+#pragma unroll
+  for (int i = 0; i < R / 4; ++i) {
+    const int e = (i * CD_LANES + l) * 4;
+    if (wide) {
+      if (e < dk) *reinterpret_cast<float4*>(sp + e) = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
+    } else {
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        if (e + x < dk) sp[e + x] = S[4 * i + x];
+    }
+  }
+}
+
+// One row of a column: S <- g S + k u with u = beta (v - (g S) . k); returns (g S) . q + u (k . q).
+template <int R>
+__device__ __forceinline__ float cd_row(float (&S)[R], const float* q, const float* k, const float* g, int l,
+                                        float v, float beta, float kq) {
+  float kk[R], d1 = 0.f, d2 = 0.f;
+#pragma unroll
+  for (int i = 0; i < R / 4; ++i) {
+    const float4 k4 = reinterpret_cast<const float4*>(k)[i * CD_LANES + l];
+    const float4 q4 = reinterpret_cast<const float4*>(q)[i * CD_LANES + l];
+    const float4 g4 = reinterpret_cast<const float4*>(g)[i * CD_LANES + l];
+    S[4 * i] *= g4.x, S[4 * i + 1] *= g4.y, S[4 * i + 2] *= g4.z, S[4 * i + 3] *= g4.w;
+    kk[4 * i] = k4.x, kk[4 * i + 1] = k4.y, kk[4 * i + 2] = k4.z, kk[4 * i + 3] = k4.w;
+    d1 = fmaf(S[4 * i], k4.x, d1), d1 = fmaf(S[4 * i + 1], k4.y, d1);
+    d1 = fmaf(S[4 * i + 2], k4.z, d1), d1 = fmaf(S[4 * i + 3], k4.w, d1);
+    d2 = fmaf(S[4 * i], q4.x, d2), d2 = fmaf(S[4 * i + 1], q4.y, d2);
+    d2 = fmaf(S[4 * i + 2], q4.z, d2), d2 = fmaf(S[4 * i + 3], q4.w, d2);
+  }
+#pragma unroll
+  for (int m = 1; m < CD_LANES; m <<= 1) {
+    d1 += __shfl_xor_sync(0xffffffffu, d1, m);
+    d2 += __shfl_xor_sync(0xffffffffu, d2, m);
+  }
+  const float u = beta * (v - d1);
+#pragma unroll
+  for (int x = 0; x < R; ++x) S[x] = fmaf(kk[x], u, S[x]);
+  return fmaf(u, kq, d2);
+}
+
+template <typename T, int R>
+__global__ void __launch_bounds__(256) channel_delta_step_kernel(const ChannelDeltaArgs a) {
+  extern __shared__ __align__(16) float sm[];     // q | k | g [DKP each] | o [dv]
+  __shared__ float scratch[32];
+  constexpr int DKP = CD_LANES * R;               // dk filled up with zeros
+  constexpr int COLS = 256 / CD_LANES;            // columns of a pass
+  pdl_launch_dependents_if_small();
+  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
+  const int H = a.H, G = a.G, dk = a.dk, dv = a.dv, kvh = h / (H / G);
+  const int Cc = cd_channels(a), C_all = cd_columns(a);
+  const int t = a.cu_q[seq], slot = a.slots[seq];
+  float *qs = sm, *ks = sm + DKP, *gs = sm + 2 * DKP, *os = sm + 3 * DKP;
+  const float rate = expf(a.a_log[h]);
+  float* head = slot >= 0 ? a.state + (size_t)slot * a.state_stride + (size_t)(a.taps - 1) * Cc + (size_t)h * dv * dk
+                          : nullptr;
+  const bool wide = (dk & 3) == 0 && (((uintptr_t)head) & 15) == 0;
+  if (head)                                       // on its way to L2 while the kernel before drains
+    for (int i = tid * 32; i < dk * dv; i += 256 * 32)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(head + i));
+  pdl_wait();
+  if (a.cu_q[seq + 1] - t <= 0) return;
+  const float* p = a.prep + (size_t)t * a.prep_stride;
+  const float* z = a.wide + (size_t)t * ((size_t)H * (dk + dv));
+  for (int d = tid; d < DKP; d += 256) {
+    const bool in = d < dk;
+    qs[d] = in ? p[kvh * dk + d] : 0.f;
+    ks[d] = in ? p[(G + kvh) * dk + d] : 0.f;
+    gs[d] = in ? expf(cd_log_decay(z[h * dk + d], a.dt_bias[h * dk + d], rate)) : 0.f;
+  }
+  const float beta = p[Cc + h], kq = p[Cc + H + kvh];
+  __syncthreads();
+  const int l = tid % CD_LANES;
+  float ss = 0.f;
+  for (int c0 = 0; c0 < dv; c0 += 2 * COLS) {     // two columns a thread group: their loads go together
+    const int ca = c0 + tid / CD_LANES, cb = ca + COLS;
+    float Sa[R], Sb[R];
+    cd_load_column<R>(Sa, head && ca < dv ? head + (size_t)ca * dk : nullptr, dk, l, wide);
+    cd_load_column<R>(Sb, head && cb < dv ? head + (size_t)cb * dk : nullptr, dk, l, wide);
+    const float va = ca < dv ? p[2 * G * dk + h * dv + ca] : 0.f, vb = cb < dv ? p[2 * G * dk + h * dv + cb] : 0.f;
+    const float oa = cd_row<R>(Sa, qs, ks, gs, l, va, beta, kq);
+    const float ob = cd_row<R>(Sb, qs, ks, gs, l, vb, beta, kq);
+    if (head && ca < dv) cd_store_column<R>(Sa, head + (size_t)ca * dk, dk, l, wide);
+    if (head && cb < dv) cd_store_column<R>(Sb, head + (size_t)cb * dk, dk, l, wide);
+    if (l == 0 && ca < dv) os[ca] = oa, ss = fmaf(oa, oa, ss);
+    if (l == 0 && cb < dv) os[cb] = ob, ss = fmaf(ob, ob, ss);
+  }
+  pdl_launch_dependents_if_large();
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dv + a.norm_eps);   // (its barriers publish os)
+  const float* gate = z + (size_t)H * dk + (size_t)h * dv;
+  T* y = (T*)a.y + ((size_t)t * H + h) * dv;
+  for (int j = tid; j < dv; j += 256) y[j] = from_f32<T>(os[j] * inv * a.norm_w[j] * cd_sigmoid(gate[j]));
+  if (a.taps > 1 && slot >= 0)                    // every reader of the old tail, the prepare kernel, has finished
+    short_conv_keep_tail(a.proj, C_all, a.taps, a.state + (size_t)slot * a.state_stride, Cc, t, 1, h * 256 + tid,
+                         H * 256);
+}
+
+template <int R>
+__global__ void __launch_bounds__(CD_LANES * CD_COLS) channel_delta_scan_kernel(const ChannelDeltaArgs a) {
+  extern __shared__ __align__(16) float sm[];     // q | k | g [CD_TT, DKP each] | v [CD_TT, CD_COLS] | beta, kq [CD_TT]
+  constexpr int DKP = CD_LANES * R;
+  pdl_launch_dependents_if_small();
+  const int seq = blockIdx.z, h = blockIdx.y, tid = threadIdx.x;
+  const int col0 = blockIdx.x * CD_COLS, col = col0 + tid / CD_LANES, l = tid % CD_LANES;
+  const int H = a.H, G = a.G, dk = a.dk, dv = a.dv, kvh = h / (H / G);
+  const int Cc = cd_channels(a);
+  float *qs = sm, *ks = qs + CD_TT * DKP, *gs = ks + CD_TT * DKP, *vs = gs + CD_TT * DKP, *bs = vs + CD_TT * CD_COLS,
+        *kqs = bs + CD_TT;
+  const float rate = expf(a.a_log[h]);
+  pdl_wait();
+  const int row0 = a.cu_q[seq], n = a.cu_q[seq + 1] - row0;
+  if (n <= 0) return;
+  const int slot = a.slots[seq];
+  const bool active = col < dv;
+  float* sp = slot >= 0 && active ? a.state + (size_t)slot * a.state_stride + (size_t)(a.taps - 1) * Cc +
+                                        ((size_t)h * dv + col) * dk
+                                  : nullptr;
+  const bool wide = (dk & 3) == 0 && (((uintptr_t)sp) & 15) == 0;
+  float S[R];
+  cd_load_column<R>(S, sp, dk, l, wide);
+  for (int t0 = 0; t0 < n; t0 += CD_TT) {
+    const int nt = min(CD_TT, n - t0);
+    __syncthreads();
+    for (int i = tid; i < nt * DKP; i += CD_LANES * CD_COLS) {
+      const int tt = i / DKP, d = i % DKP, t = row0 + t0 + tt;
+      const float* p = a.prep + (size_t)t * a.prep_stride;
+      const bool in = d < dk;
+      qs[i] = in ? p[kvh * dk + d] : 0.f;
+      ks[i] = in ? p[(G + kvh) * dk + d] : 0.f;
+      gs[i] = in ? expf(cd_log_decay(a.wide[(size_t)t * H * (dk + dv) + h * dk + d], a.dt_bias[h * dk + d], rate)) : 0.f;
+    }
+    for (int i = tid; i < nt * CD_COLS; i += CD_LANES * CD_COLS) {
+      const int c = col0 + i % CD_COLS;
+      vs[i] = c < dv ? a.prep[(size_t)(row0 + t0 + i / CD_COLS) * a.prep_stride + 2 * G * dk + h * dv + c] : 0.f;
+    }
+    if (tid < nt) {
+      const float* p = a.prep + (size_t)(row0 + t0 + tid) * a.prep_stride + Cc;
+      bs[tid] = p[h], kqs[tid] = p[H + kvh];
+    }
+    __syncthreads();
+    for (int tt = 0; tt < nt; ++tt) {
+      const float o = cd_row<R>(S, qs + tt * DKP, ks + tt * DKP, gs + tt * DKP, l, vs[tt * CD_COLS + tid / CD_LANES],
+                                bs[tt], kqs[tt]);
+      if (l == 0 && active) a.o[((size_t)(row0 + t0 + tt) * H + h) * dv + col] = o;
+    }
+  }
+  pdl_launch_dependents_if_large();
+  if (sp) cd_store_column<R>(S, sp, dk, l, wide);
+}
+
+template <typename T>
+__global__ void channel_delta_finish_kernel(const ChannelDeltaArgs a) {
+  pdl_launch_dependents_if_small();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int nwarps = blockDim.x >> 5;
+  const int H = a.H, dk = a.dk, dv = a.dv;
+  for (int h = blockIdx.y * nwarps + warp; h < H; h += gridDim.y * nwarps) {
+    const float* o = a.o + ((size_t)t * H + h) * dv;
+    const float* gate = a.wide + (size_t)t * H * (dk + dv) + (size_t)H * dk + (size_t)h * dv;
+    float ss = 0.f;
+    for (int j = lane; j < dv; j += 32) ss += o[j] * o[j];
+    ss = warp_sum(ss);
+    const float inv = 1.0f / sqrtf(ss / (float)dv + a.norm_eps);
+    T* y = (T*)a.y + ((size_t)t * H + h) * dv;
+    for (int j = lane; j < dv; j += 32) y[j] = from_f32<T>(o[j] * inv * a.norm_w[j] * cd_sigmoid(gate[j]));
+  }
+  if (a.taps > 1) {
+    const int seq = a.token_seq[t];
+    const int row0 = a.cu_q[seq], slot = a.slots[seq];
+    if (t == row0 && slot >= 0)
+      short_conv_keep_tail(a.proj, cd_columns(a), a.taps, a.state + (size_t)slot * a.state_stride, cd_channels(a), row0,
+                           a.cu_q[seq + 1] - row0, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
+  }
+  pdl_launch_dependents_if_large();
+}
+
+static int cd_check(const ChannelDeltaArgs& a) {
+  if (a.n_tokens < 0 || a.n_seqs <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dv <= 0 || a.taps <= 0 ||
+      a.n_low <= 0 || !a.proj || !a.state || !a.prep || !a.low || !a.conv_w || !a.token_seq || !a.cu_q || !a.slots)
+    return GB_ERR_BAD_ARG;
+  if (a.dk > 32 * CD_LANES || a.n_seqs > 65535 || a.H > 65535) return GB_ERR_UNSUPPORTED;
+  if (a.prep_stride != (2 * a.G * a.dk + a.H * a.dv + a.H + a.G + 3) / 4 * 4) return GB_ERR_BAD_ARG;
+  return 0;
+}
+
+template <typename T>
+static int prepare(const ChannelDeltaArgs& a, cudaStream_t s) {
+  const int e = cd_check(a);
+  if (e || a.n_tokens == 0) return e;
+  const int units = a.G + (a.H * a.dv + CD_PREP_V - 1) / CD_PREP_V;
+  return gb_launch(channel_delta_prepare_kernel<T>, dim3(a.n_tokens, units), dim3(256), (size_t)2 * a.dk * sizeof(float),
+                   s, a);
+}
+
+template <typename T, int R>
+static int run_rows(const ChannelDeltaArgs& a, cudaStream_t s) {
+  constexpr int DKP = CD_LANES * R;
+  if (a.max_rows == 1) {
+    const size_t smem = (3 * DKP + a.dv) * sizeof(float);
+    if (smem > 48 * 1024) return GB_ERR_UNSUPPORTED;
+    return gb_launch(channel_delta_step_kernel<T, R>, dim3(a.H, a.n_seqs), dim3(256), smem, s, a);
+  }
+  const size_t smem = (CD_TT * (3 * DKP + CD_COLS + 2)) * sizeof(float);
+  static bool configured = false;
+  if (smem > 48 * 1024 && !configured) {
+    cudaError_t e = cudaFuncSetAttribute(channel_delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  const int e = gb_launch(channel_delta_scan_kernel<R>, dim3((a.dv + CD_COLS - 1) / CD_COLS, a.H, a.n_seqs),
+                          dim3(CD_LANES * CD_COLS), smem, s, a);
+  if (e) return e;
+  const int warps = a.H < 8 ? a.H : 8;
+  int rows_y = (a.H + warps - 1) / warps;            // blocks of a row: enough for its heads, and
+  const int Cc = 2 * a.G * a.dk + a.H * a.dv;        //   for the tail's channels four to a thread
+  const int for_tail = a.taps > 1 ? (Cc + warps * 32 * 4 - 1) / (warps * 32 * 4) : 1;
+  if (for_tail > rows_y) rows_y = for_tail < 64 ? for_tail : 64;
+  return gb_launch(channel_delta_finish_kernel<T>, dim3(a.n_tokens, rows_y), dim3(warps * 32), 0, s, a);
+}
+
+template <typename T>
+static int run(const ChannelDeltaArgs& a, cudaStream_t s) {
+  const int e = cd_check(a);
+  if (e) return e;
+  if (!a.wide || !a.a_log || !a.dt_bias || !a.norm_w || !a.o || !a.y) return GB_ERR_BAD_ARG;
+  if (a.n_tokens == 0) return 0;
+  const int per_lane = (a.dk + CD_LANES - 1) / CD_LANES;
+  if (per_lane <= 4) return run_rows<T, 4>(a, s);
+  if (per_lane <= 8) return run_rows<T, 8>(a, s);
+  if (per_lane <= 12) return run_rows<T, 12>(a, s);
+  if (per_lane <= 16) return run_rows<T, 16>(a, s);
+  if (per_lane <= 24) return run_rows<T, 24>(a, s);
+  return run_rows<T, 32>(a, s);
+}
+
+GB_EXPORT int gb_channel_delta_prepare_f32(const ChannelDeltaArgs* a, cudaStream_t s) { return prepare<float>(*a, s); }
+GB_EXPORT int gb_channel_delta_prepare_bf16(const ChannelDeltaArgs* a, cudaStream_t s) { return prepare<bf16>(*a, s); }
+GB_EXPORT int gb_channel_delta_run_f32(const ChannelDeltaArgs* a, cudaStream_t s) { return run<float>(*a, s); }
+GB_EXPORT int gb_channel_delta_run_bf16(const ChannelDeltaArgs* a, cudaStream_t s) { return run<bf16>(*a, s); }

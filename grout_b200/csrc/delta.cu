@@ -44,6 +44,7 @@
 // convolved channels q | k | v), then S as [H, dv, dk], a column's dk elements
 // side by side.  Rows of slot < 0 (padding) read zeros and store nothing.
 #include "attn_mma.cuh"   // the asynchronous-copy helpers
+#include "short_conv.cuh"
 
 struct DeltaArgs {
   const float* proj;       // [n_tokens, C_all]
@@ -67,34 +68,13 @@ struct DeltaArgs {
                            //   step): the scan works out its one group's scalars itself, `gram` is not launched
 };
 
-__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
-
 // One block per (token, unit): unit g < G is kv head g's q and k together, the units after that are runs of
 // DELTA_PREP_V value channels; the block of unit 0 also takes beta and the decay.
 #define DELTA_PREP_V 256
-#define DELTA_MAX_TAPS 8     // taps fetched together; more are walked in turns
 
 __device__ __forceinline__ float delta_conv(const DeltaArgs& a, const float* tail, int t, int r,
                                             int c, int Cc, int C_all) {
-  const int taps = a.taps;
-  float acc = 0.f;
-  for (int j0 = 0; j0 < taps; j0 += DELTA_MAX_TAPS) {
-    float x[DELTA_MAX_TAPS], w[DELTA_MAX_TAPS];
-#pragma unroll
-    for (int jj = 0; jj < DELTA_MAX_TAPS; ++jj) {      // all loads first: one trip to memory
-      const int j = j0 + jj, rr = r - j;               // the input j tokens back
-      x[jj] = 0.f, w[jj] = 0.f;
-      if (j < taps) {
-        w[jj] = a.conv_w[(size_t)c * taps + taps - 1 - j];
-        if (rr >= 0) x[jj] = a.proj[(size_t)(t - j) * C_all + c];
-        else if (tail) x[jj] = tail[(size_t)(taps - 1 + rr) * Cc + c];
-      }
-    }
-#pragma unroll
-    for (int jj = 0; jj < DELTA_MAX_TAPS; ++jj) acc = fmaf(w[jj], x[jj], acc);
-  }
-  return silu_f(acc);
+  return short_conv_silu(a.proj, C_all, a.conv_w, a.taps, tail, Cc, t, r, c);
 }
 
 __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a) {
@@ -141,33 +121,14 @@ __global__ void __launch_bounds__(256) delta_prepare_kernel(const DeltaArgs a) {
   pdl_launch_dependents_if_large();
 }
 
-// The new tail of a sequence: the last taps - 1 inputs of its convolutions.  Entry s
-// holds the input at n - (taps - 1) + s rows from the step's first; an entry that stays
-// is read (at n + s > s) before anything at or above it is written.
+// The new tail of a sequence; the blocks of the row (blockIdx.y) share the channels.
 __device__ __forceinline__ void delta_keep_tail(const DeltaArgs& a, int seq) {
   const int slot = a.slots[seq];
   const int row0 = a.cu_q[seq], n = a.cu_q[seq + 1] - row0;
   if (slot < 0 || n <= 0) return;
-  const int taps = a.taps;
   const int Cc = 2 * a.G * a.dk + a.H * a.dv, C_all = Cc + a.H * a.dv + 2 * a.H;
-  float* tail = a.state + (size_t)slot * a.state_stride;
-  // the blocks of the row (blockIdx.y) share the channels; up to eight entries are read
-  // together before any of them is written
-  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < Cc; c += gridDim.y * blockDim.x) {
-    for (int s0 = 0; s0 < taps - 1; s0 += 8) {
-      float v[8];
-#pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        const int s = s0 + u, rr = n - (taps - 1) + s;
-        v[u] = 0.f;
-        if (s < taps - 1)
-          v[u] = rr >= 0 ? a.proj[(size_t)(row0 + rr) * C_all + c] : tail[(size_t)(taps - 1 + rr) * Cc + c];
-      }
-#pragma unroll
-      for (int u = 0; u < 8; ++u)
-        if (s0 + u < taps - 1) tail[(size_t)(s0 + u) * Cc + c] = v[u];
-    }
-  }
+  short_conv_keep_tail(a.proj, C_all, a.taps, a.state + (size_t)slot * a.state_stride, Cc, row0, n,
+                       blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
 }
 
 #define DELTA_LANES 8       // lanes that share a column of S

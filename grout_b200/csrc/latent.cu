@@ -12,6 +12,10 @@
 // serves as key and as value: attention runs as if every query head read one kv
 // head of R + dr elements, with the query [Wuk_h^T q_plain | q_rot].
 //
+// The queries may come from a latent of their own: the projection then gives q_rank numbers
+// in their place, which `prepare` RMS-normalises with a weight (cq); a product expands them,
+// and a second `prepare` turns what of the expanded queries is to be turned, if anything is.
+//
 // `prepare` does the norm and the rotations in 32-bit on the projection's 32-bit
 // sums, stores the cache row and writes the queries' two parts; the rotation
 // pairs element 2i with element 2i + 1.  `heads_mm` is the per-head product
@@ -21,7 +25,7 @@
 #include "common.cuh"
 
 struct LatentArgs {
-  const float* proj;       // [T, H (dn + dr) + R + dr + H dv] 32-bit sums: q | down | gate
+  const float* proj;       // [T, q_cols + R + dr + H dv] 32-bit sums: q (or its latent) | down | gate
   const float* norm_w;     // [R]
   const float* inv_freq;   // [dr / 2]
   const int* token_seq;    // [T]
@@ -33,10 +37,21 @@ struct LatentArgs {
   void* q_full;            // [T, H, Ds]: columns R .. R + dr get the rotated part, columns from R + dr on zeros
   int n_tokens, H, dn, dr, R, dv, Ds, max_pages, page;
   float eps;
+  int q_rank;              // > 0: the projection's first columns are the queries' latent of that size
+  const float* q_norm_w;   // [q_rank]
+  void* cq;                // [T, q_rank]: the normalised latent
+  int queries_only;        // proj holds expanded queries [T, H (dn + dr)] and nothing else
 };
 
+template <typename T>
+__device__ __forceinline__ void latent_pad(T* q_full, int nh, int Ds, int from, int tid, int step) {
+  const int w = Ds - from;
+  for (int i = tid; i < nh * w; i += step) q_full[(size_t)(i / w) * Ds + from + i % w] = from_f32<T>(0.f);
+}
+
 // A block owns one token and the heads blockIdx.y * heads_per_block ..; the block of the
-// first heads also normalises the latent and stores the token's cache row.
+// first heads also normalises the latent and stores the token's cache row.  With a latent
+// for the queries too, block 0 has the keys' latent and block 1 the queries'.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a, const int heads_per_block) {
   __shared__ float scratch[32];
@@ -45,11 +60,22 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
   const int t = blockIdx.x, tid = threadIdx.x;
   const int H = a.H, dn = a.dn, dr = a.dr, R = a.R, Ds = a.Ds;
   const int h0 = blockIdx.y * heads_per_block, nh = min(heads_per_block, H - h0);
-  const int C = H * (dn + dr) + R + dr + H * a.dv;
+  const int q_cols = a.q_rank > 0 ? a.q_rank : H * (dn + dr);
+  const int C = a.queries_only ? q_cols : q_cols + R + dr + H * a.dv;
   const float* __restrict__ row = a.proj + (size_t)t * C;
-  const float* __restrict__ down = row + H * (dn + dr);
+  const float* __restrict__ down = row + q_cols;
   const float pos = (float)a.token_pos[t];
-  if (blockIdx.y == 0) {
+  if (a.q_rank > 0 && blockIdx.y == 1) {
+    float ss = 0.f;
+    for (int i = tid; i < q_cols; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)q_cols + a.eps);
+    pdl_launch_dependents_if_large();
+    for (int i = tid; i < q_cols; i += blockDim.x)
+      ((T*)a.cq)[(size_t)t * q_cols + i] = from_f32<T>(row[i] * inv * a.q_norm_w[i]);
+    if (dr == 0) latent_pad<T>((T*)a.q_full + (size_t)t * H * Ds, H, Ds, R, tid, blockDim.x);
+    return;
+  }
+  if (blockIdx.y == 0 && !a.queries_only) {
     float ss = 0.f;
     for (int i = tid; i < R; i += blockDim.x) ss = fmaf(down[i], down[i], ss);
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)R + a.eps);
@@ -73,6 +99,7 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
     }
   }
   pdl_launch_dependents_if_large();
+  if (a.q_rank > 0) return;
   T* __restrict__ q_plain = (T*)a.q_plain + ((size_t)t * H + h0) * dn;
   T* __restrict__ q_full = (T*)a.q_full + ((size_t)t * H + h0) * Ds;
   const float* __restrict__ qrow = row + (size_t)h0 * (dn + dr);
@@ -88,21 +115,21 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
       q_full[(size_t)h * Ds + R + r] = from_f32<T>((r & 1) ? w * c + u * s : u * c - w * s);
     }
   }
-  for (int i = tid; i < nh * (Ds - R - dr); i += blockDim.x) {
-    const int h = i / (Ds - R - dr), e = i % (Ds - R - dr);
-    q_full[(size_t)h * Ds + R + dr + e] = from_f32<T>(0.f);
-  }
+  latent_pad<T>(q_full, nh, Ds, R + dr, tid, blockDim.x);
 }
 
 template <typename T>
 static int latent_prepare(const LatentArgs& a, cudaStream_t s) {
   if (a.n_tokens < 0 || a.H <= 0 || a.dn <= 0 || a.dr < 0 || a.dr % 2 || a.R <= 0 || a.dv < 0 ||
-      a.Ds < a.R + a.dr || a.page <= 0 || a.max_pages <= 0)
+      a.Ds < a.R + a.dr || (!a.queries_only && (a.page <= 0 || a.max_pages <= 0)))
     return GB_ERR_BAD_ARG;
-  if (!a.proj || !a.norm_w || !a.token_seq || !a.token_pos || !a.slots || !a.block_table || !a.pages ||
-      !a.q_plain || !a.q_full || (a.dr && !a.inv_freq))
+  if (!a.proj || !a.token_pos || !a.q_full || (a.dr && !a.inv_freq)) return GB_ERR_BAD_ARG;
+  if (!a.queries_only && (!a.norm_w || !a.token_seq || !a.slots || !a.block_table || !a.pages)) return GB_ERR_BAD_ARG;
+  if (a.q_rank < 0 || (a.q_rank > 0 && (!a.q_norm_w || !a.cq || a.queries_only)) || (a.q_rank == 0 && !a.q_plain))
     return GB_ERR_BAD_ARG;
   if (a.n_tokens == 0) return 0;
+  if (a.q_rank > 0)
+    return gb_launch(latent_prepare_kernel<T>, dim3(a.n_tokens, 2), dim3(256), 0, s, a, a.H);
   // few tokens: four heads a block, so that a step of a handful of rows fills more than a handful of SMs
   const int heads_per_block = a.n_tokens <= 64 ? min(a.H, 4) : a.H;
   return gb_launch(latent_prepare_kernel<T>, dim3(a.n_tokens, (a.H + heads_per_block - 1) / heads_per_block),

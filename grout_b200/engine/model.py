@@ -11,7 +11,7 @@ import torch
 
 from ..cache import CacheLayout, SequenceCache
 from ..parts.base import BuildContext, ParamSpec, Part, build_part
-from ..parts.norm import Averaged, with_offset
+from ..parts.norm import Averaged, HyperConnected, with_offset
 from ..parts.plan import ModelPlan
 from .batch import StepContext
 
@@ -130,6 +130,8 @@ class Model:
             if e.add is not None:
                 pending = with_offset(pending, self.stream_vectors[e.add[0]][e.add[1]])
             res, pending = self.blocks[e.layer].forward(res, pending, step, view)
+            if isinstance(pending, HyperConnected) and (history is not None or e.add is not None):
+                raise ValueError("several residual streams go with neither a depth average nor added vectors")
             if history is not None:
                 pending = Averaged(pending, history, i + 1, self.averages[i])
         if step.n_want == 0:

@@ -638,6 +638,83 @@ def qk_prepare(qkv: torch.Tensor, nq: int, nkv: int, D: int, *, q_w=None, k_w=No
     return q, kv_out
 
 
+class _QkConvArgs(ctypes.Structure):
+    _fields_ = [("proj", _P), ("n_parts", _I), ("part_stride", _L), ("bias", _P), ("conv_w", _P), ("inv_freq", _P),
+                ("cu_q", _P), ("token_pos", _P), ("slots", _P), ("block_table", _P), ("tail", _P),
+                ("tail_stride", _L), ("q_out", _P), ("k_pages", _P), ("v_pages", _P), ("T", _I), ("n_seqs", _I),
+                ("nq", _I), ("nkv", _I), ("D", _I), ("Dv", _I), ("Ds", _I), ("taps", _I), ("rot_dim", _I),
+                ("interleaved", _I), ("v_from_k", _I), ("max_pages", _I), ("page", _I), ("rot_scale", _F),
+                ("run", _I), ("one_row", _I)]
+
+
+@_profiled("qk_conv", lambda out, qkv, nq, nkv, D, **k: (
+    _nbytes(qkv, out) + out.shape[0] * 2 * nkv * D * out.element_size(), 0))
+def qk_conv(qkv: torch.Tensor, nq: int, nkv: int, D: int, *, step, block_table, k_pages, v_pages, page: int,
+            taps: int = 1, bias: Optional[torch.Tensor] = None, conv_w: Optional[torch.Tensor] = None,
+            tail: Optional[torch.Tensor] = None, v_dim: Optional[int] = None, values_are_keys: bool = False,
+            inv_freq: Optional[torch.Tensor] = None, rot_dim: int = 0, interleaved: bool = False,
+            rot_scale: float = 1.0) -> torch.Tensor:
+    """Queries and keys behind a short causal convolution.  ``qkv`` 32-bit [T, columns] or a
+    stack of partial sums [P, T, columns] (added in order): nq query heads and nkv key heads of
+    D, then nkv value heads of ``v_dim`` unless ``values_are_keys``.  Per q and k channel: + ``bias``,
+    the convolution ``conv_w`` [(nq + nkv) D, taps] over time (the last column the current
+    token's, zeros before the sequence's start), the rotation of the first ``rot_dim`` elements of
+    a head.  Returns q [T, nq, Ds] in the pages' type (Ds: the pages' row width, filled up with
+    zeros) and stores keys and values in the pages; a value that is its key is the convolved
+    one in front of the rotation.  ``tail`` [slots + 1, (taps - 1) (nq + nkv) D] 32-bit: a
+    sequence's last projected values, read and replaced for slots that are not negative."""
+    _need(qkv, "projection", torch.float32)
+    if qkv.dim() not in (2, 3):
+        raise KernelError(f"the projection is {tuple(qkv.shape)}, expected [T, columns] or partial sums of it")
+    dt = k_pages.dtype
+    T = qkv.shape[-2]
+    Dv = int(v_dim) if v_dim else D
+    Cc = (nq + nkv) * D
+    width = Cc + (0 if values_are_keys else nkv * Dv)
+    if qkv.shape[-1] != width or (values_are_keys and Dv != D):
+        raise KernelError(f"the projection has {qkv.shape[-1]} columns, expected {width}")
+    _need(k_pages, "k pages", dt, 4)
+    _need(v_pages, "v pages", dt, 4)
+    _need(block_table, "block table", torch.int32, 2)
+    Ds = int(k_pages.shape[-1])
+    if tuple(k_pages.shape[1:]) != (nkv, page, Ds) or v_pages.shape != k_pages.shape or Ds < max(D, Dv):
+        raise KernelError(f"pages are {tuple(k_pages.shape)}, expected [*, {nkv}, {page}, >= {max(D, Dv)}]")
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+    if conv_w is not None:
+        _need(conv_w, "convolution weights", torch.float32, 2)
+    if (bias is not None and bias.shape[0] != Cc) or (conv_w is not None and tuple(conv_w.shape) != (Cc, taps)):
+        raise KernelError(f"bias or convolution weights do not fit {Cc} channels and {taps} taps")
+    if taps > 1:
+        _need(tail, "kept projected values", torch.float32, 2)
+        if conv_w is None or tail.shape[1] != (taps - 1) * Cc:
+            raise KernelError(f"{taps} taps need weights and {(taps - 1) * Cc} kept values a sequence")
+    if inv_freq is not None:
+        _need(inv_freq, "inv_freq", torch.float32, 1)
+        if inv_freq.shape[0] * 2 != rot_dim:
+            raise KernelError("inv_freq must hold rot_dim / 2 entries")
+    for t, nm in ((step.token_pos, "token_pos"), (step.cu_q, "cu_q"), (step.slots, "slots")):
+        _need(t, nm, torch.int32, 1)
+    n_seqs = step.slots.shape[0]
+    if step.token_pos.shape[0] != T or step.cu_q.shape[0] != n_seqs + 1:
+        raise KernelError("token_pos, cu_q and slots do not describe the step's rows")
+    q = torch.empty((T, nq, Ds), dtype=dt, device=qkv.device)
+    a = _QkConvArgs()
+    a.proj, a.n_parts = qkv.data_ptr(), (qkv.shape[0] if qkv.dim() == 3 else 1)
+    a.part_stride = qkv.stride(0) if qkv.dim() == 3 else 0
+    a.bias, a.conv_w, a.inv_freq = _ptr(bias), _ptr(conv_w), _ptr(inv_freq if rot_dim else None)
+    a.cu_q, a.token_pos, a.slots = step.cu_q.data_ptr(), step.token_pos.data_ptr(), step.slots.data_ptr()
+    a.block_table, a.max_pages, a.page = block_table.data_ptr(), block_table.shape[1], int(page)
+    if taps > 1:
+        a.tail, a.tail_stride = tail.data_ptr(), tail.stride(0)
+    a.q_out, a.k_pages, a.v_pages = q.data_ptr(), k_pages.data_ptr(), v_pages.data_ptr()
+    a.T, a.n_seqs, a.nq, a.nkv, a.D, a.Dv, a.Ds, a.taps = T, n_seqs, nq, nkv, D, Dv, Ds, int(taps)
+    a.rot_dim, a.interleaved, a.v_from_k = int(rot_dim), int(bool(interleaved)), int(bool(values_are_keys))
+    a.rot_scale, a.one_row = float(rot_scale), int(bool(step.decode))
+    _check(_fn("qk_conv", f"gb_qk_conv_{_suffix(dt)}", "pp")(ctypes.addressof(a), _stream()), "qk_conv")
+    return q
+
+
 @_profiled("kv_write", lambda out, kv, *a, **k: (2 * _nbytes(kv), 0))
 def kv_write(kv: torch.Tensor, nkv: int, D: int, *, token_seq, token_pos, slots, block_table,
              k_pages, v_pages, page: int) -> None:
@@ -1670,6 +1747,103 @@ def delta_forward(proj: torch.Tensor, state: torch.Tensor, conv_w: torch.Tensor,
     return y
 
 
+# ---------------------------------------------------------------- delta rule, a decay per channel
+class _ChannelDeltaArgs(ctypes.Structure):
+    _fields_ = [("proj", _P), ("conv_w", _P), ("a_log", _P), ("dt_bias", _P), ("norm_w", _P), ("token_seq", _P),
+                ("cu_q", _P), ("slots", _P), ("state", _P), ("state_stride", _L), ("prep", _P), ("low", _P),
+                ("wide", _P), ("o", _P), ("y", _P), ("n_tokens", _I), ("n_seqs", _I), ("H", _I), ("G", _I),
+                ("dk", _I), ("dv", _I), ("taps", _I), ("n_low", _I), ("unit_eps", _F), ("norm_eps", _F),
+                ("prep_stride", _I), ("max_rows", _I)]
+
+
+def _channel_delta_args(proj, state, conv_w, *, H, G, dk, dv, taps, n_low, token_seq, cu_q, slots):
+    """The arguments that both halves of the mixer share, checked."""
+    _need(proj, "projection", torch.float32, 2)
+    _need(state, "state", torch.float32, 2)
+    _need(conv_w, "convolution weights", torch.float32)
+    Cc = 2 * G * dk + H * dv
+    T = proj.shape[0]
+    if proj.shape[1] != Cc + H + n_low:
+        raise KernelError(f"the projection has {proj.shape[1]} columns, expected {Cc + H + n_low}")
+    if state.shape[1] != delta_state_floats(H, G, dk, dv, taps):
+        raise KernelError(f"a sequence's state has {state.shape[1]} floats, expected "
+                          f"{delta_state_floats(H, G, dk, dv, taps)}")
+    if tuple(conv_w.shape) != (Cc, taps):
+        raise KernelError(f"convolution weights are {tuple(conv_w.shape)}, expected {(Cc, taps)}")
+    for t, nm in ((token_seq, "token_seq"), (cu_q, "cu_q"), (slots, "slots")):
+        _need(t, nm, torch.int32, 1)
+    if token_seq.shape[0] != T or cu_q.shape[0] != slots.shape[0] + 1:
+        raise KernelError("token_seq, cu_q and slots do not describe the step's rows")
+    a = _ChannelDeltaArgs()
+    a.proj, a.conv_w, a.state, a.state_stride = proj.data_ptr(), conv_w.data_ptr(), state.data_ptr(), state.stride(0)
+    a.token_seq, a.cu_q, a.slots = token_seq.data_ptr(), cu_q.data_ptr(), slots.data_ptr()
+    a.n_tokens, a.n_seqs, a.H, a.G, a.dk, a.dv, a.taps, a.n_low = T, slots.shape[0], H, G, dk, dv, taps, n_low
+    a.prep_stride = (Cc + H + G + 3) // 4 * 4
+    return a
+
+
+@_profiled("channel_delta_prepare", lambda out, proj, *a, **k: (_nbytes(proj, *out), 0))
+def channel_delta_prepare(proj: torch.Tensor, state: torch.Tensor, conv_w: torch.Tensor, *, H: int, G: int, dk: int,
+                          dv: int, taps: int, n_low: int, unit_eps: float, token_seq, cu_q, slots,
+                          dtype: torch.dtype):
+    """What comes in front of the recurrence of the delta rule with a decay per channel.  ``proj``
+    [T, C] 32-bit: the columns q [G dk] | k [G dk] | v [H dv] | beta logits [H] | the thin
+    products' inner values [n_low].  Returns (prep, low): ``prep`` [T, P] 32-bit holds what
+    ``channel_delta_run`` takes (unit q and k and v behind their convolutions, beta, k . q), ``low``
+    [T, n_low] the inner values in ``dtype``.  ``state`` is read only (the convolutions' tail)."""
+    a = _channel_delta_args(proj, state, conv_w, H=H, G=G, dk=dk, dv=dv, taps=taps, n_low=n_low,
+                            token_seq=token_seq, cu_q=cu_q, slots=slots)
+    T = proj.shape[0]
+    prep = torch.empty((T, a.prep_stride), dtype=torch.float32, device=proj.device)
+    low = torch.empty((T, n_low), dtype=dtype, device=proj.device)
+    a.prep, a.low, a.unit_eps = prep.data_ptr(), low.data_ptr(), float(unit_eps)
+    _check(_fn("channel_delta", f"gb_channel_delta_prepare_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
+           "channel_delta_prepare")
+    return prep, low
+
+
+def _cost_channel_delta(out, proj, prep, low, wide, state, *a, H, G, dk, dv, **k):
+    T = proj.shape[0]
+    return (_nbytes(prep, wide, out) + 2 * T * H * dv * 4 + 2 * k["slots"].shape[0] * H * dk * dv * 4,
+            6.0 * T * H * dk * dv)
+
+
+@_profiled("channel_delta", _cost_channel_delta)
+def channel_delta_run(proj: torch.Tensor, prep: torch.Tensor, low: torch.Tensor, wide: torch.Tensor,
+                      state: torch.Tensor, conv_w: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+                      norm_w: torch.Tensor, *, H: int, G: int, dk: int, dv: int, taps: int, norm_eps: float,
+                      token_seq, cu_q, slots, dtype: torch.dtype, max_rows: Optional[int] = None) -> torch.Tensor:
+    """The delta rule with a decay per head and key channel on the rows of a step, behind
+    ``channel_delta_prepare`` (whose ``proj``, ``prep`` and ``low`` it is given) and the second thin
+    product ``wide`` [T, H dk + H dv] 32-bit: z | gate logits.  Per head g = exp(-exp(a_log)
+    softplus(z + dt_bias)); S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.  ``state``
+    [slots + 1, delta_state_floats] 32-bit is updated in place for slots that are not negative (the
+    convolutions' tail with it).  Returns y [T, H dv] in ``dtype``: o normalised over dv, times
+    ``norm_w`` and sigmoid(gate).  ``max_rows``: the most rows any sequence brings, when the host
+    knows it; with 1 (a decode step) all of it is one kernel."""
+    n_low = low.shape[1]
+    a = _channel_delta_args(proj, state, conv_w, H=H, G=G, dk=dk, dv=dv, taps=taps, n_low=n_low,
+                            token_seq=token_seq, cu_q=cu_q, slots=slots)
+    T = proj.shape[0]
+    _need(prep, "prepared rows", torch.float32, 2)
+    _need(low, "inner values", dtype, 2)
+    _need(wide, "second thin product", torch.float32, 2)
+    if tuple(prep.shape) != (T, a.prep_stride) or tuple(wide.shape) != (T, H * (dk + dv)):
+        raise KernelError(f"prepared rows {tuple(prep.shape)} and logits {tuple(wide.shape)} do not fit the step")
+    for t, nm, n in ((a_log, "A_log", H), (dt_bias, "dt_bias", H * dk), (norm_w, "norm weight", dv)):
+        _need(t, nm, torch.float32, 1)
+        if t.shape[0] != n:
+            raise KernelError(f"{nm} has {t.shape[0]} elements, expected {n}")
+    o = torch.empty((T, H, dv), dtype=torch.float32, device=proj.device)
+    y = torch.empty((T, H * dv), dtype=dtype, device=proj.device)
+    a.a_log, a.dt_bias, a.norm_w = a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr()
+    a.prep, a.low, a.wide, a.o, a.y = (prep.data_ptr(), low.data_ptr(), wide.data_ptr(), o.data_ptr(), y.data_ptr())
+    a.norm_eps, a.max_rows = float(norm_eps), int(max_rows or 0)
+    _check(_fn("channel_delta", f"gb_channel_delta_run_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
+           "channel_delta", 1 if a.max_rows == 1 else 2)
+    return y
+
+
 # ---------------------------------------------------------------- groups of heads
 @_profiled("head_group", _cost_io)
 def head_group(x: torch.Tensor, first: int, count: int) -> torch.Tensor:
@@ -1859,13 +2033,15 @@ class _LatentArgs(ctypes.Structure):
     _fields_ = [("proj", _P), ("norm_w", _P), ("inv_freq", _P), ("token_seq", _P), ("token_pos", _P),
                 ("slots", _P), ("block_table", _P), ("pages", _P), ("q_plain", _P), ("q_full", _P),
                 ("n_tokens", _I), ("H", _I), ("dn", _I), ("dr", _I), ("R", _I), ("dv", _I), ("Ds", _I),
-                ("max_pages", _I), ("page", _I), ("eps", _F)]
+                ("max_pages", _I), ("page", _I), ("eps", _F), ("q_rank", _I), ("q_norm_w", _P), ("cq", _P),
+                ("queries_only", _I)]
 
 
 @_profiled("latent_prepare", lambda out, proj, *a, **k: (_nbytes(proj) + _nbytes(*out), 0))
 def latent_prepare(proj: torch.Tensor, norm_w: torch.Tensor, inv_freq: Optional[torch.Tensor], *,
                    H: int, dn: int, dr: int, R: int, dv: int, eps: float, token_seq, token_pos,
-                   slots, block_table, pages, page: int, dtype: torch.dtype):
+                   slots, block_table, pages, page: int, dtype: torch.dtype,
+                   q_norm_w: Optional[torch.Tensor] = None):
     """What latent attention does between its projection and its attention.  ``proj``
     [T, H (dn + dr) + R + dr + H dv] 32-bit: queries (per head dn plain, dr rotated
     elements) | the down projection | the gate.  Stores the row [c | k_rot | zeros] of
@@ -1873,15 +2049,23 @@ def latent_prepare(proj: torch.Tensor, norm_w: torch.Tensor, inv_freq: Optional[
     numbers of the down projection, RMS-normalised times ``norm_w``; k_rot: its last dr,
     rotated: element 2i with element 2i + 1 by position * inv_freq[i]).  Returns
     (q_plain [T, H, dn], q_full [T, H, Ds]) in ``dtype``; of q_full the columns from R on
-    are written (the rotated query part, then zeros), the first R are left to the caller."""
+    are written (the rotated query part, then zeros), the first R are left to the caller.
+    ``q_norm_w`` [q_rank]: the projection's first q_rank columns are the queries' latent in
+    their place; instead of q_plain it is returned, RMS-normalised, [T, q_rank], and of q_full
+    what is zero is written when there is no rotated part (``latent_queries`` does the rest)."""
     _need(proj, "projection", torch.float32, 2)
     _need(norm_w, "latent norm weight", torch.float32, 1)
     T = proj.shape[0]
     _need(pages, "latent pages", dtype, 4)
     Ds = pages.shape[-1]
-    if proj.shape[1] != H * (dn + dr) + R + dr + H * dv or norm_w.shape[0] != R:
-        raise KernelError(f"the projection has {proj.shape[1]} columns, expected "
-                          f"{H * (dn + dr) + R + dr + H * dv}; the norm weight {norm_w.shape[0]} for {R}")
+    q_rank = 0
+    if q_norm_w is not None:
+        _need(q_norm_w, "query latent norm weight", torch.float32, 1)
+        q_rank = q_norm_w.shape[0]
+    want = (q_rank or H * (dn + dr)) + R + dr + H * dv
+    if proj.shape[1] != want or norm_w.shape[0] != R:
+        raise KernelError(f"the projection has {proj.shape[1]} columns, expected {want}; the norm weight "
+                          f"{norm_w.shape[0]} for {R}")
     if tuple(pages.shape[1:]) != (1, page, Ds) or Ds < R + dr:
         raise KernelError(f"pages are {tuple(pages.shape)}, expected [*, 1, {page}, >= {R + dr}]")
     if dr:
@@ -1891,9 +2075,11 @@ def latent_prepare(proj: torch.Tensor, norm_w: torch.Tensor, inv_freq: Optional[
     for t, nm in ((token_seq, "token_seq"), (token_pos, "token_pos"), (slots, "slots")):
         _need(t, nm, torch.int32, 1)
     _need(block_table, "block table", torch.int32, 2)
-    q_plain = torch.empty((T, H, dn), dtype=dtype, device=proj.device)
+    q_plain = torch.empty((T, q_rank) if q_rank else (T, H, dn), dtype=dtype, device=proj.device)
     q_full = torch.empty((T, H, Ds), dtype=dtype, device=proj.device)
     a = _LatentArgs()
+    if q_rank:
+        a.q_rank, a.q_norm_w, a.cq = q_rank, q_norm_w.data_ptr(), q_plain.data_ptr()
     a.proj, a.norm_w, a.inv_freq = proj.data_ptr(), norm_w.data_ptr(), _ptr(inv_freq)
     a.token_seq, a.token_pos, a.slots = token_seq.data_ptr(), token_pos.data_ptr(), slots.data_ptr()
     a.block_table, a.pages = block_table.data_ptr(), pages.data_ptr()
@@ -1903,6 +2089,28 @@ def latent_prepare(proj: torch.Tensor, norm_w: torch.Tensor, inv_freq: Optional[
     _check(_fn("latent", f"gb_latent_prepare_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
            "latent_prepare")
     return q_plain, q_full
+
+
+@_profiled("latent_queries", lambda out, q, *a, **k: (2 * _nbytes(q), 0))
+def latent_queries(q: torch.Tensor, q_full: torch.Tensor, inv_freq: torch.Tensor, *, H: int, dn: int, dr: int,
+                   R: int, token_pos) -> torch.Tensor:
+    """Queries [T, H (dn + dr)] (32-bit) that a product has expanded from their latent: the dr
+    rotated elements of every head go, turned, to columns R .. R + dr of ``q_full`` [T, H, Ds]
+    (zeros behind them), the dn plain ones are returned [T, H, dn]."""
+    _need(q, "queries", torch.float32, 2)
+    _need(inv_freq, "inv_freq", torch.float32, 1)
+    _need(token_pos, "token_pos", torch.int32, 1)
+    T = q.shape[0]
+    if q.shape[1] != H * (dn + dr) or tuple(q_full.shape[:2]) != (T, H) or inv_freq.shape[0] * 2 != dr:
+        raise KernelError(f"queries {tuple(q.shape)} do not hold {H} heads of {dn} + {dr} elements")
+    q_plain = torch.empty((T, H, dn), dtype=q_full.dtype, device=q.device)
+    a = _LatentArgs()
+    a.proj, a.inv_freq, a.token_pos = q.data_ptr(), inv_freq.data_ptr(), token_pos.data_ptr()
+    a.q_plain, a.q_full, a.queries_only = q_plain.data_ptr(), q_full.data_ptr(), 1
+    a.n_tokens, a.H, a.dn, a.dr, a.R, a.Ds = T, H, dn, dr, R, q_full.shape[2]
+    _check(_fn("latent", f"gb_latent_prepare_{_suffix(q_full.dtype)}", "pp")(ctypes.addressof(a), _stream()),
+           "latent_queries")
+    return q_plain
 
 
 class _HeadsMmArgs(ctypes.Structure):
@@ -2257,6 +2465,75 @@ def gated_norm(res_in: Optional[torch.Tensor], terms, *, dtype: torch.dtype,
     _check(_fn("gated_norm", f"gb_gated_norm_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
            "gated_norm")
     return res_out, y
+
+
+# ---------------------------------------------------------------- several residual streams
+class _HyperNormArgs(ctypes.Structure):
+    _fields_ = [("res_in", _P), ("in_stride", _L), ("delta", _P), ("parts", _P), ("n_parts", _I),
+                ("part_stride", _L), ("mix", _P), ("out", _P), ("read", _P), ("rows", _P), ("norm_w", _P),
+                ("eps", _F), ("res_out", _P), ("out_stride", _L), ("y", _P), ("n_rows", _I), ("N", _I), ("S", _I)]
+
+
+HYPER_MAX_STREAMS = 16       # streams the kernel takes (HN_MAX_S)
+
+
+def _cost_hyper(out, res_in, delta, **k):
+    res, y = out
+    stored = 0 if k.get("mix") is None or k.get("rows") is not None else _nbytes(res)
+    return _nbytes(res_in, delta, y) + stored, 0
+
+
+@_profiled("hyper_norm", _cost_hyper)
+def hyper_norm(res_in: torch.Tensor, delta: Optional[torch.Tensor], *, streams: int, dtype: torch.dtype,
+               mix: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
+               read: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+               norm_w: Optional[torch.Tensor] = None, eps: float = 0.0):
+    """The boundary between two sublayers of a model with ``streams`` residual streams, in
+    32-bit: X'_t = sum_s mix[s, t] X_s + out[t] * delta; u = sum_t read[t] X'_t (the plain sum
+    without ``read``); y = rmsnorm(u) * norm_w (u itself without ``norm_w``) in ``dtype``.
+    ``res_in`` is [streams, T, N], or [T, N] when all streams are still equal; ``delta`` is
+    [T, N] in ``dtype`` or a stack of 32-bit partial sums [P, T, N], added in order, and comes
+    with ``mix`` [streams, streams] (indexed from, to) and ``out`` [streams].  Returns (X', y):
+    X' replaces ``res_in`` in place where that holds all streams; with ``rows`` the new streams
+    are not kept and X' is ``res_in``."""
+    _need(res_in, "streams", torch.float32)
+    equal = res_in.dim() == 2
+    if not equal and (res_in.dim() != 3 or res_in.shape[0] != streams):
+        raise KernelError(f"streams are {tuple(res_in.shape)}, expected [{streams}, T, N] or [T, N]")
+    T, N = res_in.shape[-2:]
+    if (delta is None) != (mix is None) or (mix is None) != (out is None):
+        raise KernelError("a sublayer's result comes with the weights that put it back")
+    a = _HyperNormArgs()
+    if delta is not None:
+        if delta.dim() == 3:
+            _need(delta, "partial sums", torch.float32, 3)
+            a.parts, a.n_parts, a.part_stride = delta.data_ptr(), delta.shape[0], delta.stride(0)
+        else:
+            _need(delta, "delta", dtype, 2)
+            a.delta = delta.data_ptr()
+        if tuple(delta.shape[-2:]) != (T, N):
+            raise KernelError(f"a result of {tuple(delta.shape)} for streams of {(T, N)}")
+    for t, nm, shape in ((mix, "mixing weights", (streams, streams)), (out, "write weights", (streams,)),
+                         (read, "read weights", (streams,)), (norm_w, "norm weight", (N,))):
+        if t is not None:
+            _need(t, nm, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"{nm} are {tuple(t.shape)}, expected {shape}")
+    if rows is not None:
+        _need(rows, "row list", torch.int32, 1)
+    n_rows = rows.shape[0] if rows is not None else T
+    res = res_in
+    if mix is not None and rows is None:
+        if equal:
+            res = torch.empty((streams, T, N), dtype=torch.float32, device=res_in.device)
+        a.res_out, a.out_stride = res.data_ptr(), res.stride(0)
+    y = torch.empty((n_rows, N), dtype=dtype, device=res_in.device)
+    a.res_in, a.in_stride = res_in.data_ptr(), 0 if equal else res_in.stride(0)
+    a.mix, a.out, a.read, a.rows, a.norm_w = _ptr(mix), _ptr(out), _ptr(read), _ptr(rows), _ptr(norm_w)
+    a.eps, a.y, a.n_rows, a.N, a.S = float(eps), y.data_ptr(), n_rows, N, int(streams)
+    _check(_fn("hyper_norm", f"gb_hyper_norm_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
+           "hyper_norm")
+    return res, y
 
 
 @_profiled("head_gate", lambda out, x, gate, *a, **k: (_nbytes(x) + out.numel() * out.element_size(), 0))

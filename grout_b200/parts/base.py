@@ -25,13 +25,23 @@ class ParamSpec:
     kind: "matrix" (a linear or embedding weight), "vector" (norm weights and
     other small tensors around one), "offset" (biases and other small tensors
     around zero), "fraction" (values inside (0, 1)), "average" (the weights of a
-    weighted sum whose last term leads) or "table" (integer tables, kept as int32).
+    weighted sum whose last term leads), "mixing" (a square matrix near the identity) or "table" (integer tables, kept as int32).
     The loader keeps bfloat16 as bfloat16 and 32-bit as 32-bit for every kind;
     only the true 32-bit path widens, and only half precision is converted.
+
+    ``free``: axes whose size no configuration states, so that the tensor decides (the inner
+    size of a product of two thin matrices, say); ``shape`` then holds the size that random
+    weights take, and the part checks that its tensors fit together.
     """
     shape: Tuple[int, ...]
     kind: str = "matrix"
     optional: bool = False
+    free: Tuple[int, ...] = ()
+
+    def takes(self, shape) -> bool:
+        """Whether a tensor of this shape fits."""
+        return len(shape) == len(self.shape) and all(
+            a == b or (i in self.free and a > 0) for i, (a, b) in enumerate(zip(shape, self.shape)))
 
 
 @dataclass(frozen=True)

@@ -16,7 +16,7 @@ from typing import Optional
 
 from .base import BuildContext, ParamSpec, Part, PartSpec, build_part, register_part
 from .linear import Linear
-from .norm import Contribution, stream_add
+from .norm import Contribution, HyperConnected, stream_add
 
 
 class Block(Part):
@@ -66,6 +66,61 @@ class PreNormBlock(Block):
             return res, a
         res, m = self.norm2.add_norm(res, a)
         return res, self.feedforward.forward(m, step)
+
+
+@register_part("block", "hyper_prenorm")
+class HyperPreNormBlock(PreNormBlock):
+    """A pre-norm layer on several residual streams ("hyper-connections").  The streams
+    X_1 .. X_s all start as the embedding; for the mixer (n = 1) and the feed-forward (n = 2)
+
+        y = sublayer(norm_n(sum_s in_n[s] X_s));   X_t <- sum_s mix_n[s, t] X_s + out_n[t] y
+
+    with learned tensors ``in``, ``out`` [streams] and ``mix`` [streams, streams] (from, to)
+    under the layer's prefix and ``hyper1`` / ``hyper2``.  A sublayer's result leaves as a
+    ``HyperConnected``: one kernel mixes the streams, puts the result back, sums up what the
+    next norm looks at and normalises it.  A model's last norm, which is given no ``read``
+    weights, sees the streams' sum."""
+
+    def __init__(self, ctx: BuildContext, norm1: PartSpec, mixer: PartSpec, streams: int,
+                 norm2: Optional[PartSpec] = None, feedforward: Optional[PartSpec] = None,
+                 hyper1: str = "hyper1.", hyper2: str = "hyper2."):
+        super().__init__(ctx, norm1, mixer, norm2, feedforward)
+        self.streams = int(streams)
+        if self.streams < 1:
+            raise ValueError("a model has at least one residual stream")
+        self.hyper = (hyper1, hyper2) if feedforward else (hyper1,)
+        self.connections = []              # per sublayer (in, mix, out), 32-bit
+
+    def param_specs(self):
+        S = self.streams
+        return {h + n: spec for h in self.hyper for n, spec in (
+            ("in", ParamSpec((S,), "average")), ("out", ParamSpec((S,), "vector")),
+            ("mix", ParamSpec((S, S), "mixing")))}
+
+    def load(self, params):
+        # 32-bit whatever the checkpoint stores: the sums into the streams are 32-bit
+        self.connections = [tuple(params[h + n].float().contiguous() for n in ("in", "mix", "out"))
+                            for h in self.hyper]
+
+    def kernel_modules(self):
+        return ("hyper_norm",)
+
+    def forward(self, res, pending, step, cache):
+        if res is None:                    # an embedding that left a first contribution
+            res, pending = pending.float(), None
+        if pending is None:
+            pending = HyperConnected(self.streams)
+        if not isinstance(pending, HyperConnected) or pending.streams != self.streams:
+            raise ValueError(f"a layer on {self.streams} residual streams was given {type(pending).__name__}")
+        read, mix, out = self.connections[0]
+        pending.read = read
+        res, n = self.norm1.add_norm(res, pending)
+        pending = HyperConnected(self.streams, self.mixer.forward(n, step, cache), mix, out)
+        if self.feedforward is None:
+            return res, pending
+        pending.read, mix, out = self.connections[1]
+        res, m = self.norm2.add_norm(res, pending)
+        return res, HyperConnected(self.streams, self.feedforward.forward(m, step), mix, out)
 
 
 @register_part("block", "sandwich")

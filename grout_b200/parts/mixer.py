@@ -21,7 +21,7 @@ from typing import Optional
 
 import torch
 
-from ..cache.spec import KVSpec, SideBySideSpec
+from ..cache.spec import KVSpec, SideBySideSpec, StateSpec
 from ..kernels import ops
 from .base import BuildContext, ParamSpec, Part, PartSpec, build_part, register_part
 from .linear import Linear
@@ -75,7 +75,15 @@ class GQAAttention(Mixer):
     [heads, hidden]; 32-bit sums, 32-bit sigmoid), before the o projection.  A rotation
     of neighbouring pairs (``rotary_interleaved``) is folded into the q/k kernel as the
     half-split one is.
-    ``names`` replaces local tensor names (keys: q, k, v, o, q_norm, k_norm, sink, g).
+    ``qk_bias``: the q and k projections have biases (tensors ``q_bias``, ``k_bias``).
+    ``conv_taps``: a causal convolution over time on every channel of q and k (tensors
+    ``q_conv``, ``k_conv`` [channels, taps], the last tap the current token's, no bias, zeros
+    before the sequence's start) comes right behind the projection and its bias, in front of the
+    rotation; values that are the keys are the convolved ones.  The last taps - 1 projected
+    values of a sequence are kept beside its keys and values (the layer's cache need is then the
+    pair of both).  Bias, convolution, rotation and the stores are one kernel.
+    ``names`` replaces local tensor names (keys: q, k, v, o, q_norm, k_norm, sink, g, q_bias,
+    k_bias, q_conv, k_conv).
 
     The mixer can run beside another one on the same input (``SideBySide``): it then names
     the rows whose 32-bit products with the input it needs (``side_weight``: the head gate's),
@@ -85,7 +93,8 @@ class GQAAttention(Mixer):
 
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight",
              "o": "o_proj.weight", "q_norm": "q_norm.weight", "k_norm": "k_norm.weight",
-             "sink": "sink", "g": "g"}
+             "sink": "sink", "g": "g", "q_bias": "q_proj.bias", "k_bias": "k_proj.bias",
+             "q_conv": "q_conv.weight", "k_conv": "k_conv.weight"}
 
     def __init__(self, ctx: BuildContext, hidden: int, n_heads: int, n_kv_heads: int,
                  head_dim: int, position: PartSpec, qk_norm_eps: Optional[float] = None,
@@ -94,8 +103,19 @@ class GQAAttention(Mixer):
                  values_are_keys: bool = False, names: Optional[dict] = None,
                  v_head_dim: Optional[int] = None, q_temp: Optional[tuple] = None,
                  sink_logit: Optional[float] = None, keep_first: int = 0, head_gate: bool = False,
-                 chunk: Optional[int] = None, reach: Optional[int] = 0):
+                 chunk: Optional[int] = None, reach: Optional[int] = 0, qk_bias: bool = False,
+                 conv_taps: Optional[int] = None):
         super().__init__(ctx)
+        self.qk_bias, self.taps = bool(qk_bias), int(conv_taps or 1)
+        self.convolves = conv_taps is not None
+        if self.taps < 1:
+            raise ValueError("a convolution has at least one tap")
+        # both are the work of one kernel, which knows no norms and no temperatures
+        self.conv_path = self.qk_bias or self.convolves
+        if self.conv_path and (shares_kv or qk_norm_eps is not None or q_temp):
+            raise ValueError("biases and convolutions of q and k go with keys of the layer's own, without "
+                             "norms and without a query temperature")
+        self.conv_bias = self.conv_w = None
         self.chunk = int(chunk or 0)
         # the keys that must stay in the cache: this layer's window or what its readers need
         self.kept_window = None if window is None or reach is None else max(int(window), int(reach))
@@ -111,7 +131,9 @@ class GQAAttention(Mixer):
         self.Dv = int(v_head_dim) if v_head_dim else self.D
         # the width of a cached row, of a query and of the attention's output
         self.Ds = max(self.D, self.Dv)
-        if self.Ds != self.D or self.Ds != self.Dv:
+        if self.conv_path and ctx.dtype == torch.bfloat16:
+            self.Ds = (self.Ds + 15) // 16 * 16   # the tensor-core kernels take multiples of 16
+        elif self.Ds != self.D or self.Ds != self.Dv:
             if values_are_keys:
                 raise ValueError("values of another size than the keys go with a v projection")
             if ctx.dtype == torch.bfloat16:       # the tensor-core kernels take multiples of 16
@@ -131,12 +153,15 @@ class GQAAttention(Mixer):
         self.shares_kv = bool(shares_kv)
         self.softcap = float(softcap) if softcap else None
         self.has_sinks, self.values_are_keys = bool(sinks), bool(values_are_keys)
-        if self.values_are_keys and (self.shares_kv or qk_norm_eps is not None):
-            raise ValueError("values that are the keys go with a cache of the layer's own and "
-                             "with keys that are not normalised")
+        if self.values_are_keys and (self.shares_kv or qk_norm_eps is not None or self.Dv != self.D):
+            raise ValueError("values that are the keys go with a cache of the layer's own, with keys that "
+                             "are not normalised and with values of their size")
         self.names = dict(self.NAMES, **(names or {}))
         self.sink = None
         self.position = build_part("position", position, ctx)
+        if self.conv_path and self.position.rotary() is None and \
+                type(self.position).apply_qk is not PositionEncoding.apply_qk:
+            raise ValueError("biases and convolutions of q and k take a rotation (or no position encoding)")
         self.qkv = self.o = None
         self.q_norm_w = self.k_norm_w = None
 
@@ -158,6 +183,11 @@ class GQAAttention(Mixer):
             specs[nm["sink"]] = ParamSpec((nq,), "offset")
         if self.head_gate:
             specs[nm["g"]] = ParamSpec((nq, H))
+        for n, rows in (("q", nq * D), ("k", nkv * D)):
+            if self.qk_bias:
+                specs[nm[n + "_bias"]] = ParamSpec((rows,), "offset")
+            if self.convolves:
+                specs[nm[n + "_conv"]] = ParamSpec((rows, self.taps), "vector")
         return specs
 
     def load(self, params):
@@ -188,9 +218,12 @@ class GQAAttention(Mixer):
                 self.k_norm_w = params[nm["k_norm"]].contiguous()
         if self.has_sinks:       # 32-bit, as the scores are
             self.sink = params[nm["sink"]].float().contiguous()
+        both = lambda n: torch.cat([params[nm["q" + n]], params[nm["k" + n]]]).float().contiguous()
+        self.conv_bias = both("_bias") if self.qk_bias else None
+        self.conv_w = both("_conv") if self.convolves else None
 
     def kernel_modules(self):
-        mods = ("qk_prepare", "attn_generic") + self.qkv.kernel_modules()
+        mods = ("qk_conv" if self.conv_path else "qk_prepare", "attn_generic") + self.qkv.kernel_modules()
         mods += self.o.kernel_modules() if self.o else ()
         if self.head_gate or self.beside:
             mods += ("elementwise",)
@@ -201,8 +234,12 @@ class GQAAttention(Mixer):
     def cache_spec(self):
         if self.shares_kv:
             return None
-        return KVSpec(self.nkv, self.Ds, self.kept_window, keep_first=self.keep_first,
-                      chunk=self.chunk or None)
+        kv = KVSpec(self.nkv, self.Ds, self.kept_window, keep_first=self.keep_first,
+                    chunk=self.chunk or None)
+        if self.taps == 1:
+            return kv
+        # what the convolution of a sequence's next token looks back to
+        return SideBySideSpec((kv, StateSpec(((self.taps - 1) * (self.nq + self.nkv) * self.D,), torch.float32)))
 
     # -- beside another mixer ------------------------------------------------
     @property
@@ -239,6 +276,11 @@ class GQAAttention(Mixer):
         """The heads' outputs [T, heads, Ds] (keys and values of the step's rows stored)."""
         T = x.shape[0]
         rot = self.position.rotary()
+        tail = None
+        if self.taps > 1:
+            if not isinstance(cache, tuple) or len(cache) != 2:
+                raise ValueError(f"attention behind a convolution was given the cache {cache!r}")
+            cache, tail = cache[0], cache[1].state
         if cache is None or (cache.spec.n_kv_heads, cache.spec.head_dim) != (self.nkv, self.Ds):
             raise ValueError(f"attention with {self.nkv} kv heads of {self.Ds} was given the cache "
                              f"{None if cache is None else cache.spec}")
@@ -246,6 +288,17 @@ class GQAAttention(Mixer):
         if not fused and (self.Ds != self.D or self.q_temp):
             raise ValueError("a position encoding with arithmetic of its own goes with neither "
                              "values of another size nor a query temperature")
+        if self.conv_path:
+            qkv = self.qkv(x, out_dtype=torch.float32, partial_ok=x.dtype == torch.bfloat16)
+            q = ops.qk_conv(qkv, self.nq, self.nkv, self.D, bias=self.conv_bias, conv_w=self.conv_w, tail=tail,
+                            taps=self.taps, v_dim=self.Dv, values_are_keys=self.values_are_keys,
+                            inv_freq=rot.inv_freq if rot else None, rot_dim=rot.rot_dim if rot else 0,
+                            interleaved=bool(rot and rot.interleaved), rot_scale=rot.amplitude if rot else 1.0,
+                            step=step, block_table=cache.block_table, k_pages=cache.k_pages,
+                            v_pages=cache.v_pages, page=cache.page)
+            return ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, step=step, page=cache.page,
+                                 scale=self.scale, window=self.window, softcap=self.softcap, sinks=self.sink,
+                                 keep_first=self.keep_first, chunk=self.chunk)
         # the q/k preparation can add the partial sums of a split-K projection itself
         qkv = self.qkv(x, partial_ok=fused and x.dtype == torch.bfloat16)
         seen = dict(step=step, page=cache.page, scale=self.scale, window=self.window, softcap=self.softcap,
@@ -486,20 +539,28 @@ class LatentAttention(Mixer):
         query sees (its own position and the ``window`` - 1 before it, or all before it)
         y = Wo [ heads * sigmoid(Wg h) ]           (the gate only with ``gated``)
 
+    With ``q_rank`` the queries come from a latent, too: q = Wuq (rmsnorm(Wdq h) * wq), the
+    norm over the q_rank numbers with the same ``norm_eps``.  ``sinks`` gives every head a
+    learned logit (tensor ``sink`` [heads]) that stands in the softmax's denominator as
+    exp(sink), is not scaled and has no value.
+
     The cache keeps [c | k_rot] per token, once for all heads; Wuk is folded into
     the query ((Wuk_i^T q_plain) . c) and Wuv applied to the attention's output over
     the latents, so the attention kernels see query heads that all read one kv head of
     kv_rank + rot_dim elements whose values are its keys.  ``position`` rotates the
     rot_dim part (neighbouring pairs).  Norm, rotation and gate are 32-bit on the
-    projection's 32-bit sums.  ``names`` replaces local tensor names (keys q, dkv,
-    dkv_norm, uk, uv, g, o)."""
+    projection's 32-bit sums.  ``names`` replaces local tensor names (keys q, dq, dq_norm,
+    uq, dkv, dkv_norm, uk, uv, sink, g, o)."""
 
-    NAMES = {"q": "q", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "g": "g", "o": "o"}
+    NAMES = {"q": "q", "dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "sink": "sink", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "g": "g", "o": "o"}
 
     def __init__(self, ctx: BuildContext, hidden: int, n_heads: int, head_dim: int, rot_dim: int,
                  v_head_dim: int, kv_rank: int, position: PartSpec, scale: float, norm_eps: float,
-                 window: Optional[int] = None, gated: bool = True, names: Optional[dict] = None):
+                 window: Optional[int] = None, gated: bool = True, q_rank: Optional[int] = None,
+                 sinks: bool = False, names: Optional[dict] = None):
         super().__init__(ctx)
+        self.q_rank, self.has_sinks = int(q_rank or 0), bool(sinks)
+        self.uq = self.q_norm_w = self.sink = None
         self.hidden, self.H, self.dn, self.dr = int(hidden), int(n_heads), int(head_dim), int(rot_dim)
         self.dv, self.R = int(v_head_dim), int(kv_rank)
         self.scale, self.norm_eps = float(scale), float(norm_eps)
@@ -521,18 +582,25 @@ class LatentAttention(Mixer):
 
     def param_specs(self):
         W, H, nm = self.hidden, self.H, self.names
-        specs = {nm["q"]: ParamSpec((H * (self.dn + self.dr), W)),
-                 nm["dkv"]: ParamSpec((self.R + self.dr, W)),
-                 nm["dkv_norm"]: ParamSpec((self.R,), "vector"),
-                 nm["uk"]: ParamSpec((H * self.dn, self.R)), nm["uv"]: ParamSpec((H * self.dv, self.R)),
-                 nm["o"]: ParamSpec((W, H * self.dv))}
+        rows = H * (self.dn + self.dr)
+        if self.q_rank:
+            specs = {nm["dq"]: ParamSpec((self.q_rank, W)), nm["dq_norm"]: ParamSpec((self.q_rank,), "vector"),
+                     nm["uq"]: ParamSpec((rows, self.q_rank))}
+        else:
+            specs = {nm["q"]: ParamSpec((rows, W))}
+        if self.has_sinks:
+            specs[nm["sink"]] = ParamSpec((H,), "offset")
+        specs.update({nm["dkv"]: ParamSpec((self.R + self.dr, W)),
+                      nm["dkv_norm"]: ParamSpec((self.R,), "vector"),
+                      nm["uk"]: ParamSpec((H * self.dn, self.R)), nm["uv"]: ParamSpec((H * self.dv, self.R)),
+                      nm["o"]: ParamSpec((W, H * self.dv))})
         if self.gated:
             specs[nm["g"]] = ParamSpec((H * self.dv, W))
         return specs
 
     def load(self, params):
         nm = self.names
-        ws = [params[nm["q"]], params[nm["dkv"]]] + ([params[nm["g"]]] if self.gated else [])
+        ws = [params[nm["dq" if self.q_rank else "q"]], params[nm["dkv"]]] + ([params[nm["g"]]] if self.gated else [])
         if len({w.dtype for w in ws}) != 1:
             raise ValueError("the projections of one mixer must be stored in one dtype to be fused")
         self.proj = Linear(torch.cat(ws, dim=0), self.ctx.products)
@@ -542,9 +610,15 @@ class LatentAttention(Mixer):
         self.uk_t = params[nm["uk"]].view(self.H, self.dn, self.R).transpose(1, 2).to(dt).contiguous()
         self.uv = params[nm["uv"]].view(self.H, self.dv, self.R).to(dt).contiguous()
         self.norm_w = params[nm["dkv_norm"]].float().contiguous()
+        if self.q_rank:
+            self.uq = Linear(params[nm["uq"]], self.ctx.products)
+            self.q_norm_w = params[nm["dq_norm"]].float().contiguous()
+        if self.has_sinks:       # 32-bit, as the scores are
+            self.sink = params[nm["sink"]].float().contiguous()
 
     def kernel_modules(self):
         mods = ("latent", "attn_generic") + self.proj.kernel_modules() + self.o.kernel_modules()
+        mods += self.uq.kernel_modules() if self.uq else ()
         if self.ctx.dtype == torch.bfloat16:
             mods += ops.fast_attention_modules(self.Ds, min(self.H, self.GROUP), 1)
         return mods
@@ -560,9 +634,10 @@ class LatentAttention(Mixer):
         kw = dict(step=step, page=cache.page, scale=self.scale, window=self.window)
         if (self.H <= self.GROUP or q.dtype != torch.bfloat16
                 or not ops.fast_attention_takes(self.Ds, self.GROUP, 1, cache.page)):
-            return ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, **kw)
+            return ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, sinks=self.sink, **kw)
+        sinks = lambda a: None if self.sink is None else self.sink[a:a + self.GROUP]
         return ops.join_heads([ops.attention(ops.head_group(q, a, min(self.GROUP, self.H - a)), cache.k_pages,
-                                             cache.v_pages, cache.block_table, **kw)
+                                             cache.v_pages, cache.block_table, sinks=sinks(a), **kw)
                                for a in range(0, self.H, self.GROUP)])
 
     def captures_prompts(self):
@@ -579,9 +654,14 @@ class LatentAttention(Mixer):
             proj, self.norm_w, rot.inv_freq if rot else None, H=H, dn=self.dn, dr=self.dr, R=self.R,
             dv=self.dv if self.gated else 0, eps=self.norm_eps, token_seq=step.token_seq,
             token_pos=step.token_pos, slots=step.slots, block_table=cache.block_table,
-            pages=cache.k_pages, page=cache.page, dtype=self.ctx.dtype)
+            pages=cache.k_pages, page=cache.page, dtype=self.ctx.dtype, q_norm_w=self.q_norm_w)
+        if self.q_rank and self.dr:         # (q_plain is the queries' latent here)
+            q_plain = ops.latent_queries(self.uq(q_plain, out_dtype=torch.float32), q, rot.inv_freq, H=H,
+                                         dn=self.dn, dr=self.dr, R=self.R, token_pos=step.token_pos)
+        elif self.q_rank:
+            q_plain = self.uq(q_plain).view(T, H, self.dn)
         ops.heads_mm(q_plain, self.uk_t, q)
         attn = self._attend(q, step, cache)
         y = ops.heads_mm(attn, self.uv, gate=proj if self.gated else None,
-                         gate_col=H * (self.dn + self.dr) + self.R + self.dr)
+                         gate_col=(self.q_rank or H * (self.dn + self.dr)) + self.R + self.dr)
         return self.o(y.view(T, H * self.dv), partial_ok=True)

@@ -15,6 +15,8 @@
   for a contribution whose own norm is an RMS norm (with, if the layer has one, a
   learned per-channel scale behind it); every other combination is resolved
   first and goes on as above.
+  Of a model with several residual streams ``res`` is their stack and ``delta`` a
+  ``HyperConnected``; ``RMSNorm`` does all of that in one kernel, too.
 * ``stream_add(res, delta, dtype) -> (res, x)``: the same sum without a norm
   behind it, for sublayers that read the stream as it is: ``x`` is the updated
   stream in the compute dtype.
@@ -94,6 +96,39 @@ class Averaged:
         return (self.weights.float()[:, None, None] * hist).sum(dim=0)
 
 
+@dataclass
+class HyperConnected:
+    """What a model with several residual streams hands to the next norm.  The stream that the
+    norm is given is then a 32-bit stack [streams, T, N] (or [T, N] while all streams are
+    still equal); ``delta``, the last sublayer's result (a tensor as in ``Contribution``, None
+    in front of the first), goes back into all of them,
+
+        X_t <- sum_s mix[s, t] X_s + out[t] * delta,
+
+    and the norm reads sum_t read[t] X_t (the streams' plain sum when ``read`` is None).  The
+    weights are 32-bit: ``mix`` [streams, streams], ``out`` and ``read`` [streams]."""
+    streams: int
+    delta: Optional[torch.Tensor] = None
+    mix: Optional[torch.Tensor] = None
+    out: Optional[torch.Tensor] = None
+    read: Optional[torch.Tensor] = None
+
+    def resolve(self, res: torch.Tensor, rows: Optional[torch.Tensor] = None):
+        """Step by step, for norms without a kernel that takes all of it: (the new streams,
+        what the norm reads), both 32-bit, of ``rows`` only when given."""
+        X = res if res.dim() == 3 else res[None].expand(self.streams, *res.shape)
+        d = self.delta
+        if rows is not None:
+            X = X.index_select(1, rows.long())
+            d = None if d is None else d.index_select(d.dim() - 2, rows.long())
+        if d is not None:
+            d = d.sum(dim=0) if d.dim() == 3 else d.float()
+            X = torch.einsum("st,sij->tij", self.mix.float(), X) + self.out.float()[:, None, None] * d
+        X = X.contiguous()
+        w = X.new_ones(self.streams) if self.read is None else self.read.float()
+        return X, (w[:, None, None] * X).sum(dim=0)
+
+
 def as_terms(pending):
     """``pending`` as a tuple of ``Contribution``s (tensors are wrapped, None is dropped)."""
     if pending is None:
@@ -130,6 +165,8 @@ class Norm(Part):
 
     def add_norm(self, res: Optional[torch.Tensor], delta: Optional[torch.Tensor],
                  rows: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+        if isinstance(delta, HyperConnected):
+            return self._add_streams(res, delta, rows)
         if isinstance(delta, Averaged):
             res, delta = delta.resolve(res, rows), None
             return res, self.forward(ops.cast(res, self.ctx.dtype))
@@ -137,6 +174,11 @@ class Norm(Part):
             delta = resolve_terms(delta)
         res = residual_add(res, delta, rows)
         return res, self.forward(ops.cast(res, self.ctx.dtype))
+
+    def _add_streams(self, res, pending, rows):
+        """Several residual streams, step by step."""
+        res, read = pending.resolve(res, rows)
+        return res, self.add_norm(read, None)[1]
 
 
 def residual_add(res, delta, rows=None) -> torch.Tensor:
@@ -195,7 +237,14 @@ class RMSNorm(Norm):
     def kernel_modules(self):
         return ("norm",)
 
+    def _add_streams(self, res, pending, rows):
+        return ops.hyper_norm(res, pending.delta, streams=pending.streams, dtype=self.ctx.dtype,
+                              mix=pending.mix, out=pending.out, read=pending.read, rows=rows,
+                              norm_w=self.weight32(), eps=self.eps)
+
     def add_norm(self, res, delta, rows=None):
+        if isinstance(delta, HyperConnected):
+            return self._add_streams(res, delta, rows)
         if isinstance(delta, (Averaged, tuple, list)) or (isinstance(delta, Contribution)
                                                           and delta.gate is not None):
             return self._add_gated(res, delta, rows)
@@ -289,6 +338,8 @@ class LayerNorm(Norm):
         return y
 
     def add_norm(self, res, delta, rows=None):
+        if isinstance(delta, HyperConnected):
+            return self._add_streams(res, delta, rows)
         post = None
         mult, offset = 1.0, None
         if isinstance(delta, Averaged):          # resolved step by step, then normalised
@@ -348,6 +399,8 @@ class DynamicTanh(Norm):
         return y
 
     def add_norm(self, res, delta, rows=None):
+        if isinstance(delta, HyperConnected):
+            return self._add_streams(res, delta, rows)
         if isinstance(delta, Averaged):          # resolved step by step, then normalised
             res, delta, rows = delta.resolve(res, rows), None, None
         elif isinstance(delta, (Contribution, tuple, list)):

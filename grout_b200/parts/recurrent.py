@@ -103,6 +103,114 @@ class GatedDelta(Mixer):
         return self.o(y, partial_ok=True)
 
 
+@register_part("mixer", "channel_delta")
+class ChannelDelta(Mixer):
+    """The delta rule with one decay per head and key channel (Kimi delta attention).  With h
+    the mixer's input,
+
+        q = Wq h, k = Wk h  (n_kv_heads x key_dim),  v = Wv h  (n_heads x value_dim)
+        each through a causal convolution over time of ``conv_taps`` taps per channel (no
+        bias, zeros before the sequence's start; the last tap is the current token's), then
+        silu;  q and k made unit vectors per head, x / sqrt(sum(x^2) + unit_eps), q also
+        times key_dim^(-1/2)
+        beta = sigmoid(Wb h)                                                     per head
+        g = exp(-exp(A_log) softplus(Wa2 (Wa1 h) + dt_bias))     per head and key channel
+        S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q       per head
+        y = Wo [ o / sqrt(mean(o^2) + norm_eps) * w * sigmoid(Wg2 (Wg1 h)) ]
+
+    Head i reads q and k of kv head i // (n_heads / n_kv_heads); the norm's weight w
+    [value_dim] is shared by the heads.  The inner sizes of the two thin products are those of
+    their tensors.  S [key_dim, value_dim] starts at zero and is kept, with the last
+    ``conv_taps - 1`` inputs of the convolutions, per sequence in 32-bit.  The projections of h
+    are one product that leaves 32-bit sums, Wa2 and Wg2 are one product with both inner
+    values side by side (its weight is zero where one's rows meet the other's columns); all else
+    up to y is 32-bit whatever the activation type.  ``names`` replaces local tensor names (keys
+    q, k, v, q_conv, k_conv, v_conv, b, A_log, a1, a2, dt_bias, g1, g2, norm, o)."""
+
+    NAMES = {"q": "q", "k": "k", "v": "v", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv",
+             "b": "b", "A_log": "A_log", "a1": "a1", "a2": "a2", "dt_bias": "dt_bias", "g1": "g1", "g2": "g2",
+             "norm": "norm", "o": "o"}
+
+    def __init__(self, ctx: BuildContext, hidden: int, n_heads: int, n_kv_heads: int, key_dim: int,
+                 value_dim: int, conv_taps: int, norm_eps: float, unit_eps: float = 1e-6, names=None):
+        super().__init__(ctx)
+        if n_heads % n_kv_heads:
+            raise ValueError(f"{n_heads} heads cannot share {n_kv_heads} kv heads")
+        if conv_taps < 1:
+            raise ValueError("a convolution has at least one tap")
+        self.hidden, self.H, self.G = int(hidden), int(n_heads), int(n_kv_heads)
+        self.dk, self.dv, self.taps = int(key_dim), int(value_dim), int(conv_taps)
+        self.norm_eps, self.unit_eps = float(norm_eps), float(unit_eps)
+        self.names = dict(self.NAMES, **(names or {}))
+        self.proj = self.thin = self.o = None
+        self.n_low = 0
+        self.conv_w = self.a_log = self.dt_bias = self.norm_w = None
+
+    def param_specs(self):
+        W, H, G, dk, dv, nm = self.hidden, self.H, self.G, self.dk, self.dv, self.names
+        thin1 = lambda n: ParamSpec((n, W), free=(0,))          # random weights take a head's size
+        thin2 = lambda rows, n: ParamSpec((rows, n), free=(1,))
+        return {nm["q"]: ParamSpec((G * dk, W)), nm["k"]: ParamSpec((G * dk, W)),
+                nm["v"]: ParamSpec((H * dv, W)), nm["b"]: ParamSpec((H, W)),
+                nm["q_conv"]: ParamSpec((G * dk, self.taps), "vector"),
+                nm["k_conv"]: ParamSpec((G * dk, self.taps), "vector"),
+                nm["v_conv"]: ParamSpec((H * dv, self.taps), "vector"),
+                nm["A_log"]: ParamSpec((H,), "offset"), nm["dt_bias"]: ParamSpec((H * dk,), "offset"),
+                nm["a1"]: thin1(dk), nm["a2"]: thin2(H * dk, dk), nm["g1"]: thin1(dv), nm["g2"]: thin2(H * dv, dv),
+                nm["norm"]: ParamSpec((dv,), "vector"), nm["o"]: ParamSpec((W, H * dv))}
+
+    def load(self, params):
+        nm = self.names
+        ws = [params[nm[k]] for k in ("q", "k", "v", "b", "a1", "g1")]
+        a2, g2 = params[nm["a2"]], params[nm["g2"]]
+        if len({w.dtype for w in ws + [a2, g2]}) != 1:
+            raise ValueError("the projections of one mixer must be stored in one dtype to be fused")
+        ra, rg = ws[4].shape[0], ws[5].shape[0]
+        if a2.shape[1] != ra or g2.shape[1] != rg:
+            raise ValueError(f"thin products of inner sizes {ra} and {rg} continue with {a2.shape[1]} and "
+                             f"{g2.shape[1]} columns")
+        # zero rows and columns fill both products up to what the tensor-core kernels take
+        self.n_low = (ra + rg + 7) // 8 * 8
+        if self.n_low > ra + rg:
+            ws.append(ws[5].new_zeros((self.n_low - ra - rg, self.hidden)))
+        self.proj = Linear(torch.cat(ws, dim=0), self.ctx.products)
+        thin = a2.new_zeros((a2.shape[0] + g2.shape[0], self.n_low))
+        thin[:a2.shape[0], :ra] = a2
+        thin[a2.shape[0]:, ra:ra + rg] = g2
+        self.thin = Linear(thin, self.ctx.products)
+        self.o = Linear(params[nm["o"]], self.ctx.products)
+        # what enters the recurrence is 32-bit whatever the checkpoint stores
+        f32 = lambda t: t.float().contiguous()
+        self.conv_w = f32(torch.cat([params[nm[k]] for k in ("q_conv", "k_conv", "v_conv")], dim=0))
+        self.a_log, self.dt_bias = f32(params[nm["A_log"]]), f32(params[nm["dt_bias"]])
+        self.norm_w = f32(params[nm["norm"]])
+
+    def kernel_modules(self):
+        return (("channel_delta",) + self.proj.kernel_modules() + self.thin.kernel_modules()
+                + self.o.kernel_modules())
+
+    def cache_spec(self):
+        return StateSpec((ops.delta_state_floats(self.H, self.G, self.dk, self.dv, self.taps),),
+                         torch.float32)
+
+    def captures_prompts(self):
+        return True
+
+    def forward(self, x, step, cache):
+        if cache is None or tuple(cache.spec.shape) != tuple(self.cache_spec().shape):
+            raise ValueError(f"the delta rule with a decay per channel was given the cache "
+                             f"{None if cache is None else cache.spec}")
+        sizes = dict(H=self.H, G=self.G, dk=self.dk, dv=self.dv, taps=self.taps, token_seq=step.token_seq,
+                     cu_q=step.cu_q, slots=step.slots, dtype=self.ctx.dtype)
+        proj = self.proj(x, out_dtype=torch.float32)
+        prep, low = ops.channel_delta_prepare(proj, cache.state, self.conv_w, n_low=self.n_low,
+                                              unit_eps=self.unit_eps, **sizes)
+        wide = self.thin(low, out_dtype=torch.float32)
+        y = ops.channel_delta_run(proj, prep, low, wide, cache.state, self.conv_w, self.a_log, self.dt_bias,
+                                  self.norm_w, norm_eps=self.norm_eps, max_rows=step.max_q_len, **sizes)
+        return self.o(y, partial_ok=True)
+
+
 @register_part("mixer", "retention")
 class Retention(Mixer):
     """Linear attention with a fixed decay per head and neither softmax nor

@@ -41,7 +41,7 @@ def check_names_and_shapes(expected: Dict[str, ParamSpec],
     missing = sorted(n for n, s in expected.items() if n not in found and not s.optional)
     unexpected = sorted(n for n in found if n not in expected)
     wrong = sorted((n, found[n], expected[n].shape) for n in expected
-                   if n in found and tuple(found[n]) != tuple(expected[n].shape))
+                   if n in found and not expected[n].takes(tuple(found[n])))
     if missing or unexpected or wrong:
         raise WeightError(missing, unexpected, wrong, where)
 

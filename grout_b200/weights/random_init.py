@@ -6,7 +6,8 @@
 to be worth writing.  Every matrix and embedding is N(0, 0.02^2), every
 vector (norm weights) 1 + N(0, 0.1^2) and every offset (biases, vectors that are
 added to something) N(0, 0.1^2); a fraction (a bound inside (0, 1)) is the sigmoid of
-N(0, 1), and the weights of an average are N(0, 0.1^2) with 1 added to the last.  Each tensor has its own generator,
+N(0, 1), the weights of an average are N(0, 0.1^2) with 1 added to the last, and a mixing
+matrix is the identity plus N(0, 0.1^2).  Each tensor has its own generator,
 seeded from (seed, tensor name), so a tensor's values do not depend on which
 other tensors are made or in which order.
 
@@ -51,6 +52,8 @@ def random_tensor(name: str, spec: ParamSpec, seed: int, dtype=torch.bfloat16,
     elif spec.kind == "average":
         x = VECTOR_STD * x
         x.reshape(-1)[-1] += 1.0
+    elif spec.kind == "mixing":
+        x = torch.eye(*spec.shape, device=device) + VECTOR_STD * x
     else:
         x = MATRIX_STD * x
     return x.to(dtype)
