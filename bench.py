@@ -21,7 +21,7 @@ weights, far more than the 126 MB L2, so nothing is flushed between timed steps.
                                        decode steps (launched one by one, an event pair
                                        around each): calls, time, GB/s, TFLOP/s, fractions
     python bench.py --requests S       the reference's request grid
-    python bench.py --designs [--design suvazen|sonalorn|zutazen|mananex|kakotar] [--design-sizes 1b,4b,8b] [--batch B] [--design-ops]
+    python bench.py --designs [--design suvazen|sonalorn|zutazen|mananex|kakotar|keralix] [--design-sizes 1b,4b,8b] [--batch B] [--design-ops]
                                        prefill and decode throughput of the Suvazen (or Sonalorn)
                                        design beside the Qwen3 decoder at equal layer sizes (random weights), and
                                        with --design-ops the per-kernel tables of both
@@ -276,6 +276,25 @@ def kakotar_config(size: str) -> dict:
     return dict(architecture="Kakotar", vocab=V, width=W, norm={"eps": 1e-6}, layers=layers)
 
 
+def keralix_config(size: str) -> dict:
+    """The Keralix model of a size: the width, heads, head size, layers, feed-forward rows and
+    vocabulary of the Qwen3 model, on four residual streams; the layers mix in turn by latent
+    attention (a latent of 128 for keys and values, which makes a cached row of the head size, and
+    one of 3/8 of the width for the queries, sinks, a gate), by the delta rule with a decay per
+    channel (as many heads, keys and values of the head size, four taps, thin products of a
+    head's inner size) and by attention behind convolutions of four taps over a window of 1,024
+    (the Qwen3 model's heads, every head rotated whole, capped scores, values that are the keys)."""
+    W, nq, nkv, D, I, L, V = DESIGN_SIZES[size]
+    lat = dict(heads=nq, dim=D, vdim=D, kv_rank=128, q_rank=3 * W // 8 // 64 * 64, scale=D ** -0.5)
+    delta = dict(heads=nq, kv_heads=nq, dim=D, vdim=D, conv=4)
+    attn = dict(heads=nq, kv_heads=nkv, dim=D, vdim=D, conv=4, scale=D ** -0.5, softcap=50.0,
+                mask={"size": 1024}, rot={"base": 1000000.0, "dims": D})
+    kinds = (("latent_attention", lat), ("channel_delta", delta), ("attention", attn))
+    layers = [dict(type=kinds[i % 3][0], mixer=kinds[i % 3][1], mlp={"kind": "dense", "ff": I}) for i in range(L)]
+    return dict(architecture="Keralix", vocab=V, width=W, streams=4, norm={"eps": 1e-6},
+                embedding={"scale": W ** 0.5}, layers=layers)
+
+
 def design_configs(size: str, design: str = "suvazen"):
     W, nq, nkv, D, I, L, V = DESIGN_SIZES[size]
     qwen = dict(QWEN3_4B, hidden_size=W, num_attention_heads=nq, num_key_value_heads=nkv, head_dim=D,
@@ -295,6 +314,9 @@ def design_configs(size: str, design: str = "suvazen"):
         return {"qwen3": qwen, "zutazen": zutazen_config(size), "mananex": mananex_config(size)}
     if design == "kakotar":       # the same two: attention, and matrix states, windows and experts
         return {"qwen3": qwen, "zutazen": zutazen_config(size), "kakotar": kakotar_config(size)}
+    if design == "keralix":       # beside attention, beside the other delta rule, beside the other latent attention
+        return {"qwen3": qwen, "sonalorn": sonalorn_config(size), "zutazen": zutazen_config(size),
+                "keralix": keralix_config(size)}
     return {"qwen3": qwen, "suvazen": suv}
 
 
@@ -600,7 +622,7 @@ def main() -> int:
     ap.add_argument("--designs", action="store_true",
                     help="instead of the default run: the Suvazen design beside the Qwen3 decoder at "
                          "equal layer sizes (--design-sizes), prefill and decode at --batch")
-    ap.add_argument("--design", default="suvazen", choices=["suvazen", "sonalorn", "zutazen", "mananex", "kakotar"],
+    ap.add_argument("--design", default="suvazen", choices=["suvazen", "sonalorn", "zutazen", "mananex", "kakotar", "keralix"],
                     help="which design --designs sets beside Qwen3")
     ap.add_argument("--design-sizes", default="1b,4b,8b",
                     help=f"which of {sorted(DESIGN_SIZES)} --designs runs")

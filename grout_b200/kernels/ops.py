@@ -2485,15 +2485,15 @@ def _cost_hyper(out, res_in, delta, **k):
 
 @_profiled("hyper_norm", _cost_hyper)
 def hyper_norm(res_in: torch.Tensor, delta: Optional[torch.Tensor], *, streams: int, dtype: torch.dtype,
-               mix: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
+               mix: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None,
                read: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
                norm_w: Optional[torch.Tensor] = None, eps: float = 0.0):
     """The boundary between two sublayers of a model with ``streams`` residual streams, in
-    32-bit: X'_t = sum_s mix[s, t] X_s + out[t] * delta; u = sum_t read[t] X'_t (the plain sum
+    32-bit: X'_t = sum_s mix[s, t] X_s + write[t] * delta; u = sum_t read[t] X'_t (the plain sum
     without ``read``); y = rmsnorm(u) * norm_w (u itself without ``norm_w``) in ``dtype``.
     ``res_in`` is [streams, T, N], or [T, N] when all streams are still equal; ``delta`` is
     [T, N] in ``dtype`` or a stack of 32-bit partial sums [P, T, N], added in order, and comes
-    with ``mix`` [streams, streams] (indexed from, to) and ``out`` [streams].  Returns (X', y):
+    with ``mix`` [streams, streams] (indexed from, to) and ``write`` [streams].  Returns (X', y):
     X' replaces ``res_in`` in place where that holds all streams; with ``rows`` the new streams
     are not kept and X' is ``res_in``."""
     _need(res_in, "streams", torch.float32)
@@ -2501,7 +2501,7 @@ def hyper_norm(res_in: torch.Tensor, delta: Optional[torch.Tensor], *, streams: 
     if not equal and (res_in.dim() != 3 or res_in.shape[0] != streams):
         raise KernelError(f"streams are {tuple(res_in.shape)}, expected [{streams}, T, N] or [T, N]")
     T, N = res_in.shape[-2:]
-    if (delta is None) != (mix is None) or (mix is None) != (out is None):
+    if (delta is None) != (mix is None) or (mix is None) != (write is None):
         raise KernelError("a sublayer's result comes with the weights that put it back")
     a = _HyperNormArgs()
     if delta is not None:
@@ -2513,7 +2513,7 @@ def hyper_norm(res_in: torch.Tensor, delta: Optional[torch.Tensor], *, streams: 
             a.delta = delta.data_ptr()
         if tuple(delta.shape[-2:]) != (T, N):
             raise KernelError(f"a result of {tuple(delta.shape)} for streams of {(T, N)}")
-    for t, nm, shape in ((mix, "mixing weights", (streams, streams)), (out, "write weights", (streams,)),
+    for t, nm, shape in ((mix, "mixing weights", (streams, streams)), (write, "write weights", (streams,)),
                          (read, "read weights", (streams,)), (norm_w, "norm weight", (N,))):
         if t is not None:
             _need(t, nm, torch.float32)
@@ -2529,7 +2529,7 @@ def hyper_norm(res_in: torch.Tensor, delta: Optional[torch.Tensor], *, streams: 
         a.res_out, a.out_stride = res.data_ptr(), res.stride(0)
     y = torch.empty((n_rows, N), dtype=dtype, device=res_in.device)
     a.res_in, a.in_stride = res_in.data_ptr(), 0 if equal else res_in.stride(0)
-    a.mix, a.out, a.read, a.rows, a.norm_w = _ptr(mix), _ptr(out), _ptr(read), _ptr(rows), _ptr(norm_w)
+    a.mix, a.out, a.read, a.rows, a.norm_w = _ptr(mix), _ptr(write), _ptr(read), _ptr(rows), _ptr(norm_w)
     a.eps, a.y, a.n_rows, a.N, a.S = float(eps), y.data_ptr(), n_rows, N, int(streams)
     _check(_fn("hyper_norm", f"gb_hyper_norm_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
            "hyper_norm")

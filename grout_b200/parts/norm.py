@@ -239,7 +239,7 @@ class RMSNorm(Norm):
 
     def _add_streams(self, res, pending, rows):
         return ops.hyper_norm(res, pending.delta, streams=pending.streams, dtype=self.ctx.dtype,
-                              mix=pending.mix, out=pending.out, read=pending.read, rows=rows,
+                              mix=pending.mix, write=pending.out, read=pending.read, rows=rows,
                               norm_w=self.weight32(), eps=self.eps)
 
     def add_norm(self, res, delta, rows=None):
