@@ -22,7 +22,9 @@
 //   scan     any other step of short sequences: the columns of S are independent recurrences; a
 //            column is held in the registers of eight lanes, 16 columns a block, and the rows are
 //            walked in order, their q, k and g staged in shared memory 16 at a time
-//   finish   after scan: one warp per (token, head) normalises and gates; the block of a sequence's
+//   local, chain   a step in which a sequence brings many rows goes chunk by chunk instead
+//            (channel_delta_chunk.cuh)
+//   finish   after these: one warp per (token, head) normalises and gates; the block of a sequence's
 //            first row keeps the new tail
 //
 // With s' = g s the two sums over dk that a row needs, s' . k and s' . q, are taken together:
@@ -33,6 +35,7 @@
 // floats: the convolutions' tail [taps - 1, Cc] (Cc = the convolved channels q | k | v), then S as
 // [H, dv, dk], a column's dk elements side by side.  Rows of slot < 0 (padding) start from zeros
 // and store nothing.
+#include "attn_mma.cuh"   // the asynchronous-copy helpers
 #include "short_conv.cuh"
 
 struct ChannelDeltaArgs {
@@ -55,6 +58,7 @@ struct ChannelDeltaArgs {
   float unit_eps, norm_eps;
   int prep_stride;         // floats between rows of prep: round4(Cc + H + G)
   int max_rows;            // the most rows any sequence brings (0: unknown)
+  float* chunks;           // [n_tokens / 32 + n_seqs, H, record] scratch of a step that goes chunk by chunk, or null
 };
 
 __device__ __forceinline__ int cd_channels(const ChannelDeltaArgs& a) { return 2 * a.G * a.dk + a.H * a.dv; }
@@ -312,6 +316,8 @@ __global__ void channel_delta_finish_kernel(const ChannelDeltaArgs a) {
   pdl_launch_dependents_if_large();
 }
 
+#include "channel_delta_chunk.cuh"
+
 static int cd_check(const ChannelDeltaArgs& a) {
   if (a.n_tokens < 0 || a.n_seqs <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dv <= 0 || a.taps <= 0 ||
       a.n_low <= 0 || !a.proj || !a.state || !a.prep || !a.low || !a.conv_w || !a.token_seq || !a.cu_q || !a.slots)
@@ -338,16 +344,21 @@ static int run_rows(const ChannelDeltaArgs& a, cudaStream_t s) {
     if (smem > 48 * 1024) return GB_ERR_UNSUPPORTED;
     return gb_launch(channel_delta_step_kernel<T, R>, dim3(a.H, a.n_seqs), dim3(256), smem, s, a);
   }
-  const size_t smem = (CD_TT * (3 * DKP + CD_COLS + 2)) * sizeof(float);
-  static bool configured = false;
-  if (smem > 48 * 1024 && !configured) {
-    cudaError_t e = cudaFuncSetAttribute(channel_delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)smem);
-    if (e != cudaSuccess) return (int)e;
-    configured = true;
+  int e;
+  if (cc_takes(a)) {
+    e = cc_run(a, s);
+  } else {
+    const size_t smem = (CD_TT * (3 * DKP + CD_COLS + 2)) * sizeof(float);
+    static bool configured = false;
+    if (smem > 48 * 1024 && !configured) {
+      cudaError_t ce = cudaFuncSetAttribute(channel_delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                            (int)smem);
+      if (ce != cudaSuccess) return (int)ce;
+      configured = true;
+    }
+    e = gb_launch(channel_delta_scan_kernel<R>, dim3((a.dv + CD_COLS - 1) / CD_COLS, a.H, a.n_seqs),
+                  dim3(CD_LANES * CD_COLS), smem, s, a);
   }
-  const int e = gb_launch(channel_delta_scan_kernel<R>, dim3((a.dv + CD_COLS - 1) / CD_COLS, a.H, a.n_seqs),
-                          dim3(CD_LANES * CD_COLS), smem, s, a);
   if (e) return e;
   const int warps = a.H < 8 ? a.H : 8;
   int rows_y = (a.H + warps - 1) / warps;            // blocks of a row: enough for its heads, and

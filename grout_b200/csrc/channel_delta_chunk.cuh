@@ -1,0 +1,381 @@
+// The delta rule with a decay per channel, chunk by chunk (included by channel_delta.cu; the
+// notation is that file's).  With L_t the sums of log g from a chunk's first row to row t
+// (per channel) and S_0 the state in front of the chunk, the rows of a chunk obey
+//
+//   u_t = beta_t (v_t - S_0^T (e^{L_t} k_t) - sum_{i<t} A_ti u_i),   A_ti = sum_d k_td k_id e^{L_td - L_id}
+//   o_t = S_0^T (e^{L_t} q_t) + sum_{i<=t} B_ti u_i,                 B_ti = sum_d q_td k_id e^{L_td - L_id}
+//   S_n = diag(e^{L_n}) S_0 + sum_i (e^{L_n - L_i} k_i) u_i^T
+//
+// The first line is a triangular system: u = X v - (W) S_0 with both X v and W from one forward
+// substitution that knows nothing of S_0.  So
+//
+//   local   takes every chunk of every head at the same time: A, B, the substitution for the dv + dk
+//           right-hand sides beta v and beta e^{L} k, and leaves the chunk's record
+//   chain   walks a sequence's chunks in order, a block per head and CC_COLS columns of S with the
+//           state in shared memory: U = U0 - W S, the read-outs, the next state: tiled 32-bit products
+//
+// Every exponent that is taken is a difference that is not positive (rows of the same half chunk
+// directly, others by way of the end of the first half), so no quotient of decays overflows however
+// strong they are.
+#pragma once
+
+#define CC_ROWS 32       // rows of a chunk
+#define CC_HALF 16
+#define CC_COLS 32       // columns of S a chain block owns
+#define CC_MIN 64        // a step goes chunk by chunk when a sequence brings this many rows
+#define CC_MAX_DK 128
+
+// A chunk's record for one head: WQ [dk][64] (per channel the 32 rows of W, then the 32 of
+// e^L q) | Kd [32][dk] (e^{L_n - L} k) | gC [dk] (e^{L_n}) | B [32][32] | U0 [32][dv]
+__host__ __device__ __forceinline__ size_t cc_record(int dk, int dv) {
+  return (size_t)dk * 64 + CC_ROWS * dk + dk + CC_ROWS * CC_ROWS + CC_ROWS * dv;
+}
+// Chunk z of a sequence whose rows start at `first` has an entry that no other chunk has.
+__host__ __device__ __forceinline__ size_t cc_entry(int first, int z, int seq) {
+  return (size_t)(first / CC_ROWS + z + seq);
+}
+
+// Sums over the warp's lanes of 32 values a lane holds: lane i gets the sum of value i.
+__device__ __forceinline__ float cc_transpose_sum(float (&v)[32], int lane) {
+#pragma unroll
+  for (int m = 16; m > 0; m >>= 1) {
+    const bool up = lane & m;
+#pragma unroll
+    for (int i = 0; i < m; ++i) {
+      const float give = up ? v[i] : v[i + m], keep = up ? v[i + m] : v[i];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, m);
+    }
+  }
+  return v[0];
+}
+
+template <int E> struct CcVec { float e[E]; };
+template <int E>
+__device__ __forceinline__ void cc_read(const float* p, float (&o)[E]) {
+  if constexpr (E == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    o[0] = x.x, o[1] = x.y, o[2] = x.z, o[3] = x.w;
+  } else if constexpr (E == 2) {
+    const float2 x = *reinterpret_cast<const float2*>(p);
+    o[0] = x.x, o[1] = x.y;
+  } else {
+    o[0] = p[0];
+  }
+}
+
+// E channels a lane: heads of up to 32 E.  The block's rows, zero beyond dk and beyond the chunk's end.
+template <int E>
+__global__ void __launch_bounds__(256) channel_delta_local_kernel(const ChannelDeltaArgs a) {
+  constexpr int DKP = 32 * E, LD = DKP + 4;      // (16-byte rows; a column's rows on different banks)
+  extern __shared__ __align__(16) float sm[];
+  float *Ks = sm, *Qs = Ks + CC_ROWS * LD, *Ls = Qs + CC_ROWS * LD, *Kr = Ls + CC_ROWS * LD;   // Kr [16][LD]
+  float *As = Kr + CC_HALF * LD, *Bs = As + CC_ROWS * CC_ROWS, *beta = Bs + CC_ROWS * CC_ROWS;
+  pdl_launch_dependents_if_small();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, seq = blockIdx.z, z = blockIdx.x;
+  const int H = a.H, G = a.G, dk = a.dk, dv = a.dv, kvh = h / (H / G), Cc = cd_channels(a);
+  const float rate = expf(a.a_log[h]);
+  pdl_wait();
+  const int first = a.cu_q[seq], n_seq = a.cu_q[seq + 1] - first;
+  const int n = min(CC_ROWS, n_seq - z * CC_ROWS), row0 = first + z * CC_ROWS;
+  if (n <= 0) return;
+  for (int i = tid; i < CC_ROWS * DKP; i += 256) {
+    const int t = i / DKP, d = i % DKP;
+    float q = 0.f, k = 0.f, lg = 0.f;
+    if (t < n && d < dk) {
+      const float* p = a.prep + (size_t)(row0 + t) * a.prep_stride;
+      q = p[kvh * dk + d], k = p[(G + kvh) * dk + d];
+      lg = cd_log_decay(a.wide[(size_t)(row0 + t) * H * (dk + dv) + h * dk + d], a.dt_bias[h * dk + d], rate);
+    }
+    Qs[t * LD + d] = q, Ks[t * LD + d] = k, Ls[t * LD + d] = lg;
+  }
+  if (tid < CC_ROWS) beta[tid] = tid < n ? a.prep[(size_t)(row0 + tid) * a.prep_stride + Cc + h] : 0.f;
+  __syncthreads();
+  if (tid < DKP) {                               // running sums of the logarithms
+    float s = 0.f;
+    for (int t = 0; t < CC_ROWS; ++t) s += Ls[t * LD + tid], Ls[t * LD + tid] = s;
+    const float mid = Ls[(CC_HALF - 1) * LD + tid];
+    for (int t = 0; t < CC_HALF; ++t) Kr[t * LD + tid] = Ks[t * LD + tid] * expf(mid - Ls[t * LD + tid]);
+  }
+  __syncthreads();
+  // A and B: a warp takes rows warp, warp + 8, ...; its lanes share the channels
+  for (int t = warp; t < CC_ROWS; t += 8) {
+    float kt[E], qt[E], lt[E], ki[E], li[E], part[32];
+    cc_read<E>(Ks + t * LD + lane * E, kt);
+    cc_read<E>(Qs + t * LD + lane * E, qt);
+    cc_read<E>(Ls + t * LD + lane * E, lt);
+    const int base = t & CC_HALF;                // the first row of t's half chunk
+#pragma unroll
+    for (int j = 0; j < CC_HALF; ++j) {
+      part[j] = part[CC_HALF + j] = 0.f;
+      if (base + j <= t) {
+        cc_read<E>(Ks + (base + j) * LD + lane * E, ki);
+        cc_read<E>(Ls + (base + j) * LD + lane * E, li);
+#pragma unroll
+        for (int x = 0; x < E; ++x) {
+          const float w = ki[x] * expf(lt[x] - li[x]);
+          part[j] = fmaf(kt[x], w, part[j]);
+          part[CC_HALF + j] = fmaf(qt[x], w, part[CC_HALF + j]);
+        }
+      }
+    }
+    float sum = cc_transpose_sum(part, lane);    // lanes 0 .. 15: A, 16 .. 31: B
+    const int j = lane & (CC_HALF - 1);
+    if (lane < CC_HALF) As[t * CC_ROWS + base + j] = base + j < t ? sum : 0.f;
+    else Bs[t * CC_ROWS + base + j] = base + j <= t ? sum : 0.f;
+    if (base) {                                  // the other half, by way of its last row
+      float mid[E];
+      cc_read<E>(Ls + (CC_HALF - 1) * LD + lane * E, mid);
+#pragma unroll
+      for (int x = 0; x < E; ++x) {
+        const float w = expf(lt[x] - mid[x]);
+        kt[x] *= w, qt[x] *= w;
+      }
+#pragma unroll
+      for (int i = 0; i < CC_HALF; ++i) {
+        part[i] = part[CC_HALF + i] = 0.f;
+        cc_read<E>(Kr + i * LD + lane * E, ki);
+#pragma unroll
+        for (int x = 0; x < E; ++x) {
+          part[i] = fmaf(kt[x], ki[x], part[i]);
+          part[CC_HALF + i] = fmaf(qt[x], ki[x], part[CC_HALF + i]);
+        }
+      }
+      sum = cc_transpose_sum(part, lane);
+      (lane < CC_HALF ? As : Bs)[t * CC_ROWS + j] = sum;
+    } else {
+      (lane < CC_HALF ? As : Bs)[t * CC_ROWS + CC_HALF + j] = 0.f;
+    }
+  }
+  __syncthreads();
+  // the substitution: a thread takes one right-hand side (dv of values, then dk of e^{L} k)
+  const size_t entry = (cc_entry(first, z, seq) * H + h) * cc_record(dk, dv);
+  float* wq = a.chunks + entry;
+  float* kd = wq + (size_t)dk * 64;
+  float* gc = kd + (size_t)CC_ROWS * dk;
+  float* bm = gc + dk;
+  float* u0 = bm + CC_ROWS * CC_ROWS;
+  for (int c = tid; c < dv + dk; c += 256) {
+    float x[CC_ROWS];
+    const int d = c - dv;
+#pragma unroll
+    for (int t = 0; t < CC_ROWS; ++t) {
+      if (d < 0) x[t] = t < n ? a.prep[(size_t)(row0 + t) * a.prep_stride + 2 * G * dk + h * dv + c] : 0.f;
+      else x[t] = Ks[t * LD + d] * expf(Ls[t * LD + d]);
+    }
+#pragma unroll
+    for (int t = 0; t < CC_ROWS; ++t) {
+      float s = x[t];
+#pragma unroll
+      for (int i0 = 0; i0 < t; i0 += 4) {        // (entries of A from the diagonal on are zero, x there still finite)
+        const float4 w = *reinterpret_cast<const float4*>(As + t * CC_ROWS + i0);
+        s = fmaf(-w.x, x[i0], s);
+        if (i0 + 1 < t) s = fmaf(-w.y, x[i0 + 1], s);
+        if (i0 + 2 < t) s = fmaf(-w.z, x[i0 + 2], s);
+        if (i0 + 3 < t) s = fmaf(-w.w, x[i0 + 3], s);
+      }
+      x[t] = beta[t] * s;
+    }
+    if (d < 0) {
+#pragma unroll
+      for (int t = 0; t < CC_ROWS; ++t) u0[(size_t)t * dv + c] = x[t];
+    } else {
+      float4* out = reinterpret_cast<float4*>(wq + (size_t)d * 64);
+#pragma unroll
+      for (int t = 0; t < CC_ROWS; t += 4) out[t / 4] = make_float4(x[t], x[t + 1], x[t + 2], x[t + 3]);
+    }
+  }
+  pdl_launch_dependents_if_large();
+  for (int i = tid; i < 8 * dk; i += 256) {      // e^{L} q, four rows of a channel a thread
+    const int d = i / 8, t = (i % 8) * 4;
+    float v[4];
+#pragma unroll
+    for (int x = 0; x < 4; ++x) v[x] = Qs[(t + x) * LD + d] * expf(Ls[(t + x) * LD + d]);
+    *reinterpret_cast<float4*>(wq + (size_t)d * 64 + CC_ROWS + t) = make_float4(v[0], v[1], v[2], v[3]);
+  }
+  // (rows beyond the chunk's end have no decay of their own: the last row's sums are the chunk's)
+  for (int i = tid; i < CC_ROWS * dk; i += 256) {
+    const int t = i / dk, d = i % dk;
+    kd[i] = Ks[t * LD + d] * expf(Ls[(CC_ROWS - 1) * LD + d] - Ls[t * LD + d]);
+  }
+  for (int d = tid; d < dk; d += 256) gc[d] = expf(Ls[(CC_ROWS - 1) * LD + d]);
+  for (int i = tid; i < CC_ROWS * CC_ROWS; i += 256) bm[i] = Bs[i];
+}
+
+__device__ __forceinline__ void cc_copy16(float* smem, const float* gmem) {
+  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem));
+}
+
+// floats of a stage: WQ | Kd | gC | B | U0's columns
+__host__ __device__ __forceinline__ int cc_stage(int dk) {
+  return dk * 64 + CC_ROWS * dk + dk + CC_ROWS * CC_ROWS + CC_ROWS * CC_COLS;
+}
+
+__global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelDeltaArgs a) {
+  extern __shared__ __align__(16) float sm[];
+  pdl_launch_dependents_if_small();
+  const int tid = threadIdx.x;
+  const int h = blockIdx.y, seq = blockIdx.z, col0 = blockIdx.x * CC_COLS;
+  const int H = a.H, dk = a.dk, dv = a.dv, Cc = cd_channels(a);
+  const int stage = cc_stage(dk);
+  float* S = sm + 2 * stage;                     // [dk][CC_COLS]
+  float* P = S + dk * CC_COLS;                   // [64][CC_COLS]: one half's part of WQ^T S, then e^{L} q S
+  float* U = P + 64 * CC_COLS;                   // [CC_ROWS][CC_COLS]
+  pdl_wait();
+  const int first = a.cu_q[seq], n_seq = a.cu_q[seq + 1] - first;
+  if (n_seq <= 0) return;
+  const int slot = a.slots[seq];
+  float* sp = slot >= 0 ? a.state + (size_t)slot * a.state_stride + (size_t)(a.taps - 1) * Cc + (size_t)h * dv * dk
+                        : nullptr;
+  const int chunks = (n_seq + CC_ROWS - 1) / CC_ROWS;
+  auto stage_in = [&](int z) {
+    float* dst = sm + (z & 1) * stage;
+    const float* src = a.chunks + (cc_entry(first, z, seq) * H + h) * cc_record(dk, dv);
+    const int whole = dk * 64 + CC_ROWS * dk + dk + CC_ROWS * CC_ROWS;      // (dk is a multiple of four)
+    for (int i = tid * 4; i < whole; i += 1024) cc_copy16(dst + i, src + i);
+    const int t = tid / 8, c = (tid % 8) * 4;
+    if (col0 + c < dv) cc_copy16(dst + whole + t * CC_COLS + c, src + whole + (size_t)t * dv + col0 + c);
+    cp_async_commit();
+  };
+  for (int s = 0; s < 2 && col0 + CC_COLS > dv; ++s)       // columns no copy brings
+    for (int i = tid; i < CC_ROWS * CC_COLS; i += 256)
+      if (col0 + i % CC_COLS >= dv) sm[s * stage + stage - CC_ROWS * CC_COLS + i] = 0.f;
+  stage_in(0);
+  // the state: element (k, c) of the head's matrix lies at c dk + k
+  for (int i = tid; i < dk * CC_COLS; i += 256) {
+    const int c = i / dk, k = i % dk;
+    S[k * CC_COLS + c] = sp && col0 + c < dv ? sp[(size_t)(col0 + c) * dk + k] : 0.f;
+  }
+  // the products' tiles: 4 rows by 4 columns of WQ^T S a thread, half the channels each; 4 by 4 of
+  // the state; 2 by 2 of the read-outs
+  const int half = tid >> 7, tr = (tid & 127) / 8 * 4, tc = (tid & 7) * 4;
+  const int k_lo = half ? dk / 2 : 0, k_hi = half ? dk : dk / 2;
+  const int sk = tid / 8 * 4, orow = tid / 16 * 2, ocol = (tid % 16) * 2;
+  for (int z = 0; z < chunks; ++z) {
+    if (z + 1 < chunks) { stage_in(z + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+    __syncthreads();
+    const float* wq = sm + (z & 1) * stage;
+    const float* kd = wq + dk * 64;
+    const float* gc = kd + CC_ROWS * dk;
+    const float* bm = gc + dk;
+    const float* u0 = bm + CC_ROWS * CC_ROWS;
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+#pragma unroll 4
+    for (int k = k_lo; k < k_hi; ++k) {
+      const float4 x = *reinterpret_cast<const float4*>(wq + k * 64 + tr);
+      const float4 y = *reinterpret_cast<const float4*>(S + k * CC_COLS + tc);
+      const float xv[4] = {x.x, x.y, x.z, x.w}, yv[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xv[i], yv[j], acc[i][j]);
+    }
+    if (half) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<float4*>(P + (tr + i) * CC_COLS + tc) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+    }
+    __syncthreads();
+    if (!half) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        float4* at = reinterpret_cast<float4*>(P + (tr + i) * CC_COLS + tc);
+        const float4 p = *at;
+        float4 s = make_float4(acc[i][0] + p.x, acc[i][1] + p.y, acc[i][2] + p.z, acc[i][3] + p.w);
+        if (tr < CC_ROWS) {                      // a row of W: U = U0 - W S
+          const float4 u = *reinterpret_cast<const float4*>(u0 + (tr + i) * CC_COLS + tc);
+          s = make_float4(u.x - s.x, u.y - s.y, u.z - s.z, u.w - s.w);
+          *reinterpret_cast<float4*>(U + (tr + i) * CC_COLS + tc) = s;
+        } else {
+          *at = s;
+        }
+      }
+    }
+    __syncthreads();
+    if (sk < dk) {                               // S <- diag(e^{L_n}) S + Kd^T U
+      float s[4][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float4 x = *reinterpret_cast<const float4*>(S + (sk + i) * CC_COLS + tc);
+        const float g = gc[sk + i];
+        s[i][0] = g * x.x, s[i][1] = g * x.y, s[i][2] = g * x.z, s[i][3] = g * x.w;
+      }
+#pragma unroll 4
+      for (int t = 0; t < CC_ROWS; ++t) {
+        const float4 x = *reinterpret_cast<const float4*>(kd + t * dk + sk);
+        const float4 y = *reinterpret_cast<const float4*>(U + t * CC_COLS + tc);
+        const float xv[4] = {x.x, x.y, x.z, x.w}, yv[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) s[i][j] = fmaf(xv[i], yv[j], s[i][j]);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<float4*>(S + (sk + i) * CC_COLS + tc) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
+    }
+    float o[2][2];                               // the read-outs: e^{L} q S_0 + B U
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int j = 0; j < 2; ++j) o[i][j] = P[(CC_ROWS + orow + i) * CC_COLS + ocol + j];
+    for (int t = 0; t <= orow + 1; ++t) {        // (B is zero behind its diagonal)
+      const float2 u = *reinterpret_cast<const float2*>(U + t * CC_COLS + ocol);
+      const float b0 = bm[orow * CC_ROWS + t], b1 = bm[(orow + 1) * CC_ROWS + t];
+      o[0][0] = fmaf(b0, u.x, o[0][0]), o[0][1] = fmaf(b0, u.y, o[0][1]);
+      o[1][0] = fmaf(b1, u.x, o[1][0]), o[1][1] = fmaf(b1, u.y, o[1][1]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int r = z * CC_ROWS + orow + i;
+      if (r < n_seq && col0 + ocol < dv)         // (dv is a multiple of four)
+        *reinterpret_cast<float2*>(a.o + ((size_t)(first + r) * H + h) * dv + col0 + ocol) = make_float2(o[i][0], o[i][1]);
+    }
+    __syncthreads();                             // S is whole, the stage and P may be overwritten
+  }
+  pdl_launch_dependents_if_large();
+  if (sp)
+    for (int i = tid; i < dk * CC_COLS; i += 256) {
+      const int c = i / dk, k = i % dk;
+      if (col0 + c < dv) sp[(size_t)(col0 + c) * dk + k] = S[k * CC_COLS + c];
+    }
+}
+
+static bool cc_takes(const ChannelDeltaArgs& a) {
+  return a.chunks && a.max_rows >= CC_MIN && a.dk <= CC_MAX_DK && a.dk % 4 == 0 && a.dv % 4 == 0 &&
+         (((uintptr_t)a.chunks | (uintptr_t)a.o) & 15) == 0;
+}
+
+template <int E>
+static int cc_local(const ChannelDeltaArgs& a, int chunks, cudaStream_t s) {
+  constexpr int LD = 32 * E + 4;
+  const size_t smem = ((3 * CC_ROWS + CC_HALF) * LD + 2 * CC_ROWS * CC_ROWS + CC_ROWS) * sizeof(float);
+  static bool configured = false;
+  if (smem > 48 * 1024 && !configured) {
+    cudaError_t e = cudaFuncSetAttribute(channel_delta_local_kernel<E>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  return gb_launch(channel_delta_local_kernel<E>, dim3(chunks, a.H, a.n_seqs), dim3(256), smem, s, a);
+}
+
+static int cc_run(const ChannelDeltaArgs& a, cudaStream_t s) {
+  const int chunks = (a.max_rows + CC_ROWS - 1) / CC_ROWS;
+  const int e = a.dk <= 32 ? cc_local<1>(a, chunks, s) : a.dk <= 64 ? cc_local<2>(a, chunks, s) : cc_local<4>(a, chunks, s);
+  if (e) return e;
+  const size_t smem = (2 * cc_stage(a.dk) + a.dk * CC_COLS + 64 * CC_COLS + CC_ROWS * CC_COLS) * sizeof(float);
+  static size_t configured = 48 * 1024;
+  if (smem > configured) {
+    cudaError_t ce = cudaFuncSetAttribute(channel_delta_chain_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                          (int)smem);
+    if (ce != cudaSuccess) return (int)ce;
+    configured = smem;
+  }
+  return gb_launch(channel_delta_chain_kernel, dim3((a.dv + CC_COLS - 1) / CC_COLS, a.H, a.n_seqs), dim3(256), smem, s, a);
+}

@@ -1753,7 +1753,11 @@ class _ChannelDeltaArgs(ctypes.Structure):
                 ("cu_q", _P), ("slots", _P), ("state", _P), ("state_stride", _L), ("prep", _P), ("low", _P),
                 ("wide", _P), ("o", _P), ("y", _P), ("n_tokens", _I), ("n_seqs", _I), ("H", _I), ("G", _I),
                 ("dk", _I), ("dv", _I), ("taps", _I), ("n_low", _I), ("unit_eps", _F), ("norm_eps", _F),
-                ("prep_stride", _I), ("max_rows", _I)]
+                ("prep_stride", _I), ("max_rows", _I), ("chunks", _P)]
+
+
+CHANNEL_DELTA_CHUNK = 32          # rows of a chunk of the kernels' chunked form (CC_ROWS)
+CHANNEL_DELTA_CHUNK_MIN = 64      # a sequence of this many rows in a step: the step goes chunk by chunk (CC_MIN)
 
 
 def _channel_delta_args(proj, state, conv_w, *, H, G, dk, dv, taps, n_low, token_seq, cu_q, slots):
@@ -1820,7 +1824,8 @@ def channel_delta_run(proj: torch.Tensor, prep: torch.Tensor, low: torch.Tensor,
     [slots + 1, delta_state_floats] 32-bit is updated in place for slots that are not negative (the
     convolutions' tail with it).  Returns y [T, H dv] in ``dtype``: o normalised over dv, times
     ``norm_w`` and sigmoid(gate).  ``max_rows``: the most rows any sequence brings, when the host
-    knows it; with 1 (a decode step) all of it is one kernel."""
+    knows it; with 1 (a decode step) all of it is one kernel, from ``CHANNEL_DELTA_CHUNK_MIN`` on the step
+    goes chunk by chunk (the same sums in another order)."""
     n_low = low.shape[1]
     a = _channel_delta_args(proj, state, conv_w, H=H, G=G, dk=dk, dv=dv, taps=taps, n_low=n_low,
                             token_seq=token_seq, cu_q=cu_q, slots=slots)
@@ -1838,9 +1843,15 @@ def channel_delta_run(proj: torch.Tensor, prep: torch.Tensor, low: torch.Tensor,
     y = torch.empty((T, H * dv), dtype=dtype, device=proj.device)
     a.a_log, a.dt_bias, a.norm_w = a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr()
     a.prep, a.low, a.wide, a.o, a.y = (prep.data_ptr(), low.data_ptr(), wide.data_ptr(), o.data_ptr(), y.data_ptr())
-    a.norm_eps, a.max_rows = float(norm_eps), int(max_rows or 0)
+    a.norm_eps, a.max_rows = float(norm_eps), int(max_rows or T)
+    chunked = a.max_rows >= CHANNEL_DELTA_CHUNK_MIN and dk <= 128 and dk % 4 == 0 and dv % 4 == 0
+    if chunked:
+        C = CHANNEL_DELTA_CHUNK
+        record = dk * 2 * C + C * dk + dk + C * C + C * dv
+        chunks = torch.empty(((T // C + slots.shape[0]) * H, record), dtype=torch.float32, device=proj.device)
+        a.chunks = chunks.data_ptr()
     _check(_fn("channel_delta", f"gb_channel_delta_run_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
-           "channel_delta", 1 if a.max_rows == 1 else 2)
+           "channel_delta", 1 if a.max_rows == 1 else (3 if chunked else 2))
     return y
 
 

@@ -155,9 +155,9 @@ def delta_head(q, k, v, beta, g, S=None):
     out = []
     for i in range(k.shape[0]):
         S = g[i].to(DT)[:, None] * S
-        u = beta[i] * (v[i] - S.T @ k[i])
+        u = beta[i] * (v[i].to(DT) - S.T @ k[i].to(DT))
         S = S + torch.outer(k[i].to(DT), u)
-        out.append(S.T @ q[i])
+        out.append(S.T @ q[i].to(DT))
     return torch.stack(out), S
 
 
