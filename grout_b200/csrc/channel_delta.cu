@@ -13,19 +13,19 @@
 // product arrive as 32-bit sums, and only y, the o projection's input, is rounded (and the thin
 // products' inner values, where activations are 16-bit).
 //
-//   prepare  one block per token and kv head (its q, its k and their product) or run of value
-//            channels: convolution, silu, unit vectors, beta; the thin products' inner values go
-//            to a tensor of their own, the second thin product's input
+//   prepare  a block per run of rows, a warp of it a kv head (its q, its k and their product) or a
+//            run of value channels, the convolutions' inputs passing through registers: convolution,
+//            silu, unit vectors, beta, the new tail; the thin products' inner values go to a tensor
+//            of their own, the second thin product's input
 //   step     a step in which every sequence brings one row: a block per (sequence, head) streams the
 //            head's state through registers once (a column's dk elements in eight lanes), and then
-//            normalises and gates the head's read-out; the heads' blocks share the new tail
+//            normalises and gates the head's read-out
 //   scan     any other step of short sequences: the columns of S are independent recurrences; a
 //            column is held in the registers of eight lanes, 16 columns a block, and the rows are
 //            walked in order, their q, k and g staged in shared memory 16 at a time
 //   local, chain   a step in which a sequence brings many rows goes chunk by chunk instead
 //            (channel_delta_chunk.cuh)
-//   finish   after these: one warp per (token, head) normalises and gates; the block of a sequence's
-//            first row keeps the new tail
+//   finish   after these: one warp per (token, head) normalises and gates
 //
 // With s' = g s the two sums over dk that a row needs, s' . k and s' . q, are taken together:
 // u = beta (v - s' . k) and o = s' . q + u (k . q), so a row costs one round of shuffles.
@@ -67,52 +67,150 @@ __device__ __forceinline__ float cd_sigmoid(float z) { return 1.0f / (1.0f + exp
 // the logarithm of a channel's decay; `rate` = exp(A_log) of its head
 __device__ __forceinline__ float cd_log_decay(float z, float bias, float rate) { return -rate * softplus_f(z + bias); }
 
-#define CD_PREP_V 256
+#define CD_RUN 8         // rows of a run (never fewer than taps - 1)
+#define CD_WARPS 8
 
-template <typename T>
-__global__ void __launch_bounds__(256) channel_delta_prepare_kernel(const ChannelDeltaArgs a) {
-  extern __shared__ float row[];   // [2 dk]: a kv head's q and k after the convolution
-  __shared__ float scratch[32];
+// E channels of a lane: c0 + lane + 32 x (those below `cols` exist).
+template <int E>
+__device__ __forceinline__ void cd_inputs(const ChannelDeltaArgs& a, const float* tail, int Cc, int C_all, int row0,
+                                          int rr, int c0, int lane, int cols, float (&o)[E]) {
+#pragma unroll
+  for (int x = 0; x < E; ++x) {
+    const int d = lane + 32 * x;
+    o[x] = 0.f;
+    if (d < cols) {
+      if (rr >= 0) o[x] = a.proj[(size_t)(row0 + rr) * C_all + c0 + d];
+      else if (tail && rr + a.taps - 1 >= 0) o[x] = tail[(size_t)(a.taps - 1 + rr) * Cc + c0 + d];
+    }
+  }
+}
+
+// The convolutions of E channels a lane over the rows of a run: holds the inputs of the last TAPS rows
+// (TAPS 0: any number of taps, whose inputs are read again for every row).
+template <int E, int TAPS>
+struct CdWalk {
+  static constexpr int W = TAPS > 0 ? TAPS : 1;
+  float w[W][E], x[W][E];
+  int c0, cols;
+  __device__ __forceinline__ void start(const ChannelDeltaArgs& a, const float* tail, int Cc, int C_all, int row0, int r0,
+                                        int first, int count, int lane) {
+    c0 = first, cols = count;
+    if (TAPS == 0) return;
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const int d = lane + 32 * e;
+        w[j][e] = d < cols ? a.conv_w[(size_t)(c0 + d) * a.taps + a.taps - 1 - j] : 0.f;
+      }
+      if (j > 0) cd_inputs<E>(a, tail, Cc, C_all, row0, r0 - j, c0, lane, cols, x[j - 1]);
+    }
+  }
+  __device__ __forceinline__ void row(const ChannelDeltaArgs& a, const float* tail, int Cc, int C_all, int row0, int rr,
+                                      int lane, float (&y)[E]) {
+    if (TAPS == 0) {
+#pragma unroll
+      for (int e = 0; e < E; ++e) y[e] = 0.f;
+      for (int j = 0; j < a.taps; ++j) {
+        cd_inputs<E>(a, tail, Cc, C_all, row0, rr - j, c0, lane, cols, x[0]);
+#pragma unroll
+        for (int e = 0; e < E; ++e)
+          if (lane + 32 * e < cols)
+            y[e] = fmaf(a.conv_w[(size_t)(c0 + lane + 32 * e) * a.taps + a.taps - 1 - j], x[0][e], y[e]);
+      }
+    } else {
+#pragma unroll
+      for (int j = W - 1; j > 0; --j)
+#pragma unroll
+        for (int e = 0; e < E; ++e) x[j][e] = x[j - 1][e];
+      cd_inputs<E>(a, tail, Cc, C_all, row0, rr, c0, lane, cols, x[0]);
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        y[e] = 0.f;
+#pragma unroll
+        for (int j = 0; j < W; ++j) y[e] = fmaf(w[j][e], x[j][e], y[e]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < E; ++e) y[e] = silu_f(y[e]);
+  }
+  // the sequence's new tail (after the rows; the owner of the channels in the first run only): entry s
+  // becomes the input at n - (taps - 1) + s rows, read before it or anything above it is written
+  __device__ __forceinline__ void keep(const ChannelDeltaArgs& a, float* tail, int Cc, int C_all, int row0, int n,
+                                       int lane) {
+    for (int s = 0; s < a.taps - 1; ++s) {
+      float v[E];
+      cd_inputs<E>(a, tail, Cc, C_all, row0, n - (a.taps - 1) + s, c0, lane, cols, v);
+#pragma unroll
+      for (int e = 0; e < E; ++e)
+        if (lane + 32 * e < cols) tail[(size_t)s * Cc + c0 + lane + 32 * e] = v[e];
+    }
+  }
+};
+
+// A block takes a run of rows, a warp of it a kv head (its q and k), 32 E value channels, or what is
+// left of the projection (beta and the inner values).
+template <typename T, int E, int TAPS>
+__global__ void __launch_bounds__(32 * CD_WARPS) channel_delta_prepare_kernel(const ChannelDeltaArgs a, const int R) {
   pdl_launch_dependents_if_small();
-  const int t = blockIdx.x, unit = blockIdx.y, tid = threadIdx.x;
-  const int H = a.H, G = a.G, dk = a.dk;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int H = a.H, G = a.G, dk = a.dk, V = H * a.dv;
   const int Cc = cd_channels(a), C_all = cd_columns(a), P = a.prep_stride;
-  const int seq = a.token_seq[t];
+  int seq, run;
+  run_of_block(a.cu_q, a.n_seqs, R, a.max_rows == 1, blockIdx.x, seq, run);
+  const int row0 = a.cu_q[seq], n_seq = a.cu_q[seq + 1] - row0;
+  const int r0 = run * R, n = min(R, n_seq - r0);
+  if (n <= 0) return;
   const int slot = a.slots[seq];
-  const int r = t - a.cu_q[seq];                 // the token's place among its sequence's rows
-  const float* tail = slot >= 0 ? a.state + (size_t)slot * a.state_stride : nullptr;
-  float* out = a.prep + (size_t)t * P;
+  float* tail = slot >= 0 && a.taps > 1 ? a.state + (size_t)slot * a.state_stride : nullptr;
+  const int v_units = (V + 32 * E - 1) / (32 * E);
+  const float q_scale = 1.0f / sqrtf((float)dk);
   pdl_wait();
-  if (unit >= G) {                               // value channels: convolution and silu
-    const int c = 2 * G * dk + (unit - G) * CD_PREP_V + tid;
-    if (tid < CD_PREP_V && c < Cc) out[c] = short_conv_silu(a.proj, C_all, a.conv_w, a.taps, tail, Cc, t, r, c);
-    return;
-  }
-  float sq = 0.f, sk = 0.f;
-  for (int i = tid; i < 2 * dk; i += blockDim.x) {
-    const int c = i < dk ? unit * dk + i : (G + unit) * dk + (i - dk);
-    const float v = short_conv_silu(a.proj, C_all, a.conv_w, a.taps, tail, Cc, t, r, c);
-    row[i] = v;
-    if (i < dk) sq += v * v; else sk += v * v;
-  }
-  sq = block_sum(sq, scratch);
-  sk = block_sum(sk, scratch);
-  const float iq = 1.0f / sqrtf(sq + a.unit_eps) * (1.0f / sqrtf((float)dk));
-  const float ik = 1.0f / sqrtf(sk + a.unit_eps);
-  float kq = 0.f;
-  for (int d = tid; d < dk; d += blockDim.x) {
-    const float q = row[d] * iq, k = row[dk + d] * ik;
-    out[unit * dk + d] = q;
-    out[(G + unit) * dk + d] = k;
-    kq = fmaf(q, k, kq);
-  }
-  kq = block_sum(kq, scratch);
-  if (tid == 0) out[Cc + H + unit] = kq;
-  if (unit == 0) {
-    const float* rest = a.proj + (size_t)t * C_all + Cc;
-    for (int h = tid; h < H; h += blockDim.x) out[Cc + h] = cd_sigmoid(rest[h]);
-    T* low = (T*)a.low + (size_t)t * a.n_low;
-    for (int i = tid; i < a.n_low; i += blockDim.x) low[i] = from_f32<T>(rest[H + i]);
+  for (int unit = blockIdx.y * CD_WARPS + warp; unit < G + v_units + 1; unit += gridDim.y * CD_WARPS) {
+    if (unit < G) {
+      CdWalk<E, TAPS> qw, kw;
+      qw.start(a, tail, Cc, C_all, row0, r0, unit * dk, dk, lane);
+      kw.start(a, tail, Cc, C_all, row0, r0, (G + unit) * dk, dk, lane);
+      for (int i = 0; i < n; ++i) {
+        float q[E], k[E], sq = 0.f, sk = 0.f, kq = 0.f;
+        qw.row(a, tail, Cc, C_all, row0, r0 + i, lane, q);
+        kw.row(a, tail, Cc, C_all, row0, r0 + i, lane, k);
+#pragma unroll
+        for (int e = 0; e < E; ++e) sq = fmaf(q[e], q[e], sq), sk = fmaf(k[e], k[e], sk), kq = fmaf(q[e], k[e], kq);
+        sq = warp_sum(sq), sk = warp_sum(sk), kq = warp_sum(kq);
+        const float iq = 1.0f / sqrtf(sq + a.unit_eps) * q_scale, ik = 1.0f / sqrtf(sk + a.unit_eps);
+        float* out = a.prep + (size_t)(row0 + r0 + i) * P;
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+          const int d = lane + 32 * e;
+          if (d < dk) out[unit * dk + d] = q[e] * iq, out[(G + unit) * dk + d] = k[e] * ik;
+        }
+        if (lane == 0) out[Cc + H + unit] = kq * iq * ik;
+      }
+      if (tail && run == 0) {
+        qw.keep(a, tail, Cc, C_all, row0, n_seq, lane);
+        kw.keep(a, tail, Cc, C_all, row0, n_seq, lane);
+      }
+    } else if (unit < G + v_units) {
+      const int c0 = 2 * G * dk + (unit - G) * 32 * E, cols = min(32 * E, Cc - c0);
+      CdWalk<E, TAPS> vw;
+      vw.start(a, tail, Cc, C_all, row0, r0, c0, cols, lane);
+      for (int i = 0; i < n; ++i) {
+        float v[E];
+        vw.row(a, tail, Cc, C_all, row0, r0 + i, lane, v);
+#pragma unroll
+        for (int e = 0; e < E; ++e)
+          if (lane + 32 * e < cols) a.prep[(size_t)(row0 + r0 + i) * P + c0 + lane + 32 * e] = v[e];
+      }
+      if (tail && run == 0) vw.keep(a, tail, Cc, C_all, row0, n_seq, lane);
+    } else {
+      for (int i = 0; i < n; ++i) {
+        const size_t t = row0 + r0 + i;
+        const float* rest = a.proj + t * C_all + Cc;
+        for (int h = lane; h < H; h += 32) a.prep[t * P + Cc + h] = cd_sigmoid(rest[h]);
+        for (int j = lane; j < a.n_low; j += 32) ((T*)a.low)[t * a.n_low + j] = from_f32<T>(rest[H + j]);
+      }
+    }
   }
   pdl_launch_dependents_if_large();
 }
@@ -231,9 +329,6 @@ __global__ void __launch_bounds__(256) channel_delta_step_kernel(const ChannelDe
   const float* gate = z + (size_t)H * dk + (size_t)h * dv;
   T* y = (T*)a.y + ((size_t)t * H + h) * dv;
   for (int j = tid; j < dv; j += 256) y[j] = from_f32<T>(os[j] * inv * a.norm_w[j] * cd_sigmoid(gate[j]));
-  if (a.taps > 1 && slot >= 0)                    // every reader of the old tail, the prepare kernel, has finished
-    short_conv_keep_tail(a.proj, C_all, a.taps, a.state + (size_t)slot * a.state_stride, Cc, t, 1, h * 256 + tid,
-                         H * 256);
 }
 
 template <int R>
@@ -306,13 +401,6 @@ __global__ void channel_delta_finish_kernel(const ChannelDeltaArgs a) {
     T* y = (T*)a.y + ((size_t)t * H + h) * dv;
     for (int j = lane; j < dv; j += 32) y[j] = from_f32<T>(o[j] * inv * a.norm_w[j] * cd_sigmoid(gate[j]));
   }
-  if (a.taps > 1) {
-    const int seq = a.token_seq[t];
-    const int row0 = a.cu_q[seq], slot = a.slots[seq];
-    if (t == row0 && slot >= 0)
-      short_conv_keep_tail(a.proj, cd_columns(a), a.taps, a.state + (size_t)slot * a.state_stride, cd_channels(a), row0,
-                           a.cu_q[seq + 1] - row0, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x);
-  }
   pdl_launch_dependents_if_large();
 }
 
@@ -327,13 +415,30 @@ static int cd_check(const ChannelDeltaArgs& a) {
   return 0;
 }
 
+template <typename T, int E, int TAPS>
+static int prepare_taps(const ChannelDeltaArgs& a, cudaStream_t s) {
+  const int R = a.taps - 1 > CD_RUN ? a.taps - 1 : CD_RUN;
+  const int blocks = a.max_rows == 1 ? a.n_seqs : a.n_tokens / R + a.n_seqs;
+  const int units = a.G + (a.H * a.dv + 32 * E - 1) / (32 * E) + 1;
+  return gb_launch(channel_delta_prepare_kernel<T, E, TAPS>, dim3(blocks, (units + CD_WARPS - 1) / CD_WARPS),
+                   dim3(32 * CD_WARPS), 0, s, a, R);
+}
+
+template <typename T, int E>
+static int prepare_size(const ChannelDeltaArgs& a, cudaStream_t s) {
+  switch (a.taps) {
+    case 2: return prepare_taps<T, E, 2>(a, s);
+    case 3: return prepare_taps<T, E, 3>(a, s);
+    case 4: return prepare_taps<T, E, 4>(a, s);
+    default: return prepare_taps<T, E, 0>(a, s);
+  }
+}
+
 template <typename T>
 static int prepare(const ChannelDeltaArgs& a, cudaStream_t s) {
   const int e = cd_check(a);
   if (e || a.n_tokens == 0) return e;
-  const int units = a.G + (a.H * a.dv + CD_PREP_V - 1) / CD_PREP_V;
-  return gb_launch(channel_delta_prepare_kernel<T>, dim3(a.n_tokens, units), dim3(256), (size_t)2 * a.dk * sizeof(float),
-                   s, a);
+  return a.dk <= 64 ? prepare_size<T, 2>(a, s) : a.dk <= 128 ? prepare_size<T, 4>(a, s) : prepare_size<T, 8>(a, s);
 }
 
 template <typename T, int R>
@@ -361,11 +466,7 @@ static int run_rows(const ChannelDeltaArgs& a, cudaStream_t s) {
   }
   if (e) return e;
   const int warps = a.H < 8 ? a.H : 8;
-  int rows_y = (a.H + warps - 1) / warps;            // blocks of a row: enough for its heads, and
-  const int Cc = 2 * a.G * a.dk + a.H * a.dv;        //   for the tail's channels four to a thread
-  const int for_tail = a.taps > 1 ? (Cc + warps * 32 * 4 - 1) / (warps * 32 * 4) : 1;
-  if (for_tail > rows_y) rows_y = for_tail < 64 ? for_tail : 64;
-  return gb_launch(channel_delta_finish_kernel<T>, dim3(a.n_tokens, rows_y), dim3(warps * 32), 0, s, a);
+  return gb_launch(channel_delta_finish_kernel<T>, dim3(a.n_tokens, (a.H + warps - 1) / warps), dim3(warps * 32), 0, s, a);
 }
 
 template <typename T>

@@ -14,9 +14,9 @@
 //   chain   walks a sequence's chunks in order, a block per head and CC_COLS columns of S with the
 //           state in shared memory: U = U0 - W S, the read-outs, the next state: tiled 32-bit products
 //
-// Every exponent that is taken is a difference that is not positive (rows of the same half chunk
-// directly, others by way of the end of the first half), so no quotient of decays overflows however
-// strong they are.
+// Every exponent that is taken is not positive and is summed up from logarithms of one sign, never a
+// difference of two running sums (rows of the same half chunk directly, others by way of the end of
+// the first half): no quotient of decays overflows, and none loses its digits behind a strong one.
 #pragma once
 
 #define CC_ROWS 32       // rows of a chunk
@@ -49,7 +49,6 @@ __device__ __forceinline__ float cc_transpose_sum(float (&v)[32], int lane) {
   return v[0];
 }
 
-template <int E> struct CcVec { float e[E]; };
 template <int E>
 __device__ __forceinline__ void cc_read(const float* p, float (&o)[E]) {
   if constexpr (E == 4) {
@@ -65,10 +64,11 @@ __device__ __forceinline__ void cc_read(const float* p, float (&o)[E]) {
 
 // E channels a lane: heads of up to 32 E.  The block's rows, zero beyond dk and beyond the chunk's end.
 template <int E>
-__global__ void __launch_bounds__(256) channel_delta_local_kernel(const ChannelDeltaArgs a) {
+__global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const ChannelDeltaArgs a) {
   constexpr int DKP = 32 * E, LD = DKP + 4;      // (16-byte rows; a column's rows on different banks)
   extern __shared__ __align__(16) float sm[];
-  float *Ks = sm, *Qs = Ks + CC_ROWS * LD, *Ls = Qs + CC_ROWS * LD, *Kr = Ls + CC_ROWS * LD;   // Kr [16][LD]
+  float *Ks = sm, *Qs = Ks + CC_ROWS * LD, *Ls = Qs + CC_ROWS * LD, *Fs = Ls + CC_ROWS * LD;
+  float *Kr = Fs + CC_ROWS * LD;                 // [16][LD]: the first half's keys, faded to its end
   float *As = Kr + CC_HALF * LD, *Bs = As + CC_ROWS * CC_ROWS, *beta = Bs + CC_ROWS * CC_ROWS;
   pdl_launch_dependents_if_small();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -91,29 +91,57 @@ __global__ void __launch_bounds__(256) channel_delta_local_kernel(const ChannelD
   }
   if (tid < CC_ROWS) beta[tid] = tid < n ? a.prep[(size_t)(row0 + tid) * a.prep_stride + Cc + h] : 0.f;
   __syncthreads();
-  if (tid < DKP) {                               // running sums of the logarithms
+  const size_t entry = (cc_entry(first, z, seq) * H + h) * cc_record(dk, dv);
+  float* wq = a.chunks + entry;
+  float* kd = wq + (size_t)dk * 64;
+  float* gc = kd + (size_t)CC_ROWS * dk;
+  float* bm = gc + dk;
+  float* u0 = bm + CC_ROWS * CC_ROWS;
+  // per channel: Fs, the logarithms summed up from the start of a row's half chunk on; and, from the
+  // chunk's end back, what is left of a row's key at the end of its half and of the chunk (rows
+  // beyond the chunk's end have no decay)
+  if (tid < DKP) {
     float s = 0.f;
-    for (int t = 0; t < CC_ROWS; ++t) s += Ls[t * LD + tid], Ls[t * LD + tid] = s;
-    const float mid = Ls[(CC_HALF - 1) * LD + tid];
-    for (int t = 0; t < CC_HALF; ++t) Kr[t * LD + tid] = Ks[t * LD + tid] * expf(mid - Ls[t * LD + tid]);
+#pragma unroll 8
+    for (int t = 0; t < CC_ROWS; ++t) {
+      if (t == CC_HALF) s = 0.f;
+      s += Ls[t * LD + tid];
+      Fs[t * LD + tid] = s;
+    }
+  } else if (tid >= 128 && tid - 128 < DKP) {
+    const int d = tid - 128;
+    float s = 0.f, in_half = 0.f;
+#pragma unroll 4
+    for (int t = CC_ROWS - 1; t >= 0; --t) {
+      const float k = Ks[t * LD + d], lg = Ls[t * LD + d];
+      if (d < dk) kd[t * dk + d] = k * expf(s);
+      if (t < CC_HALF) {
+        Kr[t * LD + d] = k * expf(in_half);
+        in_half += lg;
+      }
+      s += lg;
+    }
+    if (d < dk) gc[d] = expf(s);
   }
   __syncthreads();
   // A and B: a warp takes rows warp, warp + 8, ...; its lanes share the channels
   for (int t = warp; t < CC_ROWS; t += 8) {
-    float kt[E], qt[E], lt[E], ki[E], li[E], part[32];
+    float kt[E], qt[E], ki[E], li[E], since[E], part[32];
     cc_read<E>(Ks + t * LD + lane * E, kt);
     cc_read<E>(Qs + t * LD + lane * E, qt);
-    cc_read<E>(Ls + t * LD + lane * E, lt);
     const int base = t & CC_HALF;                // the first row of t's half chunk
 #pragma unroll
-    for (int j = 0; j < CC_HALF; ++j) {
+    for (int x = 0; x < E; ++x) since[x] = 0.f;  // the logarithms behind row base + j, up to t's
+#pragma unroll
+    for (int j = CC_HALF - 1; j >= 0; --j) {
       part[j] = part[CC_HALF + j] = 0.f;
       if (base + j <= t) {
         cc_read<E>(Ks + (base + j) * LD + lane * E, ki);
         cc_read<E>(Ls + (base + j) * LD + lane * E, li);
 #pragma unroll
         for (int x = 0; x < E; ++x) {
-          const float w = ki[x] * expf(lt[x] - li[x]);
+          const float w = ki[x] * expf(since[x]);
+          since[x] += li[x];
           part[j] = fmaf(kt[x], w, part[j]);
           part[CC_HALF + j] = fmaf(qt[x], w, part[CC_HALF + j]);
         }
@@ -124,11 +152,10 @@ __global__ void __launch_bounds__(256) channel_delta_local_kernel(const ChannelD
     if (lane < CC_HALF) As[t * CC_ROWS + base + j] = base + j < t ? sum : 0.f;
     else Bs[t * CC_ROWS + base + j] = base + j <= t ? sum : 0.f;
     if (base) {                                  // the other half, by way of its last row
-      float mid[E];
-      cc_read<E>(Ls + (CC_HALF - 1) * LD + lane * E, mid);
+      cc_read<E>(Fs + t * LD + lane * E, li);
 #pragma unroll
       for (int x = 0; x < E; ++x) {
-        const float w = expf(lt[x] - mid[x]);
+        const float w = expf(li[x]);
         kt[x] *= w, qt[x] *= w;
       }
 #pragma unroll
@@ -149,19 +176,13 @@ __global__ void __launch_bounds__(256) channel_delta_local_kernel(const ChannelD
   }
   __syncthreads();
   // the substitution: a thread takes one right-hand side (dv of values, then dk of e^{L} k)
-  const size_t entry = (cc_entry(first, z, seq) * H + h) * cc_record(dk, dv);
-  float* wq = a.chunks + entry;
-  float* kd = wq + (size_t)dk * 64;
-  float* gc = kd + (size_t)CC_ROWS * dk;
-  float* bm = gc + dk;
-  float* u0 = bm + CC_ROWS * CC_ROWS;
   for (int c = tid; c < dv + dk; c += 256) {
     float x[CC_ROWS];
     const int d = c - dv;
 #pragma unroll
     for (int t = 0; t < CC_ROWS; ++t) {
       if (d < 0) x[t] = t < n ? a.prep[(size_t)(row0 + t) * a.prep_stride + 2 * G * dk + h * dv + c] : 0.f;
-      else x[t] = Ks[t * LD + d] * expf(Ls[t * LD + d]);
+      else x[t] = Ks[t * LD + d] * expf(Fs[t * LD + d] + (t < CC_HALF ? 0.f : Fs[(CC_HALF - 1) * LD + d]));
     }
 #pragma unroll
     for (int t = 0; t < CC_ROWS; ++t) {
@@ -188,17 +209,12 @@ __global__ void __launch_bounds__(256) channel_delta_local_kernel(const ChannelD
   pdl_launch_dependents_if_large();
   for (int i = tid; i < 8 * dk; i += 256) {      // e^{L} q, four rows of a channel a thread
     const int d = i / 8, t = (i % 8) * 4;
+    const float before = t < CC_HALF ? 0.f : Fs[(CC_HALF - 1) * LD + d];
     float v[4];
 #pragma unroll
-    for (int x = 0; x < 4; ++x) v[x] = Qs[(t + x) * LD + d] * expf(Ls[(t + x) * LD + d]);
+    for (int x = 0; x < 4; ++x) v[x] = Qs[(t + x) * LD + d] * expf(Fs[(t + x) * LD + d] + before);
     *reinterpret_cast<float4*>(wq + (size_t)d * 64 + CC_ROWS + t) = make_float4(v[0], v[1], v[2], v[3]);
   }
-  // (rows beyond the chunk's end have no decay of their own: the last row's sums are the chunk's)
-  for (int i = tid; i < CC_ROWS * dk; i += 256) {
-    const int t = i / dk, d = i % dk;
-    kd[i] = Ks[t * LD + d] * expf(Ls[(CC_ROWS - 1) * LD + d] - Ls[t * LD + d]);
-  }
-  for (int d = tid; d < dk; d += 256) gc[d] = expf(Ls[(CC_ROWS - 1) * LD + d]);
   for (int i = tid; i < CC_ROWS * CC_ROWS; i += 256) bm[i] = Bs[i];
 }
 
@@ -354,7 +370,7 @@ static bool cc_takes(const ChannelDeltaArgs& a) {
 template <int E>
 static int cc_local(const ChannelDeltaArgs& a, int chunks, cudaStream_t s) {
   constexpr int LD = 32 * E + 4;
-  const size_t smem = ((3 * CC_ROWS + CC_HALF) * LD + 2 * CC_ROWS * CC_ROWS + CC_ROWS) * sizeof(float);
+  const size_t smem = ((4 * CC_ROWS + CC_HALF) * LD + 2 * CC_ROWS * CC_ROWS + CC_ROWS) * sizeof(float);
   static bool configured = false;
   if (smem > 48 * 1024 && !configured) {
     cudaError_t e = cudaFuncSetAttribute(channel_delta_local_kernel<E>, cudaFuncAttributeMaxDynamicSharedMemorySize,

@@ -11,13 +11,8 @@
 // and rotation may each be absent.
 //
 // The last taps - 1 values u of every sequence are kept (32-bit, `tail`): what a later step's
-// first rows look back to.  A step's rows are cut into runs of QC_RUN (never fewer than taps - 1)
-// rows that start at each sequence's first; only a sequence's first run looks back behind the
-// step, so the thread that owns a channel there reads the kept values and then replaces them.
-// Sequence s's runs are given the blocks cu_q[s] / RUN + s up to those of s + 1, which are never
-// fewer than it needs and are found by bisection: the host need not know how rows divide into
-// sequences.
-#include "common.cuh"
+// first rows look back to.  A block takes a run of rows (run_of_block), a warp of it a head.
+#include "short_conv.cuh"
 
 struct QkConvArgs {
   const float* proj;        // [n_parts][T, (nq + nkv) D (+ nkv Dv)] 32-bit sums
@@ -45,40 +40,48 @@ struct QkConvArgs {
 #define QC_WARPS 8
 #define QC_TAPS 4           // taps whose inputs a thread keeps in registers; with more it reads them again
 
-__device__ __forceinline__ float qc_sum(const QkConvArgs& a, size_t at) {
-  float v = 0.f;
-  for (int k0 = 0; k0 < a.n_parts; k0 += 4) {      // four partial sums requested at a time, added in order
-    float p[4];
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      const int k = k0 + u < a.n_parts ? k0 + u : a.n_parts - 1;
-      p[u] = a.proj[(size_t)k * a.part_stride + at];
+// V neighbouring values of the projection from `at` on, the partial sums added in order.
+template <int V>
+__device__ __forceinline__ void qc_sum(const QkConvArgs& a, size_t at, float (&v)[V]) {
+  auto load = [&](const float* p, float (&o)[V]) {
+    if constexpr (V == 2) {
+      const float2 x = *reinterpret_cast<const float2*>(p);
+      o[0] = x.x, o[1] = x.y;
+    } else {
+      o[0] = p[0];
     }
+  };
+  load(a.proj + at, v);
+  for (int k0 = 1; k0 < a.n_parts; k0 += 4) {      // four partial sums requested at a time
+    float p[4][V];
 #pragma unroll
     for (int u = 0; u < 4; ++u)
-      if (k0 + u < a.n_parts) v += p[u];
+      load(a.proj + (size_t)(k0 + u < a.n_parts ? k0 + u : a.n_parts - 1) * a.part_stride + at, p[u]);
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+      if (k0 + u < a.n_parts) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] += p[u][e];
+      }
   }
-  return v;
 }
 
-template <typename T, int TAPS>      // TAPS 0: any number of them
+template <typename T, int V>
+__device__ __forceinline__ void qc_store(T* p, const float (&v)[V]) {
+  if constexpr (V == 2 && sizeof(T) == 2) *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[1]);
+  else if constexpr (V == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+  else p[0] = from_f32<T>(v[0]);
+}
+
+// TAPS 0: any number of them.  V: neighbouring pairs (or pieces of what is not turned) a lane takes together
+template <typename T, int TAPS, int V>
 __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs a) {
   extern __shared__ float qc_sm[];   // the run's sines and cosines [run, rot_dim / 2] each
   pdl_launch_dependents_if_small();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int R = a.run, taps = TAPS > 0 ? TAPS : a.taps;
   int seq, run;
-  if (a.one_row) {
-    seq = blockIdx.x, run = 0;
-  } else {                           // the last sequence whose first block is not behind this one
-    int lo = 0, hi = a.n_seqs - 1;
-    const int b = blockIdx.x;
-    while (lo < hi) {
-      const int mid = (lo + hi + 1) >> 1;
-      if (a.cu_q[mid] / R + mid <= b) lo = mid; else hi = mid - 1;
-    }
-    seq = lo, run = b - (a.cu_q[lo] / R + lo);
-  }
+  run_of_block(a.cu_q, a.n_seqs, R, a.one_row, blockIdx.x, seq, run);
   const int row0 = a.cu_q[seq], n_seq = a.cu_q[seq + 1] - row0;
   const int r0 = run * R, n = min(R, n_seq - r0);        // the run: rows r0 .. r0 + n of the sequence
   if (n <= 0) return;
@@ -100,10 +103,16 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
   const int* table = slot >= 0 ? a.block_table + (size_t)slot * a.max_pages : nullptr;
   float* tail = slot >= 0 && a.tail ? a.tail + (size_t)slot * a.tail_stride : nullptr;
 
-  // u of channel c at row rr of the sequence's rows (negative: behind the step)
-  auto input = [&](int rr, int c, float b) -> float {
-    if (rr >= 0) return qc_sum(a, (size_t)(row0 + rr) * width + c) + b;
-    return tail && rr + taps - 1 >= 0 ? tail[(size_t)(taps - 1 + rr) * Cc + c] : 0.f;
+  // u of channels c .. at row rr of the sequence's rows (negative: behind the step)
+  auto input = [&](int rr, int c, const float (&b)[V], float (&u)[V]) {
+    if (rr >= 0) {
+      qc_sum<V>(a, (size_t)(row0 + rr) * width + c, u);
+#pragma unroll
+      for (int e = 0; e < V; ++e) u[e] += b[e];
+    } else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) u[e] = tail && rr + taps - 1 >= 0 ? tail[(size_t)(taps - 1 + rr) * Cc + c + e] : 0.f;
+    }
   };
   for (int head = blockIdx.y * QC_WARPS + warp; head < n_heads; head += gridDim.y * QC_WARPS) {
     if (head >= nqk) {                                   // a value head of its own: stored as it is
@@ -111,83 +120,113 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
       for (int i = 0; i < n && table; ++i) {
         const int pos = a.token_pos[row0 + r0 + i];
         T* dst = (T*)a.v_pages + paged_row(table, pos, g, a.nkv, a.page, Ds);
-        for (int d = lane; d < Ds; d += 32)
-          dst[d] = from_f32<T>(d < a.Dv ? qc_sum(a, (size_t)(row0 + r0 + i) * width + Cc + (size_t)g * a.Dv + d) : 0.f);
+        for (int d = lane; d < Ds; d += 32) {
+          float v[1] = {0.f};
+          if (d < a.Dv) qc_sum<1>(a, (size_t)(row0 + r0 + i) * width + Cc + (size_t)g * a.Dv + d, v);
+          dst[d] = from_f32<T>(v[0]);
+        }
       }
       continue;
     }
-    // an item is a rotated pair, or an element (and its neighbour) that passes unturned
-    const int pairs = half + (D - 2 * half + 1) / 2;
-    for (int it = lane; it < pairs; it += 32) {
+    // an item is V rotated pairs, or as many pairs of elements that pass unturned
+    const int turned_items = half / V;
+    const int items = turned_items + (D - 2 * half + 2 * V - 1) / (2 * V);
+    for (int it = lane; it < items; it += 32) {
       int e0, e1;
-      const bool turned = it < half;
+      const bool turned = it < turned_items;
       if (turned) {
-        e0 = a.interleaved ? 2 * it : it, e1 = a.interleaved ? 2 * it + 1 : it + half;
+        e0 = a.interleaved ? 2 * it : it * V, e1 = a.interleaved ? 2 * it + 1 : it * V + half;
       } else {
-        e0 = 2 * half + 2 * (it - half), e1 = e0 + 1;
+        e0 = 2 * half + 2 * V * (it - turned_items), e1 = e0 + V;
       }
       const bool two = e1 < D;
-      const int c0 = head * D + e0, c1 = head * D + (two ? e1 : e0);
-      const float b0 = a.bias ? a.bias[c0] : 0.f, b1 = a.bias ? a.bias[c1] : 0.f;
+      const int ch[2] = {head * D + e0, head * D + (two ? e1 : e0)};
       constexpr int W = TAPS > 0 ? TAPS : 1;
-      float w0[W], w1[W], x0[W], x1[W];      // x[j]: the input j rows back
+      float b[2][V], w[W][2][V], x[W][2][V];      // x[j]: the input j rows back
 #pragma unroll
-      for (int j = 0; j < W; ++j) {
-        w0[j] = w1[j] = 1.f, x0[j] = x1[j] = 0.f;
-        if (TAPS > 0) {
-          if (a.conv_w) {
-            w0[j] = a.conv_w[(size_t)c0 * taps + taps - 1 - j];
-            w1[j] = a.conv_w[(size_t)c1 * taps + taps - 1 - j];
-          }
-          if (j > 0) x0[j - 1] = input(r0 - j, c0, b0), x1[j - 1] = input(r0 - j, c1, b1);
+      for (int s = 0; s < 2; ++s)
+#pragma unroll
+        for (int e = 0; e < V; ++e) b[s][e] = a.bias ? a.bias[ch[s] + e] : 0.f;
+#pragma unroll
+      for (int j = 0; j < W; ++j)
+#pragma unroll
+        for (int s = 0; s < 2; ++s) {
+#pragma unroll
+          for (int e = 0; e < V; ++e)
+            w[j][s][e] = TAPS > 0 && a.conv_w ? a.conv_w[(size_t)(ch[s] + e) * taps + taps - 1 - j] : 1.f;
+          if (TAPS > 0 && j > 0) input(r0 - j, ch[s], b[s], x[j - 1][s]);
         }
-      }
-#pragma unroll 2
+#pragma unroll 4
       for (int i = 0; i < n; ++i) {
-        float y0, y1;
+        float c[2][V];
         if (TAPS > 0) {
 #pragma unroll
-          for (int j = W - 1; j > 0; --j) x0[j] = x0[j - 1], x1[j] = x1[j - 1];
-          x0[0] = input(r0 + i, c0, b0), x1[0] = input(r0 + i, c1, b1);
-          y0 = w0[0] * x0[0], y1 = w1[0] * x1[0];
+          for (int j = W - 1; j > 0; --j)
 #pragma unroll
-          for (int j = 1; j < W; ++j) y0 = fmaf(w0[j], x0[j], y0), y1 = fmaf(w1[j], x1[j], y1);
-        } else {
-          y0 = 0.f, y1 = 0.f;
-          for (int j = 0; j < taps; ++j) {
-            y0 = fmaf(a.conv_w[(size_t)c0 * taps + taps - 1 - j], input(r0 + i - j, c0, b0), y0);
-            y1 = fmaf(a.conv_w[(size_t)c1 * taps + taps - 1 - j], input(r0 + i - j, c1, b1), y1);
+            for (int s = 0; s < 2; ++s)
+#pragma unroll
+              for (int e = 0; e < V; ++e) x[j][s][e] = x[j - 1][s][e];
+#pragma unroll
+          for (int s = 0; s < 2; ++s) {
+            input(r0 + i, ch[s], b[s], x[0][s]);
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+              c[s][e] = w[0][s][e] * x[0][s][e];
+#pragma unroll
+              for (int j = 1; j < W; ++j) c[s][e] = fmaf(w[j][s][e], x[j][s][e], c[s][e]);
+            }
           }
+        } else {
+#pragma unroll
+          for (int s = 0; s < 2; ++s)
+#pragma unroll
+            for (int e = 0; e < V; ++e) c[s][e] = 0.f;
+          for (int j = 0; j < taps; ++j)
+#pragma unroll
+            for (int s = 0; s < 2; ++s) {
+              input(r0 + i - j, ch[s], b[s], x[0][s]);
+#pragma unroll
+              for (int e = 0; e < V; ++e)
+                c[s][e] = fmaf(a.conv_w[(size_t)(ch[s] + e) * taps + taps - 1 - j], x[0][s][e], c[s][e]);
+            }
         }
-        const float v0 = y0, v1 = y1;
-        if (turned) {
-          const float s = sn[i * half + it], c = cs[i * half + it];
-          y0 = v0 * c - v1 * s;
-          y1 = v1 * c + v0 * s;
-        }
+        T* dst = nullptr;
         if (head < a.nq) {
-          T* dst = (T*)a.q_out + ((size_t)(row0 + r0 + i) * a.nq + head) * Ds;
-          dst[e0] = from_f32<T>(y0);
-          if (two) dst[e1] = from_f32<T>(y1);
+          dst = (T*)a.q_out + ((size_t)(row0 + r0 + i) * a.nq + head) * Ds;
         } else if (table) {
           const size_t at = paged_row(table, a.token_pos[row0 + r0 + i], head - a.nq, a.nkv, a.page, Ds);
-          T* dst = (T*)a.k_pages + at;
-          dst[e0] = from_f32<T>(y0);
-          if (two) dst[e1] = from_f32<T>(y1);
-          if (a.v_from_k) {
-            T* dv = (T*)a.v_pages + at;
-            dv[e0] = from_f32<T>(v0);
-            if (two) dv[e1] = from_f32<T>(v1);
+          dst = (T*)a.k_pages + at;
+          if (a.v_from_k) {                      // the value: the key as it stands now
+            qc_store<T, V>((T*)a.v_pages + at + e0, c[0]);
+            if (two) qc_store<T, V>((T*)a.v_pages + at + e1, c[1]);
           }
+        }
+        if (turned) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            const int pair = a.interleaved ? it : it * V + e;
+            const float sv = sn[i * half + pair], cv = cs[i * half + pair], lo = c[0][e], hi = c[1][e];
+            c[0][e] = lo * cv - hi * sv;
+            c[1][e] = hi * cv + lo * sv;
+          }
+        }
+        if (dst) {
+          qc_store<T, V>(dst + e0, c[0]);
+          if (two) qc_store<T, V>(dst + e1, c[1]);
         }
       }
       if (tail && run == 0) {        // entry s: the input at n_seq - (taps - 1) + s; an entry that moves down
                                      // is read before it is overwritten
         for (int s = 0; s < taps - 1; ++s) {
-          const int rr = n_seq - (taps - 1) + s;
-          const float t0 = input(rr, c0, b0), t1 = input(rr, c1, b1);
-          tail[(size_t)s * Cc + c0] = t0;
-          if (two) tail[(size_t)s * Cc + c1] = t1;
+          float t[2][V];
+#pragma unroll
+          for (int k = 0; k < 2; ++k) input(n_seq - (taps - 1) + s, ch[k], b[k], t[k]);
+#pragma unroll
+          for (int k = 0; k < 2; ++k)
+            if (k == 0 || two) {
+#pragma unroll
+              for (int e = 0; e < V; ++e) tail[(size_t)s * Cc + ch[k] + e] = t[k][e];
+            }
         }
       }
     }
@@ -210,15 +249,25 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
   pdl_launch_dependents_if_large();
 }
 
-template <typename T, int TAPS>
-static int launch_taps(const QkConvArgs& a, cudaStream_t s) {
+template <typename T, int TAPS, int V>
+static int launch_items(const QkConvArgs& a, cudaStream_t s) {
   const int blocks = a.one_row ? a.n_seqs : a.T / a.run + a.n_seqs;
   const int n_heads = a.nq + a.nkv * (a.v_from_k ? 1 : 2);
   int y = (n_heads + QC_WARPS - 1) / QC_WARPS;           // few runs: a warp per head; many: fewer warps, whose
   while (y > 1 && (long long)blocks * y > 148 * 16) y = (y + 1) / 2;   // sines serve several heads
   const size_t smem = a.inv_freq ? (size_t)a.run * a.rot_dim * sizeof(float) : 0;
   if (smem > 48 * 1024) return GB_ERR_UNSUPPORTED;
-  return gb_launch(qk_conv_kernel<T, TAPS>, dim3(blocks, y), dim3(32 * QC_WARPS), smem, s, a);
+  return gb_launch(qk_conv_kernel<T, TAPS, V>, dim3(blocks, y), dim3(32 * QC_WARPS), smem, s, a);
+}
+
+template <typename T, int TAPS>
+static int launch_taps(const QkConvArgs& a, cudaStream_t s) {
+  // two pairs together where every piece of two lies on its boundary
+  const long long width = (long long)(a.nq + a.nkv) * a.D + (a.v_from_k ? 0 : (long long)a.nkv * a.Dv);
+  const bool even = !a.interleaved && a.rot_dim % 4 == 0 && (a.D - a.rot_dim) % 4 == 0 && a.Ds % 2 == 0 && width % 2 == 0 &&
+                    a.part_stride % 2 == 0 &&
+                    (((uintptr_t)a.proj | (uintptr_t)a.q_out | (uintptr_t)a.k_pages | (uintptr_t)a.v_pages) & 7) == 0;
+  return even ? launch_items<T, TAPS, 2>(a, s) : launch_items<T, TAPS, 1>(a, s);
 }
 
 template <typename T>

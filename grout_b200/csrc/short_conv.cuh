@@ -57,3 +57,21 @@ __device__ __forceinline__ void short_conv_keep_tail(const float* proj, long lon
     }
   }
 }
+
+// Rows in runs of R (never fewer than taps - 1) that start at each sequence's first row: only a
+// sequence's first run looks back behind the step, so the thread that owns a channel there can
+// read the kept inputs and replace them afterwards.  Sequence s's runs are given the blocks
+// cu_q[s] / R + s up to those of s + 1, which are never fewer than it needs and are found by
+// bisection (the host need not know how rows divide into sequences); T / R + n_seqs blocks in all.
+// `one_row`: every sequence brings one row, and block i is sequence i.
+__device__ __forceinline__ void run_of_block(const int* cu_q, int n_seqs, int R, bool one_row, int block, int& seq,
+                                             int& run) {
+  seq = block, run = 0;
+  if (one_row) return;
+  int lo = 0, hi = n_seqs - 1;
+  while (lo < hi) {                  // the last sequence whose first block is not behind this one
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu_q[mid] / R + mid <= block) lo = mid; else hi = mid - 1;
+  }
+  seq = lo, run = block - (cu_q[lo] / R + lo);
+}

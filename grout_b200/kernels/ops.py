@@ -1789,18 +1789,19 @@ def _channel_delta_args(proj, state, conv_w, *, H, G, dk, dv, taps, n_low, token
 @_profiled("channel_delta_prepare", lambda out, proj, *a, **k: (_nbytes(proj, *out), 0))
 def channel_delta_prepare(proj: torch.Tensor, state: torch.Tensor, conv_w: torch.Tensor, *, H: int, G: int, dk: int,
                           dv: int, taps: int, n_low: int, unit_eps: float, token_seq, cu_q, slots,
-                          dtype: torch.dtype):
+                          dtype: torch.dtype, max_rows: Optional[int] = None):
     """What comes in front of the recurrence of the delta rule with a decay per channel.  ``proj``
     [T, C] 32-bit: the columns q [G dk] | k [G dk] | v [H dv] | beta logits [H] | the thin
     products' inner values [n_low].  Returns (prep, low): ``prep`` [T, P] 32-bit holds what
     ``channel_delta_run`` takes (unit q and k and v behind their convolutions, beta, k . q), ``low``
-    [T, n_low] the inner values in ``dtype``.  ``state`` is read only (the convolutions' tail)."""
+    [T, n_low] the inner values in ``dtype``.  Of ``state`` the convolutions' tail is read and
+    replaced.  ``max_rows``: the most rows any sequence brings, when the host knows it."""
     a = _channel_delta_args(proj, state, conv_w, H=H, G=G, dk=dk, dv=dv, taps=taps, n_low=n_low,
                             token_seq=token_seq, cu_q=cu_q, slots=slots)
     T = proj.shape[0]
     prep = torch.empty((T, a.prep_stride), dtype=torch.float32, device=proj.device)
     low = torch.empty((T, n_low), dtype=dtype, device=proj.device)
-    a.prep, a.low, a.unit_eps = prep.data_ptr(), low.data_ptr(), float(unit_eps)
+    a.prep, a.low, a.unit_eps, a.max_rows = prep.data_ptr(), low.data_ptr(), float(unit_eps), int(max_rows or 0)
     _check(_fn("channel_delta", f"gb_channel_delta_prepare_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
            "channel_delta_prepare")
     return prep, low
@@ -1821,8 +1822,7 @@ def channel_delta_run(proj: torch.Tensor, prep: torch.Tensor, low: torch.Tensor,
     ``channel_delta_prepare`` (whose ``proj``, ``prep`` and ``low`` it is given) and the second thin
     product ``wide`` [T, H dk + H dv] 32-bit: z | gate logits.  Per head g = exp(-exp(a_log)
     softplus(z + dt_bias)); S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.  ``state``
-    [slots + 1, delta_state_floats] 32-bit is updated in place for slots that are not negative (the
-    convolutions' tail with it).  Returns y [T, H dv] in ``dtype``: o normalised over dv, times
+    [slots + 1, delta_state_floats] 32-bit is updated in place for slots that are not negative.  Returns y [T, H dv] in ``dtype``: o normalised over dv, times
     ``norm_w`` and sigmoid(gate).  ``max_rows``: the most rows any sequence brings, when the host
     knows it; with 1 (a decode step) all of it is one kernel, from ``CHANNEL_DELTA_CHUNK_MIN`` on the step
     goes chunk by chunk (the same sums in another order)."""

@@ -201,13 +201,14 @@ class ChannelDelta(Mixer):
             raise ValueError(f"the delta rule with a decay per channel was given the cache "
                              f"{None if cache is None else cache.spec}")
         sizes = dict(H=self.H, G=self.G, dk=self.dk, dv=self.dv, taps=self.taps, token_seq=step.token_seq,
-                     cu_q=step.cu_q, slots=step.slots, dtype=self.ctx.dtype)
+                     cu_q=step.cu_q, slots=step.slots, dtype=self.ctx.dtype,
+                     max_rows=step.max_q_len)
         proj = self.proj(x, out_dtype=torch.float32)
         prep, low = ops.channel_delta_prepare(proj, cache.state, self.conv_w, n_low=self.n_low,
                                               unit_eps=self.unit_eps, **sizes)
         wide = self.thin(low, out_dtype=torch.float32)
         y = ops.channel_delta_run(proj, prep, low, wide, cache.state, self.conv_w, self.a_log, self.dt_bias,
-                                  self.norm_w, norm_eps=self.norm_eps, max_rows=step.max_q_len, **sizes)
+                                  self.norm_w, norm_eps=self.norm_eps, **sizes)
         return self.o(y, partial_ok=True)
 
 
