@@ -13,7 +13,7 @@
 // product arrive as 32-bit sums, and only y, the o projection's input, is rounded (and the thin
 // products' inner values, where activations are 16-bit).
 //
-//   prepare  a block per run of rows, a warp of it a kv head (its q, its k and their product) or a
+//   prepare  a block per run of rows, a warp of it a head of q or k or a
 //            run of value channels, the convolutions' inputs passing through registers: convolution,
 //            silu, unit vectors, beta, the new tail; the thin products' inner values go to a tensor
 //            of their own, the second thin product's input
@@ -49,14 +49,14 @@ struct ChannelDeltaArgs {
   const int* slots;        // [n_seqs]
   float* state;            // [slots, state_stride]
   long long state_stride;
-  float* prep;             // [n_tokens, prep_stride]: unit q | unit k | v | beta [H] | k . q [G]
+  float* prep;             // [n_tokens, prep_stride]: unit q | unit k | v | beta [H]
   void* low;               // [n_tokens, n_low] in the activation type
   const float* wide;       // [n_tokens, H dk + H dv]: z | gate logits
   float* o;                // [n_tokens, H, dv]
   void* y;                 // [n_tokens, H dv] in the activation type
   int n_tokens, n_seqs, H, G, dk, dv, taps, n_low;
   float unit_eps, norm_eps;
-  int prep_stride;         // floats between rows of prep: round4(Cc + H + G)
+  int prep_stride;         // floats between rows of prep: round4(Cc + H)
   int max_rows;            // the most rows any sequence brings (0: unknown)
   float* chunks;           // [n_tokens / 32 + n_seqs, H, record] scratch of a step that goes chunk by chunk, or null
 };
@@ -70,88 +70,120 @@ __device__ __forceinline__ float cd_log_decay(float z, float bias, float rate) {
 #define CD_RUN 8         // rows of a run (never fewer than taps - 1)
 #define CD_WARPS 8
 
-// E channels of a lane: c0 + lane + 32 x (those below `cols` exist).
-template <int E>
-__device__ __forceinline__ void cd_inputs(const ChannelDeltaArgs& a, const float* tail, int Cc, int C_all, int row0,
-                                          int rr, int c0, int lane, int cols, float (&o)[E]) {
+// A lane's E channels among the `cols` from c0 on: E neighbours (VEC, which needs every piece on its
+// boundary and whole), or every 32nd.
+template <int E, bool VEC>
+__device__ __forceinline__ int cd_at(int lane, int e) { return VEC ? lane * E + e : lane + 32 * e; }
+
+template <int E, bool VEC>
+__device__ __forceinline__ void cd_load(const float* p, int lane, int cols, float (&o)[E]) {
+  if constexpr (VEC && E == 4) {
+    const float4 x = lane * E < cols ? *reinterpret_cast<const float4*>(p + lane * E) : make_float4(0.f, 0.f, 0.f, 0.f);
+    o[0] = x.x, o[1] = x.y, o[2] = x.z, o[3] = x.w;
+  } else if constexpr (VEC && E == 2) {
+    const float2 x = lane * E < cols ? *reinterpret_cast<const float2*>(p + lane * E) : make_float2(0.f, 0.f);
+    o[0] = x.x, o[1] = x.y;
+  } else {
 #pragma unroll
-  for (int x = 0; x < E; ++x) {
-    const int d = lane + 32 * x;
-    o[x] = 0.f;
-    if (d < cols) {
-      if (rr >= 0) o[x] = a.proj[(size_t)(row0 + rr) * C_all + c0 + d];
-      else if (tail && rr + a.taps - 1 >= 0) o[x] = tail[(size_t)(a.taps - 1 + rr) * Cc + c0 + d];
-    }
+    for (int e = 0; e < E; ++e) o[e] = cd_at<E, VEC>(lane, e) < cols ? p[cd_at<E, VEC>(lane, e)] : 0.f;
+  }
+}
+template <int E, bool VEC>
+__device__ __forceinline__ void cd_store(float* p, int lane, int cols, const float (&v)[E]) {
+  if constexpr (VEC && E == 4) {
+    if (lane * E < cols) *reinterpret_cast<float4*>(p + lane * E) = make_float4(v[0], v[1], v[2], v[3]);
+  } else if constexpr (VEC && E == 2) {
+    if (lane * E < cols) *reinterpret_cast<float2*>(p + lane * E) = make_float2(v[0], v[1]);
+  } else {
+#pragma unroll
+    for (int e = 0; e < E; ++e)
+      if (cd_at<E, VEC>(lane, e) < cols) p[cd_at<E, VEC>(lane, e)] = v[e];
   }
 }
 
+// What the rows of a run are read from.
+struct CdRows {
+  const float* proj;
+  long long ld;
+  const float* tail;       // null: zeros
+  int Cc, taps, row0;
+  // the input of channels c0 .. at row rr of the sequence's rows (negative: behind the step)
+  template <int E, bool VEC>
+  __device__ __forceinline__ void get(int rr, int c0, int cols, int lane, float (&o)[E]) const {
+    const float* p = rr >= 0 ? proj + (size_t)(row0 + rr) * ld + c0
+                             : (tail && rr + taps - 1 >= 0 ? tail + (size_t)(taps - 1 + rr) * Cc + c0 : nullptr);
+    cd_load<E, VEC>(p, lane, p ? cols : 0, o);
+  }
+};
+
 // The convolutions of E channels a lane over the rows of a run: holds the inputs of the last TAPS rows
 // (TAPS 0: any number of taps, whose inputs are read again for every row).
-template <int E, int TAPS>
+template <int E, int TAPS, bool VEC>
 struct CdWalk {
   static constexpr int W = TAPS > 0 ? TAPS : 1;
   float w[W][E], x[W][E];
   int c0, cols;
-  __device__ __forceinline__ void start(const ChannelDeltaArgs& a, const float* tail, int Cc, int C_all, int row0, int r0,
-                                        int first, int count, int lane) {
+  __device__ __forceinline__ void weights(const float* conv_w, int taps, int first, int count, int lane) {
     c0 = first, cols = count;
     if (TAPS == 0) return;
 #pragma unroll
-    for (int j = 0; j < W; ++j) {
+    for (int e = 0; e < E; ++e) {
+      const int d = cd_at<E, VEC>(lane, e);
 #pragma unroll
-      for (int e = 0; e < E; ++e) {
-        const int d = lane + 32 * e;
-        w[j][e] = d < cols ? a.conv_w[(size_t)(c0 + d) * a.taps + a.taps - 1 - j] : 0.f;
-      }
-      if (j > 0) cd_inputs<E>(a, tail, Cc, C_all, row0, r0 - j, c0, lane, cols, x[j - 1]);
+      for (int j = 0; j < W; ++j) w[j][e] = d < cols ? conv_w[(size_t)(c0 + d) * W + W - 1 - j] : 0.f;
     }
   }
-  __device__ __forceinline__ void row(const ChannelDeltaArgs& a, const float* tail, int Cc, int C_all, int row0, int rr,
-                                      int lane, float (&y)[E]) {
+  __device__ __forceinline__ void before(const CdRows& in, int r0, int lane) {
+#pragma unroll
+    for (int j = 1; j < W; ++j) in.get<E, VEC>(r0 - j, c0, cols, lane, x[j - 1]);
+  }
+  __device__ __forceinline__ void row(const CdRows& in, const float* conv_w, int rr, int lane, float (&y)[E]) {
+#pragma unroll
+    for (int e = 0; e < E; ++e) y[e] = 0.f;
     if (TAPS == 0) {
+      for (int j = 0; j < in.taps; ++j) {
+        in.get<E, VEC>(rr - j, c0, cols, lane, x[0]);
 #pragma unroll
-      for (int e = 0; e < E; ++e) y[e] = 0.f;
-      for (int j = 0; j < a.taps; ++j) {
-        cd_inputs<E>(a, tail, Cc, C_all, row0, rr - j, c0, lane, cols, x[0]);
-#pragma unroll
-        for (int e = 0; e < E; ++e)
-          if (lane + 32 * e < cols)
-            y[e] = fmaf(a.conv_w[(size_t)(c0 + lane + 32 * e) * a.taps + a.taps - 1 - j], x[0][e], y[e]);
+        for (int e = 0; e < E; ++e) {
+          const int d = cd_at<E, VEC>(lane, e);
+          if (d < cols) y[e] = fmaf(conv_w[(size_t)(c0 + d) * in.taps + in.taps - 1 - j], x[0][e], y[e]);
+        }
       }
     } else {
 #pragma unroll
       for (int j = W - 1; j > 0; --j)
 #pragma unroll
         for (int e = 0; e < E; ++e) x[j][e] = x[j - 1][e];
-      cd_inputs<E>(a, tail, Cc, C_all, row0, rr, c0, lane, cols, x[0]);
+      cd_load<E, VEC>(in.proj + (size_t)(in.row0 + rr) * in.ld + c0, lane, cols, x[0]);
 #pragma unroll
-      for (int e = 0; e < E; ++e) {
-        y[e] = 0.f;
+      for (int e = 0; e < E; ++e)
 #pragma unroll
         for (int j = 0; j < W; ++j) y[e] = fmaf(w[j][e], x[j][e], y[e]);
-      }
     }
 #pragma unroll
     for (int e = 0; e < E; ++e) y[e] = silu_f(y[e]);
   }
-  // the sequence's new tail (after the rows; the owner of the channels in the first run only): entry s
-  // becomes the input at n - (taps - 1) + s rows, read before it or anything above it is written
-  __device__ __forceinline__ void keep(const ChannelDeltaArgs& a, float* tail, int Cc, int C_all, int row0, int n,
-                                       int lane) {
-    for (int s = 0; s < a.taps - 1; ++s) {
-      float v[E];
-      cd_inputs<E>(a, tail, Cc, C_all, row0, n - (a.taps - 1) + s, c0, lane, cols, v);
+  // The sequence's new tail, after the rows: by the owner of the channels in the first run.  When the run
+  // is all of the sequence's n_seq rows the last inputs are at hand; else entry s becomes the input at
+  // n_seq - (taps - 1) + s rows, read before it or anything above it is written.
+  __device__ __forceinline__ void keep(const CdRows& in, float* tail, bool whole, int n_seq, int lane) {
+    if (TAPS > 1 && whole) {
 #pragma unroll
-      for (int e = 0; e < E; ++e)
-        if (lane + 32 * e < cols) tail[(size_t)s * Cc + c0 + lane + 32 * e] = v[e];
+      for (int j = 0; j < W - 1; ++j) cd_store<E, VEC>(tail + (size_t)(W - 2 - j) * in.Cc + c0, lane, cols, x[j]);
+      return;
+    }
+    for (int s = 0; s < in.taps - 1; ++s) {
+      float v[E];
+      in.get<E, VEC>(n_seq - (in.taps - 1) + s, c0, cols, lane, v);
+      cd_store<E, VEC>(tail + (size_t)s * in.Cc + c0, lane, cols, v);
     }
   }
 };
 
-// A block takes a run of rows, a warp of it a kv head (its q and k), 32 E value channels, or what is
+// A block takes a run of rows, a warp of it a head of q or k, 32 E value channels, or what is
 // left of the projection (beta and the inner values).
-template <typename T, int E, int TAPS>
-__global__ void __launch_bounds__(32 * CD_WARPS) channel_delta_prepare_kernel(const ChannelDeltaArgs a, const int R) {
+template <int E, int TAPS, bool VEC>
+__global__ void __launch_bounds__(32 * CD_WARPS) channel_delta_prepare_kernel(const ChannelDeltaArgs a, const int R, const int low16) {
   pdl_launch_dependents_if_small();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int H = a.H, G = a.G, dk = a.dk, V = H * a.dv;
@@ -163,55 +195,52 @@ __global__ void __launch_bounds__(32 * CD_WARPS) channel_delta_prepare_kernel(co
   if (n <= 0) return;
   const int slot = a.slots[seq];
   float* tail = slot >= 0 && a.taps > 1 ? a.state + (size_t)slot * a.state_stride : nullptr;
+  const CdRows in = {a.proj, C_all, tail, Cc, a.taps, row0};
   const int v_units = (V + 32 * E - 1) / (32 * E);
   const float q_scale = 1.0f / sqrtf((float)dk);
-  pdl_wait();
-  for (int unit = blockIdx.y * CD_WARPS + warp; unit < G + v_units + 1; unit += gridDim.y * CD_WARPS) {
-    if (unit < G) {
-      CdWalk<E, TAPS> qw, kw;
-      qw.start(a, tail, Cc, C_all, row0, r0, unit * dk, dk, lane);
-      kw.start(a, tail, Cc, C_all, row0, r0, (G + unit) * dk, dk, lane);
+  // (a warp waits for the product where it first reads it: the convolutions' weights, no kernel's
+  // output, are fetched before; further waits return at once)
+  for (int unit = blockIdx.y * CD_WARPS + warp; unit < 2 * G + v_units + 1; unit += gridDim.y * CD_WARPS) {
+    if (unit < 2 * G + v_units) {
+      const bool head = unit < 2 * G;            // a q or k head, which becomes a unit vector
+      const int c0 = head ? unit * dk : 2 * G * dk + (unit - 2 * G) * 32 * E;
+      const int cols = head ? dk : min(32 * E, Cc - c0);
+      const float scale = unit < G ? q_scale : 1.0f;
+      CdWalk<E, TAPS, VEC> walk;
+      walk.weights(a.conv_w, a.taps, c0, cols, lane);
+      pdl_wait();
+      walk.before(in, r0, lane);
+#pragma unroll 4
       for (int i = 0; i < n; ++i) {
-        float q[E], k[E], sq = 0.f, sk = 0.f, kq = 0.f;
-        qw.row(a, tail, Cc, C_all, row0, r0 + i, lane, q);
-        kw.row(a, tail, Cc, C_all, row0, r0 + i, lane, k);
+        float v[E], ss = 0.f;
+        walk.row(in, a.conv_w, r0 + i, lane, v);
+        if (head) {
 #pragma unroll
-        for (int e = 0; e < E; ++e) sq = fmaf(q[e], q[e], sq), sk = fmaf(k[e], k[e], sk), kq = fmaf(q[e], k[e], kq);
-        sq = warp_sum(sq), sk = warp_sum(sk), kq = warp_sum(kq);
-        const float iq = 1.0f / sqrtf(sq + a.unit_eps) * q_scale, ik = 1.0f / sqrtf(sk + a.unit_eps);
-        float* out = a.prep + (size_t)(row0 + r0 + i) * P;
+          for (int e = 0; e < E; ++e) {
+            if (cd_at<E, VEC>(lane, e) >= dk) v[e] = 0.f;
+            ss = fmaf(v[e], v[e], ss);
+          }
+          ss = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps) * scale;
 #pragma unroll
-        for (int e = 0; e < E; ++e) {
-          const int d = lane + 32 * e;
-          if (d < dk) out[unit * dk + d] = q[e] * iq, out[(G + unit) * dk + d] = k[e] * ik;
+          for (int e = 0; e < E; ++e) v[e] *= ss;
         }
-        if (lane == 0) out[Cc + H + unit] = kq * iq * ik;
+        cd_store<E, VEC>(a.prep + (size_t)(row0 + r0 + i) * P + c0, lane, cols, v);
       }
-      if (tail && run == 0) {
-        qw.keep(a, tail, Cc, C_all, row0, n_seq, lane);
-        kw.keep(a, tail, Cc, C_all, row0, n_seq, lane);
-      }
-    } else if (unit < G + v_units) {
-      const int c0 = 2 * G * dk + (unit - G) * 32 * E, cols = min(32 * E, Cc - c0);
-      CdWalk<E, TAPS> vw;
-      vw.start(a, tail, Cc, C_all, row0, r0, c0, cols, lane);
-      for (int i = 0; i < n; ++i) {
-        float v[E];
-        vw.row(a, tail, Cc, C_all, row0, r0 + i, lane, v);
-#pragma unroll
-        for (int e = 0; e < E; ++e)
-          if (lane + 32 * e < cols) a.prep[(size_t)(row0 + r0 + i) * P + c0 + lane + 32 * e] = v[e];
-      }
-      if (tail && run == 0) vw.keep(a, tail, Cc, C_all, row0, n_seq, lane);
+      if (tail && run == 0) walk.keep(in, tail, n == n_seq, n_seq, lane);
     } else {
+      pdl_wait();
       for (int i = 0; i < n; ++i) {
         const size_t t = row0 + r0 + i;
         const float* rest = a.proj + t * C_all + Cc;
         for (int h = lane; h < H; h += 32) a.prep[t * P + Cc + h] = cd_sigmoid(rest[h]);
-        for (int j = lane; j < a.n_low; j += 32) ((T*)a.low)[t * a.n_low + j] = from_f32<T>(rest[H + j]);
+        for (int j = lane; j < a.n_low; j += 32) {
+          if (low16) ((bf16*)a.low)[t * a.n_low + j] = from_f32<bf16>(rest[H + j]);
+          else ((float*)a.low)[t * a.n_low + j] = rest[H + j];
+        }
       }
     }
   }
+  pdl_wait();              // (a warp without a unit waits, too: a finished kernel has waited for the one before)
   pdl_launch_dependents_if_large();
 }
 
@@ -251,10 +280,11 @@ __device__ __forceinline__ void cd_store_column(const float (&S)[R], float* sp, 
 }
 
 // One row of a column: S <- g S + k u with u = beta (v - (g S) . k); returns (g S) . q + u (k . q).
+// (The lanes of every column take k . q anew: one more value in the same round of shuffles.)
 template <int R>
 __device__ __forceinline__ float cd_row(float (&S)[R], const float* q, const float* k, const float* g, int l,
-                                        float v, float beta, float kq) {
-  float kk[R], d1 = 0.f, d2 = 0.f;
+                                        float v, float beta) {
+  float kk[R], d1 = 0.f, d2 = 0.f, kq = 0.f;
 #pragma unroll
   for (int i = 0; i < R / 4; ++i) {
     const float4 k4 = reinterpret_cast<const float4*>(k)[i * CD_LANES + l];
@@ -266,11 +296,13 @@ __device__ __forceinline__ float cd_row(float (&S)[R], const float* q, const flo
     d1 = fmaf(S[4 * i + 2], k4.z, d1), d1 = fmaf(S[4 * i + 3], k4.w, d1);
     d2 = fmaf(S[4 * i], q4.x, d2), d2 = fmaf(S[4 * i + 1], q4.y, d2);
     d2 = fmaf(S[4 * i + 2], q4.z, d2), d2 = fmaf(S[4 * i + 3], q4.w, d2);
+    kq = fmaf(k4.x, q4.x, kq), kq = fmaf(k4.y, q4.y, kq), kq = fmaf(k4.z, q4.z, kq), kq = fmaf(k4.w, q4.w, kq);
   }
 #pragma unroll
   for (int m = 1; m < CD_LANES; m <<= 1) {
     d1 += __shfl_xor_sync(0xffffffffu, d1, m);
     d2 += __shfl_xor_sync(0xffffffffu, d2, m);
+    kq += __shfl_xor_sync(0xffffffffu, kq, m);
   }
   const float u = beta * (v - d1);
 #pragma unroll
@@ -307,7 +339,7 @@ __global__ void __launch_bounds__(256) channel_delta_step_kernel(const ChannelDe
     ks[d] = in ? p[(G + kvh) * dk + d] : 0.f;
     gs[d] = in ? expf(cd_log_decay(z[h * dk + d], a.dt_bias[h * dk + d], rate)) : 0.f;
   }
-  const float beta = p[Cc + h], kq = p[Cc + H + kvh];
+  const float beta = p[Cc + h];
   __syncthreads();
   const int l = tid % CD_LANES;
   float ss = 0.f;
@@ -317,8 +349,8 @@ __global__ void __launch_bounds__(256) channel_delta_step_kernel(const ChannelDe
     cd_load_column<R>(Sa, head && ca < dv ? head + (size_t)ca * dk : nullptr, dk, l, wide);
     cd_load_column<R>(Sb, head && cb < dv ? head + (size_t)cb * dk : nullptr, dk, l, wide);
     const float va = ca < dv ? p[2 * G * dk + h * dv + ca] : 0.f, vb = cb < dv ? p[2 * G * dk + h * dv + cb] : 0.f;
-    const float oa = cd_row<R>(Sa, qs, ks, gs, l, va, beta, kq);
-    const float ob = cd_row<R>(Sb, qs, ks, gs, l, vb, beta, kq);
+    const float oa = cd_row<R>(Sa, qs, ks, gs, l, va, beta);
+    const float ob = cd_row<R>(Sb, qs, ks, gs, l, vb, beta);
     if (head && ca < dv) cd_store_column<R>(Sa, head + (size_t)ca * dk, dk, l, wide);
     if (head && cb < dv) cd_store_column<R>(Sb, head + (size_t)cb * dk, dk, l, wide);
     if (l == 0 && ca < dv) os[ca] = oa, ss = fmaf(oa, oa, ss);
@@ -333,15 +365,14 @@ __global__ void __launch_bounds__(256) channel_delta_step_kernel(const ChannelDe
 
 template <int R>
 __global__ void __launch_bounds__(CD_LANES * CD_COLS) channel_delta_scan_kernel(const ChannelDeltaArgs a) {
-  extern __shared__ __align__(16) float sm[];     // q | k | g [CD_TT, DKP each] | v [CD_TT, CD_COLS] | beta, kq [CD_TT]
+  extern __shared__ __align__(16) float sm[];     // q | k | g [CD_TT, DKP each] | v [CD_TT, CD_COLS] | beta [CD_TT]
   constexpr int DKP = CD_LANES * R;
   pdl_launch_dependents_if_small();
   const int seq = blockIdx.z, h = blockIdx.y, tid = threadIdx.x;
   const int col0 = blockIdx.x * CD_COLS, col = col0 + tid / CD_LANES, l = tid % CD_LANES;
   const int H = a.H, G = a.G, dk = a.dk, dv = a.dv, kvh = h / (H / G);
   const int Cc = cd_channels(a);
-  float *qs = sm, *ks = qs + CD_TT * DKP, *gs = ks + CD_TT * DKP, *vs = gs + CD_TT * DKP, *bs = vs + CD_TT * CD_COLS,
-        *kqs = bs + CD_TT;
+  float *qs = sm, *ks = qs + CD_TT * DKP, *gs = ks + CD_TT * DKP, *vs = gs + CD_TT * DKP, *bs = vs + CD_TT * CD_COLS;
   const float rate = expf(a.a_log[h]);
   pdl_wait();
   const int row0 = a.cu_q[seq], n = a.cu_q[seq + 1] - row0;
@@ -369,14 +400,11 @@ __global__ void __launch_bounds__(CD_LANES * CD_COLS) channel_delta_scan_kernel(
       const int c = col0 + i % CD_COLS;
       vs[i] = c < dv ? a.prep[(size_t)(row0 + t0 + i / CD_COLS) * a.prep_stride + 2 * G * dk + h * dv + c] : 0.f;
     }
-    if (tid < nt) {
-      const float* p = a.prep + (size_t)(row0 + t0 + tid) * a.prep_stride + Cc;
-      bs[tid] = p[h], kqs[tid] = p[H + kvh];
-    }
+    if (tid < nt) bs[tid] = a.prep[(size_t)(row0 + t0 + tid) * a.prep_stride + Cc + h];
     __syncthreads();
     for (int tt = 0; tt < nt; ++tt) {
       const float o = cd_row<R>(S, qs + tt * DKP, ks + tt * DKP, gs + tt * DKP, l, vs[tt * CD_COLS + tid / CD_LANES],
-                                bs[tt], kqs[tt]);
+                                bs[tt]);
       if (l == 0 && active) a.o[((size_t)(row0 + t0 + tt) * H + h) * dv + col] = o;
     }
   }
@@ -411,34 +439,39 @@ static int cd_check(const ChannelDeltaArgs& a) {
       a.n_low <= 0 || !a.proj || !a.state || !a.prep || !a.low || !a.conv_w || !a.token_seq || !a.cu_q || !a.slots)
     return GB_ERR_BAD_ARG;
   if (a.dk > 32 * CD_LANES || a.n_seqs > 65535 || a.H > 65535) return GB_ERR_UNSUPPORTED;
-  if (a.prep_stride != (2 * a.G * a.dk + a.H * a.dv + a.H + a.G + 3) / 4 * 4) return GB_ERR_BAD_ARG;
+  if (a.prep_stride != (2 * a.G * a.dk + a.H * a.dv + a.H + 3) / 4 * 4) return GB_ERR_BAD_ARG;
   return 0;
 }
 
-template <typename T, int E, int TAPS>
-static int prepare_taps(const ChannelDeltaArgs& a, cudaStream_t s) {
-  const int R = a.taps - 1 > CD_RUN ? a.taps - 1 : CD_RUN;
+template <int E, int TAPS>
+static int prepare_taps(const ChannelDeltaArgs& a, int low16, cudaStream_t s) {
+  int R = a.n_tokens >= 1024 ? 2 * CD_RUN : CD_RUN;      // (long runs read fewer rows twice)
+  if (a.taps - 1 > R) R = a.taps - 1;
   const int blocks = a.max_rows == 1 ? a.n_seqs : a.n_tokens / R + a.n_seqs;
-  const int units = a.G + (a.H * a.dv + 32 * E - 1) / (32 * E) + 1;
-  return gb_launch(channel_delta_prepare_kernel<T, E, TAPS>, dim3(blocks, (units + CD_WARPS - 1) / CD_WARPS),
-                   dim3(32 * CD_WARPS), 0, s, a, R);
+  const int units = 2 * a.G + (a.H * a.dv + 32 * E - 1) / (32 * E) + 1;
+  const dim3 grid(blocks, (units + CD_WARPS - 1) / CD_WARPS), block(32 * CD_WARPS);
+  const int Cc = 2 * a.G * a.dk + a.H * a.dv;
+  const bool vec = E <= 4 && a.dk % E == 0 && (a.H * a.dv) % E == 0 && (Cc + a.H + a.n_low) % E == 0 &&
+                   a.state_stride % E == 0 && (((uintptr_t)a.proj | (uintptr_t)a.state | (uintptr_t)a.prep) & 15) == 0;
+  if constexpr (E <= 4)
+    if (vec) return gb_launch(channel_delta_prepare_kernel<E, TAPS, true>, grid, block, 0, s, a, R, low16);
+  return gb_launch(channel_delta_prepare_kernel<E, TAPS, false>, grid, block, 0, s, a, R, low16);
 }
 
-template <typename T, int E>
-static int prepare_size(const ChannelDeltaArgs& a, cudaStream_t s) {
+template <int E>
+static int prepare_size(const ChannelDeltaArgs& a, int low16, cudaStream_t s) {
   switch (a.taps) {
-    case 2: return prepare_taps<T, E, 2>(a, s);
-    case 3: return prepare_taps<T, E, 3>(a, s);
-    case 4: return prepare_taps<T, E, 4>(a, s);
-    default: return prepare_taps<T, E, 0>(a, s);
+    case 2: return prepare_taps<E, 2>(a, low16, s);
+    case 3: return prepare_taps<E, 3>(a, low16, s);
+    case 4: return prepare_taps<E, 4>(a, low16, s);
+    default: return prepare_taps<E, 0>(a, low16, s);
   }
 }
 
-template <typename T>
-static int prepare(const ChannelDeltaArgs& a, cudaStream_t s) {
+static int prepare(const ChannelDeltaArgs& a, int low16, cudaStream_t s) {
   const int e = cd_check(a);
   if (e || a.n_tokens == 0) return e;
-  return a.dk <= 64 ? prepare_size<T, 2>(a, s) : a.dk <= 128 ? prepare_size<T, 4>(a, s) : prepare_size<T, 8>(a, s);
+  return a.dk <= 128 ? prepare_size<4>(a, low16, s) : prepare_size<8>(a, low16, s);
 }
 
 template <typename T, int R>
@@ -453,7 +486,7 @@ static int run_rows(const ChannelDeltaArgs& a, cudaStream_t s) {
   if (cc_takes(a)) {
     e = cc_run(a, s);
   } else {
-    const size_t smem = (CD_TT * (3 * DKP + CD_COLS + 2)) * sizeof(float);
+    const size_t smem = (CD_TT * (3 * DKP + CD_COLS + 1)) * sizeof(float);
     static bool configured = false;
     if (smem > 48 * 1024 && !configured) {
       cudaError_t ce = cudaFuncSetAttribute(channel_delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -484,7 +517,7 @@ static int run(const ChannelDeltaArgs& a, cudaStream_t s) {
   return run_rows<T, 32>(a, s);
 }
 
-GB_EXPORT int gb_channel_delta_prepare_f32(const ChannelDeltaArgs* a, cudaStream_t s) { return prepare<float>(*a, s); }
-GB_EXPORT int gb_channel_delta_prepare_bf16(const ChannelDeltaArgs* a, cudaStream_t s) { return prepare<bf16>(*a, s); }
+GB_EXPORT int gb_channel_delta_prepare_f32(const ChannelDeltaArgs* a, cudaStream_t s) { return prepare(*a, 0, s); }
+GB_EXPORT int gb_channel_delta_prepare_bf16(const ChannelDeltaArgs* a, cudaStream_t s) { return prepare(*a, 1, s); }
 GB_EXPORT int gb_channel_delta_run_f32(const ChannelDeltaArgs* a, cudaStream_t s) { return run<float>(*a, s); }
 GB_EXPORT int gb_channel_delta_run_bf16(const ChannelDeltaArgs* a, cudaStream_t s) { return run<bf16>(*a, s); }

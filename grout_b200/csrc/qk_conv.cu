@@ -95,7 +95,6 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
     sn[i] = s * a.rot_scale, cs[i] = c * a.rot_scale;
   }
   __syncthreads();
-  pdl_wait();
   const int D = a.D, Ds = a.Ds, nqk = a.nq + a.nkv;
   const int Cc = nqk * D;                                // channels with a bias, a convolution, a kept tail
   const size_t width = (size_t)Cc + (a.v_from_k ? 0 : (size_t)a.nkv * a.Dv);
@@ -115,8 +114,11 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
     }
   };
   for (int head = blockIdx.y * QC_WARPS + warp; head < n_heads; head += gridDim.y * QC_WARPS) {
+    // (a warp waits for the product where it first reads it: what is no kernel's output, the weights,
+    // is fetched before; further waits return at once)
     if (head >= nqk) {                                   // a value head of its own: stored as it is
       const int g = head - nqk;
+      pdl_wait();
       for (int i = 0; i < n && table; ++i) {
         const int pos = a.token_pos[row0 + r0 + i];
         T* dst = (T*)a.v_pages + paged_row(table, pos, g, a.nkv, a.page, Ds);
@@ -154,8 +156,14 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
 #pragma unroll
           for (int e = 0; e < V; ++e)
             w[j][s][e] = TAPS > 0 && a.conv_w ? a.conv_w[(size_t)(ch[s] + e) * taps + taps - 1 - j] : 1.f;
-          if (TAPS > 0 && j > 0) input(r0 - j, ch[s], b[s], x[j - 1][s]);
         }
+      pdl_wait();
+      if (TAPS > 0) {
+#pragma unroll
+        for (int j = 1; j < W; ++j)
+#pragma unroll
+          for (int s = 0; s < 2; ++s) input(r0 - j, ch[s], b[s], x[j - 1][s]);
+      }
 #pragma unroll 4
       for (int i = 0; i < n; ++i) {
         float c[2][V];
@@ -168,9 +176,10 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
               for (int e = 0; e < V; ++e) x[j][s][e] = x[j - 1][s][e];
 #pragma unroll
           for (int s = 0; s < 2; ++s) {
-            input(r0 + i, ch[s], b[s], x[0][s]);
+            qc_sum<V>(a, (size_t)(row0 + r0 + i) * width + ch[s], x[0][s]);
 #pragma unroll
             for (int e = 0; e < V; ++e) {
+              x[0][s][e] += b[s][e];
               c[s][e] = w[0][s][e] * x[0][s][e];
 #pragma unroll
               for (int j = 1; j < W; ++j) c[s][e] = fmaf(w[j][s][e], x[j][s][e], c[s][e]);
@@ -215,7 +224,16 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
           if (two) qc_store<T, V>(dst + e1, c[1]);
         }
       }
-      if (tail && run == 0) {        // entry s: the input at n_seq - (taps - 1) + s; an entry that moves down
+      if (TAPS > 1 && tail && n == n_seq) {      // all of the sequence's rows: the last inputs are at hand
+#pragma unroll
+        for (int j = 0; j < W - 1; ++j)
+#pragma unroll
+          for (int k = 0; k < 2; ++k)
+            if (k == 0 || two) {
+#pragma unroll
+              for (int e = 0; e < V; ++e) tail[(size_t)(taps - 2 - j) * Cc + ch[k] + e] = x[j][k][e];
+            }
+      } else if (tail && run == 0) { // entry s: the input at n_seq - (taps - 1) + s; an entry that moves down
                                      // is read before it is overwritten
         for (int s = 0; s < taps - 1; ++s) {
           float t[2][V];
@@ -230,6 +248,7 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
         }
       }
     }
+    pdl_wait();
     for (int i = 0; i < n && Ds > D; ++i) {              // a narrower head is filled up with zeros
       T* dst = nullptr;
       T* dst2 = nullptr;
@@ -282,7 +301,8 @@ static int launch(const QkConvArgs& in, cudaStream_t s) {
     return GB_ERR_BAD_ARG;
   if (a.T == 0) return 0;
   if (!a.rot_dim) a.inv_freq = nullptr;
-  a.run = a.taps - 1 > QC_RUN ? a.taps - 1 : QC_RUN;
+  a.run = a.T >= 1024 ? 2 * QC_RUN : QC_RUN;             // (long runs read fewer rows twice)
+  if (a.taps - 1 > a.run) a.run = a.taps - 1;
   switch (a.taps) {
     case 1: return launch_taps<T, 1>(a, s);
     case 2: return launch_taps<T, 2>(a, s);

@@ -1782,7 +1782,7 @@ def _channel_delta_args(proj, state, conv_w, *, H, G, dk, dv, taps, n_low, token
     a.proj, a.conv_w, a.state, a.state_stride = proj.data_ptr(), conv_w.data_ptr(), state.data_ptr(), state.stride(0)
     a.token_seq, a.cu_q, a.slots = token_seq.data_ptr(), cu_q.data_ptr(), slots.data_ptr()
     a.n_tokens, a.n_seqs, a.H, a.G, a.dk, a.dv, a.taps, a.n_low = T, slots.shape[0], H, G, dk, dv, taps, n_low
-    a.prep_stride = (Cc + H + G + 3) // 4 * 4
+    a.prep_stride = (Cc + H + 3) // 4 * 4
     return a
 
 
@@ -1793,7 +1793,7 @@ def channel_delta_prepare(proj: torch.Tensor, state: torch.Tensor, conv_w: torch
     """What comes in front of the recurrence of the delta rule with a decay per channel.  ``proj``
     [T, C] 32-bit: the columns q [G dk] | k [G dk] | v [H dv] | beta logits [H] | the thin
     products' inner values [n_low].  Returns (prep, low): ``prep`` [T, P] 32-bit holds what
-    ``channel_delta_run`` takes (unit q and k and v behind their convolutions, beta, k . q), ``low``
+    ``channel_delta_run`` takes (unit q and k and v behind their convolutions, beta), ``low``
     [T, n_low] the inner values in ``dtype``.  Of ``state`` the convolutions' tail is read and
     replaced.  ``max_rows``: the most rows any sequence brings, when the host knows it."""
     a = _channel_delta_args(proj, state, conv_w, H=H, G=G, dk=dk, dv=dv, taps=taps, n_low=n_low,

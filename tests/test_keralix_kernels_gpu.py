@@ -346,7 +346,7 @@ def test_a_far_key_among_hundreds_is_found(dtype):
     cache = cache_for(part, dtype)
     for cuts in ([T], [T - 1, 1], [100, 299, 1]):
         got, = feed(part, cache, [x], cuts_of(cuts))
-        close(got, want, dtype, f"cuts {cuts}")
+        close(got, want, dtype, f"cuts {cuts}", bar=None if dtype == torch.float32 else 0.05)   # (sharp scores)
         apart(got[-1:], want[-1:], gone[-1:], slice(None), "the far key")
 
 
