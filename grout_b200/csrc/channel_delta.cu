@@ -69,6 +69,7 @@ __device__ __forceinline__ float cd_log_decay(float z, float bias, float rate) {
 
 #define CD_RUN 8         // rows of a run (never fewer than taps - 1)
 #define CD_WARPS 8
+#define CD_AHEAD 4       // rows requested at a time
 
 // A lane's E channels among the `cols` from c0 on: E neighbours (VEC, which needs every piece on its
 // boundary and whole), or every 32nd.
@@ -137,7 +138,9 @@ struct CdWalk {
 #pragma unroll
     for (int j = 1; j < W; ++j) in.get<E, VEC>(r0 - j, c0, cols, lane, x[j - 1]);
   }
-  __device__ __forceinline__ void row(const CdRows& in, const float* conv_w, int rr, int lane, float (&y)[E]) {
+  // row rr, whose own input `fresh` is
+  __device__ __forceinline__ void row(const CdRows& in, const float* conv_w, int rr, int lane, const float (&fresh)[E],
+                                      float (&y)[E]) {
 #pragma unroll
     for (int e = 0; e < E; ++e) y[e] = 0.f;
     if (TAPS == 0) {
@@ -154,7 +157,8 @@ struct CdWalk {
       for (int j = W - 1; j > 0; --j)
 #pragma unroll
         for (int e = 0; e < E; ++e) x[j][e] = x[j - 1][e];
-      cd_load<E, VEC>(in.proj + (size_t)(in.row0 + rr) * in.ld + c0, lane, cols, x[0]);
+#pragma unroll
+      for (int e = 0; e < E; ++e) x[0][e] = fresh[e];
 #pragma unroll
       for (int e = 0; e < E; ++e)
 #pragma unroll
@@ -210,21 +214,28 @@ __global__ void __launch_bounds__(32 * CD_WARPS) channel_delta_prepare_kernel(co
       walk.weights(a.conv_w, a.taps, c0, cols, lane);
       pdl_wait();
       walk.before(in, r0, lane);
-#pragma unroll 4
-      for (int i = 0; i < n; ++i) {
-        float v[E], ss = 0.f;
-        walk.row(in, a.conv_w, r0 + i, lane, v);
-        if (head) {
+      for (int i0 = 0; i0 < n; i0 += CD_AHEAD) {   // several rows are requested before the first is worked on
+        float fresh[CD_AHEAD][E];
 #pragma unroll
-          for (int e = 0; e < E; ++e) {
-            if (cd_at<E, VEC>(lane, e) >= dk) v[e] = 0.f;
-            ss = fmaf(v[e], v[e], ss);
+        for (int u = 0; u < CD_AHEAD; ++u)
+          cd_load<E, VEC>(a.proj + (size_t)(row0 + r0 + min(i0 + u, n - 1)) * C_all + c0, lane, cols, fresh[u]);
+#pragma unroll
+        for (int u = 0; u < CD_AHEAD; ++u) {
+          if (i0 + u >= n) break;
+          float v[E], ss = 0.f;
+          walk.row(in, a.conv_w, r0 + i0 + u, lane, fresh[u], v);
+          if (head) {
+#pragma unroll
+            for (int e = 0; e < E; ++e) {
+              if (cd_at<E, VEC>(lane, e) >= dk) v[e] = 0.f;
+              ss = fmaf(v[e], v[e], ss);
+            }
+            ss = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps) * scale;
+#pragma unroll
+            for (int e = 0; e < E; ++e) v[e] *= ss;
           }
-          ss = 1.0f / sqrtf(warp_sum(ss) + a.unit_eps) * scale;
-#pragma unroll
-          for (int e = 0; e < E; ++e) v[e] *= ss;
+          cd_store<E, VEC>(a.prep + (size_t)(row0 + r0 + i0 + u) * P + c0, lane, cols, v);
         }
-        cd_store<E, VEC>(a.prep + (size_t)(row0 + r0 + i) * P + c0, lane, cols, v);
       }
       if (tail && run == 0) walk.keep(in, tail, n == n_seq, n_seq, lane);
     } else {

@@ -24,6 +24,7 @@
 #define CC_COLS 32       // columns of S a chain block owns
 #define CC_MIN 64        // a step goes chunk by chunk when a sequence brings this many rows
 #define CC_MAX_DK 128
+#define CC_LOG2E 1.4426950408889634f   // the kernels keep logarithms to base 2: one operation less per power
 
 // A chunk's record for one head: WQ [dk][64] (per channel the 32 rows of W, then the 32 of
 // e^L q) | Kd [32][dk] (e^{L_n - L} k) | gC [dk] (e^{L_n}) | B [32][32] | U0 [32][dv]
@@ -79,13 +80,14 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
   const int first = a.cu_q[seq], n_seq = a.cu_q[seq + 1] - first;
   const int n = min(CC_ROWS, n_seq - z * CC_ROWS), row0 = first + z * CC_ROWS;
   if (n <= 0) return;
+#pragma unroll 4
   for (int i = tid; i < CC_ROWS * DKP; i += 256) {
     const int t = i / DKP, d = i % DKP;
     float q = 0.f, k = 0.f, lg = 0.f;
     if (t < n && d < dk) {
       const float* p = a.prep + (size_t)(row0 + t) * a.prep_stride;
       q = p[kvh * dk + d], k = p[(G + kvh) * dk + d];
-      lg = cd_log_decay(a.wide[(size_t)(row0 + t) * H * (dk + dv) + h * dk + d], a.dt_bias[h * dk + d], rate);
+      lg = CC_LOG2E * cd_log_decay(a.wide[(size_t)(row0 + t) * H * (dk + dv) + h * dk + d], a.dt_bias[h * dk + d], rate);
     }
     Qs[t * LD + d] = q, Ks[t * LD + d] = k, Ls[t * LD + d] = lg;
   }
@@ -114,14 +116,14 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
 #pragma unroll 4
     for (int t = CC_ROWS - 1; t >= 0; --t) {
       const float k = Ks[t * LD + d], lg = Ls[t * LD + d];
-      if (d < dk) kd[t * dk + d] = k * expf(s);
+      if (d < dk) kd[t * dk + d] = k * exp2f(s);
       if (t < CC_HALF) {
-        Kr[t * LD + d] = k * expf(in_half);
+        Kr[t * LD + d] = k * exp2f(in_half);
         in_half += lg;
       }
       s += lg;
     }
-    if (d < dk) gc[d] = expf(s);
+    if (d < dk) gc[d] = exp2f(s);
   }
   __syncthreads();
   // A and B: a warp takes rows warp, warp + 8, ...; its lanes share the channels
@@ -140,7 +142,7 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
         cc_read<E>(Ls + (base + j) * LD + lane * E, li);
 #pragma unroll
         for (int x = 0; x < E; ++x) {
-          const float w = ki[x] * expf(since[x]);
+          const float w = ki[x] * exp2f(since[x]);
           since[x] += li[x];
           part[j] = fmaf(kt[x], w, part[j]);
           part[CC_HALF + j] = fmaf(qt[x], w, part[CC_HALF + j]);
@@ -155,7 +157,7 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
       cc_read<E>(Fs + t * LD + lane * E, li);
 #pragma unroll
       for (int x = 0; x < E; ++x) {
-        const float w = expf(li[x]);
+        const float w = exp2f(li[x]);
         kt[x] *= w, qt[x] *= w;
       }
 #pragma unroll
@@ -182,7 +184,7 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
 #pragma unroll
     for (int t = 0; t < CC_ROWS; ++t) {
       if (d < 0) x[t] = t < n ? a.prep[(size_t)(row0 + t) * a.prep_stride + 2 * G * dk + h * dv + c] : 0.f;
-      else x[t] = Ks[t * LD + d] * expf(Fs[t * LD + d] + (t < CC_HALF ? 0.f : Fs[(CC_HALF - 1) * LD + d]));
+      else x[t] = Ks[t * LD + d] * exp2f(Fs[t * LD + d] + (t < CC_HALF ? 0.f : Fs[(CC_HALF - 1) * LD + d]));
     }
 #pragma unroll
     for (int t = 0; t < CC_ROWS; ++t) {
@@ -212,7 +214,7 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
     const float before = t < CC_HALF ? 0.f : Fs[(CC_HALF - 1) * LD + d];
     float v[4];
 #pragma unroll
-    for (int x = 0; x < 4; ++x) v[x] = Qs[(t + x) * LD + d] * expf(Fs[(t + x) * LD + d] + before);
+    for (int x = 0; x < 4; ++x) v[x] = Qs[(t + x) * LD + d] * exp2f(Fs[(t + x) * LD + d] + before);
     *reinterpret_cast<float4*>(wq + (size_t)d * 64 + CC_ROWS + t) = make_float4(v[0], v[1], v[2], v[3]);
   }
   for (int i = tid; i < CC_ROWS * CC_ROWS; i += 256) bm[i] = Bs[i];
@@ -264,10 +266,10 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
     S[k * CC_COLS + c] = sp && col0 + c < dv ? sp[(size_t)(col0 + c) * dk + k] : 0.f;
   }
   // the products' tiles: 4 rows by 4 columns of WQ^T S a thread, half the channels each; 4 by 4 of
-  // the state; 2 by 2 of the read-outs
+  // the state; 1 by 4 of the read-outs
   const int half = tid >> 7, tr = (tid & 127) / 8 * 4, tc = (tid & 7) * 4;
   const int k_lo = half ? dk / 2 : 0, k_hi = half ? dk : dk / 2;
-  const int sk = tid / 8 * 4, orow = tid / 16 * 2, ocol = (tid % 16) * 2;
+  const int sk = tid / 8 * 4, orow = tid / 8;
   for (int z = 0; z < chunks; ++z) {
     if (z + 1 < chunks) { stage_in(z + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
     __syncthreads();
@@ -281,7 +283,7 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
     for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-#pragma unroll 4
+#pragma unroll 8
     for (int k = k_lo; k < k_hi; ++k) {
       const float4 x = *reinterpret_cast<const float4*>(wq + k * 64 + tr);
       const float4 y = *reinterpret_cast<const float4*>(S + k * CC_COLS + tc);
@@ -321,7 +323,7 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
         const float g = gc[sk + i];
         s[i][0] = g * x.x, s[i][1] = g * x.y, s[i][2] = g * x.z, s[i][3] = g * x.w;
       }
-#pragma unroll 4
+#pragma unroll 8
       for (int t = 0; t < CC_ROWS; ++t) {
         const float4 x = *reinterpret_cast<const float4*>(kd + t * dk + sk);
         const float4 y = *reinterpret_cast<const float4*>(U + t * CC_COLS + tc);
@@ -335,22 +337,22 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
       for (int i = 0; i < 4; ++i)
         *reinterpret_cast<float4*>(S + (sk + i) * CC_COLS + tc) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
     }
-    float o[2][2];                               // the read-outs: e^{L} q S_0 + B U
+    {                                            // the read-outs: e^{L} q S_0 + B U, four columns of a row a thread
+      float4 o = *reinterpret_cast<const float4*>(P + (CC_ROWS + orow) * CC_COLS + tc);
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
+      for (int t = 0; t < CC_ROWS; t += 4) {     // (B is zero behind its diagonal)
+        const float4 w = *reinterpret_cast<const float4*>(bm + orow * CC_ROWS + t);
+        const float wv[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
-      for (int j = 0; j < 2; ++j) o[i][j] = P[(CC_ROWS + orow + i) * CC_COLS + ocol + j];
-    for (int t = 0; t <= orow + 1; ++t) {        // (B is zero behind its diagonal)
-      const float2 u = *reinterpret_cast<const float2*>(U + t * CC_COLS + ocol);
-      const float b0 = bm[orow * CC_ROWS + t], b1 = bm[(orow + 1) * CC_ROWS + t];
-      o[0][0] = fmaf(b0, u.x, o[0][0]), o[0][1] = fmaf(b0, u.y, o[0][1]);
-      o[1][0] = fmaf(b1, u.x, o[1][0]), o[1][1] = fmaf(b1, u.y, o[1][1]);
-    }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int r = z * CC_ROWS + orow + i;
-      if (r < n_seq && col0 + ocol < dv)         // (dv is a multiple of four)
-        *reinterpret_cast<float2*>(a.o + ((size_t)(first + r) * H + h) * dv + col0 + ocol) = make_float2(o[i][0], o[i][1]);
+        for (int e = 0; e < 4; ++e) {
+          const float4 u = *reinterpret_cast<const float4*>(U + (t + e) * CC_COLS + tc);
+          o.x = fmaf(wv[e], u.x, o.x), o.y = fmaf(wv[e], u.y, o.y);
+          o.z = fmaf(wv[e], u.z, o.z), o.w = fmaf(wv[e], u.w, o.w);
+        }
+      }
+      const int r = z * CC_ROWS + orow;
+      if (r < n_seq && col0 + tc < dv)           // (dv is a multiple of four)
+        *reinterpret_cast<float4*>(a.o + ((size_t)(first + r) * H + h) * dv + col0 + tc) = o;
     }
     __syncthreads();                             // S is whole, the stage and P may be overwritten
   }

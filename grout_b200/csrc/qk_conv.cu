@@ -38,6 +38,7 @@ struct QkConvArgs {
 
 #define QC_RUN 8
 #define QC_WARPS 8
+#define QC_AHEAD 4          // rows requested at a time
 #define QC_TAPS 4           // taps whose inputs a thread keeps in registers; with more it reads them again
 
 // V neighbouring values of the projection from `at` on, the partial sums added in order.
@@ -164,8 +165,19 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
 #pragma unroll
           for (int s = 0; s < 2; ++s) input(r0 - j, ch[s], b[s], x[j - 1][s]);
       }
-#pragma unroll 4
-      for (int i = 0; i < n; ++i) {
+      for (int i0 = 0; i0 < n; i0 += QC_AHEAD) {   // several rows are requested before the first is worked on
+       float fresh[QC_AHEAD][2][V];
+       if (TAPS > 0) {
+#pragma unroll
+         for (int u = 0; u < QC_AHEAD; ++u)
+#pragma unroll
+           for (int s = 0; s < 2; ++s)
+             if (u == 0 || i0 + u < n) qc_sum<V>(a, (size_t)(row0 + r0 + i0 + u) * width + ch[s], fresh[u][s]);
+       }
+#pragma unroll
+       for (int u = 0; u < QC_AHEAD; ++u) {
+        const int i = i0 + u;
+        if (i >= n) break;
         float c[2][V];
         if (TAPS > 0) {
 #pragma unroll
@@ -176,10 +188,9 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
               for (int e = 0; e < V; ++e) x[j][s][e] = x[j - 1][s][e];
 #pragma unroll
           for (int s = 0; s < 2; ++s) {
-            qc_sum<V>(a, (size_t)(row0 + r0 + i) * width + ch[s], x[0][s]);
 #pragma unroll
             for (int e = 0; e < V; ++e) {
-              x[0][s][e] += b[s][e];
+              x[0][s][e] = fresh[u][s][e] + b[s][e];
               c[s][e] = w[0][s][e] * x[0][s][e];
 #pragma unroll
               for (int j = 1; j < W; ++j) c[s][e] = fmaf(w[j][s][e], x[j][s][e], c[s][e]);
@@ -223,6 +234,7 @@ __global__ void __launch_bounds__(32 * QC_WARPS) qk_conv_kernel(const QkConvArgs
           qc_store<T, V>(dst + e0, c[0]);
           if (two) qc_store<T, V>(dst + e1, c[1]);
         }
+       }
       }
       if (TAPS > 1 && tail && n == n_seq) {      // all of the sequence's rows: the last inputs are at hand
 #pragma unroll
