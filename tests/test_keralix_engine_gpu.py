@@ -84,13 +84,13 @@ KER = {
         _layer("A", _att(4, 4, 64, 2, 0.2, 130, 8.0, (500.0, 32))),
         _layer("L", _lat(2, 64, 32, 96, 128, 0.1), 160)]),
     # odd sizes, no window, no cap, no rotation, one tap, five streams
-    "V": dict(architecture="Keralix", vocab=160, width=96, streams=5, norm={"eps": 1e-4}, embedding={"scale": 0.5}, layers=[
-        _layer("L", _lat(3, 20, 12, 33, 150, 0.35), 40),
-        _layer("A", _att(6, 2, 20, 5, 0.5, None, 5.0, (1e3, 20)), 88),
+    "V": dict(architecture="Keralix", vocab=160, width=96, streams=5, norm={"eps": 1e-4}, embedding={"scale": 2.0}, layers=[
+        _layer("L", _lat(3, 20, 12, 33, 150, 0.2), 40),
+        _layer("A", _att(6, 2, 20, 5, 0.15, None, 5.0, (1e3, 20)), 88),
         _layer("D", _delta(3, 3, 20, 10, 1), 24),
-        _layer("A", _att(3, 1, 24, 1, 0.5, 65, None, None)),
+        _layer("A", _att(3, 1, 24, 1, 0.15, 65, None, None)),
         _layer("D", _delta(2, 1, 33, 36, 9)),
-        _layer("A", _att(5, 5, 17, 12, 0.6, 2, 12.0, (1e5, 6)), 16)]),
+        _layer("A", _att(5, 5, 17, 12, 0.13, 2, 12.0, (1e5, 6)), 16)]),
     # nothing a multiple of eight; one stream
     "W": dict(architecture="Keralix", vocab=173, width=100, streams=1, norm={"eps": 2e-5}, embedding={"scale": 10.0}, layers=[
         _layer("D", _delta(5, 5, 12, 20, 3), 52),
