@@ -41,6 +41,7 @@ struct DecodeArgs {
   ScoreCap cap;            // the score cap (off when cap_log2 == 0)
   int keep_first;          // with a window: a sequence's first keep_first keys stay visible behind it
   int chunk;               // > 0: a query sees the keys of its own chunk of positions only
+  int one_kv;              // the pages hold one kv head, which all of the nkv groups of query heads read
 };
 
 template <int DT>
@@ -110,7 +111,7 @@ __global__ void __launch_bounds__(DC_THREADS) attn_decode_kernel(const DecodeArg
         const int pg = tpp_shift >= 0 ? tile >> tpp_shift : tile / tiles_per_page;
         const int in_page = tile - pg * tiles_per_page;
         const int page = table[pg];
-        const size_t base = (((size_t)page * a.nkv + kvh) * a.page + in_page * DC_BN) * D;
+        const size_t base = ((a.one_kv ? (size_t)page : (size_t)page * a.nkv + kvh) * a.page + in_page * DC_BN) * D;
         bf16* dst = my + (stage * 2 + which) * DC_BN * LD;
         const bf16* src = which ? a.v_pages : a.k_pages;
         const int valid = kv_len - tile * DC_BN;

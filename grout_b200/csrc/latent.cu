@@ -41,7 +41,23 @@ struct LatentArgs {
   const float* q_norm_w;   // [q_rank]
   void* cq;                // [T, q_rank]: the normalised latent
   int queries_only;        // proj holds expanded queries [T, H (dn + dr)] and nothing else
+  int n_parts;             // proj is that many 32-bit partial sums, added in order (a split-K projection leaves
+  long long part_stride;   //   its reduction to this kernel); floats between them
+  float* gate_out;         // with n_parts > 1 and a gate: [T, H dv], the gate's sums
 };
+
+__device__ __forceinline__ float latent_sum(const LatentArgs& a, const float* p) {
+  float v = p[0];
+  for (int k0 = 1; k0 < a.n_parts; k0 += 4) {      // four partial sums requested at a time
+    float q[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) q[u] = p[(size_t)(k0 + u < a.n_parts ? k0 + u : a.n_parts - 1) * a.part_stride];
+#pragma unroll
+    for (int u = 0; u < 4; ++u)
+      if (k0 + u < a.n_parts) v += q[u];
+  }
+  return v;
+}
 
 template <typename T>
 __device__ __forceinline__ void latent_pad(T* q_full, int nh, int Ds, int from, int tid, int step) {
@@ -51,9 +67,11 @@ __device__ __forceinline__ void latent_pad(T* q_full, int nh, int Ds, int from, 
 
 // A block owns one token and the heads blockIdx.y * heads_per_block ..; the block of the
 // first heads also normalises the latent and stores the token's cache row.  With a latent
-// for the queries too, block 0 has the keys' latent and block 1 the queries'.
+// for the queries too, block 0 has the keys' latent and block 1 the queries'.  With partial sums
+// the last gridDim.y - first_gate blocks put the gate's together.
 template <typename T>
-__global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a, const int heads_per_block) {
+__global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a, const int heads_per_block,
+                                                             const int first_gate) {
   __shared__ float scratch[32];
   pdl_launch_dependents_if_small();
   pdl_wait();
@@ -65,19 +83,32 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
   const float* __restrict__ row = a.proj + (size_t)t * C;
   const float* __restrict__ down = row + q_cols;
   const float pos = (float)a.token_pos[t];
+  if ((int)blockIdx.y >= first_gate) {
+    const int n = H * a.dv, step = (gridDim.y - first_gate) * blockDim.x;
+    pdl_launch_dependents_if_large();
+    for (int i = (blockIdx.y - first_gate) * blockDim.x + tid; i < n; i += step)
+      a.gate_out[(size_t)t * n + i] = latent_sum(a, down + R + dr + i);
+    return;
+  }
   if (a.q_rank > 0 && blockIdx.y == 1) {
     float ss = 0.f;
-    for (int i = tid; i < q_cols; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
+    for (int i = tid; i < q_cols; i += blockDim.x) {
+      const float v = latent_sum(a, row + i);
+      ss = fmaf(v, v, ss);
+    }
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)q_cols + a.eps);
     pdl_launch_dependents_if_large();
     for (int i = tid; i < q_cols; i += blockDim.x)
-      ((T*)a.cq)[(size_t)t * q_cols + i] = from_f32<T>(row[i] * inv * a.q_norm_w[i]);
+      ((T*)a.cq)[(size_t)t * q_cols + i] = from_f32<T>(latent_sum(a, row + i) * inv * a.q_norm_w[i]);
     if (dr == 0) latent_pad<T>((T*)a.q_full + (size_t)t * H * Ds, H, Ds, R, tid, blockDim.x);
     return;
   }
   if (blockIdx.y == 0 && !a.queries_only) {
     float ss = 0.f;
-    for (int i = tid; i < R; i += blockDim.x) ss = fmaf(down[i], down[i], ss);
+    for (int i = tid; i < R; i += blockDim.x) {
+      const float v = latent_sum(a, down + i);
+      ss = fmaf(v, v, ss);
+    }
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)R + a.eps);
     const int slot = a.slots[a.token_seq[t]];
     if (slot >= 0) {
@@ -86,12 +117,12 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
       T* dst = (T*)a.pages + ((size_t)pg * a.page + p % a.page) * Ds;
       for (int i = tid; i < Ds; i += blockDim.x) {
         float v = 0.f;
-        if (i < R) v = down[i] * inv * a.norm_w[i];
+        if (i < R) v = latent_sum(a, down + i) * inv * a.norm_w[i];
         else if (i < R + dr) {
           const int e = i - R, pair = e >> 1;
           float s, c;
           sincosf(pos * a.inv_freq[pair], &s, &c);
-          const float u = down[R + 2 * pair], w = down[R + 2 * pair + 1];
+          const float u = latent_sum(a, down + R + 2 * pair), w = latent_sum(a, down + R + 2 * pair + 1);
           v = (e & 1) ? w * c + u * s : u * c - w * s;
         }
         dst[i] = from_f32<T>(v);
@@ -106,12 +137,13 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
   for (int i = tid; i < nh * (dn + dr); i += blockDim.x) {
     const int h = i / (dn + dr), e = i % (dn + dr);
     if (e < dn) {
-      q_plain[(size_t)h * dn + e] = from_f32<T>(qrow[i]);
+      q_plain[(size_t)h * dn + e] = from_f32<T>(latent_sum(a, qrow + i));
     } else {
       const int r = e - dn, pair = r >> 1;
       float s, c;
       sincosf(pos * a.inv_freq[pair], &s, &c);
-      const float u = qrow[h * (dn + dr) + dn + 2 * pair], w = qrow[h * (dn + dr) + dn + 2 * pair + 1];
+      const float* at = qrow + h * (dn + dr) + dn + 2 * pair;
+      const float u = latent_sum(a, at), w = latent_sum(a, at + 1);
       q_full[(size_t)h * Ds + R + r] = from_f32<T>((r & 1) ? w * c + u * s : u * c - w * s);
     }
   }
@@ -128,12 +160,13 @@ static int latent_prepare(const LatentArgs& a, cudaStream_t s) {
   if (a.q_rank < 0 || (a.q_rank > 0 && (!a.q_norm_w || !a.cq || a.queries_only)) || (a.q_rank == 0 && !a.q_plain))
     return GB_ERR_BAD_ARG;
   if (a.n_tokens == 0) return 0;
-  if (a.q_rank > 0)
-    return gb_launch(latent_prepare_kernel<T>, dim3(a.n_tokens, 2), dim3(256), 0, s, a, a.H);
+  if (a.n_parts < 1 || (a.n_parts > 1 && a.dv > 0 && !a.queries_only && !a.gate_out)) return GB_ERR_BAD_ARG;
   // few tokens: four heads a block, so that a step of a handful of rows fills more than a handful of SMs
-  const int heads_per_block = a.n_tokens <= 64 ? min(a.H, 4) : a.H;
-  return gb_launch(latent_prepare_kernel<T>, dim3(a.n_tokens, (a.H + heads_per_block - 1) / heads_per_block),
-                   dim3(256), 0, s, a, heads_per_block);
+  const int heads_per_block = a.q_rank > 0 ? a.H : (a.n_tokens <= 64 ? min(a.H, 4) : a.H);
+  const int first_gate = a.q_rank > 0 ? 2 : (a.H + heads_per_block - 1) / heads_per_block;
+  const int gates = a.n_parts > 1 && a.dv > 0 && !a.queries_only ? min(8, (a.H * a.dv + 511) / 512) : 0;
+  return gb_launch(latent_prepare_kernel<T>, dim3(a.n_tokens, first_gate + gates), dim3(256), 0, s, a, heads_per_block,
+                   first_gate);
 }
 GB_EXPORT int gb_latent_prepare_f32(const LatentArgs* a, cudaStream_t s) { return latent_prepare<float>(*a, s); }
 GB_EXPORT int gb_latent_prepare_bf16(const LatentArgs* a, cudaStream_t s) { return latent_prepare<bf16>(*a, s); }
@@ -148,6 +181,8 @@ struct HeadsMmArgs {
   void* out;
   const float* g;
   int T, H, K, N, ldx, ldo, ldg;
+  const float* x_parts;    // instead of x: n_parts 32-bit partial sums [T, H, K] of it, added in order (bfloat16 only)
+  int n_parts;
 };
 
 #define HM_BM 16
@@ -242,6 +277,31 @@ __device__ __forceinline__ void ht_stage(bf16 (*dst)[HT_LD], const bf16* src, si
   }
 }
 
+// The same from 32-bit partial sums, which are added in order and rounded once.
+template <int ITERS, int THREADS>
+__device__ __forceinline__ void ht_stage_parts(bf16 (*dst)[HT_LD], const float* src, size_t ld, int n_parts, size_t stride,
+                                               int rows_here, int k0, int K, int tid) {
+#pragma unroll
+  for (int it = 0; it < ITERS; ++it) {
+    const int i = tid + it * THREADS;
+    const int r = i / (HT_BK / 8), kv = (i % (HT_BK / 8)) * 8;
+    float s[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s[j] = 0.f;
+    if (r < rows_here) {
+      const float* p = src + (size_t)r * ld + k0 + kv;
+      for (int q = 0; q < n_parts; ++q, p += stride)
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+          if (k0 + kv + j < K) s[j] += p[j];
+    }
+    __align__(16) bf16 e[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) e[j] = __float2bfloat16_rn(s[j]);
+    *reinterpret_cast<uint4*>(&dst[r][kv]) = *reinterpret_cast<const uint4*>(e);
+  }
+}
+
 template <int MW>
 __global__ void __launch_bounds__(MW * 64) heads_mm_tc_kernel(const HeadsMmArgs a, const int vec) {
   constexpr int BM = 32 * MW, THREADS = MW * 64;
@@ -264,7 +324,11 @@ __global__ void __launch_bounds__(MW * 64) heads_mm_tc_kernel(const HeadsMmArgs 
       for (int c = 0; c < 4; ++c) acc[i][j][c] = 0.f;
   for (int k0 = 0; k0 < K; k0 += HT_BK) {
     if (k0) __syncthreads();
-    ht_stage<BM * (HT_BK / 8) / THREADS, THREADS>(As, x, (size_t)a.H * a.ldx, min(BM, a.T - t0), k0, K, vec & 1, tid);
+    if (a.x_parts)
+      ht_stage_parts<BM * (HT_BK / 8) / THREADS, THREADS>(As, a.x_parts + ((size_t)t0 * a.H + h) * K, (size_t)a.H * K,
+                                                          a.n_parts, (size_t)a.T * a.H * K, min(BM, a.T - t0), k0, K, tid);
+    else
+      ht_stage<BM * (HT_BK / 8) / THREADS, THREADS>(As, x, (size_t)a.H * a.ldx, min(BM, a.T - t0), k0, K, vec & 1, tid);
     ht_stage<HT_BN * (HT_BK / 8) / THREADS, THREADS>(Bs, w, (size_t)K, min(HT_BN, N - n0), k0, K, vec & 2, tid);
     __syncthreads();
 #pragma unroll
@@ -329,7 +393,8 @@ template <typename T>
 static int heads_mm(const HeadsMmArgs& a, cudaStream_t s) {
   if (a.T < 0 || a.H <= 0 || a.K <= 0 || a.N <= 0 || a.ldx < a.K || a.ldo < a.N || a.H > 65535)
     return GB_ERR_BAD_ARG;
-  if (!a.x || !a.w || !a.out) return GB_ERR_BAD_ARG;
+  if ((!a.x && !a.x_parts) || !a.w || !a.out) return GB_ERR_BAD_ARG;
+  if (a.x_parts && (sizeof(T) != 2 || a.n_parts < 1)) return GB_ERR_UNSUPPORTED;
   if (a.T == 0) return 0;
   if (sizeof(T) == 2) {
     // bit 0: rows of x can be read 16 bytes at a time; bit 1: rows of w; bit 2: pairs of the result stored as one word

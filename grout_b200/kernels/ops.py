@@ -1044,6 +1044,7 @@ def _gate_code(gate_act: str, bias, silu_mul: bool, n_fused: int):
     return _GATE_CODES[gate_act]
 
 
+TC_WHOLE_K = 512        # up to this inner size a 32-bit result is made of whole tiles
 _TC_PLANS = {}
 _TC_ERRORS = {}
 _TC_ERROR_NAMES = {111: "a role of the tcgen05 attention kernel waited 2 s on a barrier",
@@ -1153,8 +1154,15 @@ def gemm_tc_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype=torch.bfloat16,
     with torch.cuda.device(x.device):
         plan = _tc_plan(A.shape[0], B.shape[0], K)
         split = plan[4] if (split_out and swap and not silu_mul) else 0
+        # a short inner size: a block takes a whole tile (no two blocks share one and meet at its end):
+        # 10 against 14 us at 8192 x 256 with 8 rows
+        whole = (not split and swap and not silu_mul and not relu_squared and K <= TC_WHOLE_K
+                 and (out_dtype == torch.float32 or into is not None))
+        split = 1 if whole else split
         y = (_result((split, M, N), torch.float32, x.device, into) if split
              else _result((M, n_out), out_dtype, x.device, into))
+        if whole:
+            y = y[0]
         ws = _WORKSPACES.setdefault(x.device.index or 0, _Workspace())
         scratch, counters = ws.get(x.device, plan[2], plan[3])
         a = _TcArgs()
@@ -1170,7 +1178,7 @@ def gemm_tc_bf16(x: torch.Tensor, w: torch.Tensor, out_dtype=torch.bfloat16,
         _check(_fn("gemm_tc", "gb_gemm_tc_bf16", "pppp")(
             A.data_ptr(), B.data_ptr(), ctypes.addressof(a), _stream()), "gemm_tc_bf16",
             detail=f" {N}x{K}" + ((" " + gate_act) if silu_mul else "") + (" relu2" if relu_squared else "") +
-            (f" split {split}" if split else ""))
+            (f" split {split}" if split > 1 else ""))
     return y
 
 
@@ -1268,7 +1276,7 @@ class _DecodeArgs(ctypes.Structure):
                 ("kv_len", _P), ("out", _P), ("part_o", _P), ("part_ml", _P), ("n_seqs", _I),
                 ("nq", _I), ("nkv", _I), ("max_pages", _I), ("page", _I), ("window", _I),
                 ("n_splits", _I), ("scale_log2", _F), ("sinks", _P), ("cap_log2", _F),
-                ("cap_inv", _F), ("keep_first", _I), ("chunk", _I)]
+                ("cap_inv", _F), ("keep_first", _I), ("chunk", _I), ("one_kv", _I)]
 
 
 def _set_cap_and_sinks(a, scale: float, softcap: Optional[float], sinks, nq: int) -> None:
@@ -1309,6 +1317,13 @@ def _sm_count(device) -> int:
 def fast_attention_takes(D: int, nq: int, nkv: int, page: int) -> bool:
     """Shapes the tensor-core kernels accept; others go to the plain kernel."""
     return D % 16 == 0 and 16 <= D <= 128 and page == 64 and nq % nkv == 0 and nq // nkv <= 16
+
+
+def groups_on_one_head(nq: int) -> int:
+    """The fewest equal groups of at most sixteen that ``nq`` query heads form (0: none with fewer than
+    twice the groups that they need)."""
+    least = (nq + 15) // 16
+    return next((g for g in range(least, 2 * least) if nq % g == 0), 0)
 
 
 def _q_blocks(q_lens, n_qblocks, rows: int, T: int, n_seqs: int) -> int:
@@ -1466,9 +1481,11 @@ def attn_decode_bf16(q, k_pages, v_pages, block_table, *, slots, kv_len, page: i
                      max_kv_len: int, window: Optional[int] = None,
                      n_splits: Optional[int] = None, softcap: Optional[float] = None,
                      sinks: Optional[torch.Tensor] = None, keep_first: int = 0,
-                    chunk: int = 0) -> torch.Tensor:
+                    chunk: int = 0, groups: int = 0) -> torch.Tensor:
     """Attention of one new token per sequence over its cached keys (split-K).
-    ``keep_first``: with a window, a sequence's first keys that stay visible behind it."""
+    ``keep_first``: with a window, a sequence's first keys that stay visible behind it.
+    ``groups``: the pages hold one kv head, and the query heads read it in that many equal groups (of
+    at most sixteen), a block each."""
     _need(q, "q", torch.bfloat16, 3)
     B, nq, D = q.shape
     _need(k_pages, "k pages", torch.bfloat16, 4)
@@ -1476,6 +1493,10 @@ def attn_decode_bf16(q, k_pages, v_pages, block_table, *, slots, kv_len, page: i
     nkv = k_pages.shape[1]
     if tuple(k_pages.shape[1:]) != (nkv, page, D) or v_pages.shape != k_pages.shape:
         raise KernelError(f"pages are {tuple(k_pages.shape)}, expected [*, nkv, {page}, {D}]")
+    if groups:
+        if nkv != 1 or nq % groups:
+            raise KernelError(f"{nq} query heads do not form {groups} groups on one kv head")
+        nkv = int(groups)
     for t, nm in ((block_table, "block table"), (slots, "slots"), (kv_len, "kv_len")):
         _need(t, nm, torch.int32)
     if slots.shape[0] != B or kv_len.shape[0] != B:
@@ -1498,6 +1519,7 @@ def attn_decode_bf16(q, k_pages, v_pages, block_table, *, slots, kv_len, page: i
     a.n_seqs, a.nq, a.nkv, a.max_pages, a.page = B, nq, nkv, block_table.shape[1], page
     a.window, a.n_splits, a.scale_log2 = int(window or 0), ns, float(scale) * _LOG2E
     a.keep_first, a.chunk = int(keep_first or 0), _chunk_arg(chunk, keep_first)
+    a.one_kv = int(bool(groups))
     _set_cap_and_sinks(a, scale, softcap, sinks, nq)
     _check(_fn("attn_decode_bf16", "gb_attn_decode_bf16", "pip")(
         ctypes.addressof(a), D, _stream()), "attn_decode_bf16", 2 if ns > 1 else 1)
@@ -1625,6 +1647,13 @@ def attention(q, k_pages, v_pages, block_table, *, step, page: int, scale: float
     _T, nq, D = q.shape
     keep_first = int(keep_first or 0) if window else 0
     extra = dict(softcap=softcap, sinks=sinks, keep_first=keep_first, chunk=chunk)
+    if (q.dtype == torch.bfloat16 and not step.decode and PREFILL_ATTENTION == "tc"
+            and attn_prefill_tc_takes(D, nq, k_pages.shape[1], page)):
+        # the grid comes from the host's copy of the lengths; a captured step has
+        # none, and the kernels then take the most blocks its rows can make
+        return attn_prefill_tc(q, k_pages, v_pages, block_table, cu_q=step.cu_q,
+                               slots=step.slots, kv_len=step.kv_len, q_lens=step.q_lens,
+                               page=page, scale=scale, window=window, **extra)
     if q.dtype == torch.bfloat16 and fast_attention_takes(D, nq, k_pages.shape[1], page):
         nkv = k_pages.shape[1]
         if step.decode and attn_decode_tma_takes(D, nq, nkv, page) and (
@@ -1637,12 +1666,6 @@ def attention(q, k_pages, v_pages, block_table, *, step, page: int, scale: float
             return attn_decode_bf16(q, k_pages, v_pages, block_table, slots=step.slots,
                                     kv_len=step.kv_len, page=page, scale=scale,
                                     max_kv_len=step.max_kv_len, window=window, **extra)
-        # the grid comes from the host's copy of the lengths; a captured step has
-        # none, and the kernels then take the most blocks its rows can make
-        if PREFILL_ATTENTION == "tc" and attn_prefill_tc_takes(D, nq, k_pages.shape[1], page):
-            return attn_prefill_tc(q, k_pages, v_pages, block_table, cu_q=step.cu_q,
-                                   slots=step.slots, kv_len=step.kv_len, q_lens=step.q_lens,
-                                   page=page, scale=scale, window=window, **extra)
         return attn_prefill_bf16(q, k_pages, v_pages, block_table, cu_q=step.cu_q,
                                  slots=step.slots, kv_len=step.kv_len, q_lens=step.q_lens,
                                  page=page, scale=scale, window=window, **extra)
@@ -2045,7 +2068,19 @@ class _LatentArgs(ctypes.Structure):
                 ("slots", _P), ("block_table", _P), ("pages", _P), ("q_plain", _P), ("q_full", _P),
                 ("n_tokens", _I), ("H", _I), ("dn", _I), ("dr", _I), ("R", _I), ("dv", _I), ("Ds", _I),
                 ("max_pages", _I), ("page", _I), ("eps", _F), ("q_rank", _I), ("q_norm_w", _P), ("cq", _P),
-                ("queries_only", _I)]
+                ("queries_only", _I), ("n_parts", _I), ("part_stride", _L), ("gate_out", _P)]
+
+
+def _latent_parts(a, proj, dv_cols: int = 0):
+    """``proj`` [T, C] or partial sums of it [P, T, C] into the arguments; the gate's sums [T, dv_cols]
+    (a tensor that the kernel fills) when there are several, else None."""
+    a.proj, a.n_parts = proj.data_ptr(), (proj.shape[0] if proj.dim() == 3 else 1)
+    a.part_stride = proj.stride(0) if proj.dim() == 3 else 0
+    if a.n_parts == 1 or not dv_cols:
+        return None
+    gate = torch.empty((proj.shape[-2], dv_cols), dtype=torch.float32, device=proj.device)
+    a.gate_out = gate.data_ptr()
+    return gate
 
 
 @_profiled("latent_prepare", lambda out, proj, *a, **k: (_nbytes(proj) + _nbytes(*out), 0))
@@ -2063,10 +2098,12 @@ def latent_prepare(proj: torch.Tensor, norm_w: torch.Tensor, inv_freq: Optional[
     are written (the rotated query part, then zeros), the first R are left to the caller.
     ``q_norm_w`` [q_rank]: the projection's first q_rank columns are the queries' latent in
     their place; instead of q_plain it is returned, RMS-normalised, [T, q_rank], and of q_full
-    what is zero is written when there is no rotated part (``latent_queries`` does the rest)."""
-    _need(proj, "projection", torch.float32, 2)
+    what is zero is written when there is no rotated part (``latent_queries`` does the rest).
+    ``proj`` may be a stack of partial sums [P, T, C], added in order.  A third result is the
+    gate as ``heads_mm`` takes it: (logits, their first column), (None, 0) without a gate."""
+    _need(proj, "projection", torch.float32)
     _need(norm_w, "latent norm weight", torch.float32, 1)
-    T = proj.shape[0]
+    T = proj.shape[-2]
     _need(pages, "latent pages", dtype, 4)
     Ds = pages.shape[-1]
     q_rank = 0
@@ -2074,8 +2111,8 @@ def latent_prepare(proj: torch.Tensor, norm_w: torch.Tensor, inv_freq: Optional[
         _need(q_norm_w, "query latent norm weight", torch.float32, 1)
         q_rank = q_norm_w.shape[0]
     want = (q_rank or H * (dn + dr)) + R + dr + H * dv
-    if proj.shape[1] != want or norm_w.shape[0] != R:
-        raise KernelError(f"the projection has {proj.shape[1]} columns, expected {want}; the norm weight "
+    if proj.dim() not in (2, 3) or proj.shape[-1] != want or norm_w.shape[0] != R:
+        raise KernelError(f"the projection is {tuple(proj.shape)}, expected {want} columns; the norm weight "
                           f"{norm_w.shape[0]} for {R}")
     if tuple(pages.shape[1:]) != (1, page, Ds) or Ds < R + dr:
         raise KernelError(f"pages are {tuple(pages.shape)}, expected [*, 1, {page}, >= {R + dr}]")
@@ -2091,7 +2128,8 @@ def latent_prepare(proj: torch.Tensor, norm_w: torch.Tensor, inv_freq: Optional[
     a = _LatentArgs()
     if q_rank:
         a.q_rank, a.q_norm_w, a.cq = q_rank, q_norm_w.data_ptr(), q_plain.data_ptr()
-    a.proj, a.norm_w, a.inv_freq = proj.data_ptr(), norm_w.data_ptr(), _ptr(inv_freq)
+    gate = _latent_parts(a, proj, H * dv)
+    a.norm_w, a.inv_freq = norm_w.data_ptr(), _ptr(inv_freq)
     a.token_seq, a.token_pos, a.slots = token_seq.data_ptr(), token_pos.data_ptr(), slots.data_ptr()
     a.block_table, a.pages = block_table.data_ptr(), pages.data_ptr()
     a.q_plain, a.q_full = q_plain.data_ptr(), q_full.data_ptr()
@@ -2099,24 +2137,27 @@ def latent_prepare(proj: torch.Tensor, norm_w: torch.Tensor, inv_freq: Optional[
     a.max_pages, a.page, a.eps = block_table.shape[1], int(page), float(eps)
     _check(_fn("latent", f"gb_latent_prepare_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
            "latent_prepare")
-    return q_plain, q_full
+    if not dv:
+        return q_plain, q_full, (None, 0)
+    return q_plain, q_full, ((gate, 0) if gate is not None else (proj.view(T, want), want - H * dv))
 
 
 @_profiled("latent_queries", lambda out, q, *a, **k: (2 * _nbytes(q), 0))
 def latent_queries(q: torch.Tensor, q_full: torch.Tensor, inv_freq: torch.Tensor, *, H: int, dn: int, dr: int,
                    R: int, token_pos) -> torch.Tensor:
-    """Queries [T, H (dn + dr)] (32-bit) that a product has expanded from their latent: the dr
+    """Queries [T, H (dn + dr)] (32-bit, or partial sums of them) that a product has expanded from their latent: the dr
     rotated elements of every head go, turned, to columns R .. R + dr of ``q_full`` [T, H, Ds]
     (zeros behind them), the dn plain ones are returned [T, H, dn]."""
-    _need(q, "queries", torch.float32, 2)
+    _need(q, "queries", torch.float32)
     _need(inv_freq, "inv_freq", torch.float32, 1)
     _need(token_pos, "token_pos", torch.int32, 1)
-    T = q.shape[0]
-    if q.shape[1] != H * (dn + dr) or tuple(q_full.shape[:2]) != (T, H) or inv_freq.shape[0] * 2 != dr:
+    T = q.shape[-2]
+    if q.shape[-1] != H * (dn + dr) or tuple(q_full.shape[:2]) != (T, H) or inv_freq.shape[0] * 2 != dr:
         raise KernelError(f"queries {tuple(q.shape)} do not hold {H} heads of {dn} + {dr} elements")
     q_plain = torch.empty((T, H, dn), dtype=q_full.dtype, device=q.device)
     a = _LatentArgs()
-    a.proj, a.inv_freq, a.token_pos = q.data_ptr(), inv_freq.data_ptr(), token_pos.data_ptr()
+    _latent_parts(a, q)
+    a.inv_freq, a.token_pos = inv_freq.data_ptr(), token_pos.data_ptr()
     a.q_plain, a.q_full, a.queries_only = q_plain.data_ptr(), q_full.data_ptr(), 1
     a.n_tokens, a.H, a.dn, a.dr, a.R, a.Ds = T, H, dn, dr, R, q_full.shape[2]
     _check(_fn("latent", f"gb_latent_prepare_{_suffix(q_full.dtype)}", "pp")(ctypes.addressof(a), _stream()),
@@ -2126,7 +2167,7 @@ def latent_queries(q: torch.Tensor, q_full: torch.Tensor, inv_freq: torch.Tensor
 
 class _HeadsMmArgs(ctypes.Structure):
     _fields_ = [("x", _P), ("w", _P), ("out", _P), ("g", _P), ("T", _I), ("H", _I), ("K", _I),
-                ("N", _I), ("ldx", _I), ("ldo", _I), ("ldg", _I)]
+                ("N", _I), ("ldx", _I), ("ldo", _I), ("ldg", _I), ("x_parts", _P), ("n_parts", _I)]
 
 
 @_profiled("heads_mm", lambda out, x, w, *a, **k: (_nbytes(x, w) + x.shape[0] * w.shape[0] * w.shape[1] * x.element_size(),
@@ -2136,27 +2177,35 @@ def heads_mm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = Non
     """A product per head: out[t, h, :N] = w[h] x[t, h, :K] with x [T, H, ldx >= K], w [H, N, K]
     and out [T, H, ldo >= N] (made [T, H, N] when not given; columns from N on are left as
     they are).  ``gate`` [T, ld] 32-bit: the result is multiplied, on its 32-bit sums, by
-    sigmoid(gate[t, gate_col + h N + n])."""
+    sigmoid(gate[t, gate_col + h N + n]).  ``x`` may also be a stack of 32-bit partial sums
+    [P, T, H K] of a bfloat16 tensor, which are added in order and rounded once."""
+    parts = None
+    if x.dtype == torch.float32 and w.dtype == torch.bfloat16:
+        _need(x, "partial sums", torch.float32, 3)
+        parts, x = x, x[0].view(x.shape[1], w.shape[0], -1)
+    else:
+        _need(w, "weights per head", x.dtype, 3)
     _need(x, "rows per head", ndim=3)
-    _need(w, "weights per head", x.dtype, 3)
     T, H, ldx = x.shape
     Hw, N, K = w.shape
-    if Hw != H or K > ldx or not x.is_contiguous() or not w.is_contiguous():
+    if Hw != H or K > ldx or (parts is not None and K != ldx) or not x.is_contiguous() or not w.is_contiguous():
         raise KernelError(f"rows {tuple(x.shape)} and weights {tuple(w.shape)} do not fit together")
     if out is None:
-        out = torch.empty((T, H, N), dtype=x.dtype, device=x.device)
-    _need(out, "result", x.dtype, 3)
+        out = torch.empty((T, H, N), dtype=w.dtype, device=x.device)
+    _need(out, "result", w.dtype, 3)
     if out.shape[0] != T or out.shape[1] != H or out.shape[2] < N or not out.is_contiguous():
         raise KernelError(f"the result is {tuple(out.shape)}, expected [{T}, {H}, >= {N}]")
     a = _HeadsMmArgs()
     a.x, a.w, a.out = x.data_ptr(), w.data_ptr(), out.data_ptr()
     a.T, a.H, a.K, a.N, a.ldx, a.ldo = T, H, K, N, ldx, out.shape[2]
+    if parts is not None:
+        a.x_parts, a.n_parts = parts.data_ptr(), parts.shape[0]
     if gate is not None:
         _need(gate, "gate", torch.float32, 2)
         if gate.shape[0] != T or gate_col + H * N > gate.shape[1] or gate.stride(1) != 1:
             raise KernelError("the gate's rows do not hold the heads' columns")
         a.g, a.ldg = gate.data_ptr() + 4 * int(gate_col), gate.stride(0)
-    _check(_fn("latent", f"gb_heads_mm_{_suffix(x.dtype)}", "pp")(ctypes.addressof(a), _stream()),
+    _check(_fn("latent", f"gb_heads_mm_{_suffix(w.dtype)}", "pp")(ctypes.addressof(a), _stream()),
            "heads_mm")
     return out
 

@@ -630,11 +630,19 @@ class LatentAttention(Mixer):
 
     def _attend(self, q, step, cache):
         """Attention of all heads over the one shared row per token.  More heads than the
-        tensor-core kernels let share a kv head go in groups, each a call of its own."""
+        tensor-core kernels let share a kv head go in groups, each a call of its own (the tcgen05
+        kernel of a prompt takes any number, and a decode step's groups are one call where they are
+        equal)."""
         kw = dict(step=step, page=cache.page, scale=self.scale, window=self.window)
         if (self.H <= self.GROUP or q.dtype != torch.bfloat16
+                or (not step.decode and ops.attn_prefill_tc_takes(self.Ds, self.H, 1, cache.page))
                 or not ops.fast_attention_takes(self.Ds, self.GROUP, 1, cache.page)):
             return ops.attention(q, cache.k_pages, cache.v_pages, cache.block_table, sinks=self.sink, **kw)
+        groups = ops.groups_on_one_head(self.H)
+        if step.decode and groups:
+            return ops.attn_decode_bf16(q, cache.k_pages, cache.v_pages, cache.block_table, slots=step.slots,
+                                        kv_len=step.kv_len, max_kv_len=step.max_kv_len, page=cache.page,
+                                        scale=self.scale, window=self.window, sinks=self.sink, groups=groups)
         sinks = lambda a: None if self.sink is None else self.sink[a:a + self.GROUP]
         return ops.join_heads([ops.attention(ops.head_group(q, a, min(self.GROUP, self.H - a)), cache.k_pages,
                                              cache.v_pages, cache.block_table, sinks=sinks(a), **kw)
@@ -649,19 +657,21 @@ class LatentAttention(Mixer):
                              f"{None if cache is None else cache.spec}")
         T, H = x.shape[0], self.H
         rot = self.position.rotary()
-        proj = self.proj(x, out_dtype=torch.float32)
-        q_plain, q = ops.latent_prepare(
+        # (the preparation and the products per head can add the partial sums of split-K products)
+        parts = x.dtype == torch.bfloat16
+        proj = self.proj(x, out_dtype=torch.float32, partial_ok=parts)
+        q_plain, q, gate = ops.latent_prepare(
             proj, self.norm_w, rot.inv_freq if rot else None, H=H, dn=self.dn, dr=self.dr, R=self.R,
             dv=self.dv if self.gated else 0, eps=self.norm_eps, token_seq=step.token_seq,
             token_pos=step.token_pos, slots=step.slots, block_table=cache.block_table,
             pages=cache.k_pages, page=cache.page, dtype=self.ctx.dtype, q_norm_w=self.q_norm_w)
         if self.q_rank and self.dr:         # (q_plain is the queries' latent here)
-            q_plain = ops.latent_queries(self.uq(q_plain, out_dtype=torch.float32), q, rot.inv_freq, H=H,
+            q_plain = ops.latent_queries(self.uq(q_plain, out_dtype=torch.float32, partial_ok=parts), q, rot.inv_freq, H=H,
                                          dn=self.dn, dr=self.dr, R=self.R, token_pos=step.token_pos)
         elif self.q_rank:
-            q_plain = self.uq(q_plain).view(T, H, self.dn)
+            q_plain = self.uq(q_plain, partial_ok=parts)
+            q_plain = q_plain.view(T, H, self.dn) if q_plain.dim() == 2 else q_plain
         ops.heads_mm(q_plain, self.uk_t, q)
         attn = self._attend(q, step, cache)
-        y = ops.heads_mm(attn, self.uv, gate=proj if self.gated else None,
-                         gate_col=(self.q_rank or H * (self.dn + self.dr)) + self.R + self.dr)
+        y = ops.heads_mm(attn, self.uv, gate=gate[0], gate_col=gate[1])
         return self.o(y.view(T, H * self.dv), partial_ok=True)
