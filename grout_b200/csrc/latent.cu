@@ -46,8 +46,10 @@ struct LatentArgs {
   float* gate_out;         // with n_parts > 1 and a gate: [T, H dv], the gate's sums
 };
 
+template <bool PARTS>
 __device__ __forceinline__ float latent_sum(const LatentArgs& a, const float* p) {
   float v = p[0];
+  if constexpr (!PARTS) return v;
   for (int k0 = 1; k0 < a.n_parts; k0 += 4) {      // four partial sums requested at a time
     float q[4];
 #pragma unroll
@@ -69,7 +71,7 @@ __device__ __forceinline__ void latent_pad(T* q_full, int nh, int Ds, int from, 
 // first heads also normalises the latent and stores the token's cache row.  With a latent
 // for the queries too, block 0 has the keys' latent and block 1 the queries'.  With partial sums
 // the last gridDim.y - first_gate blocks put the gate's together.
-template <typename T>
+template <typename T, bool PARTS>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a, const int heads_per_block,
                                                              const int first_gate) {
   __shared__ float scratch[32];
@@ -83,30 +85,30 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
   const float* __restrict__ row = a.proj + (size_t)t * C;
   const float* __restrict__ down = row + q_cols;
   const float pos = (float)a.token_pos[t];
-  if ((int)blockIdx.y >= first_gate) {
+  if (PARTS && (int)blockIdx.y >= first_gate) {
     const int n = H * a.dv, step = (gridDim.y - first_gate) * blockDim.x;
     pdl_launch_dependents_if_large();
     for (int i = (blockIdx.y - first_gate) * blockDim.x + tid; i < n; i += step)
-      a.gate_out[(size_t)t * n + i] = latent_sum(a, down + R + dr + i);
+      a.gate_out[(size_t)t * n + i] = latent_sum<PARTS>(a, down + R + dr + i);
     return;
   }
   if (a.q_rank > 0 && blockIdx.y == 1) {
     float ss = 0.f;
     for (int i = tid; i < q_cols; i += blockDim.x) {
-      const float v = latent_sum(a, row + i);
+      const float v = latent_sum<PARTS>(a, row + i);
       ss = fmaf(v, v, ss);
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)q_cols + a.eps);
     pdl_launch_dependents_if_large();
     for (int i = tid; i < q_cols; i += blockDim.x)
-      ((T*)a.cq)[(size_t)t * q_cols + i] = from_f32<T>(latent_sum(a, row + i) * inv * a.q_norm_w[i]);
+      ((T*)a.cq)[(size_t)t * q_cols + i] = from_f32<T>(latent_sum<PARTS>(a, row + i) * inv * a.q_norm_w[i]);
     if (dr == 0) latent_pad<T>((T*)a.q_full + (size_t)t * H * Ds, H, Ds, R, tid, blockDim.x);
     return;
   }
   if (blockIdx.y == 0 && !a.queries_only) {
     float ss = 0.f;
     for (int i = tid; i < R; i += blockDim.x) {
-      const float v = latent_sum(a, down + i);
+      const float v = latent_sum<PARTS>(a, down + i);
       ss = fmaf(v, v, ss);
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)R + a.eps);
@@ -117,12 +119,12 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
       T* dst = (T*)a.pages + ((size_t)pg * a.page + p % a.page) * Ds;
       for (int i = tid; i < Ds; i += blockDim.x) {
         float v = 0.f;
-        if (i < R) v = latent_sum(a, down + i) * inv * a.norm_w[i];
+        if (i < R) v = latent_sum<PARTS>(a, down + i) * inv * a.norm_w[i];
         else if (i < R + dr) {
           const int e = i - R, pair = e >> 1;
           float s, c;
           sincosf(pos * a.inv_freq[pair], &s, &c);
-          const float u = latent_sum(a, down + R + 2 * pair), w = latent_sum(a, down + R + 2 * pair + 1);
+          const float u = latent_sum<PARTS>(a, down + R + 2 * pair), w = latent_sum<PARTS>(a, down + R + 2 * pair + 1);
           v = (e & 1) ? w * c + u * s : u * c - w * s;
         }
         dst[i] = from_f32<T>(v);
@@ -137,13 +139,13 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentArgs a,
   for (int i = tid; i < nh * (dn + dr); i += blockDim.x) {
     const int h = i / (dn + dr), e = i % (dn + dr);
     if (e < dn) {
-      q_plain[(size_t)h * dn + e] = from_f32<T>(latent_sum(a, qrow + i));
+      q_plain[(size_t)h * dn + e] = from_f32<T>(latent_sum<PARTS>(a, qrow + i));
     } else {
       const int r = e - dn, pair = r >> 1;
       float s, c;
       sincosf(pos * a.inv_freq[pair], &s, &c);
       const float* at = qrow + h * (dn + dr) + dn + 2 * pair;
-      const float u = latent_sum(a, at), w = latent_sum(a, at + 1);
+      const float u = latent_sum<PARTS>(a, at), w = latent_sum<PARTS>(a, at + 1);
       q_full[(size_t)h * Ds + R + r] = from_f32<T>((r & 1) ? w * c + u * s : u * c - w * s);
     }
   }
@@ -165,8 +167,9 @@ static int latent_prepare(const LatentArgs& a, cudaStream_t s) {
   const int heads_per_block = a.q_rank > 0 ? a.H : (a.n_tokens <= 64 ? min(a.H, 4) : a.H);
   const int first_gate = a.q_rank > 0 ? 2 : (a.H + heads_per_block - 1) / heads_per_block;
   const int gates = a.n_parts > 1 && a.dv > 0 && !a.queries_only ? min(8, (a.H * a.dv + 511) / 512) : 0;
-  return gb_launch(latent_prepare_kernel<T>, dim3(a.n_tokens, first_gate + gates), dim3(256), 0, s, a, heads_per_block,
-                   first_gate);
+  const dim3 grid(a.n_tokens, first_gate + gates);
+  return a.n_parts > 1 ? gb_launch(latent_prepare_kernel<T, true>, grid, dim3(256), 0, s, a, heads_per_block, first_gate)
+                       : gb_launch(latent_prepare_kernel<T, false>, grid, dim3(256), 0, s, a, heads_per_block, first_gate);
 }
 GB_EXPORT int gb_latent_prepare_f32(const LatentArgs* a, cudaStream_t s) { return latent_prepare<float>(*a, s); }
 GB_EXPORT int gb_latent_prepare_bf16(const LatentArgs* a, cudaStream_t s) { return latent_prepare<bf16>(*a, s); }
@@ -302,7 +305,7 @@ __device__ __forceinline__ void ht_stage_parts(bf16 (*dst)[HT_LD], const float* 
   }
 }
 
-template <int MW>
+template <int MW, bool PARTS>
 __global__ void __launch_bounds__(MW * 64) heads_mm_tc_kernel(const HeadsMmArgs a, const int vec) {
   constexpr int BM = 32 * MW, THREADS = MW * 64;
   __shared__ __align__(16) bf16 As[BM][HT_LD];
@@ -324,7 +327,7 @@ __global__ void __launch_bounds__(MW * 64) heads_mm_tc_kernel(const HeadsMmArgs 
       for (int c = 0; c < 4; ++c) acc[i][j][c] = 0.f;
   for (int k0 = 0; k0 < K; k0 += HT_BK) {
     if (k0) __syncthreads();
-    if (a.x_parts)
+    if constexpr (PARTS)
       ht_stage_parts<BM * (HT_BK / 8) / THREADS, THREADS>(As, a.x_parts + ((size_t)t0 * a.H + h) * K, (size_t)a.H * K,
                                                           a.n_parts, (size_t)a.T * a.H * K, min(BM, a.T - t0), k0, K, tid);
     else
@@ -402,9 +405,10 @@ static int heads_mm(const HeadsMmArgs& a, cudaStream_t s) {
                     ((a.K % 8 == 0 && (uintptr_t)a.w % 16 == 0) ? 2 : 0) |
                     ((a.ldo % 2 == 0 && (uintptr_t)a.out % 4 == 0) ? 4 : 0);
     const unsigned ny = (a.N + HT_BN - 1) / HT_BN;
-    if (a.T <= 32) return gb_launch(heads_mm_tc_kernel<1>, dim3(1, ny, a.H), dim3(64), 0, s, a, vec);
-    if (a.T <= 64) return gb_launch(heads_mm_tc_kernel<2>, dim3(1, ny, a.H), dim3(128), 0, s, a, vec);
-    return gb_launch(heads_mm_tc_kernel<4>, dim3((a.T + 127) / 128, ny, a.H), dim3(256), 0, s, a, vec);
+    if (a.x_parts) return gb_launch(heads_mm_tc_kernel<1, true>, dim3((a.T + 31) / 32, ny, a.H), dim3(64), 0, s, a, vec);
+    if (a.T <= 32) return gb_launch(heads_mm_tc_kernel<1, false>, dim3(1, ny, a.H), dim3(64), 0, s, a, vec);
+    if (a.T <= 64) return gb_launch(heads_mm_tc_kernel<2, false>, dim3(1, ny, a.H), dim3(128), 0, s, a, vec);
+    return gb_launch(heads_mm_tc_kernel<4, false>, dim3((a.T + 127) / 128, ny, a.H), dim3(256), 0, s, a, vec);
   }
   return gb_launch(heads_mm_kernel<T>, dim3((a.T + HM_BM - 1) / HM_BM, (a.N + HM_BN - 1) / HM_BN, a.H),
                    dim3(256), 0, s, a);
