@@ -23,9 +23,9 @@
 //   scan     any other step of short sequences: the columns of S are independent recurrences; a
 //            column is held in the registers of eight lanes, 16 columns a block, and the rows are
 //            walked in order, their q, k and g staged in shared memory 16 at a time
-//   local, chain   a step in which a sequence brings many rows goes chunk by chunk instead
+//   local, chain, out   a step in which a sequence brings many rows goes chunk by chunk instead
 //            (channel_delta_chunk.cuh)
-//   finish   after these: one warp per (token, head) normalises and gates
+//   finish   after scan: one warp per (token, head) normalises and gates
 //
 // With s' = g s the two sums over dk that a row needs, s' . k and s' . q, are taken together:
 // u = beta (v - s' . k) and o = s' . q + u (k . q), so a row costs one round of shuffles.
@@ -493,21 +493,17 @@ static int run_rows(const ChannelDeltaArgs& a, cudaStream_t s) {
     if (smem > 48 * 1024) return GB_ERR_UNSUPPORTED;
     return gb_launch(channel_delta_step_kernel<T, R>, dim3(a.H, a.n_seqs), dim3(256), smem, s, a);
   }
-  int e;
-  if (cc_takes(a)) {
-    e = cc_run(a, s);
-  } else {
-    const size_t smem = (CD_TT * (3 * DKP + CD_COLS + 1)) * sizeof(float);
-    static bool configured = false;
-    if (smem > 48 * 1024 && !configured) {
-      cudaError_t ce = cudaFuncSetAttribute(channel_delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                            (int)smem);
-      if (ce != cudaSuccess) return (int)ce;
-      configured = true;
-    }
-    e = gb_launch(channel_delta_scan_kernel<R>, dim3((a.dv + CD_COLS - 1) / CD_COLS, a.H, a.n_seqs),
-                  dim3(CD_LANES * CD_COLS), smem, s, a);
+  if (cc_takes(a)) return cc_run<T>(a, s);
+  const size_t smem = (CD_TT * (3 * DKP + CD_COLS + 1)) * sizeof(float);
+  static bool configured = false;
+  if (smem > 48 * 1024 && !configured) {
+    cudaError_t ce = cudaFuncSetAttribute(channel_delta_scan_kernel<R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                          (int)smem);
+    if (ce != cudaSuccess) return (int)ce;
+    configured = true;
   }
+  const int e = gb_launch(channel_delta_scan_kernel<R>, dim3((a.dv + CD_COLS - 1) / CD_COLS, a.H, a.n_seqs),
+                          dim3(CD_LANES * CD_COLS), smem, s, a);
   if (e) return e;
   const int warps = a.H < 8 ? a.H : 8;
   return gb_launch(channel_delta_finish_kernel<T>, dim3(a.n_tokens, (a.H + warps - 1) / warps), dim3(warps * 32), 0, s, a);

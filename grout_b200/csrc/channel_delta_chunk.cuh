@@ -12,7 +12,10 @@
 //   local   takes every chunk of every head at the same time: A, B, the substitution for the dv + dk
 //           right-hand sides beta v and beta e^{L} k, and leaves the chunk's record
 //   chain   walks a sequence's chunks in order, a block per head and CC_COLS columns of S with the
-//           state in shared memory: U = U0 - W S, the read-outs, the next state: tiled 32-bit products
+//           state in shared memory: U = U0 - W S and the next state, tiled 32-bit products; it leaves
+//           U and the state in front of every chunk in the record
+//   out     takes every chunk of every head at the same time again: the read-outs, one product of
+//           the record's [e^{L} q | B] with [S_0 ; U], and their norm and gate
 //
 // Every exponent that is taken is not positive and is summed up from logarithms of one sign, never a
 // difference of two running sums (rows of the same half chunk directly, others by way of the end of
@@ -24,13 +27,17 @@
 #define CC_COLS 32       // columns of S a chain block owns
 #define CC_MIN 64        // a step goes chunk by chunk when a sequence brings this many rows
 #define CC_MAX_DK 128
+#define CC_MAX_DV 1024
 #define CC_LOG2E 1.4426950408889634f   // the kernels keep logarithms to base 2: one operation less per power
 
-// A chunk's record for one head: WQ [dk][64] (per channel the 32 rows of W, then the 32 of
-// e^L q) | Kd [32][dk] (e^{L_n - L} k) | gC [dk] (e^{L_n}) | B [32][32] | U0 [32][dv]
+// A chunk's record for one head: W [dk][32] (per channel the 32 rows) | Kd [32][dk] (e^{L_n - L} k) |
+// gC [dk] (e^{L_n}) | QB [dk + 32][32] (per channel the rows of e^L q, then per row i the column of
+// B) | SU [dk + 32][dv] (S_0, then U0, which becomes U)
 __host__ __device__ __forceinline__ size_t cc_record(int dk, int dv) {
-  return (size_t)dk * 64 + CC_ROWS * dk + dk + CC_ROWS * CC_ROWS + CC_ROWS * dv;
+  return (size_t)2 * dk * CC_ROWS + dk + (size_t)(dk + CC_ROWS) * (CC_ROWS + dv);
 }
+__host__ __device__ __forceinline__ int cc_at_qb(int dk) { return 2 * dk * CC_ROWS + dk; }
+__host__ __device__ __forceinline__ int cc_at_su(int dk) { return cc_at_qb(dk) + (dk + CC_ROWS) * CC_ROWS; }
 // Chunk z of a sequence whose rows start at `first` has an entry that no other chunk has.
 __host__ __device__ __forceinline__ size_t cc_entry(int first, int z, int seq) {
   return (size_t)(first / CC_ROWS + z + seq);
@@ -95,10 +102,10 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
   __syncthreads();
   const size_t entry = (cc_entry(first, z, seq) * H + h) * cc_record(dk, dv);
   float* wq = a.chunks + entry;
-  float* kd = wq + (size_t)dk * 64;
+  float* kd = wq + (size_t)dk * CC_ROWS;
   float* gc = kd + (size_t)CC_ROWS * dk;
-  float* bm = gc + dk;
-  float* u0 = bm + CC_ROWS * CC_ROWS;
+  float* qb = wq + cc_at_qb(dk);
+  float* u0 = wq + cc_at_su(dk) + (size_t)dk * dv;
   // per channel: Fs, the logarithms summed up from the start of a row's half chunk on; and, from the
   // chunk's end back, what is left of a row's key at the end of its half and of the chunk (rows
   // beyond the chunk's end have no decay)
@@ -203,7 +210,7 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
 #pragma unroll
       for (int t = 0; t < CC_ROWS; ++t) u0[(size_t)t * dv + c] = x[t];
     } else {
-      float4* out = reinterpret_cast<float4*>(wq + (size_t)d * 64);
+      float4* out = reinterpret_cast<float4*>(wq + (size_t)d * CC_ROWS);
 #pragma unroll
       for (int t = 0; t < CC_ROWS; t += 4) out[t / 4] = make_float4(x[t], x[t + 1], x[t + 2], x[t + 3]);
     }
@@ -215,9 +222,10 @@ __global__ void __launch_bounds__(256, 2) channel_delta_local_kernel(const Chann
     float v[4];
 #pragma unroll
     for (int x = 0; x < 4; ++x) v[x] = Qs[(t + x) * LD + d] * exp2f(Fs[(t + x) * LD + d] + before);
-    *reinterpret_cast<float4*>(wq + (size_t)d * 64 + CC_ROWS + t) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(qb + (size_t)d * CC_ROWS + t) = make_float4(v[0], v[1], v[2], v[3]);
   }
-  for (int i = tid; i < CC_ROWS * CC_ROWS; i += 256) bm[i] = Bs[i];
+  for (int i = tid; i < CC_ROWS * CC_ROWS; i += 256)     // B by columns
+    qb[(size_t)dk * CC_ROWS + i] = Bs[(i % CC_ROWS) * CC_ROWS + i / CC_ROWS];
 }
 
 __device__ __forceinline__ void cc_copy16(float* smem, const float* gmem) {
@@ -225,10 +233,8 @@ __device__ __forceinline__ void cc_copy16(float* smem, const float* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(s), "l"(gmem));
 }
 
-// floats of a stage: WQ | Kd | gC | B | U0's columns
-__host__ __device__ __forceinline__ int cc_stage(int dk) {
-  return dk * 64 + CC_ROWS * dk + dk + CC_ROWS * CC_ROWS + CC_ROWS * CC_COLS;
-}
+// floats of a chain block's stage: W | Kd | gC | U0's columns
+__host__ __device__ __forceinline__ int cc_stage(int dk) { return 2 * dk * CC_ROWS + dk + CC_ROWS * CC_COLS; }
 
 __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelDeltaArgs a) {
   extern __shared__ __align__(16) float sm[];
@@ -238,8 +244,8 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
   const int H = a.H, dk = a.dk, dv = a.dv, Cc = cd_channels(a);
   const int stage = cc_stage(dk);
   float* S = sm + 2 * stage;                     // [dk][CC_COLS]
-  float* P = S + dk * CC_COLS;                   // [64][CC_COLS]: one half's part of WQ^T S, then e^{L} q S
-  float* U = P + 64 * CC_COLS;                   // [CC_ROWS][CC_COLS]
+  float* P = S + dk * CC_COLS;                   // [4][CC_ROWS][CC_COLS]: a quarter of the channels' part of W S each
+  float* U = P + 4 * CC_ROWS * CC_COLS;          // [CC_ROWS][CC_COLS]
   pdl_wait();
   const int first = a.cu_q[seq], n_seq = a.cu_q[seq + 1] - first;
   if (n_seq <= 0) return;
@@ -247,37 +253,38 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
   float* sp = slot >= 0 ? a.state + (size_t)slot * a.state_stride + (size_t)(a.taps - 1) * Cc + (size_t)h * dv * dk
                         : nullptr;
   const int chunks = (n_seq + CC_ROWS - 1) / CC_ROWS;
+  auto record = [&](int z) { return a.chunks + (cc_entry(first, z, seq) * H + h) * cc_record(dk, dv); };
+  const int whole = 2 * dk * CC_ROWS + dk;                 // (dk is a multiple of four)
   auto stage_in = [&](int z) {
     float* dst = sm + (z & 1) * stage;
-    const float* src = a.chunks + (cc_entry(first, z, seq) * H + h) * cc_record(dk, dv);
-    const int whole = dk * 64 + CC_ROWS * dk + dk + CC_ROWS * CC_ROWS;      // (dk is a multiple of four)
+    const float* src = record(z);
     for (int i = tid * 4; i < whole; i += 1024) cc_copy16(dst + i, src + i);
     const int t = tid / 8, c = (tid % 8) * 4;
-    if (col0 + c < dv) cc_copy16(dst + whole + t * CC_COLS + c, src + whole + (size_t)t * dv + col0 + c);
+    if (col0 + c < dv) cc_copy16(dst + whole + t * CC_COLS + c, src + cc_at_su(dk) + (size_t)(dk + t) * dv + col0 + c);
     cp_async_commit();
   };
   for (int s = 0; s < 2 && col0 + CC_COLS > dv; ++s)       // columns no copy brings
     for (int i = tid; i < CC_ROWS * CC_COLS; i += 256)
-      if (col0 + i % CC_COLS >= dv) sm[s * stage + stage - CC_ROWS * CC_COLS + i] = 0.f;
+      if (col0 + i % CC_COLS >= dv) sm[s * stage + whole + i] = 0.f;
   stage_in(0);
   // the state: element (k, c) of the head's matrix lies at c dk + k
   for (int i = tid; i < dk * CC_COLS; i += 256) {
     const int c = i / dk, k = i % dk;
     S[k * CC_COLS + c] = sp && col0 + c < dv ? sp[(size_t)(col0 + c) * dk + k] : 0.f;
   }
-  // the products' tiles: 4 rows by 4 columns of WQ^T S a thread, half the channels each; 4 by 4 of
-  // the state; 1 by 4 of the read-outs
-  const int half = tid >> 7, tr = (tid & 127) / 8 * 4, tc = (tid & 7) * 4;
-  const int k_lo = half ? dk / 2 : 0, k_hi = half ? dk : dk / 2;
-  const int sk = tid / 8 * 4, orow = tid / 8;
+  // tiles: 4 rows by 4 columns of W S a thread, a quarter of the channels each; 4 by 4 of the state
+  const int quarter = tid >> 6, tr = (tid & 63) / 8 * 4, tc = (tid & 7) * 4;
+  const int per = (dk + 3) / 4, k_lo = quarter * per, k_hi = min(dk, k_lo + per);
+  const int sk = tid / 8 * 4, urow = tid / 8;
+  const bool col_in = col0 + tc < dv;                      // (dv is a multiple of four)
   for (int z = 0; z < chunks; ++z) {
     if (z + 1 < chunks) { stage_in(z + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
     __syncthreads();
-    const float* wq = sm + (z & 1) * stage;
-    const float* kd = wq + dk * 64;
+    const float* w = sm + (z & 1) * stage;
+    const float* kd = w + dk * CC_ROWS;
     const float* gc = kd + CC_ROWS * dk;
-    const float* bm = gc + dk;
-    const float* u0 = bm + CC_ROWS * CC_ROWS;
+    const float* u0 = gc + dk;
+    float* su = record(z) + cc_at_su(dk) + col0 + tc;
     float acc[4][4];
 #pragma unroll
     for (int i = 0; i < 4; ++i)
@@ -285,7 +292,7 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
       for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
 #pragma unroll 8
     for (int k = k_lo; k < k_hi; ++k) {
-      const float4 x = *reinterpret_cast<const float4*>(wq + k * 64 + tr);
+      const float4 x = *reinterpret_cast<const float4*>(w + k * CC_ROWS + tr);
       const float4 y = *reinterpret_cast<const float4*>(S + k * CC_COLS + tc);
       const float xv[4] = {x.x, x.y, x.z, x.w}, yv[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
@@ -293,26 +300,20 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xv[i], yv[j], acc[i][j]);
     }
-    if (half) {
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-        *reinterpret_cast<float4*>(P + (tr + i) * CC_COLS + tc) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
-    }
+    for (int i = 0; i < 4; ++i)
+      *reinterpret_cast<float4*>(P + (quarter * CC_ROWS + tr + i) * CC_COLS + tc) =
+          make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
     __syncthreads();
-    if (!half) {
+    {                                            // U = U0 - W S, four columns of a row a thread
+      float4 u = *reinterpret_cast<const float4*>(u0 + urow * CC_COLS + tc);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        float4* at = reinterpret_cast<float4*>(P + (tr + i) * CC_COLS + tc);
-        const float4 p = *at;
-        float4 s = make_float4(acc[i][0] + p.x, acc[i][1] + p.y, acc[i][2] + p.z, acc[i][3] + p.w);
-        if (tr < CC_ROWS) {                      // a row of W: U = U0 - W S
-          const float4 u = *reinterpret_cast<const float4*>(u0 + (tr + i) * CC_COLS + tc);
-          s = make_float4(u.x - s.x, u.y - s.y, u.z - s.z, u.w - s.w);
-          *reinterpret_cast<float4*>(U + (tr + i) * CC_COLS + tc) = s;
-        } else {
-          *at = s;
-        }
+      for (int q = 0; q < 4; ++q) {
+        const float4 x = *reinterpret_cast<const float4*>(P + (q * CC_ROWS + urow) * CC_COLS + tc);
+        u.x -= x.x, u.y -= x.y, u.z -= x.z, u.w -= x.w;
       }
+      *reinterpret_cast<float4*>(U + urow * CC_COLS + tc) = u;
+      if (col_in) *reinterpret_cast<float4*>(su + (size_t)(dk + urow) * dv) = u;
     }
     __syncthreads();
     if (sk < dk) {                               // S <- diag(e^{L_n}) S + Kd^T U
@@ -320,6 +321,7 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float4 x = *reinterpret_cast<const float4*>(S + (sk + i) * CC_COLS + tc);
+        if (col_in) *reinterpret_cast<float4*>(su + (size_t)(sk + i) * dv) = x;
         const float g = gc[sk + i];
         s[i][0] = g * x.x, s[i][1] = g * x.y, s[i][2] = g * x.z, s[i][3] = g * x.w;
       }
@@ -337,23 +339,6 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
       for (int i = 0; i < 4; ++i)
         *reinterpret_cast<float4*>(S + (sk + i) * CC_COLS + tc) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
     }
-    {                                            // the read-outs: e^{L} q S_0 + B U, four columns of a row a thread
-      float4 o = *reinterpret_cast<const float4*>(P + (CC_ROWS + orow) * CC_COLS + tc);
-#pragma unroll
-      for (int t = 0; t < CC_ROWS; t += 4) {     // (B is zero behind its diagonal)
-        const float4 w = *reinterpret_cast<const float4*>(bm + orow * CC_ROWS + t);
-        const float wv[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float4 u = *reinterpret_cast<const float4*>(U + (t + e) * CC_COLS + tc);
-          o.x = fmaf(wv[e], u.x, o.x), o.y = fmaf(wv[e], u.y, o.y);
-          o.z = fmaf(wv[e], u.z, o.z), o.w = fmaf(wv[e], u.w, o.w);
-        }
-      }
-      const int r = z * CC_ROWS + orow;
-      if (r < n_seq && col0 + tc < dv)           // (dv is a multiple of four)
-        *reinterpret_cast<float4*>(a.o + ((size_t)(first + r) * H + h) * dv + col0 + tc) = o;
-    }
     __syncthreads();                             // S is whole, the stage and P may be overwritten
   }
   pdl_launch_dependents_if_large();
@@ -364,9 +349,92 @@ __global__ void __launch_bounds__(256) channel_delta_chain_kernel(const ChannelD
     }
 }
 
+// The read-outs of a chunk: [32 x (dk + 32)] times [(dk + 32) x dv], 128 columns at a time, a thread 4 rows
+// (its warp's) by 4 columns, 32 elements of the sum staged together (two stages); then the norm
+// over a row's dv numbers, the weight and the gate.
+#define CO_COLS 128
+#define CO_STAGE (CC_ROWS * (CC_ROWS + CO_COLS))
+template <typename T>
+__global__ void __launch_bounds__(256) channel_delta_out_kernel(const ChannelDeltaArgs a) {
+  extern __shared__ __align__(16) float sm[];    // two stages [A: 32 x 32 | B: 32 x CO_COLS] | the read-outs [32][dv]
+  pdl_launch_dependents_if_small();
+  const int tid = threadIdx.x, lane = tid & 31, row = tid / 32 * 4;
+  const int h = blockIdx.y, seq = blockIdx.z, z = blockIdx.x;
+  const int H = a.H, dk = a.dk, dv = a.dv, K = dk + CC_ROWS;
+  float* os = sm + 2 * CO_STAGE;
+  pdl_wait();
+  const int first = a.cu_q[seq], n = min(CC_ROWS, a.cu_q[seq + 1] - first - z * CC_ROWS);
+  if (n <= 0) return;
+  const float* rec = a.chunks + (cc_entry(first, z, seq) * H + h) * cc_record(dk, dv);
+  const float* qb = rec + cc_at_qb(dk);
+  const float* su = rec + cc_at_su(dk);
+  const int tiles = (K + CC_ROWS - 1) / CC_ROWS, col_tiles = (dv + CO_COLS - 1) / CO_COLS;
+  auto stage_in = [&](int s) {                   // stage s: column tile s / tiles, rows (s % tiles) 32 ..
+    float* as = sm + (s & 1) * CO_STAGE;
+    float* bs = as + CC_ROWS * CC_ROWS;
+    const int k0 = s % tiles * CC_ROWS, c0 = s / tiles * CO_COLS;
+    {
+      const int k = tid / 8, r = (tid % 8) * 4;
+      if (k0 + k < K) cc_copy16(as + k * CC_ROWS + r, qb + (size_t)(k0 + k) * CC_ROWS + r);
+    }
+#pragma unroll
+    for (int it = 0; it < 4; ++it) {
+      const int k = tid / 32 + 8 * it, c = lane * 4;
+      if (k0 + k < K && c0 + c < dv) cc_copy16(bs + k * CO_COLS + c, su + (size_t)(k0 + k) * dv + c0 + c);
+    }
+    cp_async_commit();
+  };
+  float acc[4][4];
+  stage_in(0);
+  const int stages = tiles * col_tiles;
+  for (int s = 0; s < stages; ++s) {
+    if (s + 1 < stages) { stage_in(s + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+    __syncthreads();
+    const float* as = sm + (s & 1) * CO_STAGE;
+    const float* bs = as + CC_ROWS * CC_ROWS;
+    if (s % tiles == 0) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    }
+    const int nk = min(CC_ROWS, K - s % tiles * CC_ROWS);
+#pragma unroll 8
+    for (int k = 0; k < nk; ++k) {               // (columns beyond dv hold what no one reads)
+      const float4 x = *reinterpret_cast<const float4*>(as + k * CC_ROWS + row);
+      const float4 y = *reinterpret_cast<const float4*>(bs + k * CO_COLS + lane * 4);
+      const float xv[4] = {x.x, x.y, x.z, x.w}, yv[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xv[i], yv[j], acc[i][j]);
+    }
+    const int c = s / tiles * CO_COLS + lane * 4;
+    if (s % tiles == tiles - 1 && c < dv) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<float4*>(os + (row + i) * dv + c) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+    }
+    __syncthreads();
+  }
+  pdl_launch_dependents_if_large();
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {                  // (a warp finishes the rows it has made)
+    const int r = row + i;
+    if (r >= n) break;
+    const size_t t = (size_t)first + z * CC_ROWS + r;
+    float ss = 0.f;
+    for (int j = lane; j < dv; j += 32) ss = fmaf(os[r * dv + j], os[r * dv + j], ss);
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + a.norm_eps);
+    const float* gate = a.wide + t * H * (dk + dv) + (size_t)H * dk + (size_t)h * dv;
+    T* y = (T*)a.y + (t * H + h) * dv;
+    for (int j = lane; j < dv; j += 32) y[j] = from_f32<T>(os[r * dv + j] * inv * a.norm_w[j] * cd_sigmoid(gate[j]));
+  }
+}
+
 static bool cc_takes(const ChannelDeltaArgs& a) {
   return a.chunks && a.max_rows >= CC_MIN && a.dk <= CC_MAX_DK && a.dk % 4 == 0 && a.dv % 4 == 0 &&
-         (((uintptr_t)a.chunks | (uintptr_t)a.o) & 15) == 0;
+         a.dv <= CC_MAX_DV && (((uintptr_t)a.chunks) & 15) == 0;
 }
 
 template <int E>
@@ -383,17 +451,27 @@ static int cc_local(const ChannelDeltaArgs& a, int chunks, cudaStream_t s) {
   return gb_launch(channel_delta_local_kernel<E>, dim3(chunks, a.H, a.n_seqs), dim3(256), smem, s, a);
 }
 
+template <typename T>
 static int cc_run(const ChannelDeltaArgs& a, cudaStream_t s) {
   const int chunks = (a.max_rows + CC_ROWS - 1) / CC_ROWS;
-  const int e = a.dk <= 32 ? cc_local<1>(a, chunks, s) : a.dk <= 64 ? cc_local<2>(a, chunks, s) : cc_local<4>(a, chunks, s);
+  int e = a.dk <= 32 ? cc_local<1>(a, chunks, s) : a.dk <= 64 ? cc_local<2>(a, chunks, s) : cc_local<4>(a, chunks, s);
   if (e) return e;
-  const size_t smem = (2 * cc_stage(a.dk) + a.dk * CC_COLS + 64 * CC_COLS + CC_ROWS * CC_COLS) * sizeof(float);
-  static size_t configured = 48 * 1024;
-  if (smem > configured) {
+  size_t smem = (2 * cc_stage(a.dk) + a.dk * CC_COLS + 5 * CC_ROWS * CC_COLS) * sizeof(float);
+  static size_t chain_smem = 48 * 1024, out_smem = 48 * 1024;    // (out_smem: per activation type)
+  if (smem > chain_smem) {
     cudaError_t ce = cudaFuncSetAttribute(channel_delta_chain_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                           (int)smem);
     if (ce != cudaSuccess) return (int)ce;
-    configured = smem;
+    chain_smem = smem;
   }
-  return gb_launch(channel_delta_chain_kernel, dim3((a.dv + CC_COLS - 1) / CC_COLS, a.H, a.n_seqs), dim3(256), smem, s, a);
+  e = gb_launch(channel_delta_chain_kernel, dim3((a.dv + CC_COLS - 1) / CC_COLS, a.H, a.n_seqs), dim3(256), smem, s, a);
+  if (e) return e;
+  smem = (2 * CO_STAGE + CC_ROWS * a.dv) * sizeof(float);
+  if (smem > out_smem) {
+    cudaError_t ce = cudaFuncSetAttribute(channel_delta_out_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                          (int)smem);
+    if (ce != cudaSuccess) return (int)ce;
+    out_smem = smem;
+  }
+  return gb_launch(channel_delta_out_kernel<T>, dim3(chunks, a.H, a.n_seqs), dim3(256), smem, s, a);
 }

@@ -1867,10 +1867,11 @@ def channel_delta_run(proj: torch.Tensor, prep: torch.Tensor, low: torch.Tensor,
     a.a_log, a.dt_bias, a.norm_w = a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr()
     a.prep, a.low, a.wide, a.o, a.y = (prep.data_ptr(), low.data_ptr(), wide.data_ptr(), o.data_ptr(), y.data_ptr())
     a.norm_eps, a.max_rows = float(norm_eps), int(max_rows or T)
-    chunked = a.max_rows >= CHANNEL_DELTA_CHUNK_MIN and dk <= 128 and dk % 4 == 0 and dv % 4 == 0
+    chunked = (a.max_rows >= CHANNEL_DELTA_CHUNK_MIN and dk <= 128 and dk % 4 == 0 and dv <= 1024
+               and dv % 4 == 0)
     if chunked:
         C = CHANNEL_DELTA_CHUNK
-        record = dk * 2 * C + C * dk + dk + C * C + C * dv
+        record = 2 * dk * C + dk + (dk + C) * (C + dv)
         chunks = torch.empty(((T // C + slots.shape[0]) * H, record), dtype=torch.float32, device=proj.device)
         a.chunks = chunks.data_ptr()
     _check(_fn("channel_delta", f"gb_channel_delta_run_{_suffix(dtype)}", "pp")(ctypes.addressof(a), _stream()),
