@@ -457,6 +457,9 @@ static int cc_run(const ChannelDeltaArgs& a, cudaStream_t s) {
   int e = a.dk <= 32 ? cc_local<1>(a, chunks, s) : a.dk <= 64 ? cc_local<2>(a, chunks, s) : cc_local<4>(a, chunks, s);
   if (e) return e;
   size_t smem = (2 * cc_stage(a.dk) + a.dk * CC_COLS + 5 * CC_ROWS * CC_COLS) * sizeof(float);
+  // a grid that has an SM for every block: one block an SM, wherever it finds room first (two would
+  // halve each other's pace while other SMs stand idle)
+  if ((long long)((a.dv + CC_COLS - 1) / CC_COLS) * a.H * a.n_seqs <= 148 && smem < 120 * 1024) smem = 120 * 1024;
   static size_t chain_smem = 48 * 1024, out_smem = 48 * 1024;    // (out_smem: per activation type)
   if (smem > chain_smem) {
     cudaError_t ce = cudaFuncSetAttribute(channel_delta_chain_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
