@@ -96,7 +96,7 @@ def in_layer(w, dtype):
 
 # ------------------------------------------------------------------ residual streams
 @BOTH
-@pytest.mark.parametrize("sizes", [(1, 24, 5), (2, 100, 3), (3, 1024, 70), (4, 256, 9), (4, 2560, 130), (5, 512, 8),
+@pytest.mark.parametrize("sizes", [(1, 24, 5), (2, 100, 3), (3, 1024, 70), (4, 288, 9), (4, 2560, 130), (5, 512, 8),
                                    (8, 96, 4), (8, 1024, 2), (11, 36, 6), (4, 37, 3)])
 def test_streams_mixed_read_and_normalised_in_one_kernel(dtype, sizes):
     from grout_b200.kernels import ops
@@ -182,7 +182,7 @@ def _conv(H, G, D, taps, window, cap, dims, base=1e4):
                 mask={"size": window} if window else None, rot={"base": base, "dims": dims} if dims else None)
 
 
-CONV_SHAPES = [_conv(4, 2, 48, 3, 17, 20.0, 48), _conv(6, 3, 64, 4, 64, None, 32), _conv(2, 1, 128, 2, 65, 5.0, 128),
+CONV_SHAPES = [_conv(6, 2, 48, 3, 17, 20.0, 48), _conv(6, 3, 64, 4, 64, None, 32), _conv(2, 1, 128, 2, 65, 5.0, 128),
                _conv(3, 3, 40, 5, 63, 30.0, 16), _conv(4, 1, 24, 1, None, 8.0, 0), _conv(2, 2, 20, 12, 130, None, 20),
                _conv(5, 5, 17, 3, 2, 15.0, 6)]
 
@@ -212,7 +212,7 @@ def test_attention_behind_convolutions_in_every_cut(dtype, m):
 @BOTH
 def test_attention_behind_convolutions_in_mixed_batches(dtype):
     """Requests of unequal lengths together and alone; one-token and many-token rows in one step."""
-    m, W = _conv(4, 2, 48, 4, 30, 20.0, 24), 40
+    m, W = _conv(6, 2, 32, 4, 30, 20.0, 24), 40
     w, pw = in_layer(_conv_weights(m, W, seed=3, sharp=3.0), dtype)
     xs = [rnd(n, W, seed=50 + n).to(dtype) for n in (1, 75, 3, 34)]
     part = _conv_part(m, W, w, dtype)
@@ -302,7 +302,7 @@ def _lat(H, D, Dv, Rq, R, scale=None):
 
 
 @BOTH
-@pytest.mark.parametrize("m", [_lat(4, 32, 48, 96, 128), _lat(3, 24, 16, 20, 40), _lat(20, 16, 24, 36, 64), _lat(2, 128, 32, 64, 150),
+@pytest.mark.parametrize("m", [_lat(5, 24, 40, 88, 128), _lat(3, 24, 16, 20, 40), _lat(20, 16, 24, 36, 64), _lat(2, 128, 32, 64, 150),
                                _lat(2, 8, 8, 8, 8, 0.6), _lat(17, 16, 16, 33, 24)])
 def test_latent_queries_and_sinks_in_every_cut(dtype, m):
     from grout_b200.parts import PartSpec
@@ -412,7 +412,7 @@ def _delta_part(m, W, w, dtype, eps=1e-5):
 
 
 # heads of 64 and 128 and odd ones, several heads on one key, one tap, more taps than rows of a step
-DELTA_SHAPES = [_delta(4, 4, 64, 32, 3), _delta(4, 2, 128, 128, 4, 24, 24), _delta(3, 1, 20, 36, 2, 5, 3), _delta(2, 2, 16, 10, 1),
+DELTA_SHAPES = [_delta(3, 3, 64, 48, 3), _delta(4, 2, 128, 128, 4, 24, 24), _delta(3, 1, 20, 36, 2, 5, 3), _delta(2, 2, 16, 10, 1),
                 _delta(2, 1, 33, 17, 5), _delta(1, 1, 96, 160, 10), _delta(2, 2, 200, 24, 3)]
 
 
